@@ -34,8 +34,11 @@ extern "C" {
  * sequence slots and the ragged step (b200_engine_step, b200_engine_slot_*), the per-mechanism stack ops;  5: + sandwich
  * blocks, latent attention, mLSTM, routed experts;  6: + post-norm blocks, the prepared attention (b200_attn_prep_desc), the
  * generalized delta rule, Mamba-2, softmax-routed experts (fields appended to b200_moe_desc and b200_stack_layer),
- * b200_stack_lin_scan, b200_stack_attn_prep.  All additive: callers of an older version keep working. */
-#define B200_ABI_VERSION 7
+ * b200_stack_lin_scan, b200_stack_attn_prep;  8: + hyper-connected blocks, Mamba's selective scan, RWKV-style time mixing, the
+ * pooled-block attention (fields appended to b200_moe_desc, b200_stack_layer and b200_stack_desc), b200_stack_hyper_step,
+ * b200_stack_input_conv, b200_stack_pool_attention, b200_stack_wkv, b200_stack_mamba1.  All additive: callers of an older version
+ * keep working once they are compiled against this header. */
+#define B200_ABI_VERSION 8
 
 typedef enum b200_status {
   B200_OK = 0,
@@ -295,8 +298,13 @@ int64_t b200_engine_bytes_per_token(const b200_engine* eng, int64_t ctx);
 typedef enum b200_dtype { B200_BF16 = 0, B200_F32 = 1 } b200_dtype;
 /* PARALLEL: x += m·(mixer(h) + ff(h)), h = norm(x), one norm.  SANDWICH: x += post_norm(mixer(norm(x))), then
  * x += ff_post_norm(ff(ff_norm(x))) — a norm before and after every sublayer.  POSTNORM: x += post_norm(mixer(x)), then
- * x += ff_post_norm(ff(x)) — the sublayers read the stream itself, the norm sits on their output only. */
-typedef enum b200_block_kind { B200_BLOCK_PARALLEL = 0, B200_BLOCK_SANDWICH = 1, B200_BLOCK_POSTNORM = 2 } b200_block_kind;
+ * x += ff_post_norm(ff(x)) — the sublayers read the stream itself, the norm sits on their output only.  HYPER: `streams` copies
+ * of the residual stream, all equal to the embedding at the start; a sublayer reads u = Σ_s in[s]·x_s and its output
+ * y = sublayer(norm(u)) goes back as x_d <- Σ_s mix[s][d]·x_s + m·out[d]·y (all copies at once from the old ones); at the end x
+ * is the sum of the copies.  With one copy and unit weights this is the plain pre-norm block x += m·sublayer(norm(x)). */
+typedef enum b200_block_kind {
+  B200_BLOCK_PARALLEL = 0, B200_BLOCK_SANDWICH = 1, B200_BLOCK_POSTNORM = 2, B200_BLOCK_HYPER = 3
+} b200_block_kind;
 /* RELU2: max(z, 0)²; TANH: tanh(z) (the bottleneck of a low-rank decay projection). */
 typedef enum b200_ff_act {
   B200_ACT_GELU_TANH = 0, B200_ACT_SILU = 1, B200_ACT_GELU_ERF = 2, B200_ACT_RELU2 = 3, B200_ACT_TANH = 4
@@ -311,14 +319,19 @@ typedef enum b200_norm_kind { B200_NORM_RMS = 0, B200_NORM_LAYER = 1 } b200_norm
  * of the state.  In sandwich and post-norm blocks ATTENTION is the windowed attention of b200_attn_desc behind the
  * per-token preparation of b200_attn_prep_desc (query / key norms, rotary positions, value norm, value mix-in).
  * GATED_DELTA: the gated delta rule — a key × value matrix per head with one decay per head and a removal along the unit
- * key weighted by a per-head write strength, behind short causal convolutions (b200_gdelta_desc). */
+ * key weighted by a per-head write strength, behind short causal convolutions (b200_gdelta_desc).
+ * In hyper-connected blocks: MAMBA1: a selective scan with a decay per channel and state entry (b200_mamba1_desc).  WKV: time
+ * mixing with a decay per key channel and a bonus for the current token (b200_wkv_desc).  POOL_ATTENTION: attention behind
+ * short convolutions, with pooled blocks behind its window and mixed heads (b200_pool_attn_desc).  PARALLEL: left_scale ·
+ * (a POOL_ATTENTION) + right_scale · (a WKV) over the same input. */
 typedef enum b200_mixer_kind {
   B200_MIX_ATTENTION = 0, B200_MIX_LATENT = 1, B200_MIX_MLSTM = 2, B200_MIX_DELTA = 3, B200_MIX_MAMBA2 = 4,
-  B200_MIX_GATED_DELTA = 5
+  B200_MIX_GATED_DELTA = 5, B200_MIX_MAMBA1 = 6, B200_MIX_WKV = 7, B200_MIX_POOL_ATTENTION = 8, B200_MIX_PARALLEL = 9
 } b200_mixer_kind;
 /* GATED: act(gate)·up → down (merged into w_in / w_out).  DENSE: act(up) → down.  MOE: routed clamped gated experts
- * (+ optional gated shared expert), b200_moe_desc. */
-typedef enum b200_ff_kind { B200_FF_GATED = 0, B200_FF_DENSE = 1, B200_FF_MOE = 2 } b200_ff_kind;
+ * (+ optional gated shared expert), b200_moe_desc.  GLU_CLAMP: one clamped gated unit, g = min(gate·h, limit),
+ * u = clamp(up·h, ±limit), down·(g·sigmoid(1.702 g)·(u + 1)) (hyper-connected blocks). */
+typedef enum b200_ff_kind { B200_FF_GATED = 0, B200_FF_DENSE = 1, B200_FF_MOE = 2, B200_FF_GLU_CLAMP = 3 } b200_ff_kind;
 
 typedef struct b200_attn_desc {
   int32_t heads;       /* query heads */
@@ -375,12 +388,14 @@ typedef struct b200_moe_desc {
   const void* w_exp_out;    /* [experts][width, expert_ff] */
   /* variants (all 0: the form above) */
   int32_t router_kind;      /* 0: weight = sigmoid(logit).  1: scores = softmax over all experts, the chosen scores are divided
-                             * by their sum (+ 1e-20) and multiplied by route_scale */
+                             * by their sum (+ 1e-20) and multiplied by route_scale.  2: softmax over the chosen logits only */
   int32_t weight_output;    /* 0: the weight multiplies the expert's input, 1: its output */
   int32_t expert_act;       /* 0: the clamped gated unit.  else a b200_ff_act applied to up·h alone (no gate rows, no clamp);
                              * the shared expert has the same form: w_ff_in [up8(shared_ff), width] */
   int32_t shared_plain;     /* 0: shared expert × sigmoid(sg·h).  1: added as it is (no gate row) */
   float route_scale;
+  int32_t expert_gated;     /* 1: down·(act(gate·h)·(up·h)) with act = expert_act (a b200_ff_act) and no clamp; w_exp_in holds gate
+                             * and up rows, the shared expert has the same form: w_ff_in [up8(2·shared_ff), width] */
 } b200_moe_desc;
 
 /* What happens to q | k | v of an attention mixer between the in-projection and the cache, per token, in fp32:
@@ -445,6 +460,64 @@ typedef struct b200_gdelta_desc {
   const float* head_norm;   /* [vdim], shared by the heads */
 } b200_gdelta_desc;
 
+/* Weights of one sublayer's hyper-connection over `streams` copies. */
+typedef struct b200_hyper_desc {
+  const float* in;          /* [streams] */
+  const float* out;         /* [streams] */
+  const float* mix;         /* [streams][streams], from × to */
+} b200_hyper_desc;
+
+/* Attention of POOL_ATTENTION mixers and of the left half of PARALLEL ones (sizes heads / kv_heads / dim / vdim / scale / window
+ * in b200_attn_desc; keep_first = out_gate = sink = 0).  w_in rows [q: heads·dim | k: kv_heads·dim | v: kv_heads·vdim] at
+ * off_q / off_k / off_v, biases in b_in.  Every row passes a causal convolution of `taps` taps per channel (no bias; zeros
+ * before the sequence); then, in fp32, q and k are RMS-normed per head and multiplied by q_norm / k_norm (shared by the
+ * heads) and the first rot_dims entries of every head turn (entry i with i + rot_dims/2, angles as in b200_attn_prep_desc).
+ * score = (q·k)·scale, then softcap·tanh(score / softcap).  Position i sees the tokens of its window and, with pool > 0, one
+ * key and one value for every block of `pool` positions that ends before the window — the means of the block's cached keys and
+ * of its cached values.  One softmax over both; with `sink` its denominator also holds exp(sink[head]).  With `talk` the
+ * weights of head h become Σ_g talk[h][g]·(weights of head g) before they meet head h's own key/value head's values. */
+typedef struct b200_pool_attn_desc {
+  int32_t taps, rot_dims, pool;
+  float softcap;            /* 0: no cap */
+  const float* conv_w;      /* [taps][n_in]: row taps − 1 meets the current token; columns are rows of w_in.  NULL: no convolution */
+  const float* q_norm;      /* [dim] or NULL: no head norms */
+  const float* k_norm;      /* [dim] */
+  const float* rot_table;   /* [max_ctx][rot_dims/2][2] fp32 */
+  const float* sink;        /* [heads] or NULL */
+  const float* talk;        /* [heads][heads] or NULL */
+} b200_pool_attn_desc;
+
+/* RWKV-style time mixing.  Five blends of the mixer's input with the previous token's, mix_s = h + (h' − h)·mu_s for
+ * s = r, k, v, g, w (h' = 0 at the start); r, k, v, gate logits = their blends through w_rkvg; decay
+ * w = exp(−exp(w2·tanh(w1·mix_w) + w0)).  Per head with state S [dim][dim]: o = (S + diag(u) k vᵀ)ᵀ r, then
+ * S <- diag(w) S + k vᵀ; then o / rms(o) per head · norm · silu(gate).  The state (fp32) lives in the slot, beside the rows
+ * h' is built from. */
+typedef struct b200_wkv_desc {
+  int32_t heads, dim, rank;
+  const float* mu;          /* [5][width]: r, k, v, g, w */
+  const void* w_rkvg;       /* [4][heads·dim][width] */
+  const void* w1;           /* [up8(rank)][width] (padding rows zero) */
+  const void* w2;           /* [heads·dim][up8(rank)] (padding columns zero) */
+  const float* w0;          /* [heads·dim] */
+  const float* u;           /* [heads·dim] */
+  const float* norm;        /* [heads·dim] */
+} b200_wkv_desc;
+
+/* Mamba's selective scan.  w_in rows [x: inner | z: inner] at off_v / off_g.  x passes a causal convolution of `taps` taps per
+ * channel with a bias and SiLU; w_x·x gives [dt | B | C]; dt = softplus(w_dt·dt + dt_b) per channel, A = −exp(A_log);
+ * S[c][n] <- exp(dt_c·A[c][n])·S[c][n] + dt_c·x_c·B_n,  y_c = Σ_n S[c][n]·C_n + D_c·x_c;  then y·silu(z).  The state (fp32) and
+ * the convolution's last taps − 1 inputs live in the slot. */
+typedef struct b200_mamba1_desc {
+  int32_t inner, state, dt_rank, taps;
+  const float* conv_w;      /* [taps][inner], last row the current token's */
+  const float* conv_b;      /* [inner] */
+  const void* w_x;          /* [up8(up8(dt_rank) + 2·state)][inner]: dt rows, zero rows up to a multiple of 8, B rows, C rows */
+  const void* w_dt;         /* [inner][up8(dt_rank)] (padding columns zero) */
+  const float* dt_b;        /* [inner] */
+  const float* A_log;       /* [inner][state] */
+  const float* D;           /* [inner] */
+} b200_mamba1_desc;
+
 typedef struct b200_stack_layer {
   b200_attn_desc attn;
   int32_t ff;          /* feed-forward width; 0 = the layer has none */
@@ -481,6 +554,17 @@ typedef struct b200_stack_layer {
   int32_t kv_share;      /* attention mixers: > 0: this layer has no key / value rows in w_in and no cache of its own — it
                           * reads the rows that layer kv_share − 1 (an earlier attention layer with equal kv_heads, dim and
                           * vdim) cached for the same positions */
+  /* ---- hyper-connected blocks (zero / NULL for the others).  norm and ff_norm are the norms in front of the sublayers; w_in may
+   * be NULL (n_in 0) for WKV mixers; w_out [width, k_out] = [left | right] for PARALLEL ones, the right half's columns from
+   * up8(heads·vdim) on; GLU_CLAMP: w_ff_in [2·ff, width] = [gate | up], w_ff_out [width, ff] */
+  b200_hyper_desc hc1, hc2; /* the mixer's and the feed-forward's connections */
+  int32_t canon_taps;       /* taps of the convolution the mixer's normed input h passes: h + conv(h); 0: none */
+  const float* canon_w;     /* [canon_taps][width], last row the current token's */
+  float ff_limit;           /* GLU_CLAMP */
+  float left_scale, right_scale; /* PARALLEL (POOL_ATTENTION and WKV alone: 1) */
+  b200_pool_attn_desc pool;
+  b200_wkv_desc wkv;
+  b200_mamba1_desc mamba1;
 } b200_stack_layer;
 
 typedef struct b200_stack_desc {
@@ -501,6 +585,7 @@ typedef struct b200_stack_desc {
   const b200_stack_layer* layers_host;
   int32_t norm_kind;     /* b200_norm_kind of the block and final norms */
   float logit_softcap;   /* > 0: logits <- cap·tanh(logits / cap) */
+  int32_t streams;       /* copies of the residual stream of hyper-connected blocks (0 or 1: one) */
 } b200_stack_desc;
 
 /* Build a stack engine (single GPU).  Borrows the weights; owns the caches [slot][run][max_ctx][kv_heads·dim | ·vdim],

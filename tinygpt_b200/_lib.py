@@ -57,7 +57,7 @@ class MoeDesc(C.Structure):
                 ("limit", C.c_float), ("shared_limit", C.c_float),
                 ("router", C.c_void_p), ("w_exp_in", C.c_void_p), ("w_exp_out", C.c_void_p),
                 ("router_kind", C.c_int32), ("weight_output", C.c_int32), ("expert_act", C.c_int32),
-                ("shared_plain", C.c_int32), ("route_scale", C.c_float)]
+                ("shared_plain", C.c_int32), ("route_scale", C.c_float), ("expert_gated", C.c_int32)]
 
 
 class AttnPrepDesc(C.Structure):
@@ -82,6 +82,27 @@ class GatedDeltaDesc(C.Structure):
                 ("dt_bias", C.c_void_p), ("head_norm", C.c_void_p)]
 
 
+class HyperDesc(C.Structure):
+    _fields_ = [("w_in", C.c_void_p), ("w_out", C.c_void_p), ("mix", C.c_void_p)]
+
+
+class PoolAttnDesc(C.Structure):
+    _fields_ = [("taps", C.c_int32), ("rot_dims", C.c_int32), ("pool", C.c_int32), ("softcap", C.c_float),
+                ("conv_w", C.c_void_p), ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("rot_table", C.c_void_p),
+                ("sink", C.c_void_p), ("talk", C.c_void_p)]
+
+
+class WkvDesc(C.Structure):
+    _fields_ = [("heads", C.c_int32), ("dim", C.c_int32), ("rank", C.c_int32), ("mu", C.c_void_p), ("w_rkvg", C.c_void_p),
+                ("w1", C.c_void_p), ("w2", C.c_void_p), ("w0", C.c_void_p), ("u", C.c_void_p), ("norm", C.c_void_p)]
+
+
+class Mamba1Desc(C.Structure):
+    _fields_ = [("inner", C.c_int32), ("state", C.c_int32), ("dt_rank", C.c_int32), ("taps", C.c_int32),
+                ("conv_w", C.c_void_p), ("conv_b", C.c_void_p), ("w_x", C.c_void_p), ("w_dt", C.c_void_p), ("dt_b", C.c_void_p),
+                ("A_log", C.c_void_p), ("D", C.c_void_p)]
+
+
 class StackLayer(C.Structure):
     _fields_ = [("attn", AttnDesc), ("ff", C.c_int32), ("ff_act", C.c_int32),
                 ("off_q", C.c_int32), ("off_k", C.c_int32), ("off_v", C.c_int32), ("off_g", C.c_int32),
@@ -94,7 +115,9 @@ class StackLayer(C.Structure):
                 ("w_ff_in", C.c_void_p), ("w_ff_out", C.c_void_p),
                 ("lat", LatentDesc), ("rec", MlstmDesc), ("moe", MoeDesc),
                 ("prep", AttnPrepDesc), ("delta", DeltaDesc), ("mamba", MambaDesc), ("gdelta", GatedDeltaDesc),
-                ("b_out", C.c_void_p), ("kv_share", C.c_int32)]
+                ("b_out", C.c_void_p), ("kv_share", C.c_int32),
+                ("hc1", HyperDesc), ("hc2", HyperDesc), ("canon_taps", C.c_int32), ("canon_w", C.c_void_p), ("ff_limit", C.c_float),
+                ("left_scale", C.c_float), ("right_scale", C.c_float), ("pool", PoolAttnDesc), ("wkv", WkvDesc), ("mamba1", Mamba1Desc)]
 
 
 class StackDesc(C.Structure):
@@ -106,7 +129,7 @@ class StackDesc(C.Structure):
                 ("max_ctx", C.c_int32), ("max_slots", C.c_int32),
                 ("embed", C.c_void_p), ("mix_in", C.c_void_p), ("side_table", C.c_void_p), ("final_norm", C.c_void_p),
                 ("head", C.c_void_p), ("layers_host", C.POINTER(StackLayer)),
-                ("norm_kind", C.c_int32), ("logit_softcap", C.c_float)]
+                ("norm_kind", C.c_int32), ("logit_softcap", C.c_float), ("streams", C.c_int32)]
 
 
 # name -> (restype, argtypes); every symbol include/b200_decode.h declares (tests/test_abi.py checks the two agree)

@@ -36,6 +36,13 @@
 // Sandwich blocks also take the prepared attention (biases, either rotary layout, a sink in the softmax; a layer may read the
 // keys and values an earlier layer cached instead of projecting its own), the latent attention with a query latent, a
 // sliding window and an element-wise output gate, and the gated delta rule behind short convolutions.
+//
+// Per run of a layer (hyper-connected block: `streams` copies of the stream):
+//   one pass per sublayer boundary: x_d <- Σ mix·x_s + m·out_d·y of the sublayer before, u = Σ in_s·x_s, n = norm(u)·(offset + w)
+//   mixer:  h = n + conv(n) (the last normed rows live in the slot), its token-shift blends, then Mamba's selective scan,
+//           RWKV-style time mixing, an attention with pooled blocks and mixed heads, or the sum of the last two (one
+//           out-projection over both halves' columns)
+//   feed-forward: a clamped gated unit, or routed gated experts; what both leave is the next pass's y
 #include <algorithm>
 #include <cstring>
 #include <map>
@@ -43,7 +50,10 @@
 #include <vector>
 
 #include "engine.cuh"
+#include "ops.cuh"
+#include "stack_hyper.cuh"
 #include "stack_mix.cuh"
+#include "stack_pool.cuh"
 #include "stack_rec.cuh"
 
 namespace b200 {
@@ -141,7 +151,27 @@ struct StackEngine {
     bool ok_in = false, ok_out = false, ok_ff_in = false, ok_ff_out = false, ok_lora = false, ok_uq = false;
   };
   std::vector<SPlans> splans;
+  // ---- hyper-connected blocks
+  int streams = 1;
+  float* hy_hn = nullptr;          // [tok, width]: normed rows in front of the input convolution
+  void *hmix = nullptr, *p4 = nullptr;   // [5][tok][width] token-shift blends; [4][tok][heads·dim] r | k | v | gate logits
+  float *pool_scores = nullptr, *pool_parts = nullptr, *pool_outs = nullptr;
+  int64_t pool_row_floats = 0, pool_score_floats = 0;
+  int pool_heads_max = 0, pool_hv_max = 0, wkv_max = 0;
+  void* m1_xc = nullptr;
+  float *m1_xd = nullptr, *m1_dt = nullptr;
+  int m1_inner_max = 0, m1_xd_max = 0;
+  const void* hy_y = nullptr;      // the previous sublayer's output, not yet in the copies, and its connection
+  bool hy_y_bf16 = false;
+  b200_hyper_desc hy_prev{};
+  // where a run's pieces lie behind run_s_off: the input convolution's rows come first
+  struct HyperState {
+    size_t pool_conv = 0, wkv = 0, m1_conv = 0, m1 = 0, total = 0;
+  };
+  std::vector<HyperState> hstate;  // per layer
 };
+constexpr int64_t kPoolScoreFloats = 32ll << 20;   // score workspace of prompts on the general kernels (rows go in portions)
+constexpr int kPoolSplitCtas = 4 * 148;            // split launches aim at this many CTAs
 static inline int up8i(int n) { return (n + 7) / 8 * 8; }
 constexpr int kGemmRows = 32;
 
@@ -207,7 +237,7 @@ static int stack_workspace(StackEngine* s, int tok, int rows) {
     return o;
   };
   const size_t W = d.width, T = tok;
-  const size_t o_x = take(T * W * 4), o_xa = take(T * W * 4), o_x0 = take(T * W * 4), o_y = take(T * W * 4);
+  const size_t o_x = take(T * W * 4 * s->streams), o_xa = take(T * W * 4), o_x0 = take(T * W * 4), o_y = take(T * W * 4);
   const size_t o_h = take(T * W * s->esz), o_proj = take(T * s->n_in_max * s->esz);
   const size_t o_mid = take(T * s->k_out_max * s->esz), o_sg = take(T * std::max(1, d.side_dim) * s->esz);
   const size_t o_hn = take((size_t)rows * W * s->esz), o_lg = take((size_t)rows * d.vocab * 4);
@@ -217,7 +247,7 @@ static int stack_workspace(StackEngine* s, int tok, int rows) {
   const size_t o_aws = take((size_t)kStackSplitRows * s->max_heads * kStackMaxSplits * (2 + s->max_vdim) * 4);
   const size_t o_tick = take((size_t)kStackSplitRows * s->max_heads * 4);
   // sandwich blocks
-  const bool sw = d.block != B200_BLOCK_PARALLEL;
+  const bool sw = d.block != B200_BLOCK_PARALLEL;   // blocks whose sublayers have products of their own
   const size_t o_qa = take(sw ? T * s->qa_max * s->esz : 0), o_ol = take(sw ? T * s->ol_max * s->esz : 0);
   const size_t o_lt = take(sw ? T * s->lin_max * 2 : 0);
   const size_t o_pf = take(s->any_rec ? (size_t)kMaxBatch * s->n_in_max * 4 + T * 2 * s->max_heads * 4 : 0);
@@ -238,6 +268,15 @@ static int stack_workspace(StackEngine* s, int tok, int rows) {
   const size_t o_rf = take(T * s->rec_f_max * 4), o_rw = take(T * s->rec_wl_max * 4);
   const size_t o_rl = take(T * s->rec_lr_max * s->esz), o_vk = take(T * s->vkeep_max * s->esz);
   const size_t o_lqq = take(T * s->latq_max * s->esz);
+  // hyper-connected blocks
+  const bool hy = d.block == B200_BLOCK_HYPER;
+  const size_t o_hhn = take(hy ? T * W * 4 : 0), o_hmx = take(s->wkv_max > 0 ? kShiftMixes * T * W * s->esz : 0);
+  const size_t o_p4 = take(4 * T * s->wkv_max * s->esz);
+  s->pool_score_floats = s->pool_row_floats > 0 ? std::max<int64_t>(s->pool_row_floats, std::min<int64_t>((int64_t)T * s->pool_row_floats, kPoolScoreFloats)) : 0;
+  const size_t prow = T + kPoolSplitCtas;
+  const size_t o_psc = take((size_t)s->pool_score_floats * 4), o_ppt = take(prow * s->pool_heads_max * 2 * 4);
+  const size_t o_po = take((size_t)kPoolSplitCtas * s->pool_hv_max * 4);
+  const size_t o_mxc = take(T * s->m1_inner_max * s->esz), o_mxd = take(T * s->m1_xd_max * 4), o_mdt = take(T * s->m1_inner_max * 4);
   B200_CUDA(cudaMalloc((void**)&s->ws, off));
   B200_CUDA(cudaMemset(s->ws, 0, off));
   s->lat_c = lx ? (__nv_bfloat16*)(s->ws + o_lc) : nullptr;
@@ -250,6 +289,15 @@ static int stack_workspace(StackEngine* s, int tok, int rows) {
   s->rec_lr = s->ws + o_rl;
   s->vkeep = s->ws + o_vk;
   s->latq = s->ws + o_lqq;
+  s->hy_hn = (float*)(s->ws + o_hhn);
+  s->hmix = s->ws + o_hmx;
+  s->p4 = s->ws + o_p4;
+  s->pool_scores = (float*)(s->ws + o_psc);
+  s->pool_parts = (float*)(s->ws + o_ppt);
+  s->pool_outs = (float*)(s->ws + o_po);
+  s->m1_xc = s->ws + o_mxc;
+  s->m1_xd = (float*)(s->ws + o_mxd);
+  s->m1_dt = (float*)(s->ws + o_mdt);
   s->ws_tok = tok;
   s->ws_rows = rows;
   s->x = (float*)(s->ws + o_x);
@@ -513,7 +561,8 @@ static int stack_side(StackEngine* s, int li, float* cur, int n_tok, cudaStream_
 // ---------------------------------------------------------------------------------------------------- sandwich blocks
 // C = A·Wᵀ + bias for dense T-typed rows A [M, K]: out_t (T [M, N]) and / or out_f (fp32 [M, N]).  bf16 engines stream W
 // once for steps of up to kMaxBatch rows (GEMV; both outputs from the same fp32 sums), use the tcgen05 GEMM from kGemmRows
-// rows on (bf16 out, widened when fp32 is asked for), and the general kernel otherwise.
+// rows on (bias in its epilogue; fp32 alone is handed out unrounded, beside T it is the widened T), and the general kernel
+// otherwise.
 static int stack_lin(StackEngine* s, const void* A, const void* Wt, const float* bias, int M, int N, int K, const GemvPlan* plan,
                      void* out_t, float* out_f, cudaStream_t st) {
   int rc;
@@ -527,10 +576,9 @@ static int stack_lin(StackEngine* s, const void* A, const void* Wt, const float*
     return gemv_launch(pl, st, s->pdl);
   }
   if (s->fast && M >= kGemmRows && gemm_shape_ok(N, K)) {
-    __nv_bfloat16* o = (__nv_bfloat16*)(out_t ? out_t : s->lin_tmp);
-    if ((rc = launch_gemm_bf16(o, A, Wt, M, N, K, st)) != B200_OK) return rc;
-    if (bias && (rc = launch_stack_bias_add(o, bias, M, N, st)) != B200_OK) return rc;
-    return out_f ? launch_stack_axpy(out_f, o, 1.f, false, (int64_t)M * N, st) : B200_OK;
+    if (out_t == nullptr) return launch_gemm_bf16_f32(out_f, A, Wt, bias, M, N, K, st);
+    if ((rc = launch_gemm_bf16_bias(out_t, A, Wt, bias, M, N, K, st)) != B200_OK) return rc;
+    return out_f ? launch_stack_axpy(out_f, (const __nv_bfloat16*)out_t, 1.f, false, (int64_t)M * N, st) : B200_OK;
   }
   StackGemm g;
   g.a = A; g.lda = K; g.k1 = K;
@@ -566,12 +614,46 @@ static int stack_lin_norm_add(StackEngine* s, const void* A, const void* Wt, int
   const int W = s->d.width;
   int rc;
   if (s->fast && !(M <= kMaxBatch && plan != nullptr) && M >= kGemmRows && gemm_shape_ok(W, K)) {
-    if ((rc = launch_gemm_bf16(s->lin_tmp, A, Wt, M, W, K, st)) != B200_OK) return rc;
-    if (bias && (rc = launch_stack_bias_add((__nv_bfloat16*)s->lin_tmp, bias, M, W, st)) != B200_OK) return rc;
+    if ((rc = launch_gemm_bf16_bias(s->lin_tmp, A, Wt, bias, M, W, K, st)) != B200_OK) return rc;
     return stack_norm_add_next(s, x, s->lin_tmp, true, norm_w, next_w, M, st);
   }
   if ((rc = stack_lin(s, A, Wt, bias, M, W, K, plan, nullptr, s->y, st)) != B200_OK) return rc;
   return stack_norm_add_next(s, x, s->y, false, norm_w, next_w, M, st);
+}
+
+// Routed experts (and the shared one) of layer L on the rows hin → s->y (fp32).  proj, mid and y2 are scratch.
+static int stack_moe_ff(StackEngine* s, const b200_stack_layer& L, const StackEngine::SPlans& pl, const void* hin, int n_tok, cudaStream_t st) {
+  const int W = s->d.width, dt = s->dtype;
+  const size_t esz = s->esz;
+  int rc;
+  MoeRun m = s->moe_ws;
+  m.m = L.moe; m.width = W; m.n_tok = n_tok; m.h = hin; m.y = s->y;
+  m.small = n_tok <= kSmallRows;
+  m.plan_stride = s->moe_e_max;
+  m.tc = s->fast && n_tok >= kGemmRows && gemm_shape_ok(moe_up_rows(L.moe), W) &&
+         gemm_shape_ok(W, L.moe.expert_ff);
+  if (m.tc) {   // that path reads the group sizes back: not inside a stream capture
+    cudaStreamCaptureStatus cs = cudaStreamCaptureStatusNone;
+    B200_CUDA(cudaStreamIsCapturing(st, &cs));
+    m.tc = cs == cudaStreamCaptureStatusNone;
+  }
+  if (L.moe.shared_ff > 0) {
+    const bool plain = L.moe.expert_act != 0 && !L.moe.expert_gated;   // up alone behind a plain activation, no gate row
+    const int fs = L.moe.shared_ff, n_sh = moe_shared_rows(L.moe);
+    if ((rc = stack_lin(s, hin, L.w_ff_in, nullptr, n_tok, n_sh, W, pl.ok_ff_in ? &pl.ff_in : nullptr, s->proj, nullptr, st)) != B200_OK)
+      return rc;
+    if (L.moe.expert_gated) rc = launch_stack_glu(s->mid, fs, s->proj, n_sh, n_tok, fs, L.moe.expert_act, dt, st);
+    else if (plain) rc = launch_stack_act_mul(s->mid, fs, s->proj, nullptr, n_sh, n_tok, fs, L.moe.expert_act, dt, st);
+    else rc = launch_stack_glu_clamp(s->mid, fs, s->proj, n_sh, n_tok, fs, L.moe.shared_limit, dt, st);
+    if (rc != B200_OK) return rc;
+    if ((rc = stack_lin(s, s->mid, L.w_ff_out, nullptr, n_tok, W, fs, pl.ok_ff_out ? &pl.ff_out : nullptr, nullptr, s->y2, st)) != B200_OK)
+      return rc;
+    m.shared = s->y2; m.shared_f32 = true;
+    if (!L.moe.shared_plain) {
+      m.sg = (const uint8_t*)s->proj + (size_t)2 * fs * esz; m.ld_sg = n_sh;
+    }
+  }
+  return run_moe(m, dt, st);
 }
 
 static int stack_run_sandwich(StackEngine* s, int r, float* x, int n_tok, cudaStream_t st) {
@@ -805,34 +887,219 @@ static int stack_run_sandwich(StackEngine* s, int r, float* x, int n_tok, cudaSt
     return stack_lin_norm_add(s, s->mid, L.w_ff_out, n_tok, L.ff, pl.ok_ff_out ? &pl.ff_out : nullptr, L.ff_post_norm, x,
                               next_run_w, st);
   }
-  MoeRun m = s->moe_ws;
-  m.m = L.moe; m.width = W; m.n_tok = n_tok; m.h = hin; m.y = s->y;
-  m.small = n_tok <= kSmallRows;
-  m.plan_stride = s->moe_e_max;
-  m.tc = s->fast && n_tok >= kGemmRows && gemm_shape_ok((L.moe.expert_act != 0 ? 1 : 2) * L.moe.expert_ff, W) &&
-         gemm_shape_ok(W, L.moe.expert_ff);
-  if (m.tc) {   // that path reads the group sizes back: not inside a stream capture
-    cudaStreamCaptureStatus cs = cudaStreamCaptureStatusNone;
-    B200_CUDA(cudaStreamIsCapturing(st, &cs));
-    m.tc = cs == cudaStreamCaptureStatusNone;
-  }
-  if (L.moe.shared_ff > 0) {
-    const bool plain = L.moe.expert_act != 0;   // up alone behind a plain activation, no gate row
-    const int fs = L.moe.shared_ff, n_sh = plain ? up8i(fs) : up8i(2 * fs + 1);
-    if ((rc = stack_lin(s, hin, L.w_ff_in, nullptr, n_tok, n_sh, W, pl.ok_ff_in ? &pl.ff_in : nullptr, s->proj, nullptr, st)) != B200_OK)
-      return rc;
-    if (plain) rc = launch_stack_act_mul(s->mid, fs, s->proj, nullptr, n_sh, n_tok, fs, L.moe.expert_act, dt, st);
-    else rc = launch_stack_glu_clamp(s->mid, fs, s->proj, n_sh, n_tok, fs, L.moe.shared_limit, dt, st);
-    if (rc != B200_OK) return rc;
-    if ((rc = stack_lin(s, s->mid, L.w_ff_out, nullptr, n_tok, W, fs, pl.ok_ff_out ? &pl.ff_out : nullptr, nullptr, s->y2, st)) != B200_OK)
-      return rc;
-    m.shared = s->y2; m.shared_f32 = true;
-    if (!L.moe.shared_plain) {
-      m.sg = (const uint8_t*)s->proj + (size_t)2 * fs * esz; m.ld_sg = n_sh;
-    }
-  }
-  if ((rc = run_moe(m, dt, st)) != B200_OK) return rc;
+  if ((rc = stack_moe_ff(s, L, pl, hin, n_tok, st)) != B200_OK) return rc;
   return stack_norm_add_next(s, x, s->y, false, L.ff_post_norm, next_run_w, n_tok, st);
+}
+
+// Attention with pooled blocks over the step's rows: few rows split their key lists over CTAs; many go whole, in portions the
+// score workspace holds.
+static int stack_pool_attention(StackEngine* s, const PoolAttn& p0, cudaStream_t st) {
+  const int nk = pool_keys_max(s->d.max_ctx, p0.a.window, p0.d.pool), tiles = (nk + kPoolTile - 1) / kPoolTile;
+  const int64_t row = (int64_t)p0.a.heads * nk;
+  const int portion = (int)std::max<int64_t>(1, std::min<int64_t>(p0.n_tok, s->pool_score_floats / row));
+  int rc;
+  for (int r0 = 0; r0 < p0.n_tok; r0 += portion) {
+    PoolAttn p = p0;
+    p.n_tok = std::min(portion, p0.n_tok - r0);
+    p.q = (uint8_t*)p0.q + (size_t)r0 * p0.a.heads * p0.a.dim * s->esz;
+    p.mid = (uint8_t*)p0.mid + (size_t)r0 * p0.ld_mid * s->esz;
+    p.slot = p0.slot + r0; p.pos = p0.pos + r0;
+    p.scores = s->pool_scores; p.parts = s->pool_parts; p.outs = s->pool_outs;
+    p.nk_max = nk;
+    const int splits = std::max(1, std::min({kPoolMaxSplits, tiles, kPoolSplitCtas / p.n_tok}));
+    p.keys_per_split = (tiles + splits - 1) / splits * kPoolTile;
+    p.nsplit = (nk + p.keys_per_split - 1) / p.keys_per_split;
+    if ((rc = launch_pool_attention(p, s->dtype, st)) != B200_OK) return rc;
+  }
+  return B200_OK;
+}
+
+// ---------------------------------------------------------------------------------------------- hyper-connected blocks
+// A sublayer's out-projection; what it leaves joins the copies in the next pass over them.
+static int hyper_out(StackEngine* s, const void* A, const void* Wt, int M, int K, const GemvPlan* plan, const b200_hyper_desc& hc,
+                     cudaStream_t st) {
+  const int W = s->d.width;
+  s->hy_prev = hc;
+  s->hy_y_bf16 = s->fast && !(M <= kMaxBatch && plan != nullptr) && M >= kGemmRows && gemm_shape_ok(W, K);
+  s->hy_y = s->hy_y_bf16 ? s->lin_tmp : (const void*)s->y;
+  return s->hy_y_bf16 ? launch_gemm_bf16(s->lin_tmp, A, Wt, M, W, K, st)
+                      : stack_lin(s, A, Wt, nullptr, M, W, K, plan, nullptr, s->y, st);
+}
+
+static HyperStep hyper_step(StackEngine* s, float* x, int n_tok) {
+  HyperStep p;
+  p.streams = s->streams; p.width = s->d.width; p.n_tok = n_tok; p.x = x;
+  p.y = s->hy_y; p.y_bf16 = s->hy_y_bf16; p.prev = s->hy_prev; p.mult = s->d.residual_mult;
+  p.eps = s->d.norm_eps; p.offset = s->d.norm_offset;
+  p.slot = s->m_slot; p.pos = s->m_pos;
+  s->hy_y = nullptr;
+  return p;
+}
+
+// Time mixing of the step's rows: the blends lie in hmix; r | k | v | gate logits are four products of equal shape.
+static int stack_wkv(StackEngine* s, const b200_stack_layer& L, float* state, void* mid, int64_t ld_mid, int n_pad, int n_tok,
+                     const LinScan& seq, cudaStream_t st) {
+  const b200_wkv_desc& q = L.wkv;
+  const int W = s->d.width, dt = s->dtype, hd = q.heads * q.dim, rk = up8i(q.rank);
+  const size_t esz = s->esz;
+  const uint8_t* mix = (const uint8_t*)s->hmix;
+  const void* mix_w = mix + (size_t)4 * n_tok * W * esz;
+  int rc;
+  if (n_tok <= kSmallRows) {
+    SmallGemv g;
+    g.a = mix; g.lda = W; g.sa = (int64_t)n_tok * W;
+    g.w = q.w_rkvg; g.sw = (int64_t)hd * W;
+    g.c = s->p4; g.ldc = hd; g.sc = (int64_t)n_tok * hd;
+    g.M = n_tok; g.N = hd; g.K = W; g.items = 4;
+    if ((rc = launch_small_gemv(g, dt, st)) != B200_OK) return rc;
+    SmallGemv w1;
+    w1.a = mix_w; w1.lda = W; w1.w = q.w1; w1.c = s->rec_lr; w1.ldc = rk;
+    w1.M = n_tok; w1.N = rk; w1.K = W; w1.act = B200_ACT_TANH;
+    if ((rc = launch_small_gemv(w1, dt, st)) != B200_OK) return rc;
+    SmallGemv w2;
+    w2.a = s->rec_lr; w2.lda = rk; w2.w = q.w2; w2.bias = q.w0; w2.c = s->rec_wl; w2.ldc = hd; w2.c_f32 = true;
+    w2.M = n_tok; w2.N = hd; w2.K = rk;
+    if ((rc = launch_small_gemv(w2, dt, st)) != B200_OK) return rc;
+  } else {
+    if (s->fast && n_tok >= kGemmRows && gemm_shape_ok(hd, W)) {
+      for (int z = 0; z < 4; ++z)
+        if ((rc = launch_gemm_bf16((uint8_t*)s->p4 + (size_t)z * n_tok * hd * 2, mix + (size_t)z * n_tok * W * 2,
+                                   (const uint8_t*)q.w_rkvg + (size_t)z * hd * W * 2, n_tok, hd, W, st)) != B200_OK)
+          return rc;
+    } else {
+      StackGemm g;
+      g.a = mix; g.lda = W; g.k1 = W; g.sa = (int64_t)n_tok * W;
+      g.w = q.w_rkvg; g.sw = (int64_t)hd * W;
+      g.M = n_tok; g.N = hd; g.K = W; g.batch = 4;
+      g.epi = SEPI_STORE; g.c = s->p4; g.ldc = hd; g.sc = (int64_t)n_tok * hd;
+      if ((rc = launch_stack_gemm(g, dt, st)) != B200_OK) return rc;
+    }
+    // the decay's bottleneck stays fp32 up to the operand of its second stage
+    if ((rc = stack_lin(s, mix_w, q.w1, nullptr, n_tok, rk, W, nullptr, nullptr, s->rec_wl, st)) != B200_OK) return rc;
+    if ((rc = launch_stack_cast_rows(s->rec_lr, rk, s->rec_wl, rk, n_tok, rk, true, dt, st)) != B200_OK) return rc;
+    if ((rc = stack_lin(s, s->rec_lr, q.w2, q.w0, n_tok, hd, rk, nullptr, nullptr, s->rec_wl, st)) != B200_OK) return rc;
+  }
+  WkvRun m;
+  m.d = q; m.eps = s->d.norm_eps; m.scale = L.right_scale;
+  m.p4 = s->p4; m.wl = s->rec_wl; m.f = s->rec_f;
+  m.scan = seq;
+  m.scan.ld = wkv_row_floats(q.heads, q.dim);
+  m.scan.state = state; m.scan.slot_stride = (int64_t)s->s_slot;
+  m.scan.o = s->rec_o; m.scan.ld_o = hd;
+  m.mid = mid; m.ld_mid = ld_mid; m.n_pad = n_pad;
+  return run_wkv(m, dt, st);
+}
+
+static int stack_run_hyper(StackEngine* s, int r, float* x, int n_tok, cudaStream_t st) {
+  const b200_stack_desc& d = s->d;
+  const int li = s->run_layer[r];
+  const b200_stack_layer& L = s->layers[li];
+  const StackEngine::SPlans& pl = s->splans[li];
+  const StackEngine::HyperState& hs = s->hstate[li];
+  const int W = d.width, dt = s->dtype;
+  const size_t esz = s->esz;
+  int rc;
+  bool single = true;   // every row is its sequence's only new row: states move on inside the kernels that read them
+  for (const StackEngine::Seg& g : s->segs) single = single && g.count == 1;
+  LinScan seq;
+  seq.slot = s->m_slot; seq.pos = s->m_pos; seq.n_tok = n_tok; seq.n_seg = n_tok;
+  if (!s->segs.empty()) {
+    seq.n_seg = (int)s->segs.size(); seq.seg_row0 = s->m_seg_row0; seq.seg_count = s->m_seg_count;
+  }
+  float* state = s->rstate + s->run_s_off[r];
+  ShiftState shift;
+  shift.seg_row0 = s->m_seg_row0; shift.seg_count = s->m_seg_count; shift.slot = s->m_slot; shift.pos = s->m_pos;
+  shift.n_seg = (int)s->segs.size(); shift.slot_stride = (int64_t)s->s_slot;
+  auto keep_rows = [&](const void* rows, bool f32, int64_t ld, int channels, int keep, float* to) {
+    if (single || keep <= 0) return;
+    shift.src[shift.n_src++] = ShiftSource{rows, f32, ld, channels, keep, to};
+  };
+  // ---- the previous sublayer joins the copies; the mixer's input
+  const bool has_left = L.mixer == B200_MIX_POOL_ATTENTION || L.mixer == B200_MIX_PARALLEL;
+  const bool has_wkv = L.mixer == B200_MIX_WKV || L.mixer == B200_MIX_PARALLEL;
+  InputConv c;
+  c.taps = std::max(1, L.canon_taps);
+  c.w = L.canon_taps > 0 ? L.canon_w : nullptr;
+  c.mu = has_wkv ? L.wkv.mu : nullptr;
+  c.h = L.mixer == B200_MIX_WKV ? nullptr : s->h;
+  c.mix = s->hmix;
+  c.state = state; c.slot_stride = (int64_t)s->s_slot;
+  HyperStep a = hyper_step(s, x, n_tok);
+  a.in = L.hc1.in; a.norm_w = L.norm;
+  if (single) {
+    a.conv = true; a.c = c;
+  } else {
+    a.hn = s->hy_hn;
+  }
+  if ((rc = launch_hyper_step(a, dt, st)) != B200_OK) return rc;
+  if (!single && (rc = launch_input_conv(c, s->hy_hn, s->m_slot, s->m_pos, n_tok, W, dt, st)) != B200_OK) return rc;
+  keep_rows(s->hy_hn, true, W, W, c.taps, state);
+  // ---- mixer
+  if (L.n_in > 0 && (rc = stack_lin(s, s->h, L.w_in, L.b_in, n_tok, L.n_in, W, pl.ok_in ? &pl.in : nullptr, s->proj, nullptr, st)) != B200_OK)
+    return rc;
+  const int right_off = has_left ? up8i(L.attn.heads * L.attn.vdim) : 0;
+  if (has_left) {
+    PoolAttn p;
+    p.a = L.attn; p.d = L.pool; p.eps = d.norm_eps;
+    p.proj = s->proj; p.ld_proj = L.n_in; p.off_q = L.off_q; p.off_k = L.off_k; p.off_v = L.off_v;
+    p.q = s->qa;
+    p.kcache = s->kbase + s->run_k_off[r] * esz; p.vcache = s->vbase + s->run_v_off[r] * esz;
+    p.k_slot_stride = (int64_t)s->k_slot; p.v_slot_stride = (int64_t)s->v_slot; p.max_ctx = d.max_ctx;
+    p.conv_state = state + hs.pool_conv; p.conv_slot_stride = (int64_t)s->s_slot;
+    p.single = single ? 1 : 0;
+    p.slot = s->m_slot; p.pos = s->m_pos; p.n_tok = n_tok;
+    p.mid = s->mid; p.ld_mid = L.k_out; p.n_pad = right_off; p.out_scale = L.left_scale;
+    if ((rc = launch_pool_prep(p, dt, st)) != B200_OK) return rc;
+    if (!single && (rc = launch_pool_blocks(p, dt, st)) != B200_OK) return rc;
+    if (L.pool.conv_w != nullptr) keep_rows(s->proj, false, L.n_in, L.n_in, L.pool.taps - 1, state + hs.pool_conv);
+    if ((rc = stack_pool_attention(s, p, st)) != B200_OK) return rc;
+  }
+  if (has_wkv) {
+    if ((rc = stack_wkv(s, L, state + hs.wkv, (uint8_t*)s->mid + (size_t)right_off * esz, L.k_out, L.k_out - right_off, n_tok, seq, st)) != B200_OK)
+      return rc;
+  }
+  if (L.mixer == B200_MIX_MAMBA1) {
+    const b200_mamba1_desc& q = L.mamba1;
+    const int rk = up8i(q.dt_rank), nx = up8i(rk + 2 * q.state);
+    Mamba1Run m;
+    m.d = q;
+    m.proj = s->proj; m.ld_proj = L.n_in; m.off_x = L.off_v; m.off_z = L.off_g;
+    m.conv_state = state + hs.m1_conv; m.state = state + hs.m1; m.slot_stride = (int64_t)s->s_slot;
+    m.advance = single ? 1 : 0;
+    m.xc = s->m1_xc; m.xd = s->m1_xd; m.ld_xd = nx; m.dt = s->m1_dt;
+    m.slot = s->m_slot; m.pos = s->m_pos; m.n_tok = n_tok; m.n_seg = seq.n_seg; m.seg_row0 = seq.seg_row0; m.seg_count = seq.seg_count;
+    m.mid = s->mid; m.ld_mid = L.k_out;
+    if ((rc = launch_mamba1_conv(m, dt, st)) != B200_OK) return rc;
+    keep_rows((const uint8_t*)s->proj + (size_t)L.off_v * esz, false, L.n_in, q.inner, q.taps - 1, state + hs.m1_conv);
+    if (n_tok <= kSmallRows) {
+      SmallGemv g;
+      g.a = s->m1_xc; g.lda = q.inner; g.w = q.w_x; g.c = s->m1_xd; g.ldc = nx; g.c_f32 = true;
+      g.M = n_tok; g.N = nx; g.K = q.inner;
+      if ((rc = launch_small_gemv(g, dt, st)) != B200_OK) return rc;
+      if ((rc = launch_mamba1_dt(m, dt, st)) != B200_OK) return rc;
+    } else {
+      if ((rc = stack_lin(s, s->m1_xc, q.w_x, nullptr, n_tok, nx, q.inner, nullptr, nullptr, s->m1_xd, st)) != B200_OK) return rc;
+      if ((rc = launch_stack_cast_rows(s->rec_lr, rk, s->m1_xd, nx, n_tok, rk, false, dt, st)) != B200_OK) return rc;
+      if ((rc = stack_lin(s, s->rec_lr, q.w_dt, q.dt_b, n_tok, q.inner, rk, nullptr, nullptr, s->m1_dt, st)) != B200_OK) return rc;
+    }
+    if ((rc = launch_mamba1_scan(m, dt, st)) != B200_OK) return rc;
+  }
+  if ((rc = launch_shift_state(shift, dt, st)) != B200_OK) return rc;
+  if ((rc = hyper_out(s, s->mid, L.w_out, n_tok, L.k_out, pl.ok_out ? &pl.out : nullptr, L.hc1, st)) != B200_OK) return rc;
+  // ---- feed-forward
+  if (L.ff_kind != B200_FF_MOE && L.ff <= 0) return B200_OK;
+  HyperStep f = hyper_step(s, x, n_tok);
+  f.in = L.hc2.in; f.norm_w = L.ff_norm; f.h = s->h;
+  if ((rc = launch_hyper_step(f, dt, st)) != B200_OK) return rc;
+  if (L.ff_kind == B200_FF_MOE) {
+    if ((rc = stack_moe_ff(s, L, pl, s->h, n_tok, st)) != B200_OK) return rc;
+    s->hy_y = s->y; s->hy_y_bf16 = false; s->hy_prev = L.hc2;
+    return B200_OK;
+  }
+  if ((rc = stack_lin(s, s->h, L.w_ff_in, nullptr, n_tok, 2 * L.ff, W, pl.ok_ff_in ? &pl.ff_in : nullptr, s->proj, nullptr, st)) != B200_OK)
+    return rc;
+  if ((rc = launch_stack_glu_clamp(s->mid, L.ff, s->proj, 2 * L.ff, n_tok, L.ff, L.ff_limit, dt, st)) != B200_OK) return rc;
+  return hyper_out(s, s->mid, L.w_ff_out, n_tok, L.ff, pl.ok_ff_out ? &pl.ff_out : nullptr, L.hc2, st);
 }
 
 // One pass: n_tok rows {m_tok, m_slot, m_pos} through every run, then the head for the n_rows rows listed in m_want.
@@ -842,8 +1109,11 @@ static int stack_pass(b200_engine* e, int n_tok, int n_rows, cudaStream_t st, bo
   const b200_stack_desc& d = s->d;
   const int W = d.width, dt = s->dtype;
   int rc;
-  if ((rc = launch_stack_embed(s->x, s->x0, d.embed, s->m_tok, n_tok, d.vocab, W, d.embed_scale, dt, st)) != B200_OK)
+  const bool hyper = d.block == B200_BLOCK_HYPER;
+  if ((rc = hyper ? launch_hyper_embed(s->x, d.embed, s->m_tok, n_tok, d.vocab, W, s->streams, d.embed_scale, dt, st)
+                  : launch_stack_embed(s->x, s->x0, d.embed, s->m_tok, n_tok, d.vocab, W, d.embed_scale, dt, st)) != B200_OK)
     return rc;
+  s->hy_y = nullptr;
   float *cur = s->x, *other = s->x_alt;
   s->h_ready = false;
   if (s->any_rec && !s->segs.empty()) {   // the recurrences walk every sequence's rows in order
@@ -857,6 +1127,10 @@ static int stack_pass(b200_engine* e, int n_tok, int n_rows, cudaStream_t st, bo
   }
   for (int r = 0; r < d.n_runs; ++r) {
     const b200_stack_layer& L = s->layers[s->run_layer[r]];
+    if (hyper) {
+      if ((rc = stack_run_hyper(s, r, cur, n_tok, st)) != B200_OK) return rc;
+      continue;
+    }
     if (d.block != B200_BLOCK_PARALLEL) {
       if ((rc = stack_run_sandwich(s, r, cur, n_tok, st)) != B200_OK) return rc;
       continue;
@@ -892,6 +1166,12 @@ static int stack_pass(b200_engine* e, int n_tok, int n_rows, cudaStream_t st, bo
     }
     if ((rc = stack_product_out(s, s->run_layer[r], cur, n_tok, st)) != B200_OK) return rc;
     if (L.side_gate != nullptr && (rc = stack_side(s, s->run_layer[r], cur, n_tok, st)) != B200_OK) return rc;
+  }
+  if (hyper && n_rows > 0) {   // the last sublayer joins the copies, and the head reads their sum
+    HyperStep p = hyper_step(s, cur, n_tok);
+    p.hn = s->x0;
+    if ((rc = launch_hyper_step(p, dt, st)) != B200_OK) return rc;
+    cur = s->x0;
   }
   if (n_rows > 0 && (rc = stack_product_head(s, cur, rows_in_order ? nullptr : s->m_want, n_rows, st)) != B200_OK) return rc;
   return B200_OK;
@@ -1167,6 +1447,21 @@ int64_t stack_bytes_per_token(const b200_engine* e, int64_t ctx) {
   for (int r = 0; r < d.n_runs; ++r) {
     const b200_stack_layer& L = s->layers[s->run_layer[r]];
     bytes += ((int64_t)L.n_in * d.width + (int64_t)d.width * L.k_out) * s->esz;
+    if (d.block == B200_BLOCK_HYPER) {
+      const b200_attn_desc& a = L.attn;
+      const int64_t hd = (int64_t)L.wkv.heads * L.wkv.dim;
+      if (L.mixer == B200_MIX_POOL_ATTENTION || L.mixer == B200_MIX_PARALLEL) {
+        const int64_t keys = pool_keys_max((int)ctx + 1, a.window, L.pool.pool);
+        bytes += (keys + 1) * a.kv_heads * (a.dim + a.vdim) * s->esz;
+      }
+      if (L.mixer == B200_MIX_WKV || L.mixer == B200_MIX_PARALLEL)
+        bytes += (4 * hd * d.width + (int64_t)L.wkv.rank * (d.width + hd)) * s->esz + 2 * hd * L.wkv.dim * 4;
+      if (L.mixer == B200_MIX_MAMBA1)
+        bytes += (int64_t)L.mamba1.inner * (2 * L.mamba1.dt_rank + 2 * L.mamba1.state) * s->esz + 2ll * L.mamba1.inner * L.mamba1.state * 4;
+      if (L.ff_kind == B200_FF_MOE) bytes += ((int64_t)L.moe.experts + 3ll * L.moe.top * L.moe.expert_ff + 3ll * L.moe.shared_ff) * d.width * s->esz;
+      else bytes += 3ll * L.ff * d.width * s->esz;
+      continue;
+    }
     if (d.block == B200_BLOCK_SANDWICH) {
       const b200_attn_desc& a = L.attn;
       if (L.mixer == B200_MIX_ATTENTION) {
@@ -1201,6 +1496,105 @@ int64_t stack_bytes_per_token(const b200_engine* e, int64_t ctx) {
   return bytes;
 }
 
+// Layer l of a hyper-connected model: its description, the workspace it needs and where its state's pieces lie.
+static int stack_check_hyper(StackEngine* s, int l) {
+  const b200_stack_layer& L = s->layers[l];
+  const b200_attn_desc& a = L.attn;
+  const int W = s->d.width;
+  const bool left = L.mixer == B200_MIX_POOL_ATTENTION || L.mixer == B200_MIX_PARALLEL;
+  const bool wkv = L.mixer == B200_MIX_WKV || L.mixer == B200_MIX_PARALLEL;
+  B200_CHECK_ARG(left || wkv || L.mixer == B200_MIX_MAMBA1, "engine_create_stack: layer %d: mixer kind %d is not built for hyper-connected blocks", l, L.mixer);
+  B200_CHECK_ARG(L.norm && L.w_out && L.k_out > 0 && L.n_in >= 0 && (L.n_in == 0 || L.w_in), "engine_create_stack: layer %d: null weight", l);
+  for (const b200_hyper_desc* h : {&L.hc1, &L.hc2})
+    B200_CHECK_ARG(s->streams == 1 || (h == &L.hc2 && L.ff_kind != B200_FF_MOE && L.ff <= 0) || (h->in && h->out && h->mix),
+                   "engine_create_stack: layer %d: %d streams need their connection weights", l, s->streams);
+  B200_CHECK_ARG(L.canon_taps >= 0 && L.canon_taps <= kConvMaxTaps && (L.canon_taps == 0 || L.canon_w),
+                 "engine_create_stack: layer %d: input convolution of %d taps (0 … %d)", l, L.canon_taps, kConvMaxTaps);
+  StackEngine::HyperState& st = s->hstate[l];
+  st.total = (size_t)std::max(1, L.canon_taps) * W;
+  if (left) {
+    const b200_pool_attn_desc& q = L.pool;
+    B200_CHECK_ARG(a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.dim > 0 && a.vdim > 0 && a.window >= 0 &&
+                       a.keep_first == 0 && !a.out_gate && !a.sink && q.pool >= 0 && q.softcap >= 0.f,
+                   "engine_create_stack: layer %d: bad attention description", l);
+    B200_CHECK_ARG(L.off_q >= 0 && L.off_q + a.heads * a.dim <= L.n_in && L.off_k + a.kv_heads * a.dim <= L.n_in &&
+                       L.off_v + a.kv_heads * a.vdim <= L.n_in,
+                   "engine_create_stack: layer %d: segment offsets do not fit", l);
+    B200_CHECK_ARG(q.rot_dims >= 0 && q.rot_dims % 2 == 0 && q.rot_dims <= a.dim && (q.rot_dims == 0 || q.rot_table) &&
+                       (q.q_norm == nullptr) == (q.k_norm == nullptr) &&
+                       (q.conv_w == nullptr || (q.taps >= 1 && q.taps <= kConvMaxTaps)),
+                   "engine_create_stack: layer %d: attention preparation", l);
+    B200_CHECK_ARG((size_t)((a.heads / a.kv_heads + 1) * a.dim + a.vdim) * 4 <= 48 * 1024 && (size_t)a.heads * a.dim * 4 <= 200 * 1024 &&
+                       (size_t)(2 * a.heads + 2 * a.heads * (kPoolTile + 1) + a.heads * a.vdim) * 4 <= 200 * 1024,
+                   "engine_create_stack: layer %d: heads · head size above one CTA's shared memory", l);
+    st.pool_conv = st.total;
+    st.total += q.conv_w != nullptr ? (size_t)(q.taps - 1) * L.n_in : 0;
+    s->qa_max = std::max(s->qa_max, a.heads * a.dim);
+    s->pool_row_floats = std::max(s->pool_row_floats, (int64_t)a.heads * pool_keys_max(s->d.max_ctx, a.window, q.pool));
+    s->pool_heads_max = std::max(s->pool_heads_max, a.heads);
+    s->pool_hv_max = std::max(s->pool_hv_max, a.heads * a.vdim);
+  }
+  if (wkv) {
+    const b200_wkv_desc& q = L.wkv;
+    B200_CHECK_ARG(q.heads > 0 && q.dim > 0 && q.dim <= kScanMaxDim && q.rank > 0 && q.mu && q.w_rkvg && q.w1 && q.w2 && q.w0 && q.u && q.norm,
+                   "engine_create_stack: layer %d: time-mixing description (head size up to %d)", l, kScanMaxDim);
+    const int hd = q.heads * q.dim;
+    st.wkv = st.total;
+    st.total += (size_t)hd * q.dim;
+    s->wkv_max = std::max(s->wkv_max, hd);
+    s->rec_f_max = std::max(s->rec_f_max, (int)wkv_row_floats(q.heads, q.dim));
+    s->rec_o_max = std::max(s->rec_o_max, hd);
+    s->rec_wl_max = std::max(s->rec_wl_max, std::max(hd, up8i(q.rank)));
+    s->rec_lr_max = std::max(s->rec_lr_max, up8i(q.rank));
+    s->lin_max = std::max(s->lin_max, hd);
+  }
+  if (L.mixer == B200_MIX_MAMBA1) {
+    const b200_mamba1_desc& q = L.mamba1;
+    B200_CHECK_ARG(q.inner > 0 && q.state > 0 && q.state <= kMamba1MaxState && q.dt_rank > 0 && q.taps >= 1 && q.taps <= kMambaMaxTaps &&
+                       q.conv_w && q.conv_b && q.w_x && q.w_dt && q.dt_b && q.A_log && q.D && L.k_out == q.inner &&
+                       L.off_v >= 0 && L.off_v + q.inner <= L.n_in && L.off_g >= 0 && L.off_g + q.inner <= L.n_in,
+                   "engine_create_stack: layer %d: Mamba description (state up to %d, up to %d taps)", l, kMamba1MaxState, kMambaMaxTaps);
+    st.m1_conv = st.total;
+    st.total += (size_t)(q.taps - 1) * q.inner;
+    st.m1 = st.total;
+    st.total += (size_t)q.inner * q.state;
+    s->m1_inner_max = std::max(s->m1_inner_max, q.inner);
+    s->m1_xd_max = std::max(s->m1_xd_max, up8i(up8i(q.dt_rank) + 2 * q.state));
+    s->rec_lr_max = std::max(s->rec_lr_max, up8i(q.dt_rank));
+    s->lin_max = std::max(s->lin_max, std::max(q.inner, s->m1_xd_max));
+  } else {
+    const int right = wkv ? L.wkv.heads * L.wkv.dim : 0, from = left ? up8i(a.heads * a.vdim) : 0;
+    B200_CHECK_ARG(L.k_out >= from + right, "engine_create_stack: layer %d: k_out %d below its columns", l, L.k_out);
+  }
+  int ff_rows = 0, ff_mid = 0;
+  if (L.ff_kind == B200_FF_MOE) {
+    const b200_moe_desc& m = L.moe;
+    B200_CHECK_ARG(m.experts > 0 && m.top > 0 && m.top <= m.experts && m.expert_ff > 0 && m.shared_ff >= 0 && m.router && m.w_exp_in &&
+                       m.w_exp_out && L.ff_norm && (m.shared_ff == 0 || (L.w_ff_in && L.w_ff_out)) && m.router_kind >= 0 && m.router_kind <= 2 &&
+                       m.expert_act >= 0 && m.expert_act <= B200_ACT_TANH &&
+                       ((m.expert_act == 0 && !m.expert_gated) || m.shared_ff == 0 || m.shared_plain),
+                   "engine_create_stack: layer %d: mixture-of-experts description", l);
+    s->any_moe = true;
+    s->moe_e_max = std::max(s->moe_e_max, m.experts);
+    s->moe_top_max = std::max(s->moe_top_max, m.top);
+    s->moe_ff_max = std::max(s->moe_ff_max, m.expert_ff);
+    ff_rows = m.shared_ff > 0 ? moe_shared_rows(m) : 0;
+    ff_mid = m.shared_ff;
+  } else {
+    B200_CHECK_ARG(L.ff_kind == B200_FF_GLU_CLAMP && L.ff >= 0 && (L.ff == 0 || (L.ff_norm && L.w_ff_in && L.w_ff_out)),
+                   "engine_create_stack: layer %d: feed-forward kind %d", l, L.ff_kind);
+    ff_rows = 2 * L.ff;
+    ff_mid = L.ff;
+  }
+  st.total = (st.total + 3) / 4 * 4;
+  s->any_rec = s->recurrent = true;
+  s->max_heads = std::max(s->max_heads, a.heads);
+  s->n_in_max = std::max(s->n_in_max, std::max(L.n_in, ff_rows));
+  s->k_out_max = std::max(s->k_out_max, std::max(L.k_out, ff_mid));
+  s->lin_max = std::max(s->lin_max, std::max(W, std::max(L.n_in, ff_rows)));
+  return B200_OK;
+}
+
 static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
   B200_CHECK_ARG(desc && out, "engine_create_stack: null argument");
   *out = nullptr;
@@ -1208,7 +1602,8 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
   if (rc != B200_OK) return rc;
   const b200_stack_desc& d = *desc;
   B200_CHECK_ARG(d.dtype == B200_BF16 || d.dtype == B200_F32, "engine_create_stack: unknown dtype %d", d.dtype);
-  B200_CHECK_ARG(d.block == B200_BLOCK_PARALLEL || d.block == B200_BLOCK_SANDWICH || d.block == B200_BLOCK_POSTNORM,
+  B200_CHECK_ARG(d.block == B200_BLOCK_PARALLEL || d.block == B200_BLOCK_SANDWICH || d.block == B200_BLOCK_POSTNORM ||
+                     d.block == B200_BLOCK_HYPER,
                  "engine_create_stack: block kind %d not built", d.block);
   B200_CHECK_ARG(d.block != B200_BLOCK_POSTNORM || d.norm_kind == B200_NORM_RMS,
                  "engine_create_stack: post-norm blocks are built with RMS norms");
@@ -1244,7 +1639,16 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
   s->run_mix.assign(d.run_mix_host, d.run_mix_host + d.n_runs);
   s->d.layers_host = nullptr;
   s->d.run_layer_host = s->d.run_mix_host = nullptr;
-  const bool sandwich = d.block != B200_BLOCK_PARALLEL;   // a norm per sublayer: in front and behind, or behind only
+  const bool hyper = d.block == B200_BLOCK_HYPER;
+  if (hyper) {
+    s->streams = std::max(1, d.streams);
+    B200_CHECK_ARG(d.norm_kind == B200_NORM_RMS && s->streams <= kMaxStreams && !d.mix_in && !d.side_table,
+                   "engine_create_stack: hyper-connected blocks are built with RMS norms, 1 … %d streams, no mix-in and no token table", kMaxStreams);
+    s->hstate.resize(d.n_layers);
+    for (int l = 0; l < d.n_layers; ++l)
+      if ((rc = stack_check_hyper(s, l)) != B200_OK) return rc;
+  }
+  const bool sandwich = d.block != B200_BLOCK_PARALLEL && !hyper;   // a norm per sublayer: in front and behind, or behind only
   for (int l = 0; sandwich && l < d.n_layers; ++l) {
     const b200_stack_layer& L = s->layers[l];
     const b200_attn_desc& a = L.attn;
@@ -1365,7 +1769,7 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
                          m.w_exp_in && m.w_exp_out && (L.ff_norm || d.block == B200_BLOCK_POSTNORM) && L.ff_post_norm &&
                          (m.shared_ff == 0 || (L.w_ff_in && L.w_ff_out)),
                      "engine_create_stack: layer %d: mixture-of-experts description", l);
-      B200_CHECK_ARG((m.router_kind == 0 || m.router_kind == 1) && m.expert_act >= 0 && m.expert_act <= B200_ACT_TANH &&
+      B200_CHECK_ARG((m.router_kind >= 0 && m.router_kind <= 2) && !m.expert_gated && m.expert_act >= 0 && m.expert_act <= B200_ACT_TANH &&
                          (m.expert_act == 0 || m.shared_ff == 0 || m.shared_plain),
                      "engine_create_stack: layer %d: router kind %d / expert activation %d (a plain activation takes a plain shared expert)",
                      l, m.router_kind, m.expert_act);
@@ -1381,7 +1785,7 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
     s->k_out_max = std::max(s->k_out_max, std::max(L.k_out, ff_mid));
     s->lin_max = std::max(s->lin_max, std::max(W, std::max(L.n_in, ff_rows)));
   }
-  for (int l = 0; !sandwich && l < d.n_layers; ++l) {
+  for (int l = 0; !sandwich && !hyper && l < d.n_layers; ++l) {
     const b200_stack_layer& L = s->layers[l];
     const b200_attn_desc& a = L.attn;
     B200_CHECK_ARG(L.mixer == B200_MIX_ATTENTION && L.ff_kind == B200_FF_GATED,
@@ -1417,7 +1821,14 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
     s->run_k_off[r] = s->k_slot;
     s->run_v_off[r] = s->v_slot;
     s->run_s_off[r] = s->s_slot;
-    if (RL.mixer == B200_MIX_ATTENTION && sandwich && RL.kv_share > 0) {
+    if (hyper) {   // token rows, block rows behind them, and a fixed-size state
+      if (RL.mixer == B200_MIX_POOL_ATTENTION || RL.mixer == B200_MIX_PARALLEL) {
+        const size_t rows = (size_t)d.max_ctx + pool_rows(d.max_ctx, RL.pool.pool);
+        s->k_slot += (rows * a.kv_heads * a.dim + 7) / 8 * 8;   // every run starts on a 16-byte boundary
+        s->v_slot += (rows * a.kv_heads * a.vdim + 7) / 8 * 8;
+      }
+      s->s_slot += s->hstate[s->run_layer[r]].total;
+    } else if (RL.mixer == B200_MIX_ATTENTION && sandwich && RL.kv_share > 0) {
       // the cache of the latest earlier run of the source layer (the pass of a loop this run belongs to, or the last one)
       int src = -1;
       for (int q = 0; q < r; ++q)
@@ -1458,7 +1869,20 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
       if (k % 8 != 0 || (reinterpret_cast<uintptr_t>(w) & 15) != 0) return false;
       return gemv_make_plan(pl, w, n, n, k, 1, pro, epi, s->num_sms) == B200_OK;
     };
-    for (int l = 0; !sandwich && l < d.n_layers; ++l) {
+    for (int l = 0; hyper && l < d.n_layers; ++l) {
+      const b200_stack_layer& L = s->layers[l];
+      StackEngine::SPlans& sp = s->splans[l];
+      sp.ok_in = L.n_in > 0 && plan(&sp.in, L.w_in, L.n_in, d.width, EPI_BIAS_F32);
+      sp.ok_out = plan(&sp.out, L.w_out, d.width, L.k_out, EPI_BIAS_F32);
+      if (L.ff_kind == B200_FF_GLU_CLAMP && L.ff > 0) {
+        sp.ok_ff_in = plan(&sp.ff_in, L.w_ff_in, 2 * (int64_t)L.ff, d.width, EPI_BIAS_F32);
+        sp.ok_ff_out = plan(&sp.ff_out, L.w_ff_out, d.width, L.ff, EPI_BIAS_F32);
+      } else if (L.ff_kind == B200_FF_MOE && L.moe.shared_ff > 0) {
+        sp.ok_ff_in = plan(&sp.ff_in, L.w_ff_in, moe_shared_rows(L.moe), d.width, EPI_BIAS_F32);
+        sp.ok_ff_out = plan(&sp.ff_out, L.w_ff_out, d.width, L.moe.shared_ff, EPI_BIAS_F32);
+      }
+    }
+    for (int l = 0; !sandwich && !hyper && l < d.n_layers; ++l) {
       const b200_stack_layer& L = s->layers[l];
       s->plans[l].ok_in = plan(&s->plans[l].in, L.w_in, L.n_in, d.width, EPI_BIAS_F32, PRO_F32);
       s->plans[l].ok_out = plan(&s->plans[l].out, L.w_out, d.width, L.k_out, EPI_RESID_F32);

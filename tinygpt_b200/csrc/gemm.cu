@@ -71,9 +71,53 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
   asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 }
 
+// sixteen consecutive columns of one output row (`left` of them exist): bf16(acc + bias) or fp32 acc + bias
+template <typename OT>
+__device__ __forceinline__ void store16(OT* dst, uint32_t (&r)[16], int left, const float* bias);
+template <>
+__device__ __forceinline__ void store16<__nv_bfloat16>(__nv_bfloat16* dst, uint32_t (&r)[16], int left, const float* bias) {
+  if (bias != nullptr) {
+#pragma unroll
+    for (int j = 0; j < 16; ++j)
+      if (j < left) r[j] = __float_as_uint(__uint_as_float(r[j]) + bias[j]);
+  }
+  if (left >= 16 && ((reinterpret_cast<uintptr_t>(dst) & 15) == 0)) {
+    uint4 o0, o1;
+    o0.x = pack2(__uint_as_float(r[0]), __uint_as_float(r[1]));
+    o0.y = pack2(__uint_as_float(r[2]), __uint_as_float(r[3]));
+    o0.z = pack2(__uint_as_float(r[4]), __uint_as_float(r[5]));
+    o0.w = pack2(__uint_as_float(r[6]), __uint_as_float(r[7]));
+    o1.x = pack2(__uint_as_float(r[8]), __uint_as_float(r[9]));
+    o1.y = pack2(__uint_as_float(r[10]), __uint_as_float(r[11]));
+    o1.z = pack2(__uint_as_float(r[12]), __uint_as_float(r[13]));
+    o1.w = pack2(__uint_as_float(r[14]), __uint_as_float(r[15]));
+    reinterpret_cast<uint4*>(dst)[0] = o0;
+    reinterpret_cast<uint4*>(dst)[1] = o1;
+  } else {
+#pragma unroll
+    for (int j = 0; j < 16; ++j)
+      if (j < left) dst[j] = f_to_bf16(__uint_as_float(r[j]));
+  }
+}
+template <>
+__device__ __forceinline__ void store16<float>(float* dst, uint32_t (&r)[16], int left, const float* bias) {
+  float v[16];
+#pragma unroll
+  for (int j = 0; j < 16; ++j) v[j] = __uint_as_float(r[j]) + (bias != nullptr && j < left ? bias[j] : 0.f);
+  if (left >= 16 && ((reinterpret_cast<uintptr_t>(dst) & 15) == 0)) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) reinterpret_cast<float4*>(dst)[j] = make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
+  } else {
+#pragma unroll
+    for (int j = 0; j < 16; ++j)
+      if (j < left) dst[j] = v[j];
+  }
+}
+
+template <typename OT>
 __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_b,
-                    __nv_bfloat16* __restrict__ C, int M, int N, int K) {
+                    OT* __restrict__ C, const float* __restrict__ bias, int M, int N, int K) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   uint8_t* sA = smem;                                   // [stages][128 × 64 bf16], 1024-byte aligned (swizzle atom)
@@ -157,26 +201,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
     for (int c = 0; c < kBN; c += 16) {
       uint32_t r[16];
       tmem_ld16(tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)c, r);
-      if (row < M) {
-        __nv_bfloat16* dst = C + (size_t)row * N + n0 + c;
-        if (n0 + c + 16 <= N && ((reinterpret_cast<uintptr_t>(dst) & 15) == 0)) {
-          uint4 o0, o1;
-          o0.x = pack2(__uint_as_float(r[0]), __uint_as_float(r[1]));
-          o0.y = pack2(__uint_as_float(r[2]), __uint_as_float(r[3]));
-          o0.z = pack2(__uint_as_float(r[4]), __uint_as_float(r[5]));
-          o0.w = pack2(__uint_as_float(r[6]), __uint_as_float(r[7]));
-          o1.x = pack2(__uint_as_float(r[8]), __uint_as_float(r[9]));
-          o1.y = pack2(__uint_as_float(r[10]), __uint_as_float(r[11]));
-          o1.z = pack2(__uint_as_float(r[12]), __uint_as_float(r[13]));
-          o1.w = pack2(__uint_as_float(r[14]), __uint_as_float(r[15]));
-          reinterpret_cast<uint4*>(dst)[0] = o0;
-          reinterpret_cast<uint4*>(dst)[1] = o1;
-        } else {
-#pragma unroll
-          for (int j = 0; j < 16; ++j)
-            if (n0 + c + j < N) dst[j] = f_to_bf16(__uint_as_float(r[j]));
-        }
-      }
+      if (row < M && n0 + c < N)
+        store16<OT>(C + (size_t)row * N + n0 + c, r, N - n0 - c, bias != nullptr ? bias + n0 + c : nullptr);
     }
   }
 
@@ -219,9 +245,10 @@ __device__ __forceinline__ void mbar_wait_bounded(uint64_t* bar, uint32_t parity
   }
 }
 
+template <typename OT>
 __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_b,
-                               __nv_bfloat16* __restrict__ C, int M, int N, int K) {
+                               OT* __restrict__ C, const float* __restrict__ bias, int M, int N, int K) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   uint8_t* sA = smem;                                   // [stages][128 × 64 bf16]
@@ -322,26 +349,8 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap tmap_a, const
       for (int c = 0; c < kPBN; c += 16) {
         uint32_t r[16];
         tmem_ld16(tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(acc * kPBN + c), r);
-        if (row < M && n0 + c < N) {
-          __nv_bfloat16* dst = C + (size_t)row * N + n0 + c;
-          if (n0 + c + 16 <= N && ((reinterpret_cast<uintptr_t>(dst) & 15) == 0)) {
-            uint4 o0, o1;
-            o0.x = pack2(__uint_as_float(r[0]), __uint_as_float(r[1]));
-            o0.y = pack2(__uint_as_float(r[2]), __uint_as_float(r[3]));
-            o0.z = pack2(__uint_as_float(r[4]), __uint_as_float(r[5]));
-            o0.w = pack2(__uint_as_float(r[6]), __uint_as_float(r[7]));
-            o1.x = pack2(__uint_as_float(r[8]), __uint_as_float(r[9]));
-            o1.y = pack2(__uint_as_float(r[10]), __uint_as_float(r[11]));
-            o1.z = pack2(__uint_as_float(r[12]), __uint_as_float(r[13]));
-            o1.w = pack2(__uint_as_float(r[14]), __uint_as_float(r[15]));
-            reinterpret_cast<uint4*>(dst)[0] = o0;
-            reinterpret_cast<uint4*>(dst)[1] = o1;
-          } else {
-#pragma unroll
-            for (int j = 0; j < 16; ++j)
-              if (n0 + c + j < N) dst[j] = f_to_bf16(__uint_as_float(r[j]));
-          }
-        }
+        if (row < M && n0 + c < N)
+          store16<OT>(C + (size_t)row * N + n0 + c, r, N - n0 - c, bias != nullptr ? bias + n0 + c : nullptr);
       }
       // all of this thread's tcgen05.ld have completed (tmem_ld16 waits): hand the buffer back to the MMA warp
       tc_fence_before();
@@ -387,7 +396,8 @@ int make_tmap_sw128(CUtensorMap* out, const void* base, int64_t rows, int64_t co
 
 }  // namespace
 
-int launch_gemm_bf16(void* C, const void* A, const void* B, int64_t M, int64_t N, int64_t K, cudaStream_t st) {
+template <typename OT>
+static int launch_gemm_t(OT* C, const void* A, const void* B, const float* bias, int64_t M, int64_t N, int64_t K, cudaStream_t st) {
   B200_CHECK_ARG(C && A && B && M > 0 && N > 0 && K > 0, "gemm: bad arguments");
   B200_CHECK_ARG(K % 8 == 0 && N % 8 == 0, "gemm: K=%lld and N=%lld must be multiples of 8 (16-byte rows)", (long long)K,
                  (long long)N);
@@ -396,7 +406,7 @@ int launch_gemm_bf16(void* C, const void* A, const void* B, int64_t M, int64_t N
   B200_CHECK_ARG(M < (1ll << 31) && N < (1ll << 31) && K < (1ll << 31), "gemm: shape out of range");
   static bool attr_set = false;
   if (!attr_set) {
-    B200_CUDA(cudaFuncSetAttribute(gemm_tcgen05_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kGemmSmem));
+    B200_CUDA(cudaFuncSetAttribute(gemm_tcgen05_kernel<OT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGemmSmem));
     attr_set = true;
   }
   CUtensorMap ta, tb;
@@ -410,7 +420,7 @@ int launch_gemm_bf16(void* C, const void* A, const void* B, int64_t M, int64_t N
     static cudaError_t p_err = cudaSuccess;
     static int sms = 0;
     std::call_once(p_once, [] {
-      p_err = cudaFuncSetAttribute(gemm_tcgen05_persistent_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kPGemmSmem);
+      p_err = cudaFuncSetAttribute(gemm_tcgen05_persistent_kernel<OT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPGemmSmem);
       int dev = 0;
       if (p_err == cudaSuccess) p_err = cudaGetDevice(&dev);
       if (p_err == cudaSuccess) p_err = cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
@@ -420,8 +430,8 @@ int launch_gemm_bf16(void* C, const void* A, const void* B, int64_t M, int64_t N
     if ((rc = make_tmap_sw128(&tb, B, N, K, kPBN)) != B200_OK) return rc;
     const int64_t tiles = ((M + kBM - 1) / kBM) * ((N + kPBN - 1) / kPBN);
     g_launches.fetch_add(1);
-    gemm_tcgen05_persistent_kernel<<<(unsigned)std::min<int64_t>(tiles, sms), kGemmThreads, kPGemmSmem, st>>>(
-        ta, tb, (__nv_bfloat16*)C, (int)M, (int)N, (int)K);
+    gemm_tcgen05_persistent_kernel<OT><<<(unsigned)std::min<int64_t>(tiles, sms), kGemmThreads, kPGemmSmem, st>>>(
+        ta, tb, C, bias, (int)M, (int)N, (int)K);
     B200_CUDA(cudaGetLastError());
     return B200_OK;
   }
@@ -429,9 +439,19 @@ int launch_gemm_bf16(void* C, const void* A, const void* B, int64_t M, int64_t N
   if ((rc = make_tmap_sw128(&tb, B, N, K)) != B200_OK) return rc;
   dim3 grid((unsigned)((N + kBN - 1) / kBN), (unsigned)((M + kBM - 1) / kBM));
   g_launches.fetch_add(1);
-  gemm_tcgen05_kernel<<<grid, kGemmThreads, kGemmSmem, st>>>(ta, tb, (__nv_bfloat16*)C, (int)M, (int)N, (int)K);
+  gemm_tcgen05_kernel<OT><<<grid, kGemmThreads, kGemmSmem, st>>>(ta, tb, C, bias, (int)M, (int)N, (int)K);
   B200_CUDA(cudaGetLastError());
   return B200_OK;
+}
+
+int launch_gemm_bf16(void* C, const void* A, const void* B, int64_t M, int64_t N, int64_t K, cudaStream_t st) {
+  return launch_gemm_t<__nv_bfloat16>((__nv_bfloat16*)C, A, B, nullptr, M, N, K, st);
+}
+int launch_gemm_bf16_bias(void* C, const void* A, const void* B, const float* bias, int64_t M, int64_t N, int64_t K, cudaStream_t st) {
+  return launch_gemm_t<__nv_bfloat16>((__nv_bfloat16*)C, A, B, bias, M, N, K, st);
+}
+int launch_gemm_bf16_f32(float* C, const void* A, const void* B, const float* bias, int64_t M, int64_t N, int64_t K, cudaStream_t st) {
+  return launch_gemm_t<float>(C, A, B, bias, M, N, K, st);
 }
 
 }  // namespace b200

@@ -47,6 +47,10 @@ int launch_sample(int64_t* token_out, const void* logits, int64_t V, float tempe
 
 // ---- tcgen05 prefill GEMM (gemm.cu)
 int launch_gemm_bf16(void* C, const void* A, const void* B, int64_t M, int64_t N, int64_t K, cudaStream_t st);
+// C = bf16(A·Bᵀ + bias), one rounding
+int launch_gemm_bf16_bias(void* C, const void* A, const void* B, const float* bias, int64_t M, int64_t N, int64_t K, cudaStream_t st);
+// the same products handed out as fp32 sums: C = A·Bᵀ + bias (bias may be null)
+int launch_gemm_bf16_f32(float* C, const void* A, const void* B, const float* bias, int64_t M, int64_t N, int64_t K, cudaStream_t st);
 
 // ---- prefill helpers (prefill.cu)
 int launch_bias_add(void* y, const void* b, int64_t rows, int64_t n, cudaStream_t st);

@@ -135,6 +135,25 @@ __global__ void __launch_bounds__(256) stack_glu_clamp_kernel(T* __restrict__ y,
   }
 }
 
+// y[r, j] = T(act(gu[r, j])·gu[r, n + j]): a gated unit without a clamp, one rounding
+template <typename T>
+__global__ void __launch_bounds__(256) stack_glu_kernel(T* __restrict__ y, int64_t ld_y, const T* __restrict__ gu, int64_t ld_gu,
+                                                        int n, int act, int64_t total) {
+  pdl_trigger();
+  pdl_wait();
+  for (int64_t e = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t r = e / n;
+    const int j = (int)(e % n);
+    const float g = ldf<T>(gu + r * ld_gu + j), u = ldf<T>(gu + r * ld_gu + n + j);
+    const float a = act == B200_ACT_SILU ? g / (1.f + expf(-g))
+                    : act == B200_ACT_GELU_ERF ? 0.5f * g * (1.f + erff(g * 0.70710678118654752f))
+                    : act == B200_ACT_RELU2 ? fmaxf(g, 0.f) * fmaxf(g, 0.f)
+                    : act == B200_ACT_TANH ? tanhf(g)
+                    : 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+    y[r * ld_y + j] = cvt<T>(a * u);
+  }
+}
+
 __global__ void __launch_bounds__(256) stack_softcap_kernel(float* __restrict__ lg, __nv_bfloat16* __restrict__ lb,
                                                             int64_t total, float cap) {
   pdl_trigger();
@@ -744,7 +763,8 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const MoeRun p) {
   if (t >= p.n_tok) return;
   const int E = p.m.experts, top = p.m.top;
   const float* z = p.z + (int64_t)t * E;
-  // softmax routing: the scores' common denominator (the order of the scores is that of the logits)
+  // softmax routing: the scores' common denominator (the order of the scores is that of the logits); kind 2 normalises over the
+  // chosen logits alone, so it needs the first choice's logit only
   float zmax = -INFINITY, zsum = 0.f, picked = 0.f;
   if (p.m.router_kind == 1) {
     for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, z[e]);
@@ -777,7 +797,8 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const MoeRun p) {
     if (bi == 0x7fffffff) bi = 0;   // fewer finite logits than choices: cannot happen with top <= experts
     if (lane == 0) {
       p.sel_e[(int64_t)t * top + k] = bi;
-      const float score = p.m.router_kind == 1 ? expf(bv - zmax) / zsum : 1.f / (1.f + expf(-bv));
+      if (k == 0 && p.m.router_kind == 2) zmax = bv;
+      const float score = p.m.router_kind == 1 ? expf(bv - zmax) / zsum : p.m.router_kind == 2 ? expf(bv - zmax) : 1.f / (1.f + expf(-bv));
       p.sel_w[(int64_t)t * top + k] = score;
       picked += score;
       if (p.small) p.pair_slot[(int64_t)t * top + k] = t * top + k;   // no sorting: a pair stays where it is
@@ -788,6 +809,8 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const MoeRun p) {
   }
   if (p.m.router_kind == 1 && lane == 0)   // the chosen scores over their sum, times the design's scale
     for (int k = 0; k < top; ++k) p.sel_w[(int64_t)t * top + k] = p.sel_w[(int64_t)t * top + k] / (picked + 1e-20f) * p.m.route_scale;
+  if (p.m.router_kind == 2 && lane == 0)
+    for (int k = 0; k < top; ++k) p.sel_w[(int64_t)t * top + k] = p.sel_w[(int64_t)t * top + k] / picked;
 }
 
 // One CTA: counts → group ends, the row tiles of every group, and a sorted position for every pair.
@@ -926,6 +949,19 @@ int launch_stack_glu_clamp(void* y, int64_t ld_y, const void* gu, int64_t ld_gu,
   else
     B200_CUDA(launch_pdl(stack_glu_clamp_kernel<__nv_bfloat16>, dim3(grid_cap(total, 256)), dim3(256), 0, st, stack_pdl(),
                          (__nv_bfloat16*)y, ld_y, (const __nv_bfloat16*)gu, ld_gu, n, limit, total));
+  return B200_OK;
+}
+
+int launch_stack_glu(void* y, int64_t ld_y, const void* gu, int64_t ld_gu, int64_t rows, int n, int act, int dtype, cudaStream_t st) {
+  MIX_DTYPE_CHECK(dtype);
+  B200_CHECK_ARG(y && gu && rows > 0 && n > 0 && act >= B200_ACT_GELU_TANH && act <= B200_ACT_TANH, "stack glu: bad arguments");
+  const int64_t total = rows * n;
+  if (dtype == B200_F32)
+    B200_CUDA(launch_pdl(stack_glu_kernel<float>, dim3(grid_cap(total, 256)), dim3(256), 0, st, stack_pdl(), (float*)y, ld_y,
+                         (const float*)gu, ld_gu, n, act, total));
+  else
+    B200_CUDA(launch_pdl(stack_glu_kernel<__nv_bfloat16>, dim3(grid_cap(total, 256)), dim3(256), 0, st, stack_pdl(),
+                         (__nv_bfloat16*)y, ld_y, (const __nv_bfloat16*)gu, ld_gu, n, act, total));
   return B200_OK;
 }
 
@@ -1137,11 +1173,12 @@ int run_moe(const MoeRun& p, int dtype, cudaStream_t st) {
   B200_CHECK_ARG(m.experts <= 8192, "moe: more than 8192 experts not built");
   const int P = p.n_tok * m.top, n_tiles = moe_tiles(P, m.experts), E = m.experts, S = p.plan_stride > 0 ? p.plan_stride : E;
   B200_CHECK_ARG(S >= E, "moe: plan stride below the expert count");
-  B200_CHECK_ARG(m.router_kind == 0 || m.router_kind == 1, "moe: router kind %d", m.router_kind);
+  B200_CHECK_ARG(m.router_kind >= 0 && m.router_kind <= 2, "moe: router kind %d", m.router_kind);
   int rc;
   // rows of an expert's in-projection: gate | up of the clamped gated unit, or up alone under a plain activation
-  const int n_up = m.expert_act != 0 ? m.expert_ff : 2 * m.expert_ff;
+  const int n_up = moe_up_rows(m);
   auto hidden = [&]() -> int {
+    if (m.expert_gated) return launch_stack_glu(p.act, m.expert_ff, p.gu, n_up, P, m.expert_ff, m.expert_act, dtype, st);
     if (m.expert_act != 0) return launch_stack_act_mul(p.act, m.expert_ff, p.gu, nullptr, n_up, P, m.expert_ff, m.expert_act, dtype, st);
     return launch_stack_glu_clamp(p.act, m.expert_ff, p.gu, n_up, P, m.expert_ff, m.limit, dtype, st);
   };
@@ -1162,7 +1199,7 @@ int run_moe(const MoeRun& p, int dtype, cudaStream_t st) {
     }
     g.w = m.w_exp_in; g.sw = (int64_t)n_up * p.width; g.item_mat = p.sel_e;
     g.M = 1; g.N = n_up; g.K = p.width; g.items = P;
-    const bool act_in_product = m.expert_act == B200_ACT_RELU2 || m.expert_act == B200_ACT_TANH || m.expert_act == B200_ACT_SILU;
+    const bool act_in_product = !m.expert_gated && (m.expert_act == B200_ACT_RELU2 || m.expert_act == B200_ACT_TANH || m.expert_act == B200_ACT_SILU);
     if (act_in_product) {   // a plain activation rides on the product's store: the hidden rows leave in one launch
       g.c = p.act; g.sc = m.expert_ff; g.act = m.expert_act;
       if ((rc = launch_small_gemv(g, dtype, st)) != B200_OK) return rc;

@@ -19,6 +19,8 @@ int launch_stack_norm_add_norm(float* x, const void* y, bool y_bf16, const float
 // y[r, j] = T(min(g, limit)·sigmoid(1.702·min(g, limit))·(clamp(u, ±limit) + 1)), g = gu[r, j], u = gu[r, n + j]
 int launch_stack_glu_clamp(void* y, int64_t ld_y, const void* gu, int64_t ld_gu, int64_t rows, int n, float limit, int dtype,
                            cudaStream_t st);
+// y[r, j] = T( act(gu[r, j])·gu[r, n + j] ), act a b200_ff_act
+int launch_stack_glu(void* y, int64_t ld_y, const void* gu, int64_t ld_gu, int64_t rows, int n, int act, int dtype, cudaStream_t st);
 // logits (fp32) and their bf16 copy <- cap·tanh(logits / cap)
 int launch_stack_softcap(float* logits, __nv_bfloat16* logits_bf, int64_t total, float cap, cudaStream_t st);
 
@@ -164,6 +166,13 @@ struct MoeRun {
   bool tc = false;
   __nv_bfloat16* outp_bf = nullptr;   // [P, width]
 };
+// rows of one expert's in-projection: gate and up of a gated unit (clamped, or expert_gated), or up alone
+inline int moe_up_rows(const b200_moe_desc& m) { return m.expert_act != 0 && !m.expert_gated ? m.expert_ff : 2 * m.expert_ff; }
+// rows of the shared expert's in-projection (padded to 8): gate | up | gate logit, gate | up, or up alone
+inline int moe_shared_rows(const b200_moe_desc& m) {
+  const int n = m.expert_gated ? 2 * m.shared_ff : m.expert_act != 0 ? m.shared_ff : 2 * m.shared_ff + 1;
+  return (n + 7) / 8 * 8;
+}
 __host__ __device__ inline int moe_tiles(int pairs, int experts) { return (pairs + 63) / 64 + experts; }
 inline int64_t moe_plan_ints(int pairs, int experts) { return 2 * (int64_t)experts + 2 * moe_tiles(pairs, experts); }   // experts = the stride
 int run_moe(const MoeRun& p, int dtype, cudaStream_t st);

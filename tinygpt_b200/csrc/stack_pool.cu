@@ -1,0 +1,426 @@
+// stack_pool.cu — attention with pooled blocks and mixed heads as plain kernels: any head counts and sizes, storage type
+// T = bf16 or fp32.  Every kernel starts with griddepcontrol.launch_dependents + griddepcontrol.wait.
+#include "stack_pool.cuh"
+
+#include <algorithm>
+
+#include "stack_hyper.cuh"
+
+namespace b200 {
+
+namespace {
+
+template <typename T> __device__ __forceinline__ float ldf(const T* p);
+template <> __device__ __forceinline__ float ldf<float>(const float* p) { return *p; }
+template <> __device__ __forceinline__ float ldf<__nv_bfloat16>(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+template <typename T> __device__ __forceinline__ T cvt(float v);
+template <> __device__ __forceinline__ float cvt<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 cvt<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+// One CTA per (token, key/value head g): the channels of the query heads that read g, of key head g and of value head g.  The
+// convolution of every channel goes to shared memory; then one warp per query / key head takes the head's norm and turns
+// its first rot_dims entries.  Queries leave for q, keys and values for the slot's cache rows.
+template <typename T>
+__global__ void __launch_bounds__(256) pool_prep_kernel(const PoolAttn p) {
+  pdl_trigger();
+  pdl_wait();
+  extern __shared__ float sm[];   // [per·dk: q | dk: k | dv: v]
+  const int t = blockIdx.x, g = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int H = p.a.heads, G = p.a.kv_heads, dk = p.a.dim, dv = p.a.vdim, per = H / G, taps = p.d.conv_w != nullptr ? p.d.taps : 1;
+  const int nq = per * dk, mine = nq + dk + dv, ps = p.pos[t];
+  const T* row = static_cast<const T*>(p.proj) + (int64_t)t * p.ld_proj;
+  float* cs = p.conv_state + (int64_t)p.slot[t] * p.conv_slot_stride;
+  const int front = p.single ? 0 : rows_in_front(p.slot, p.pos, t, taps - 1);
+  for (int e = tid; e < mine; e += 256) {
+    const int col = e < nq ? p.off_q + g * nq + e : e < nq + dk ? p.off_k + g * dk + (e - nq) : p.off_v + g * dv + (e - nq - dk);
+    auto back = [&](int j) {
+      if (j <= front) return ldf<T>(row - (int64_t)j * p.ld_proj + col);
+      return ps - j >= 0 ? cs[(int64_t)(taps - 1 - (j - front)) * p.ld_proj + col] : 0.f;
+    };
+    float acc = back(0);
+    if (p.d.conv_w != nullptr) {
+      acc = 0.f;
+      for (int j = 0; j < taps; ++j) acc = fmaf(p.d.conv_w[(int64_t)(taps - 1 - j) * p.ld_proj + col], back(j), acc);
+      if (p.single)
+        for (int i = 0; i < taps - 1; ++i) {   // entry i: the row taps − 2 − i positions back, further along than what is written
+          const float v = back(taps - 2 - i);
+          cs[(int64_t)i * p.ld_proj + col] = v;
+        }
+    }
+    sm[e] = acc;
+  }
+  __syncthreads();
+  const int half = p.d.rot_dims / 2;
+  const float* tab = half > 0 ? p.d.rot_table + (int64_t)ps * half * 2 : nullptr;
+  T* kc = static_cast<T*>(p.kcache) + (int64_t)p.slot[t] * p.k_slot_stride;
+  T* vc = static_cast<T*>(p.vcache) + (int64_t)p.slot[t] * p.v_slot_stride;
+  for (int hh = warp; hh <= per; hh += 8) {   // hh < per: query head g·per + hh; per: the key head
+    float* x = sm + hh * dk;
+    const float* w = hh < per ? p.d.q_norm : p.d.k_norm;
+    float inv = 1.f;
+    if (p.d.q_norm != nullptr) {
+      float ss = 0.f;
+      for (int i = lane; i < dk; i += 32) ss += x[i] * x[i];
+      inv = 1.f / sqrtf(warp_sum(ss) / (float)dk + p.eps);
+    }
+    T* dst = hh < per ? static_cast<T*>(p.q) + ((int64_t)t * H + g * per + hh) * dk : kc + ((int64_t)ps * G + g) * dk;
+    for (int i = lane; i < dk - half; i += 32) {   // half pairs, then the entries that do not turn
+      if (i < half) {
+        float u = x[i] * inv, v = x[i + half] * inv;
+        if (p.d.q_norm != nullptr) {
+          u *= w[i];
+          v *= w[i + half];
+        }
+        const float c = tab[2 * i], s = tab[2 * i + 1];
+        const T a = cvt<T>(u * c - v * s), b = cvt<T>(v * c + u * s);
+        dst[i] = a;
+        dst[i + half] = b;
+        if (hh == per) {   // what the block mean below reads: the key as the cache holds it
+          x[i] = ldf<T>(&a);
+          x[i + half] = ldf<T>(&b);
+        }
+      } else {
+        float u = x[i + half] * inv;
+        if (p.d.q_norm != nullptr) u *= w[i + half];
+        const T a = cvt<T>(u);
+        dst[i + half] = a;
+        if (hh == per) x[i + half] = ldf<T>(&a);
+      }
+    }
+  }
+  float* v = sm + nq + dk;
+  for (int i = tid; i < dv; i += 256) {
+    const T a = cvt<T>(v[i]);
+    vc[((int64_t)ps * G + g) * dv + i] = a;
+    v[i] = ldf<T>(&a);
+  }
+  if (!p.single || p.d.pool <= 0 || (ps + 1) % p.d.pool != 0) return;
+  __syncthreads();
+  const int P = p.d.pool, b = ps / P;
+  const float inv = 1.f / (float)P;
+  for (int e = tid; e < dk + dv; e += 256) {   // the block's earlier rows were cached by earlier steps
+    const bool key = e < dk;
+    const int n = key ? dk : dv, i = key ? e : e - dk;
+    T* c = key ? kc : vc;
+    float s = 0.f;
+    for (int j = 0; j < P - 1; ++j) s += ldf<T>(c + ((int64_t)(b * P + j) * G + g) * n + i);
+    s += sm[nq + e];
+    c[((int64_t)(p.max_ctx + b) * G + g) * n + i] = cvt<T>(s * inv);
+  }
+}
+
+// Rows whose position ends a block: the means of the block's cached keys and values (rows of this step or of earlier ones).
+template <typename T>
+__global__ void __launch_bounds__(256) pool_blocks_kernel(const PoolAttn p) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, P = p.d.pool, ps = p.pos[t];
+  if ((ps + 1) % P != 0) return;
+  const int b = ps / P, nk = p.a.kv_heads * p.a.dim, nv = p.a.kv_heads * p.a.vdim;
+  T* kc = static_cast<T*>(p.kcache) + (int64_t)p.slot[t] * p.k_slot_stride;
+  T* vc = static_cast<T*>(p.vcache) + (int64_t)p.slot[t] * p.v_slot_stride;
+  const float inv = 1.f / (float)P;
+  for (int e = threadIdx.x; e < nk + nv; e += 256) {
+    const bool key = e < nk;
+    const int n = key ? nk : nv, i = key ? e : e - nk;
+    T* c = key ? kc : vc;
+    float s = 0.f;
+    for (int j = 0; j < P; ++j) s += ldf<T>(c + (int64_t)(b * P + j) * n + i);
+    c[(int64_t)(p.max_ctx + b) * n + i] = cvt<T>(s * inv);
+  }
+}
+
+__device__ __forceinline__ float capped(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
+
+// One CTA of eight warps per (row, split of the key list): the capped scores of every head, and each head's running maximum and
+// sum over the split.  A warp takes one key per lane and up to kPoolHC query heads of one key/value head at a time: the key row's
+// entries are loaded once for all of them, the queries come from shared memory.
+constexpr int kPoolHC = 4;
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) pool_scores_kernel(const PoolAttn p) {
+  pdl_trigger();
+  pdl_wait();
+  extern __shared__ float qs[];   // [H·dk]
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int H = p.a.heads, G = p.a.kv_heads, dk = p.a.dim, per = H / G, i = p.pos[t];
+  const int lo = pool_lo(i, p.a.window), nb = pool_nb(i, p.a.window, p.d.pool), total = nb + i - lo + 1;
+  const int begin = blockIdx.y * p.keys_per_split, end = min(total, begin + p.keys_per_split);
+  if (begin >= end) return;
+  const T* q = static_cast<const T*>(p.q) + (int64_t)t * H * dk;
+  for (int e = threadIdx.x; e < H * dk; e += 256) qs[e] = ldf<T>(q + e) * p.a.scale;
+  __syncthreads();
+  const T* K = static_cast<const T*>(p.kcache) + (int64_t)p.slot[t] * p.k_slot_stride;
+  const int chunks = (per + kPoolHC - 1) / kPoolHC;
+  for (int un = warp; un < G * chunks; un += 8) {
+    const int g = un / chunks, h0 = g * per + (un % chunks) * kPoolHC, nh = min(kPoolHC, (g + 1) * per - h0);
+    float m[kPoolHC], l[kPoolHC];
+#pragma unroll
+    for (int u = 0; u < kPoolHC; ++u) {
+      m[u] = -INFINITY;
+      l[u] = 0.f;
+    }
+    for (int k0 = begin; k0 < end; k0 += 32) {
+      const int idx = k0 + lane;
+      if (idx < end) {
+        const int r = idx < nb ? p.max_ctx + idx : lo + (idx - nb);
+        const T* kr = K + ((int64_t)r * G + g) * dk;
+        float s[kPoolHC];
+#pragma unroll
+        for (int u = 0; u < kPoolHC; ++u) s[u] = 0.f;
+        if constexpr (VEC) {   // sixteen-byte pieces of the key row, eight requested together
+          const uint4* k4 = reinterpret_cast<const uint4*>(kr);
+          for (int d0 = 0; d0 < dk >> 3; d0 += 8) {
+            uint4 kq[8];
+#pragma unroll
+            for (int w = 0; w < 8; ++w) kq[w] = d0 + w < (dk >> 3) ? k4[d0 + w] : make_uint4(0, 0, 0, 0);
+#pragma unroll
+            for (int w = 0; w < 8; ++w) {
+              if (d0 + w >= (dk >> 3)) break;
+              float kf[8];
+              unpack8(kq[w], kf);
+#pragma unroll
+              for (int u = 0; u < kPoolHC; ++u) {
+                if (u < nh) {
+                  const float* qq = qs + (h0 + u) * dk + (d0 + w) * 8;
+#pragma unroll
+                  for (int x = 0; x < 8; ++x) s[u] = fmaf(qq[x], kf[x], s[u]);
+                }
+              }
+            }
+          }
+        } else {
+          for (int d = 0; d < dk; ++d) {
+            const float kv = ldf<T>(kr + d);
+#pragma unroll
+            for (int u = 0; u < kPoolHC; ++u)
+              if (u < nh) s[u] = fmaf(qs[(h0 + u) * dk + d], kv, s[u]);
+          }
+        }
+#pragma unroll
+        for (int u = 0; u < kPoolHC; ++u) {
+          if (u < nh) {
+            const float v = capped(s[u], p.d.softcap);
+            p.scores[((int64_t)t * H + h0 + u) * p.nk_max + idx] = v;
+            const float mn = fmaxf(m[u], v);
+            l[u] = l[u] * expf(m[u] - mn) + expf(v - mn);   // first key: exp(−inf) = 0
+            m[u] = mn;
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < kPoolHC; ++u) {
+      if (u >= nh) break;
+      const float mt = warp_max(m[u]);
+      const float lt = warp_sum(m[u] == -INFINITY ? 0.f : l[u] * expf(m[u] - mt));
+      if (lane == 0) {
+        float* o = p.parts + (((int64_t)t * H + h0 + u) * p.nsplit + blockIdx.y) * 2;
+        o[0] = mt;
+        o[1] = lt;
+      }
+    }
+  }
+}
+
+// One CTA per (row, split): every head's maximum and denominator over all splits (and the sink), then tile by tile of
+// kPoolTile keys the weights of all heads, their mix, and the weighted values — a thread owns value columns and the query heads
+// that read them; the sums over tiles sit in shared memory.
+template <typename T, int VC>
+__global__ void __launch_bounds__(256) pool_values_kernel(const PoolAttn p) {
+  pdl_trigger();
+  pdl_wait();
+  extern __shared__ float sm[];
+  const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int H = p.a.heads, G = p.a.kv_heads, dv = p.a.vdim, per = H / G, i = p.pos[t];
+  constexpr int KP = kPoolTile + 1;
+  float* s_m = sm;                    // [H]
+  float* s_il = s_m + H;              // [H]
+  float* s_w = s_il + H;              // [H][KP]
+  float* s_x = s_w + H * KP;          // [H][KP] mixed
+  float* s_o = s_x + H * KP;          // [H·dv]
+  const int lo = pool_lo(i, p.a.window), nb = pool_nb(i, p.a.window, p.d.pool), total = nb + i - lo + 1;
+  const int begin = blockIdx.y * p.keys_per_split, end = min(total, begin + p.keys_per_split);
+  if (begin >= end) return;
+  const int live = (total + p.keys_per_split - 1) / p.keys_per_split;   // splits that hold keys
+  for (int h = warp; h < H; h += 8) {
+    const float* o = p.parts + ((int64_t)t * H + h) * p.nsplit * 2;
+    float m = p.d.sink != nullptr ? p.d.sink[h] : -INFINITY;
+    for (int s = lane; s < live; s += 32) m = fmaxf(m, o[2 * s]);
+    m = warp_max(m);
+    float l = 0.f;
+    for (int s = lane; s < live; s += 32) l += o[2 * s + 1] * expf(o[2 * s] - m);
+    l = warp_sum(l);
+    if (p.d.sink != nullptr) l += expf(p.d.sink[h] - m);
+    if (lane == 0) {
+      s_m[h] = m;
+      s_il[h] = 1.f / l;
+    }
+  }
+  for (int e = tid; e < H * dv; e += 256) s_o[e] = 0.f;
+  __syncthreads();
+  const T* V = static_cast<const T*>(p.vcache) + (int64_t)p.slot[t] * p.v_slot_stride;
+  for (int k0 = begin; k0 < end; k0 += kPoolTile) {
+    const int n = min(kPoolTile, end - k0);
+    for (int h = warp; h < H; h += 8)
+      s_w[h * KP + lane] = lane < n ? expf(p.scores[((int64_t)t * H + h) * p.nk_max + k0 + lane] - s_m[h]) * s_il[h] : 0.f;
+    __syncthreads();
+    const float* wm = s_w;
+    if (p.d.talk != nullptr) {
+      for (int h = warp; h < H; h += 8) {
+        const float* T0 = p.d.talk + (int64_t)h * H;
+        float a = 0.f;
+        for (int g = 0; g < H; ++g) a = fmaf(T0[g], s_w[g * KP + lane], a);
+        s_x[h * KP + lane] = a;
+      }
+      wm = s_x;
+      __syncthreads();
+    }
+    const int cols = G * dv / VC;
+    for (int e = tid; e < cols; e += 256) {
+      const int c = e * VC, g = c / dv, cc = c % dv;   // VC columns of one head (dv is a multiple of VC)
+      for (int u0 = 0; u0 < per; u0 += kPoolHC) {
+        const int nh = min(kPoolHC, per - u0), h0 = g * per + u0;
+        float acc[kPoolHC][VC];
+#pragma unroll
+        for (int u = 0; u < kPoolHC; ++u)
+#pragma unroll
+          for (int x = 0; x < VC; ++x) acc[u][x] = 0.f;
+#pragma unroll 8
+        for (int k = 0; k < n; ++k) {
+          const int idx = k0 + k, r = idx < nb ? p.max_ctx + idx : lo + (idx - nb);
+          const T* vr = V + ((int64_t)r * G) * dv + c;
+          float v[VC];
+          if constexpr (VC == 2) {
+            const uint32_t b = *reinterpret_cast<const uint32_t*>(vr);
+            v[0] = bf16_lo(b);
+            v[1] = bf16_hi(b);
+          } else {
+            v[0] = ldf<T>(vr);
+          }
+#pragma unroll
+          for (int u = 0; u < kPoolHC; ++u) {
+            if (u < nh) {
+              const float w = wm[(h0 + u) * KP + k];
+#pragma unroll
+              for (int x = 0; x < VC; ++x) acc[u][x] = fmaf(w, v[x], acc[u][x]);
+            }
+          }
+        }
+#pragma unroll
+        for (int u = 0; u < kPoolHC; ++u)
+          if (u < nh)
+#pragma unroll
+            for (int x = 0; x < VC; ++x) s_o[(h0 + u) * dv + cc + x] += acc[u][x];
+      }
+    }
+    __syncthreads();
+  }
+  if (p.nsplit > 1) {
+    float* o = p.outs + ((int64_t)t * p.nsplit + blockIdx.y) * H * dv;
+    for (int e = tid; e < H * dv; e += 256) o[e] = s_o[e];
+    return;
+  }
+  T* y = static_cast<T*>(p.mid) + (int64_t)t * p.ld_mid;
+  for (int e = tid; e < max(H * dv, p.n_pad); e += 256) y[e] = cvt<T>(e < H * dv ? s_o[e] * p.out_scale : 0.f);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) pool_merge_kernel(const PoolAttn p) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, e = blockIdx.y * 128 + threadIdx.x, n = p.a.heads * p.a.vdim, i = p.pos[t];
+  if (e >= max(n, p.n_pad)) return;
+  const int total = pool_nb(i, p.a.window, p.d.pool) + i - pool_lo(i, p.a.window) + 1;
+  const int live = (total + p.keys_per_split - 1) / p.keys_per_split;
+  float a = 0.f;
+  if (e < n) {
+    const float* o = p.outs + (int64_t)t * p.nsplit * n + e;
+#pragma unroll 8
+    for (int s = 0; s < live; ++s) a += o[(int64_t)s * n];
+  }
+  static_cast<T*>(p.mid)[(int64_t)t * p.ld_mid + e] = cvt<T>(a * p.out_scale);
+}
+
+int check_pool(const PoolAttn& p) {
+  const b200_attn_desc& a = p.a;
+  B200_CHECK_ARG(a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.dim > 0 && a.vdim > 0 && a.window >= 0 && p.d.pool >= 0,
+                 "pool attention: bad sizes (heads %d, kv_heads %d, dim %d, vdim %d)", a.heads, a.kv_heads, a.dim, a.vdim);
+  B200_CHECK_ARG(p.d.rot_dims >= 0 && p.d.rot_dims % 2 == 0 && p.d.rot_dims <= a.dim && (p.d.rot_dims == 0 || p.d.rot_table),
+                 "pool attention: rot_dims %d must be even, at most the head size %d, with a table", p.d.rot_dims, a.dim);
+  B200_CHECK_ARG((p.d.q_norm == nullptr) == (p.d.k_norm == nullptr), "pool attention: one of the two head norms is missing");
+  B200_CHECK_ARG(p.d.softcap >= 0.f, "pool attention: negative softcap");
+  B200_CHECK_ARG(p.q && p.kcache && p.vcache && p.slot && p.pos && p.n_tok > 0 && p.max_ctx > 0, "pool attention: null argument");
+  return B200_OK;
+}
+
+}  // namespace
+
+#define POOL_DTYPE_CHECK(dtype) \
+  B200_CHECK_ARG((dtype) == B200_BF16 || (dtype) == B200_F32, "stack op: unknown dtype %d", (int)(dtype))
+
+int launch_pool_prep(const PoolAttn& p, int dtype, cudaStream_t st) {
+  POOL_DTYPE_CHECK(dtype);
+  int rc = check_pool(p);
+  if (rc != B200_OK) return rc;
+  B200_CHECK_ARG(p.proj != nullptr, "pool attention: null projection");
+  B200_CHECK_ARG(p.d.conv_w == nullptr || (p.d.taps >= 1 && p.d.taps <= kConvMaxTaps && (p.d.taps == 1 || p.conv_state)),
+                 "pool attention: 1 … %d convolution taps with a state", kConvMaxTaps);
+  const size_t smem = (size_t)((p.a.heads / p.a.kv_heads + 1) * p.a.dim + p.a.vdim) * 4;
+  B200_CHECK_ARG(smem <= 48 * 1024, "pool attention: the heads that share one key/value head exceed 12288 channels");
+  const dim3 grid(p.n_tok, p.a.kv_heads);
+  if (dtype == B200_F32) B200_CUDA(launch_pdl(pool_prep_kernel<float>, grid, dim3(256), smem, st, stack_pdl(), p));
+  else B200_CUDA(launch_pdl(pool_prep_kernel<__nv_bfloat16>, grid, dim3(256), smem, st, stack_pdl(), p));
+  return B200_OK;
+}
+
+int launch_pool_blocks(const PoolAttn& p, int dtype, cudaStream_t st) {
+  POOL_DTYPE_CHECK(dtype);
+  int rc = check_pool(p);
+  if (rc != B200_OK) return rc;
+  if (p.d.pool <= 0) return B200_OK;
+  if (dtype == B200_F32) B200_CUDA(launch_pdl(pool_blocks_kernel<float>, dim3(p.n_tok), dim3(256), 0, st, stack_pdl(), p));
+  else B200_CUDA(launch_pdl(pool_blocks_kernel<__nv_bfloat16>, dim3(p.n_tok), dim3(256), 0, st, stack_pdl(), p));
+  return B200_OK;
+}
+
+int launch_pool_attention(const PoolAttn& p, int dtype, cudaStream_t st) {
+  POOL_DTYPE_CHECK(dtype);
+  int rc = check_pool(p);
+  if (rc != B200_OK) return rc;
+  const int H = p.a.heads, dk = p.a.dim, dv = p.a.vdim;
+  B200_CHECK_ARG(p.scores && p.parts && p.mid && p.nk_max > 0 && p.nsplit >= 1 && p.nsplit <= kPoolMaxSplits && p.keys_per_split > 0 &&
+                     (int64_t)p.nsplit * p.keys_per_split >= p.nk_max && (p.nsplit == 1 || p.outs),
+                 "pool attention: bad workspace");
+  const size_t sm_q = (size_t)H * dk * 4, sm_v = (size_t)(2 * H + 2 * H * (kPoolTile + 1) + H * dv) * 4;
+  B200_CHECK_ARG(sm_q <= 200 * 1024 && sm_v <= 200 * 1024, "pool attention: heads · head size exceeds one CTA's shared memory");
+  static bool attr_done = false;
+  if (!attr_done) {
+    B200_CUDA(cudaFuncSetAttribute(pool_scores_kernel<float, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    B200_CUDA(cudaFuncSetAttribute(pool_scores_kernel<__nv_bfloat16, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    B200_CUDA(cudaFuncSetAttribute(pool_scores_kernel<__nv_bfloat16, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    B200_CUDA(cudaFuncSetAttribute(pool_values_kernel<float, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    B200_CUDA(cudaFuncSetAttribute(pool_values_kernel<__nv_bfloat16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    B200_CUDA(cudaFuncSetAttribute(pool_values_kernel<__nv_bfloat16, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    attr_done = true;
+  }
+  const dim3 grid(p.n_tok, p.nsplit);
+  const bool kvec = dtype == B200_BF16 && dk % 8 == 0 && p.k_slot_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(p.kcache) & 15) == 0;
+  const bool vvec = dtype == B200_BF16 && dv % 2 == 0 && p.v_slot_stride % 2 == 0 && (reinterpret_cast<uintptr_t>(p.vcache) & 3) == 0;
+  if (dtype == B200_F32) {
+    B200_CUDA(launch_pdl(pool_scores_kernel<float, false>, grid, dim3(256), sm_q, st, stack_pdl(), p));
+    B200_CUDA(launch_pdl(pool_values_kernel<float, 1>, grid, dim3(256), sm_v, st, stack_pdl(), p));
+  } else {
+    if (kvec) B200_CUDA(launch_pdl(pool_scores_kernel<__nv_bfloat16, true>, grid, dim3(256), sm_q, st, stack_pdl(), p));
+    else B200_CUDA(launch_pdl(pool_scores_kernel<__nv_bfloat16, false>, grid, dim3(256), sm_q, st, stack_pdl(), p));
+    if (vvec) B200_CUDA(launch_pdl(pool_values_kernel<__nv_bfloat16, 2>, grid, dim3(256), sm_v, st, stack_pdl(), p));
+    else B200_CUDA(launch_pdl(pool_values_kernel<__nv_bfloat16, 1>, grid, dim3(256), sm_v, st, stack_pdl(), p));
+  }
+  if (p.nsplit > 1) {
+    const dim3 mg(p.n_tok, (std::max(H * dv, p.n_pad) + 127) / 128);
+    if (dtype == B200_F32) B200_CUDA(launch_pdl(pool_merge_kernel<float>, mg, dim3(128), 0, st, stack_pdl(), p));
+    else B200_CUDA(launch_pdl(pool_merge_kernel<__nv_bfloat16>, mg, dim3(128), 0, st, stack_pdl(), p));
+  }
+  return B200_OK;
+}
+
+}  // namespace b200

@@ -7,6 +7,8 @@
 
 #include <algorithm>
 
+#include "stack_hyper.cuh"
+
 namespace b200 {
 
 namespace {
@@ -111,7 +113,8 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnPrep p) {
 // multiply-adds per operand and column, and the output's dot with the NEW columns.  Columns never read each other, so
 // the result of a sequence does not depend on what else is in the step; the order of the sums inside a column is fixed by
 // dk alone (lane l sums rows l, l + 32, …, then the butterfly), whatever NC is.
-template <int DR, bool REMOVE, int NC>
+// OLD: the output reads the columns BEFORE the token joins them, plus the token's bonus times its value.
+template <int DR, bool REMOVE, int NC, bool OLD = false>
 __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
   pdl_trigger();
   pdl_wait();
@@ -126,6 +129,7 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
   constexpr int NVR = (CH * COLS + 255) / 256;            // staged values per thread and chunk
   __shared__ float s_x[CH][NV][DK];
   __shared__ float s_v[CH][COLS];
+  __shared__ float s_bonus[CH];
   const int seg = blockIdx.x, hd = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
   const int dk = p.dk, dv = p.dv;
   const int j0 = blockIdx.z * COLS, jw = j0 + warp * NC;
@@ -148,7 +152,7 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
   const float* src_r = p.r + (int64_t)hs * dk;
   const float* src_p = REMOVE ? p.p + (int64_t)hd * dk : nullptr;
   const float* src_q = REMOVE ? p.q + (int64_t)(p.q_shared ? hs : hd) * dk : nullptr;
-  float r_x[NQ], r_v[NVR];
+  float r_x[NQ], r_v[NVR], r_b = 0.f;
   auto fetch = [&](int c0) {
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
@@ -172,6 +176,7 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
       }
       r_v[i] = val;
     }
+    if constexpr (OLD) r_b = tid < CH && c0 + tid < cnt ? p.bonus[(int64_t)(r0 + c0 + tid) * p.ld + hd] : 0.f;
   };
   fetch(0);
   for (int c0 = 0; c0 < cnt; c0 += CH) {
@@ -182,6 +187,7 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
 #pragma unroll
     for (int i = 0; i < NVR; ++i)
       if (tid + 256 * i < CH * COLS) (&s_v[0][0])[tid + 256 * i] = r_v[i];
+    if (OLD && tid < CH) s_bonus[tid] = r_b;
     __syncthreads();
     if (c0 + CH < cnt) fetch(c0 + CH);
     if (jw >= dv) continue;   // warps past the last column only help with the staging
@@ -220,11 +226,12 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
           if constexpr (REMOVE) pp = s_x[t][3][d];
 #pragma unroll
           for (int c = 0; c < NC; ++c) {
+            if constexpr (OLD) dot[u][c] = fmaf(S[c][i], rr, dot[u][c]);
             float sn = dd * S[c][i];
             if constexpr (REMOVE) sn = fmaf(-pp, rem[c], sn);
             sn = fmaf(bb, vj[c], sn);
             S[c][i] = sn;
-            dot[u][c] = fmaf(sn, rr, dot[u][c]);
+            if constexpr (!OLD) dot[u][c] = fmaf(sn, rr, dot[u][c]);
           }
         }
       }
@@ -244,6 +251,7 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
 #pragma unroll
           for (int cc = 0; cc < NC; ++cc) mine = (uu == u && cc == c) ? dot[uu][cc] : mine;
         }
+        if constexpr (OLD) mine = fmaf(s_bonus[t4 + u], s_v[t4 + u][warp * NC + c], mine);   // t4 + u < CH
         if (t4 + u < n && jw + c < dv) p.o[(int64_t)(r0 + c0 + t4 + u) * p.ld_o + (int64_t)hd * dv + jw + c] = mine;
       }
     }
@@ -315,7 +323,7 @@ __global__ void __launch_bounds__(128) delta_out_kernel(const DeltaRun p) {
 // exactly when it has the same slot and that position.  Inputs from before the step's first row come from the slot's
 // state, which holds the last taps − 1 inputs, oldest first (zeros before position 0).
 __device__ __forceinline__ bool same_seq(const int32_t* slot, const int32_t* pos, int t, int j) {
-  return t - j >= 0 && slot[t - j] == slot[t] && pos[t - j] == pos[t] - j;
+  return row_same_seq(slot, pos, t, j);
 }
 
 // One thread per (row, channel): convolution over the row's own input and the taps − 1 before it + bias + SiLU into the
@@ -522,6 +530,212 @@ __global__ void __launch_bounds__(256) gdelta_out_kernel(const GatedDeltaRun p) 
   }
 }
 
+// --------------------------------------------------------------------------------------------------------- time mixing
+// One warp per (token, head): decay exp(−exp(wl)), the bonus Σ r·u·k; the scan's fp32 rows [decay | k | r | v | bonus].
+template <typename T>
+__global__ void __launch_bounds__(128) wkv_prep_kernel(const WkvRun p) {
+  pdl_trigger();
+  pdl_wait();
+  const int pair = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int H = p.d.heads, dk = p.d.dim;
+  if (pair >= p.scan.n_tok * H) return;
+  const int t = pair / H, hd = pair % H;
+  const int64_t n = (int64_t)H * dk, seg = (int64_t)p.scan.n_tok * n;
+  const T* r = static_cast<const T*>(p.p4) + (int64_t)t * n;
+  float* f = p.f + (int64_t)t * p.scan.ld;
+  float b = 0.f;
+  for (int i = lane; i < dk; i += 32) {
+    const int c = hd * dk + i;
+    const float rv = ldf<T>(r + c), kv = ldf<T>(r + seg + c);
+    f[c] = expf(-expf(p.wl[(int64_t)t * n + c]));
+    f[n + c] = kv;
+    f[2 * n + c] = rv;
+    f[3 * n + c] = ldf<T>(r + 2 * seg + c);
+    b = fmaf(rv * p.d.u[c], kv, b);
+  }
+  b = warp_sum(b);
+  if (lane == 0) f[4 * n + hd] = b;
+}
+
+// One warp per (token, head): o / rms(o) · norm · silu(gate) · scale; the last head's warp also clears the padding columns.
+template <typename T>
+__global__ void __launch_bounds__(128) wkv_out_kernel(const WkvRun p) {
+  pdl_trigger();
+  pdl_wait();
+  const int pair = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int H = p.d.heads, dv = p.d.dim;
+  if (pair >= p.scan.n_tok * H) return;
+  const int t = pair / H, hd = pair % H;
+  const int64_t n = (int64_t)H * dv;
+  const float* o = p.scan.o + (int64_t)t * p.scan.ld_o + hd * dv;
+  float ss = 0.f;
+  for (int c = lane; c < dv; c += 32) ss += o[c] * o[c];
+  const float inv = p.scale / sqrtf(warp_sum(ss) / (float)dv + p.eps);
+  const T* g = static_cast<const T*>(p.p4) + ((int64_t)3 * p.scan.n_tok + t) * n + hd * dv;
+  T* y = static_cast<T*>(p.mid) + (int64_t)t * p.ld_mid + hd * dv;
+  for (int c = lane; c < dv; c += 32) y[c] = cvt<T>(o[c] * inv * p.d.norm[hd * dv + c] * siluf(ldf<T>(g + c)));
+  if (hd == H - 1)
+    for (int c = (int)n + lane; c < p.n_pad; c += 32) static_cast<T*>(p.mid)[(int64_t)t * p.ld_mid + c] = cvt<T>(0.f);
+}
+
+// ------------------------------------------------------------------------------------------------------ selective scan
+// One thread per (row, channel): convolution over the row's own input and the taps − 1 before it, bias, SiLU.
+template <typename T>
+__global__ void __launch_bounds__(128) mamba1_conv_kernel(const Mamba1Run p) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, c = blockIdx.y * 128 + threadIdx.x, inner = p.d.inner, taps = p.d.taps;
+  if (c >= inner) return;
+  const T* x = static_cast<const T*>(p.proj) + p.off_x + c;
+  float* cs = p.conv_state + (int64_t)p.slot[t] * p.slot_stride;
+  const int front = rows_in_front(p.slot, p.pos, t, taps - 1), ps = p.pos[t];
+  auto back = [&](int j) {
+    if (j <= front) return ldf<T>(x + (int64_t)(t - j) * p.ld_proj);
+    return ps - j >= 0 ? cs[(int64_t)(taps - 1 - (j - front)) * inner + c] : 0.f;
+  };
+  float acc = p.d.conv_b[c];
+  for (int j = 0; j < taps; ++j) acc = fmaf(p.d.conv_w[(int64_t)(taps - 1 - j) * inner + c], back(j), acc);
+  static_cast<T*>(p.xc)[(int64_t)t * inner + c] = cvt<T>(siluf(acc));
+  if (p.advance)
+    for (int e = 0; e < taps - 1; ++e) {   // entry e: the row taps − 2 − e positions back, further along than what is written
+      const float v = back(taps - 2 - e);
+      cs[(int64_t)e * inner + c] = v;
+    }
+}
+
+// One warp per (row, channel): dt logit = Σ_r w_dt[c][r]·T(dt_r) + dt_b
+template <typename T>
+__global__ void __launch_bounds__(256) mamba1_dt_kernel(const Mamba1Run p) {
+  pdl_trigger();
+  pdl_wait();
+  const int c = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, t = blockIdx.y;
+  if (c >= p.d.inner) return;
+  const int rk8 = (p.d.dt_rank + 7) / 8 * 8;
+  const T* w = static_cast<const T*>(p.d.w_dt) + (int64_t)c * rk8;
+  const float* x = p.xd + (int64_t)t * p.ld_xd;
+  float a = 0.f;
+  for (int i = lane; i < p.d.dt_rank; i += 32) a = fmaf(ldf<T>(w + i), x[i], a);
+  a = warp_sum(a);
+  if (lane == 0) p.dt[(int64_t)t * p.d.inner + c] = a + p.d.dt_b[c];
+}
+
+// LPC lanes share a channel, NPT state entries each; 128 threads = 128 / LPC channels per CTA.  The CTA walks its sequence CH
+// tokens at a time: the chunk's B and C rows (fp32) and its channels' step sizes, inputs and gates sit in shared memory,
+// while the next chunk's values are already on their way into registers.  The state is in registers for the whole walk; a
+// token costs a thread NPT exponentials and 3·NPT multiply-adds, and the lanes' partial sums of four tokens meet side by
+// side, off the state's chain.  Entries past the state's size hold zeros (decay 1, B = C = 0).
+template <typename T, int LPC, int NPT>
+__global__ void __launch_bounds__(128) mamba1_scan_kernel(const Mamba1Run p) {
+  pdl_trigger();
+  pdl_wait();
+  constexpr int NS = LPC * NPT, CPB = 128 / LPC;
+  constexpr int CH = NS <= 32 ? 32 : NS <= 64 ? 16 : 8;         // tokens per chunk
+  constexpr int NBC = CH * 2 * NS / 128;                        // staged B | C entries per thread
+  constexpr int NX = (CH * CPB + 127) / 128;                    // staged (token, channel) triples per thread
+  __shared__ float s_b[CH][NS], s_c[CH][NS];
+  __shared__ float s_dt[CH][CPB], s_x[CH][CPB], s_z[CH][CPB];
+  const int seg = blockIdx.x, tid = threadIdx.x, ch = tid / LPC, ln = tid % LPC;
+  const int c0 = blockIdx.y * CPB, c = c0 + ch, inner = p.d.inner, N = p.d.state;
+  const int r0 = p.seg_row0 != nullptr ? p.seg_row0[seg] : seg;
+  const int cnt = p.seg_count != nullptr ? p.seg_count[seg] : 1;
+  float* st = p.state + (int64_t)p.slot[r0] * p.slot_stride + (int64_t)c * N;
+  const bool fresh = p.pos[r0] == 0, live = c < inner;
+  float S[NPT], A[NPT];
+#pragma unroll
+  for (int i = 0; i < NPT; ++i) {   // lane ln holds entries ln·NPT …: consecutive B / C entries per thread
+    const int n = ln * NPT + i;
+    S[i] = live && n < N && !fresh ? st[n] : 0.f;
+    A[i] = live && n < N ? -expf(p.d.A_log[(int64_t)c * N + n]) * 1.4426950408889634f : 0.f;   // exp(dt·A) = 2^(dt·A·log2 e)
+  }
+  const float D = live ? p.d.D[c] : 0.f;
+  const int off_b = (p.d.dt_rank + 7) / 8 * 8;
+  float r_bc[NBC], r_dt[NX], r_x[NX], r_z[NX];
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int i = 0; i < NBC; ++i) {
+      const int e = tid + 128 * i, t = e / (2 * NS), w = (e / NS) & 1, n = e % NS;
+      r_bc[i] = t0 + t < cnt && n < N ? p.xd[(int64_t)(r0 + t0 + t) * p.ld_xd + off_b + w * N + n] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < NX; ++i) {
+      const int e = tid + 128 * i, t = e / CPB, cc = c0 + e % CPB;
+      r_dt[i] = r_x[i] = r_z[i] = 0.f;
+      if (e < CH * CPB && t0 + t < cnt && cc < inner) {
+        const int64_t row = r0 + t0 + t;
+        r_dt[i] = softplusf(p.dt[row * inner + cc]);
+        r_x[i] = ldf<T>(static_cast<const T*>(p.xc) + row * inner + cc);
+        r_z[i] = siluf(ldf<T>(static_cast<const T*>(p.proj) + row * p.ld_proj + p.off_z + cc));
+      }
+    }
+  };
+  fetch(0);
+  for (int t0 = 0; t0 < cnt; t0 += CH) {
+    const int n_t = min(CH, cnt - t0);
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < NBC; ++i) {
+      const int e = tid + 128 * i, t = e / (2 * NS), w = (e / NS) & 1, n = e % NS;
+      (w ? s_c : s_b)[t][n] = r_bc[i];
+    }
+#pragma unroll
+    for (int i = 0; i < NX; ++i) {
+      const int e = tid + 128 * i;
+      if (e < CH * CPB) {
+        (&s_dt[0][0])[e] = r_dt[i];
+        (&s_x[0][0])[e] = r_x[i];
+        (&s_z[0][0])[e] = r_z[i];
+      }
+    }
+    __syncthreads();
+    if (t0 + CH < cnt) fetch(t0 + CH);
+    for (int t4 = 0; t4 < n_t; t4 += 4) {   // rows past the end hold dt = 0, x = 0: the state stays (2^0·S + 0)
+      float y[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int t = t4 + u;
+        const float dt = s_dt[t][ch], dx = dt * s_x[t][ch];
+        float a = 0.f;
+#pragma unroll
+        for (int i = 0; i < NPT; ++i) {
+          S[i] = fmaf(exp2f(dt * A[i]), S[i], dx * s_b[t][ln * NPT + i]);
+          a = fmaf(S[i], s_c[t][ln * NPT + i], a);
+        }
+        y[u] = a;
+      }
+#pragma unroll
+      for (int o = LPC / 2; o > 0; o >>= 1) {
+#pragma unroll
+        for (int u = 0; u < 4; ++u) y[u] += __shfl_xor_sync(0xffffffffu, y[u], o);
+      }
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int t = t4 + u;
+        if (ln == (u & (LPC - 1)) && t < n_t && live) {
+          const float v = fmaf(D, s_x[t][ch], y[u]) * s_z[t][ch];
+          static_cast<T*>(p.mid)[(int64_t)(r0 + t0 + t) * p.ld_mid + c] = cvt<T>(v);
+        }
+      }
+    }
+  }
+  if (!live) return;
+#pragma unroll
+  for (int i = 0; i < NPT; ++i) {
+    const int n = ln * NPT + i;
+    if (n < N) st[n] = S[i];
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) stack_cast_rows_kernel(T* __restrict__ y, int64_t ld_y, const float* __restrict__ x, int64_t ld_x,
+                                                              int n, int tanh_of, int64_t total) {
+  pdl_trigger();
+  pdl_wait();
+  for (int64_t e = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (int64_t)gridDim.x * blockDim.x) {
+    const float v = x[e / n * ld_x + e % n];
+    y[e / n * ld_y + e % n] = cvt<T>(tanh_of ? tanhf(v) : v);
+  }
+}
+
 // --------------------------------------------------------------------------------- post-norm + residual + operand copy
 template <typename YT>
 __global__ void __launch_bounds__(256) stack_rms_add_cast_kernel(float* __restrict__ x, const YT* __restrict__ y,
@@ -599,6 +813,7 @@ int launch_lin_scan(const LinScan& p, cudaStream_t st) {
                  "linear scan: null argument");
   B200_CHECK_ARG((p.p == nullptr) == (p.q == nullptr), "linear scan: the removal needs both of its vectors");
   B200_CHECK_ARG(p.heads > 0 && p.dk > 0 && p.dv > 0 && p.share > 0 && p.heads % p.share == 0, "linear scan: bad sizes");
+  B200_CHECK_ARG(!p.read_old || (p.p == nullptr && p.bonus && p.vscale == nullptr), "linear scan: reading the old state takes a bonus and no removal");
   B200_CHECK_ARG(p.dk <= kScanMaxDim, "linear scan: more than %d key channels not built", kScanMaxDim);
   // two columns per warp where the value size fills them and the registers hold them: half the CTAs stage the same rows
   const int nc = (p.dv >= 32 && p.dk <= 256) ? 2 : 1;
@@ -606,6 +821,7 @@ int launch_lin_scan(const LinScan& p, cudaStream_t st) {
 #define B200_SCAN_NC(DR, NC)                                                                                       \
   do {                                                                                                             \
     if (p.p != nullptr) B200_CUDA(launch_pdl(lin_scan_kernel<DR, true, NC>, grid, dim3(256), 0, st, stack_pdl(), p));  \
+    else if (p.read_old) B200_CUDA(launch_pdl(lin_scan_kernel<DR, false, NC, true>, grid, dim3(256), 0, st, stack_pdl(), p)); \
     else B200_CUDA(launch_pdl(lin_scan_kernel<DR, false, NC>, grid, dim3(256), 0, st, stack_pdl(), p));           \
   } while (0)
 #define B200_SCAN(DR)              \
@@ -696,6 +912,78 @@ int run_mamba(const MambaRun& p, int dtype, cudaStream_t st) {
   const dim3 og(p.scan.n_tok, m.taps > 1 ? 1 + std::min((ch + 255) / 256, 16) : 1);
   if (dtype == B200_F32) B200_CUDA(launch_pdl(mamba_out_kernel<float>, og, dim3(256), 0, st, stack_pdl(), p));
   else B200_CUDA(launch_pdl(mamba_out_kernel<__nv_bfloat16>, og, dim3(256), 0, st, stack_pdl(), p));
+  return B200_OK;
+}
+
+int run_wkv(const WkvRun& p, int dtype, cudaStream_t st) {
+  REC_DTYPE_CHECK(dtype);
+  const int H = p.d.heads, dk = p.d.dim;
+  B200_CHECK_ARG(p.p4 && p.wl && p.f && p.mid && p.scan.n_tok > 0 && H > 0 && dk > 0, "time mixing: null argument");
+  B200_CHECK_ARG(p.d.u && p.d.norm, "time mixing: null weight");
+  const dim3 grid((unsigned)(((int64_t)p.scan.n_tok * H + 3) / 4));
+  if (dtype == B200_F32) B200_CUDA(launch_pdl(wkv_prep_kernel<float>, grid, dim3(128), 0, st, stack_pdl(), p));
+  else B200_CUDA(launch_pdl(wkv_prep_kernel<__nv_bfloat16>, grid, dim3(128), 0, st, stack_pdl(), p));
+  LinScan s = p.scan;
+  const int64_t n = (int64_t)H * dk;
+  s.heads = H; s.dk = dk; s.dv = dk; s.share = 1; s.d_scalar = 0; s.read_old = 1;
+  s.d = p.f; s.b = p.f + n; s.r = p.f + 2 * n; s.v = p.f + 3 * n; s.bonus = p.f + 4 * n;
+  s.p = s.q = s.vscale = nullptr;
+  int rc = launch_lin_scan(s, st);
+  if (rc != B200_OK) return rc;
+  if (dtype == B200_F32) B200_CUDA(launch_pdl(wkv_out_kernel<float>, grid, dim3(128), 0, st, stack_pdl(), p));
+  else B200_CUDA(launch_pdl(wkv_out_kernel<__nv_bfloat16>, grid, dim3(128), 0, st, stack_pdl(), p));
+  return B200_OK;
+}
+
+int launch_mamba1_conv(const Mamba1Run& p, int dtype, cudaStream_t st) {
+  REC_DTYPE_CHECK(dtype);
+  const b200_mamba1_desc& d = p.d;
+  B200_CHECK_ARG(p.proj && p.xc && p.slot && p.pos && p.n_tok > 0 && d.inner > 0 && d.conv_w && d.conv_b && d.taps >= 1 && d.taps <= kMambaMaxTaps,
+                 "mamba1 convolution: bad arguments (1 … %d taps)", kMambaMaxTaps);
+  B200_CHECK_ARG(d.taps == 1 || p.conv_state, "mamba1 convolution: null state");
+  const dim3 grid(p.n_tok, (d.inner + 127) / 128);
+  if (dtype == B200_F32) B200_CUDA(launch_pdl(mamba1_conv_kernel<float>, grid, dim3(128), 0, st, stack_pdl(), p));
+  else B200_CUDA(launch_pdl(mamba1_conv_kernel<__nv_bfloat16>, grid, dim3(128), 0, st, stack_pdl(), p));
+  return B200_OK;
+}
+
+int launch_mamba1_dt(const Mamba1Run& p, int dtype, cudaStream_t st) {
+  REC_DTYPE_CHECK(dtype);
+  B200_CHECK_ARG(p.xd && p.dt && p.d.w_dt && p.d.dt_b && p.d.dt_rank > 0 && p.n_tok > 0 && p.n_tok <= 65535, "mamba1 step sizes: bad arguments");
+  const dim3 grid((p.d.inner + 7) / 8, p.n_tok);
+  if (dtype == B200_F32) B200_CUDA(launch_pdl(mamba1_dt_kernel<float>, grid, dim3(256), 0, st, stack_pdl(), p));
+  else B200_CUDA(launch_pdl(mamba1_dt_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, stack_pdl(), p));
+  return B200_OK;
+}
+
+int launch_mamba1_scan(const Mamba1Run& p, int dtype, cudaStream_t st) {
+  REC_DTYPE_CHECK(dtype);
+  const b200_mamba1_desc& d = p.d;
+  B200_CHECK_ARG(p.xd && p.dt && p.xc && p.proj && p.state && p.mid && p.slot && p.pos && p.n_seg > 0 && p.n_tok > 0 && d.A_log && d.D,
+                 "mamba1 scan: null argument");
+  B200_CHECK_ARG(d.inner > 0 && d.state > 0 && d.state <= kMamba1MaxState, "mamba1 scan: state 1 … %d", kMamba1MaxState);
+#define B200_M1(LPC, NPT)                                                                                                  do {                                                                                                                       const dim3 grid(p.n_seg, (d.inner + 128 / LPC - 1) / (128 / LPC));                                                       if (dtype == B200_F32) B200_CUDA(launch_pdl(mamba1_scan_kernel<float, LPC, NPT>, grid, dim3(128), 0, st, stack_pdl(), p));     else B200_CUDA(launch_pdl(mamba1_scan_kernel<__nv_bfloat16, LPC, NPT>, grid, dim3(128), 0, st, stack_pdl(), p));       } while (0)
+  if (d.state <= 8) B200_M1(2, 4);
+  else if (d.state <= 16) B200_M1(4, 4);
+  else if (d.state <= 32) B200_M1(8, 4);
+  else if (d.state <= 64) B200_M1(16, 4);
+  else if (d.state <= 128) B200_M1(32, 4);
+  else B200_M1(32, 8);
+#undef B200_M1
+  return B200_OK;
+}
+
+int launch_stack_cast_rows(void* y, int64_t ld_y, const float* x, int64_t ld_x, int64_t rows, int n, bool tanh_of, int dtype,
+                           cudaStream_t st) {
+  REC_DTYPE_CHECK(dtype);
+  B200_CHECK_ARG(y && x && rows > 0 && n > 0, "stack cast rows: bad arguments");
+  const int64_t total = rows * n;
+  const unsigned grid = (unsigned)std::min<int64_t>((total + 255) / 256, 148 * 8);
+  if (dtype == B200_F32)
+    B200_CUDA(launch_pdl(stack_cast_rows_kernel<float>, dim3(grid), dim3(256), 0, st, stack_pdl(), (float*)y, ld_y, x, ld_x, n, tanh_of ? 1 : 0, total));
+  else
+    B200_CUDA(launch_pdl(stack_cast_rows_kernel<__nv_bfloat16>, dim3(grid), dim3(256), 0, st, stack_pdl(), (__nv_bfloat16*)y, ld_y, x,
+                         ld_x, n, tanh_of ? 1 : 0, total));
   return B200_OK;
 }
 

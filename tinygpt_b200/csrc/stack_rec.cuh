@@ -4,6 +4,8 @@
 // delta rule: all terms; Mamba-2: a scalar d per head, no removal, b and r shared by a group of heads), with the
 // design-specific passes before it (gates, decays, unit keys, the short convolution) and behind it (head norms, gates).
 // Storage type T = bf16 or fp32; everything that enters a recurrence, its state and every norm are fp32.
+// Also the recurrences of hyper-connected blocks: RWKV-style time mixing (the same scan, its output read from the state
+// before the token joins it) and Mamba's selective scan (a decay per channel and state entry, a kernel of its own).
 #pragma once
 #include "stack.cuh"
 
@@ -32,8 +34,11 @@ int launch_attn_prep(const AttnPrep& p, int dtype, cudaStream_t st);
 // row or null.  State of a slot: [heads][dk][dv] fp32 at state + slot·slot_stride; a sequence whose first row has
 // position 0 starts from zero.
 constexpr int kScanMaxDim = 512;
+//   read_old (no removal):  o_j = s·r + bonus·v_j with the s from BEFORE the update; bonus: [heads] per row
 struct LinScan {
   int heads = 0, dk = 0, dv = 0, share = 1, d_scalar = 0;
+  int read_old = 0;
+  const float* bonus = nullptr;
   int q_shared = 0;   // 1: q is [heads / share][dk] like b and r (the removal reads along a shared key)
   const float *d = nullptr, *p = nullptr, *q = nullptr, *b = nullptr, *r = nullptr, *v = nullptr, *vscale = nullptr;
   int64_t ld = 0;
@@ -115,6 +120,55 @@ inline int64_t gdelta_state_floats(int heads, int kv_heads, int dim, int vdim, i
   return (int64_t)heads * dim * vdim + (int64_t)(taps - 1) * (2ll * kv_heads * dim + (int64_t)heads * vdim);
 }
 int run_gdelta(const GatedDeltaRun& p, int dtype, cudaStream_t st);
+
+// ---- RWKV-style time mixing around the scan (read_old): everything between the five blended inputs' products and the
+// out-projection
+struct WkvRun {
+  b200_wkv_desc d{};
+  float eps = 1e-5f, scale = 1.f;   // scale: a factor of the mixer's output (fp32, before it is rounded)
+  const void* p4 = nullptr;      // [4][n_tok][heads·dim] T: r | k | v | gate logits
+  const float* wl = nullptr;     // [n_tok, heads·dim] fp32: w2·tanh(bottleneck) + w0
+  float* f = nullptr;            // [n_tok, wkv_row_floats] fp32 workspace: decay | k | r | v | bonus
+  LinScan scan{};                // state, slots, positions, sequences, o
+  void* mid = nullptr;           // [n_tok, ld_mid] T, the mixer's columns from column 0 on; columns [heads·dim, n_pad) get zeros
+  int64_t ld_mid = 0;
+  int n_pad = 0;
+};
+inline int64_t wkv_row_floats(int heads, int dim) { return (int64_t)heads * (4 * dim + 1); }
+int run_wkv(const WkvRun& p, int dtype, cudaStream_t st);
+
+// ---- Mamba's selective scan: the convolution in front of w_x, then everything between the step-size logits and the
+// out-projection
+struct Mamba1Run {
+  b200_mamba1_desc d{};
+  const void* proj = nullptr;    // [n_tok, ld_proj] T: x at off_x, z at off_z
+  int64_t ld_proj = 0;
+  int off_x = 0, off_z = 0;
+  float* conv_state = nullptr;   // slot 0's [taps − 1][inner] fp32
+  float* state = nullptr;        // slot 0's [inner][state] fp32
+  int64_t slot_stride = 0;
+  int advance = 0;               // 1: every row is its sequence's only new one — the convolution moves its state on itself
+  void* xc = nullptr;            // [n_tok, inner] T: convolved channels
+  const float* xd = nullptr;     // [n_tok, ld_xd] fp32: dt | B | C rows of w_x·xc (B from column up8(dt_rank) on)
+  int64_t ld_xd = 0;
+  float* dt = nullptr;           // [n_tok, inner] fp32: w_dt·dt + dt_b (before softplus)
+  const int32_t* seg_row0 = nullptr;   // null: every row is a sequence
+  const int32_t* seg_count = nullptr;
+  const int32_t* slot = nullptr;
+  const int32_t* pos = nullptr;
+  int n_seg = 0, n_tok = 0;
+  void* mid = nullptr;           // [n_tok, ld_mid] T
+  int64_t ld_mid = 0;
+};
+constexpr int kMamba1MaxState = 256;
+inline int64_t mamba1_state_floats(int inner, int state, int taps) { return (int64_t)inner * (state + taps - 1); }
+int launch_mamba1_conv(const Mamba1Run& p, int dtype, cudaStream_t st);
+// dt from xd by plain dot products (a few rows, or shapes the matrix paths do not take)
+int launch_mamba1_dt(const Mamba1Run& p, int dtype, cudaStream_t st);
+int launch_mamba1_scan(const Mamba1Run& p, int dtype, cudaStream_t st);
+// y[r, :n] = T(x[r, :n]) of fp32 rows, or T(tanh(x[r, :n]))
+int launch_stack_cast_rows(void* y, int64_t ld_y, const float* x, int64_t ld_x, int64_t rows, int n, bool tanh_of, int dtype,
+                           cudaStream_t st);
 
 // x[r, :] += mult · rmsnorm(y[r, :]) · w  (fp32 stream), and h[r, :] = bf16(x[r, :]) — a sublayer's post-norm, the
 // residual sum and the next sublayer's operand copy in one pass; h may be null

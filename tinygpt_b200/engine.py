@@ -17,8 +17,8 @@ from typing import Callable, Dict, Iterable, List, Optional, Tuple
 import torch
 
 from . import models
-from ._lib import (AttnDesc, AttnPrepDesc, B200Error, DeltaDesc, GatedDeltaDesc, LatentDesc, LayerWeights, MambaDesc, MlstmDesc, ModelDesc,
-                   MoeDesc, StackDesc, StackLayer, WeightTable, check, lib, require_device)
+from ._lib import (AttnDesc, AttnPrepDesc, B200Error, DeltaDesc, GatedDeltaDesc, HyperDesc, LatentDesc, LayerWeights, Mamba1Desc,
+                   MambaDesc, MlstmDesc, ModelDesc, MoeDesc, PoolAttnDesc, WkvDesc, StackDesc, StackLayer, WeightTable, check, lib, require_device)
 
 
 def align_prompts(token_lists, context_size: int, pad_token: int):
@@ -158,7 +158,8 @@ class DecodeEngine:
         self._rot_tables = {}
         self._mix_seen = False
         for i, L in enumerate(spec.layers if sandwich else ()):
-            arr[i] = (self._postnorm_layer if spec.block == "postnorm" else self._sandwich_layer)(spec, i, L, ptr, mdt, acts)
+            build = {"postnorm": self._postnorm_layer, "hyper": self._hyper_layer}.get(spec.block, self._sandwich_layer)
+            arr[i] = build(spec, i, L, ptr, mdt, acts)
         for i, L in enumerate(() if sandwich else spec.layers):
             a, lay, p = L.attn, spec.layout(i), f"l{i}."
             side = spec.side_dim > 0
@@ -173,11 +174,11 @@ class DecodeEngine:
         runs = spec.runs()
         run_layer = (C.c_int32 * len(runs))(*[r[0] for r in runs])
         run_mix = (C.c_int32 * len(runs))(*[int(r[1]) for r in runs])
-        desc = StackDesc(1 if mdt == torch.float32 else 0, {"parallel": 0, "sandwich": 1, "postnorm": 2}[spec.block], spec.width, spec.vocab, len(spec.layers), len(runs),
+        desc = StackDesc(1 if mdt == torch.float32 else 0, {"parallel": 0, "sandwich": 1, "postnorm": 2, "hyper": 3}[spec.block], spec.width, spec.vocab, len(spec.layers), len(runs),
                          run_layer, run_mix, spec.embed_scale, spec.residual_mult, spec.norm_eps, spec.norm_offset,
                          spec.side_dim, spec.side_dim * len(spec.layers), spec.max_ctx, spec.max_slots,
                          ptr("embed", mdt), ptr("mix_in", mdt), ptr("side_table", mdt), ptr("final_norm", torch.float32),
-                         ptr("head", mdt), arr, {"rms": 0, "layer": 1}[spec.norm_kind], spec.logit_softcap)
+                         ptr("head", mdt), arr, {"rms": 0, "layer": 1}[spec.norm_kind], spec.logit_softcap, spec.streams)
         h = C.c_void_p()
         with torch.cuda.device(dev):
             check(lib().b200_engine_create_stack(C.byref(desc), C.byref(h)), "b200_engine_create_stack")
@@ -290,6 +291,51 @@ class DecodeEngine:
                           0, None, None, None, mixer, 2 if L.ff_kind == "moe" else 1, ptr(p + "post_norm", f32),
                           None, ptr(p + "ff_post_norm", f32) if has_ff else None,
                           ptr(p + "w_ff_in", mdt), ptr(p + "w_ff_out", mdt), LatentDesc(), MlstmDesc(), moe, prep, delta, mamba)
+
+    def _hyper_layer(self, spec, i, L, ptr, mdt, acts) -> StackLayer:
+        """Descriptor of layer i of a hyper-connected model (selective scan, time mixing, pooled-block attention or the sum of the
+        last two; clamped gated or routed feed-forward, or none)."""
+        lay, p = spec.mix_layout(i), f"l{i}."
+        f32 = torch.float32
+        attn, pool, wkv, mamba1, moe = AttnDesc(), PoolAttnDesc(), WkvDesc(), Mamba1Desc(), MoeDesc()
+        if L.pool is not None:
+            a = L.pool
+            attn = AttnDesc(a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.window, 0, 0)
+            tab = None
+            if a.rot is not None:
+                tab = self._rot_tables.get(a.rot)
+                if tab is None:
+                    tab = self._rot_tables[a.rot] = a.rot.table(spec.max_ctx).contiguous().to(self.device)
+            pool = PoolAttnDesc(a.conv, a.rot.dims if a.rot is not None else 0, a.pool, a.softcap, ptr(p + "left.conv_w", f32),
+                                ptr(p + "left.q_norm", f32), ptr(p + "left.k_norm", f32), tab.data_ptr() if tab is not None else None,
+                                ptr(p + "left.sink", f32), ptr(p + "left.talk", f32))
+        if L.wkv is not None:
+            a = L.wkv
+            wkv = WkvDesc(a.heads, a.dim, a.rank, ptr(p + "mu", f32), ptr(p + "w_rkvg", mdt), ptr(p + "w1", mdt), ptr(p + "w2", mdt),
+                          ptr(p + "w0", f32), ptr(p + "u", f32), ptr(p + "head_norm", f32))
+        if L.mamba1 is not None:
+            a = L.mamba1
+            mamba1 = Mamba1Desc(a.inner, a.state, a.dt_rank, a.conv, ptr(p + "conv_w", f32), ptr(p + "conv_b", f32), ptr(p + "w_x", mdt),
+                                ptr(p + "w_dt", mdt), ptr(p + "dt_b", f32), ptr(p + "A_log", f32), ptr(p + "D", f32))
+        if L.ff_kind == "moe":
+            m = L.moe
+            moe = MoeDesc(m.experts, m.top, m.expert_ff, m.shared_ff, m.limit, m.shared_limit, ptr(p + "router", mdt),
+                          ptr(p + "w_exp_in", mdt), ptr(p + "w_exp_out", mdt), {"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}[m.router],
+                          int(m.weight_output), acts[m.act[4:]] if m.act.startswith("glu_") and m.act != "glu_clamp" else
+                          0 if m.act == "glu_clamp" else acts[m.act], int(m.shared_plain), m.route_scale,
+                          int(m.act.startswith("glu_") and m.act != "glu_clamp"))
+        has_ff = L.ff_kind == "moe" or L.ff > 0
+
+        def hc(q):
+            return HyperDesc(ptr(p + q + "in", f32), ptr(p + q + "out", f32), ptr(p + q + "mix", f32))
+
+        return StackLayer(attn, L.ff, 0, lay.off_q, lay.off_k, lay.off_v, lay.off_g, 0, 0, lay.n_in, 0, lay.k_out, ptr(p + "norm", f32),
+                          ptr(p + "w_in", mdt), ptr(p + "b_in", f32), ptr(p + "w_out", mdt), 0, None, None, None,
+                          {"mamba1": 6, "wkv": 7, "pool_attention": 8, "parallel": 9}[L.mixer], 2 if L.ff_kind == "moe" else 3, None,
+                          ptr(p + "ff_norm", f32) if has_ff else None, None, ptr(p + "w_ff_in", mdt), ptr(p + "w_ff_out", mdt),
+                          LatentDesc(), MlstmDesc(), moe, AttnPrepDesc(), DeltaDesc(), MambaDesc(), GatedDeltaDesc(), None, 0,
+                          hc("hc1."), hc("hc2."), L.canon, ptr(p + "canon_w", f32), L.ff_limit, L.left_scale, L.right_scale, pool, wkv,
+                          mamba1)
 
     # --------------------------------------------------------------------------------- ragged steps (stack engines)
     def step(self, entries, greedy: bool = False) -> torch.Tensor:

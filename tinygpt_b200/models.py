@@ -269,7 +269,8 @@ class MoeSpec:
     "softmax": scores are a softmax over all experts and the chosen ones are divided by their sum (+ 1e-20) and multiplied by
     route_scale.  The weight multiplies the expert's input, or (weight_output) its output.  act "glu_clamp": clamped gated
     experts of width expert_ff (clamp `limit`); "relu2": down·relu(up·h)², no gate rows.  shared_ff > 0: a shared expert of
-    that width (clamp shared_limit) behind a per-token sigmoid gate, or (shared_plain) added as it is."""
+    that width (clamp shared_limit) behind a per-token sigmoid gate, or (shared_plain) added as it is.  router "softmax_chosen":
+    a softmax over the chosen logits alone; act "glu_silu": down·(silu(gate·h)·(up·h))."""
     experts: int
     top: int
     expert_ff: int
@@ -373,19 +374,70 @@ class GatedDeltaSpec:
 
 
 @dataclass(frozen=True)
+class PoolAttnSpec:
+    """Attention behind short convolutions: grouped heads with biases, a causal convolution of `conv` taps on q, k and v, per-head
+    query / key norms, rotate-half rotary positions, tanh-capped scores (softcap 0: none), a sliding window of `window` tokens
+    and behind it one mean key / value per block of `pool` tokens (0: none), a learned sink per head, and heads whose softmax
+    weights are mixed by a heads × heads matrix."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    conv: int
+    window: int = 0
+    pool: int = 0
+    rot: Optional[HalfRotarySpec] = None
+    softcap: float = 0.0
+
+    def visible(self, i: int, j: int) -> bool:
+        return j <= i and (self.window <= 0 or i - j < self.window)
+
+    def visible_block(self, i: int, b: int) -> bool:
+        return self.window > 0 and self.pool > 0 and b * self.pool + self.pool - 1 <= i - self.window
+
+
+@dataclass(frozen=True)
+class WkvSpec:
+    """RWKV-style time mixing: per head a dim × dim state with a decay per key channel (from a tanh bottleneck of `rank`), a
+    bonus for the current token, head norms and a silu gate; its inputs are blends of a token's row and the row before it."""
+    heads: int
+    dim: int
+    rank: int
+
+
+@dataclass(frozen=True)
+class Mamba1Spec:
+    """Mamba's selective scan: `inner` channels with a state of `state` entries each, step sizes through a bottleneck of
+    `dt_rank`, a causal convolution of `conv` taps with a bias."""
+    inner: int
+    state: int
+    dt_rank: int
+    conv: int
+
+
+@dataclass(frozen=True)
 class StackLayerSpec:
     attn: Optional[AttnSpec] = None  # mixer "attention"
     ff: int = 0                      # feed-forward width (gated / dense), 0 = none
     ff_act: str = "gelu_tanh"        # gelu_tanh | silu | gelu_erf
-    mixer: str = "attention"         # attention | latent_attention | mlstm | general_delta | mamba2 | gated_delta
+    mixer: str = "attention"         # attention | latent_attention | mlstm | general_delta | mamba2 | gated_delta; of
+                                     # hyper-connected blocks: mamba1 | wkv | pool_attention | parallel
     latent: Optional[LatentSpec] = None
     mlstm: Optional[MlstmSpec] = None
-    ff_kind: str = "gated"           # gated | dense | moe
+    ff_kind: str = "gated"           # gated | dense | moe | glu_clamp
     moe: Optional[MoeSpec] = None
     prep: Optional[AttnPrepSpec] = None   # attention mixers of sandwich / post-norm blocks
     delta: Optional[DeltaSpec] = None
     mamba: Optional[Mamba2Spec] = None
     gdelta: Optional[GatedDeltaSpec] = None
+    pool: Optional[PoolAttnSpec] = None   # mixers pool_attention and (left half) parallel
+    wkv: Optional[WkvSpec] = None         # mixers wkv and (right half) parallel
+    mamba1: Optional[Mamba1Spec] = None
+    left_scale: float = 1.0          # mixer parallel: left_scale·left + right_scale·right
+    right_scale: float = 1.0
+    canon: int = 0                   # taps of the convolution over the mixer's normed input, h + conv(h); 0 = none
+    ff_limit: float = 0.0            # ff_kind glu_clamp: the clamp
     kv_from: Optional[int] = None    # attention mixers: read the keys and values layer kv_from cached (no projections of its own)
 
 
@@ -443,9 +495,12 @@ class StackSpec:
     max_ctx: int = 4096              # cache rows per slot
     max_slots: int = 8               # sequences the engine holds at a time
     block: str = "parallel"          # parallel: x += m·(mixer(h) + ff(h)), one norm | sandwich: a norm before and after
-    norm_kind: str = "rms"           # each sublayer | postnorm: a norm behind each sublayer only.  rms | layer (weight-only)
+                                     # each sublayer | postnorm: a norm behind each sublayer only | hyper: a norm before each
+                                     # sublayer, which reads and writes `streams` copies of x through small matrices
+    norm_kind: str = "rms"           # rms | layer (weight-only)
     loop_mix: bool = True            # every pass of the loop starts with x <- mix_in·[x; x0]
     logit_softcap: float = 0.0       # > 0: logits <- cap·tanh(logits / cap)
+    streams: int = 1                 # hyper blocks: copies of the residual stream
     layer_scale: bool = False        # every sublayer's normed output is multiplied by a per-channel vector (the packer folds
                                      # it into the post-norm's weight: both are element-wise factors of the same product)
 
@@ -516,6 +571,17 @@ class StackSpec:
             off_gate = _up8(off_q + a.groups * a.state)
             return MixLayout(off_q=off_q, off_k=off_k, off_v=off_v, off_g=0, off_gate=off_gate, n_in=off_gate + _up8(a.heads),
                              k_out=a.inner)
+        if L.mixer in ("pool_attention", "parallel"):   # [q | k | v]; out columns [left | right]
+            a = L.pool
+            off_k = _up8(a.heads * a.dim)
+            off_v = off_k + _up8(a.kv_heads * a.dim)
+            return MixLayout(off_q=0, off_k=off_k, off_v=off_v, n_in=off_v + _up8(a.kv_heads * a.vdim),
+                             k_out=_up8(a.heads * a.vdim) + (_up8(L.wkv.heads * L.wkv.dim) if L.mixer == "parallel" else 0))
+        if L.mixer == "wkv":   # its products read five blends of the input: no merged in-projection
+            return MixLayout(k_out=_up8(L.wkv.heads * L.wkv.dim))
+        if L.mixer == "mamba1":   # [x | z]
+            a = L.mamba1
+            return MixLayout(off_v=0, off_g=_up8(a.inner), n_in=2 * _up8(a.inner), k_out=a.inner)
         raise ValueError(f"mix_layout: layer {i} has mixer {L.mixer!r}")
 
     def with_ctx(self, max_ctx: int, max_slots: Optional[int] = None) -> "StackSpec":
@@ -526,6 +592,21 @@ class StackSpec:
         n = self.vocab * self.width
         for i, mix in self.runs():
             L, a = self.layers[i], self.layers[i].attn
+            if self.block == "hyper":
+                if L.pool is not None:
+                    q = L.pool
+                    n += self.width * (q.heads * (q.dim + q.vdim) + q.kv_heads * (q.dim + q.vdim))
+                if L.wkv is not None:
+                    q = L.wkv
+                    n += self.width * (5 * q.heads * q.dim + q.rank) + q.heads * q.dim * q.rank
+                if L.mamba1 is not None:
+                    q = L.mamba1
+                    n += 3 * self.width * q.inner + q.inner * (2 * q.dt_rank + 2 * q.state)
+                if L.ff_kind == "moe":
+                    n += self.width * (L.moe.experts + 3 * L.moe.top * L.moe.expert_ff + 3 * L.moe.shared_ff)
+                else:
+                    n += 3 * L.ff * self.width
+                continue
             if L.mixer == "latent_attention":
                 q = L.latent
                 hq = q.heads * (q.dim + q.rot_dim)
@@ -1240,6 +1321,275 @@ def pack_tarudra_weights(spec: StackSpec, named: Dict[str, torch.Tensor], device
     return out
 
 
+# ---------------------------------------------------------------------------------------------------------- Bibezen
+def bibezen_from_config(doc: dict, name: str = "Bibezen", shapes: Optional[Dict[str, Tuple[int, ...]]] = None) -> StackSpec:
+    """config.json of the Bibezen design → StackSpec.  Bibezen: hyper-connected blocks (`streams` copies of the residual stream)
+    with zero-centred RMS norms and a short convolution over every mixer's input; mixers are Mamba's selective scan, RWKV-style
+    time mixing, or the weighted sum of a pooled-block attention and a time mixing; feed-forwards are a clamped gated unit or
+    softmax-routed SwiGLU experts with a shared expert; scaled embedding, whose table is also the head.  `shapes` (tensor name
+    → shape, from the checkpoint's header) gives the one size config.json leaves to the tensors: the rank of the decay
+    bottlenecks (without it a default stands in, for synthetic checkpoints)."""
+    def wkv_spec(i: int, m: dict, key: str) -> WkvSpec:
+        rank = int(shapes[f"l{i}.mix.{key}w1"][0]) if shapes and f"l{i}.mix.{key}w1" in shapes else int(m.get("rank", 16))
+        return WkvSpec(heads=int(m["heads"]), dim=int(m["dim"]), rank=rank)
+
+    canon = int((doc.get("canon") or {}).get("taps", 0))
+    layers = []
+    for i, lc in enumerate(doc["layers"]):
+        kind, m = lc.get("type"), lc["mixer"]
+        if kind == "mamba1":
+            kw = dict(mamba1=Mamba1Spec(inner=int(m["inner"]), state=int(m["state"]), dt_rank=int(m["dt_rank"]), conv=int(m["conv"])))
+            if min(kw["mamba1"].inner, kw["mamba1"].state, kw["mamba1"].dt_rank, kw["mamba1"].conv) < 1:
+                raise ValueError(f"Bibezen: layer {i}: Mamba sizes must be positive")
+        elif kind == "wkv":
+            kw = dict(wkv=wkv_spec(i, m, ""))
+        elif kind == "parallel":
+            q = m["left"]
+            heads, kv = int(q["heads"]), int(q["kv_heads"])
+            if kv < 1 or heads % kv:
+                raise ValueError(f"Bibezen: layer {i}: {heads} heads over {kv} kv_heads")
+            rot = None
+            if q.get("rot") and int(q["rot"]["dims"]) > 0:
+                rot = HalfRotarySpec(dims=int(q["rot"]["dims"]), base=float(q["rot"]["base"]))
+                if rot.dims % 2 or rot.dims > int(q["dim"]):
+                    raise ValueError(f"Bibezen: layer {i}: rot.dims {rot.dims} must be even and at most dim")
+            mask = q.get("mask") or {}
+            kw = dict(pool=PoolAttnSpec(heads=heads, kv_heads=kv, dim=int(q["dim"]), vdim=int(q["vdim"]), scale=float(q["scale"]),
+                                        conv=int(q["conv"]), window=int(mask.get("size", 0)), pool=int(mask.get("pool", 0)), rot=rot,
+                                        softcap=float(q.get("softcap") or 0.0)),
+                      wkv=wkv_spec(i, m["right"], "right."), left_scale=float(m["left_scale"]), right_scale=float(m["right_scale"]))
+            if kw["pool"].conv < 1:
+                raise ValueError(f"Bibezen: layer {i}: {q['conv']} taps")
+        else:
+            raise ValueError(f"Bibezen: layer {i}: mixer type {kind!r} is not part of the design")
+        mlp = lc.get("mlp")
+        if mlp is None:
+            kw.update(ff_kind="glu_clamp", ff=0)
+        elif mlp.get("kind") == "dense":
+            kw.update(ff_kind="glu_clamp", ff=int(mlp["ff"]), ff_limit=float(mlp["limit"]))
+        elif mlp.get("kind") == "moe":
+            sh = mlp.get("shared") or {}
+            kw.update(ff_kind="moe", moe=MoeSpec(experts=int(mlp["router"]["experts"]), top=int(mlp["router"]["top"]),
+                                                 expert_ff=int(mlp["expert"]["ff"]), shared_ff=int(sh.get("ff", 0)),
+                                                 router="softmax_chosen", weight_output=True, act="glu_silu", shared_plain=True))
+            if not 1 <= kw["moe"].top <= kw["moe"].experts:
+                raise ValueError(f"Bibezen: layer {i}: top {kw['moe'].top} of {kw['moe'].experts} experts")
+        else:
+            raise ValueError(f"Bibezen: layer {i}: feed-forward kind {mlp.get('kind')!r} is not part of the design")
+        layers.append(StackLayerSpec(mixer=kind, canon=canon, **kw))
+    streams = int(doc["streams"])
+    if streams < 1:
+        raise ValueError(f"Bibezen: streams {streams}")
+    return StackSpec(name=name, architecture="Bibezen", width=int(doc["width"]), vocab=int(doc["vocab"]), layers=tuple(layers),
+                     embed_scale=float((doc.get("embedding") or {}).get("scale", 1.0)), residual_mult=float(doc.get("residual_mult", 1.0)),
+                     norm_eps=float(doc["norm"]["eps"]), norm_offset=1.0, block="hyper", norm_kind="rms", loop_mix=False, streams=streams)
+
+
+def bibezen_config(spec: StackSpec) -> dict:
+    """The config.json a Bibezen StackSpec is read from (inverse of bibezen_from_config; the decay bottlenecks' ranks travel in
+    the tensors' shapes)."""
+    doc = {"architecture": "Bibezen", "canon": {"taps": spec.layers[0].canon if spec.layers else 0},
+           "embedding": {"scale": spec.embed_scale}, "layers": [], "norm": {"eps": spec.norm_eps}, "residual_mult": spec.residual_mult,
+           "streams": spec.streams, "vocab": spec.vocab, "width": spec.width}
+    for L in spec.layers:
+        if L.mixer == "mamba1":
+            a = L.mamba1
+            mixer = {"conv": a.conv, "dt_rank": a.dt_rank, "inner": a.inner, "state": a.state}
+        elif L.mixer == "wkv":
+            mixer = {"dim": L.wkv.dim, "heads": L.wkv.heads}
+        else:
+            a = L.pool
+            left = {"conv": a.conv, "dim": a.dim, "heads": a.heads, "kv_heads": a.kv_heads, "scale": a.scale, "softcap": a.softcap,
+                    "vdim": a.vdim}
+            if a.window > 0:
+                left["mask"] = {"pool": a.pool, "size": a.window}
+            if a.rot is not None:
+                left["rot"] = {"base": a.rot.base, "dims": a.rot.dims}
+            mixer = {"left": left, "left_scale": L.left_scale, "right": {"dim": L.wkv.dim, "heads": L.wkv.heads},
+                     "right_scale": L.right_scale}
+        mlp = None
+        if L.ff_kind == "moe":
+            mlp = {"expert": {"ff": L.moe.expert_ff}, "kind": "moe", "router": {"experts": L.moe.experts, "top": L.moe.top}}
+            if L.moe.shared_ff > 0:
+                mlp["shared"] = {"ff": L.moe.shared_ff}
+        elif L.ff > 0:
+            mlp = {"ff": L.ff, "kind": "dense", "limit": L.ff_limit}
+        doc["layers"].append({"mixer": mixer, "mlp": mlp, "type": L.mixer})
+    return doc
+
+
+def bibezen_tensor_shapes(spec: StackSpec) -> Dict[str, Tuple[int, ...]]:
+    """Checkpoint tensor names and shapes of a Bibezen model (Linear weights are [out, in])."""
+    W, S, out = spec.width, spec.streams, {}
+    out["embed"] = (spec.vocab, W)
+
+    def wkv(p, a):
+        n = a.heads * a.dim
+        for nm in "rkvgw":
+            out[p + "mu." + nm] = (W,)
+        for nm in "rkvg":
+            out[p + nm] = (n, W)
+        out[p + "w1"], out[p + "w2"], out[p + "w0"] = (a.rank, W), (n, a.rank), (n,)
+        out[p + "u"], out[p + "norm"], out[p + "o"] = (a.heads, a.dim), (n,), (W, n)
+
+    def gated(p, ff):
+        out[p + "gate"], out[p + "up"], out[p + "down"] = (ff, W), (ff, W), (W, ff)
+
+    for i, L in enumerate(spec.layers):
+        p = f"l{i}."
+        has_ff = L.ff_kind == "moe" or L.ff > 0
+        out[p + "norm1"] = (W,)
+        if L.canon > 0:
+            out[p + "canon1"] = (W, L.canon)
+        for q in ("hc1.", "hc2.") if has_ff else ("hc1.",):
+            out[p + q + "in"], out[p + q + "out"], out[p + q + "mix"] = (S,), (S,), (S, S)
+        if L.mixer == "mamba1":
+            a = L.mamba1
+            out[p + "mix.in"], out[p + "mix.conv"], out[p + "mix.conv.b"] = (2 * a.inner, W), (a.inner, a.conv), (a.inner,)
+            out[p + "mix.x"], out[p + "mix.dt"], out[p + "mix.dt.b"] = (a.dt_rank + 2 * a.state, a.inner), (a.inner, a.dt_rank), (a.inner,)
+            out[p + "mix.A_log"], out[p + "mix.D"], out[p + "mix.o"] = (a.inner, a.state), (a.inner,), (W, a.inner)
+        elif L.mixer == "wkv":
+            wkv(p + "mix.", L.wkv)
+        else:
+            a, q = L.pool, p + "mix.left."
+            for nm, rows in (("q", a.heads * a.dim), ("k", a.kv_heads * a.dim), ("v", a.kv_heads * a.vdim)):
+                out[q + nm], out[q + nm + ".b"], out[q + nm + ".conv"] = (rows, W), (rows,), (rows, a.conv)
+            out[q + "q.norm"], out[q + "k.norm"] = (a.dim,), (a.dim,)
+            out[q + "sink"], out[q + "talk"], out[q + "o"] = (a.heads,), (a.heads, a.heads), (W, a.heads * a.vdim)
+            wkv(p + "mix.right.", L.wkv)
+        if has_ff:
+            out[p + "norm2"] = (W,)
+        if L.ff_kind == "moe":
+            for e in range(L.moe.experts):
+                gated(f"{p}mlp.e{e}.", L.moe.expert_ff)
+            out[p + "mlp.router"] = (L.moe.experts, W)
+            if L.moe.shared_ff > 0:
+                gated(p + "mlp.shared.", L.moe.shared_ff)
+        elif L.ff > 0:
+            gated(p + "mlp.", L.ff)
+    out["final.norm"] = (W,)
+    return out
+
+
+def synth_bibezen_weights(spec: StackSpec, seed: int = 0, std: float = 0.05) -> Dict[str, torch.Tensor]:
+    """Seeded synthetic Bibezen checkpoint (bf16, checkpoint names): matrices N(0, std·√(64/in)) (routers four times wider, so that
+    the choice does not hang on the last bit), zero-centred norm weights N(0, 0.1), other norm weights 1 + N(0, 0.1),
+    connection weights near an even read and an identity-like write, decays and step sizes in the range where the state
+    both keeps and forgets."""
+    g = torch.Generator().manual_seed(seed)
+    w = {}
+    for name, shape in bibezen_tensor_shapes(spec).items():
+        t = torch.randn(shape, generator=g)
+        last = name.rsplit(".", 1)[-1]
+        if ".hc" in name:
+            t = torch.eye(shape[0]) * 0.8 + 0.15 * t if last == "mix" else (1.0 / spec.streams if last == "in" else 1.0) + 0.3 * t
+        elif name.endswith("norm1") or name.endswith("norm2") or name == "final.norm":
+            t = 0.1 * t
+        elif name.endswith(".norm") or last == "D":
+            t = 1.0 + 0.1 * t
+        elif ".mu." in name:
+            t = torch.sigmoid(t)
+        elif last == "A_log":
+            t = 0.5 * t
+        elif name.endswith("dt.b"):
+            t = t - 1.0
+        elif last == "w0":
+            t = t - 1.0
+        elif last == "talk":
+            t = torch.eye(shape[0]) * 0.8 + t * (0.4 / shape[0] ** 0.5)
+        elif last in ("sink", "u") or last == "b" and len(shape) == 1:
+            t = t * 0.5
+        elif last in ("conv", "canon1"):
+            t = t * 0.4
+        elif name == "embed":
+            t = t * 0.2
+        elif len(shape) == 2:
+            t = t * (std * (64.0 / shape[1]) ** 0.5) * (4.0 if last == "router" else 1.0)
+        w[name] = t.to(torch.bfloat16)
+    return w
+
+
+def pack_bibezen_weights(spec: StackSpec, named: Dict[str, torch.Tensor], device="cuda",
+                         dtype: torch.dtype = torch.bfloat16) -> Dict[str, torch.Tensor]:
+    """Checkpoint tensors (Bibezen names) → the engine's layout on `device`.  Per layer: w_in = the in-projections that read the
+    mixer's input itself, merged by rows (attention [q | k | v] with b_in, Mamba [x | z]); time mixing: its four products' matrices as
+    one [4, heads·dim, width] block, the bottleneck padded to 8; w_out = [left.o | right.o] by columns; taps of every
+    convolution with the tap as the slow index; gate | up rows of the gated units merged; vectors in fp32, matrices in `dtype`.
+    The head is the embedding table."""
+    W = spec.width
+    out: Dict[str, torch.Tensor] = {}
+
+    def mat(t):
+        return t.to(dtype).contiguous().to(device)
+
+    def vec(t):
+        return t.to(torch.float32).reshape(-1).contiguous().to(device)
+
+    def padded(rows, cols, *pieces):
+        """[rows, cols] of zeros with (row, column, tensor) pieces put in."""
+        t = torch.zeros(rows, cols, dtype=dtype)
+        for r, c, x in pieces:
+            t[r:r + x.shape[0], c:c + x.shape[1]] = x.to(dtype)
+        return t.to(device)
+
+    out["embed"] = mat(named["embed"])
+    out["head"], out["final_norm"] = out["embed"], vec(named["final.norm"])
+    for i, L in enumerate(spec.layers):
+        lay, p = spec.mix_layout(i), f"l{i}."
+        q = p + "mix."
+        if L.mixer == "mamba1":
+            a, rk = L.mamba1, _up8(L.mamba1.dt_rank)
+            t, x = named[q + "in"], named[q + "x"]
+            out[p + "w_in"] = padded(lay.n_in, W, (lay.off_v, 0, t[:a.inner]), (lay.off_g, 0, t[a.inner:]))
+            out[p + "conv_w"], out[p + "conv_b"] = vec(named[q + "conv"].t()), vec(named[q + "conv.b"])
+            out[p + "w_x"] = padded(_up8(rk + 2 * a.state), a.inner, (0, 0, x[:a.dt_rank]), (rk, 0, x[a.dt_rank:]))
+            out[p + "w_dt"], out[p + "dt_b"] = padded(a.inner, rk, (0, 0, named[q + "dt"])), vec(named[q + "dt.b"])
+            out[p + "A_log"], out[p + "D"], out[p + "w_out"] = vec(named[q + "A_log"]), vec(named[q + "D"]), mat(named[q + "o"])
+        if L.wkv is not None:
+            a, r = L.wkv, q + ("right." if L.mixer == "parallel" else "")
+            n, rk = a.heads * a.dim, _up8(a.rank)
+            out[p + "mu"] = vec(torch.stack([named[r + "mu." + s] for s in "rkvgw"]))
+            out[p + "w_rkvg"] = mat(torch.stack([named[r + s] for s in "rkvg"]))
+            out[p + "w1"], out[p + "w2"] = padded(rk, W, (0, 0, named[r + "w1"])), padded(n, rk, (0, 0, named[r + "w2"]))
+            out[p + "w0"], out[p + "u"], out[p + "head_norm"] = vec(named[r + "w0"]), vec(named[r + "u"]), vec(named[r + "norm"])
+            if L.mixer == "wkv":
+                out[p + "w_out"] = padded(W, lay.k_out, (0, 0, named[r + "o"]))
+        if L.pool is not None:
+            a, r = L.pool, q + "left."
+            offs = (("q", lay.off_q), ("k", lay.off_k), ("v", lay.off_v))
+            out[p + "w_in"] = padded(lay.n_in, W, *[(o, 0, named[r + s]) for s, o in offs])
+            b_in, conv = torch.zeros(lay.n_in), torch.zeros(a.conv, lay.n_in)
+            for s, o in offs:
+                n = named[r + s].shape[0]
+                b_in[o:o + n], conv[:, o:o + n] = named[r + s + ".b"].float(), named[r + s + ".conv"].t().float()
+            out[p + "b_in"], out[p + "left.conv_w"] = b_in.to(device), vec(conv)
+            out[p + "left.q_norm"], out[p + "left.k_norm"] = vec(named[r + "q.norm"]), vec(named[r + "k.norm"])
+            out[p + "left.sink"], out[p + "left.talk"] = vec(named[r + "sink"]), vec(named[r + "talk"])
+            out[p + "w_out"] = padded(W, lay.k_out, (0, 0, named[r + "o"]),
+                                      *([(0, _up8(a.heads * a.vdim), named[q + "right.o"])] if L.wkv is not None else []))
+        out[p + "norm"] = vec(named[p + "norm1"])
+        if L.canon > 0:
+            out[p + "canon_w"] = vec(named[p + "canon1"].t())
+        has_ff = L.ff_kind == "moe" or L.ff > 0
+        for h in ("hc1.", "hc2.") if has_ff else ("hc1.",):
+            for s in ("in", "out", "mix"):
+                out[p + h + s] = vec(named[p + h + s])
+        if has_ff:
+            out[p + "ff_norm"] = vec(named[p + "norm2"])
+        if L.ff_kind == "moe":
+            m, q = L.moe, p + "mlp."
+            out[p + "router"] = mat(named[q + "router"])
+            out[p + "w_exp_in"] = mat(torch.stack([torch.cat([named[f"{q}e{e}.gate"], named[f"{q}e{e}.up"]], 0) for e in range(m.experts)]))
+            out[p + "w_exp_out"] = mat(torch.stack([named[f"{q}e{e}.down"] for e in range(m.experts)]))
+            if m.shared_ff > 0:
+                out[p + "w_ff_in"] = padded(_up8(2 * m.shared_ff), W, (0, 0, named[q + "shared.gate"]), (m.shared_ff, 0, named[q + "shared.up"]))
+                out[p + "w_ff_out"] = mat(named[q + "shared.down"])
+        elif L.ff > 0:
+            out[p + "w_ff_in"] = mat(torch.cat([named[p + "mlp.gate"], named[p + "mlp.up"]], 0))
+            out[p + "w_ff_out"] = mat(named[p + "mlp.down"])
+    return out
+
+
 @dataclass(frozen=True)
 class Architecture:
     """One design of the layer-stack registry: its config reader and writer, checkpoint tensor list, synthetic checkpoint
@@ -1399,6 +1749,8 @@ ARCHITECTURES["Tekosun"] = Architecture(tekosun_from_config, tekosun_config, tek
                                         pack_tekosun_weights, with_shapes=True)
 ARCHITECTURES["Tarudra"] = Architecture(tarudra_from_config, tarudra_config, tarudra_tensor_shapes, synth_tarudra_weights,
                                         pack_tarudra_weights)
+ARCHITECTURES["Bibezen"] = Architecture(bibezen_from_config, bibezen_config, bibezen_tensor_shapes, synth_bibezen_weights,
+                                        pack_bibezen_weights, with_shapes=True)
 
 
 # ------------------------------------------------------------------------------------------- checkpoint writer

@@ -113,7 +113,8 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnPrep p) {
 // multiply-adds per operand and column, and the output's dot with the NEW columns.  Columns never read each other, so
 // the result of a sequence does not depend on what else is in the step; the order of the sums inside a column is fixed by
 // dk alone (lane l sums rows l, l + 32, …, then the butterfly), whatever NC is.
-// OLD: the output reads the columns BEFORE the token joins them, plus the token's bonus times its value.
+// OLD: the output reads the columns BEFORE the token joins them, plus the token's bonus times its value; d holds the decay
+// minus one, so that a decay close to one keeps all its digits.
 template <int DR, bool REMOVE, int NC, bool OLD = false>
 __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
   pdl_trigger();
@@ -227,7 +228,7 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
 #pragma unroll
           for (int c = 0; c < NC; ++c) {
             if constexpr (OLD) dot[u][c] = fmaf(S[c][i], rr, dot[u][c]);
-            float sn = dd * S[c][i];
+            float sn = OLD ? fmaf(dd, S[c][i], S[c][i]) : dd * S[c][i];
             if constexpr (REMOVE) sn = fmaf(-pp, rem[c], sn);
             sn = fmaf(bb, vj[c], sn);
             S[c][i] = sn;
@@ -531,7 +532,8 @@ __global__ void __launch_bounds__(256) gdelta_out_kernel(const GatedDeltaRun p) 
 }
 
 // --------------------------------------------------------------------------------------------------------- time mixing
-// One warp per (token, head): decay exp(−exp(wl)), the bonus Σ r·u·k; the scan's fp32 rows [decay | k | r | v | bonus].
+// One warp per (token, head): decay exp(−exp(wl)) (minus one), the bonus Σ r·u·k; the scan's fp32 rows
+// [decay − 1 | k | r | v | bonus].
 template <typename T>
 __global__ void __launch_bounds__(128) wkv_prep_kernel(const WkvRun p) {
   pdl_trigger();
@@ -547,7 +549,7 @@ __global__ void __launch_bounds__(128) wkv_prep_kernel(const WkvRun p) {
   for (int i = lane; i < dk; i += 32) {
     const int c = hd * dk + i;
     const float rv = ldf<T>(r + c), kv = ldf<T>(r + seg + c);
-    f[c] = expf(-expf(p.wl[(int64_t)t * n + c]));
+    f[c] = expm1f(-expf(p.wl[(int64_t)t * n + c]));
     f[n + c] = kv;
     f[2 * n + c] = rv;
     f[3 * n + c] = ldf<T>(r + 2 * seg + c);
@@ -623,7 +625,8 @@ __global__ void __launch_bounds__(256) mamba1_dt_kernel(const Mamba1Run p) {
 // tokens at a time: the chunk's B and C rows (fp32) and its channels' step sizes, inputs and gates sit in shared memory,
 // while the next chunk's values are already on their way into registers.  The state is in registers for the whole walk; a
 // token costs a thread NPT exponentials and 3·NPT multiply-adds, and the lanes' partial sums of four tokens meet side by
-// side, off the state's chain.  Entries past the state's size hold zeros (decay 1, B = C = 0).
+// side, off the state's chain.  The decay is 2^(dt·A·log2 e); fp32 engines take exp(dt·A) − 1 instead, so that thousands of
+// decays close to one do not add up a rounding of their own.  Entries past the state's size hold zeros (decay 1, B = C = 0).
 template <typename T, int LPC, int NPT>
 __global__ void __launch_bounds__(128) mamba1_scan_kernel(const Mamba1Run p) {
   pdl_trigger();
@@ -645,7 +648,7 @@ __global__ void __launch_bounds__(128) mamba1_scan_kernel(const Mamba1Run p) {
   for (int i = 0; i < NPT; ++i) {   // lane ln holds entries ln·NPT …: consecutive B / C entries per thread
     const int n = ln * NPT + i;
     S[i] = live && n < N && !fresh ? st[n] : 0.f;
-    A[i] = live && n < N ? -expf(p.d.A_log[(int64_t)c * N + n]) * 1.4426950408889634f : 0.f;   // exp(dt·A) = 2^(dt·A·log2 e)
+    A[i] = live && n < N ? -expf(p.d.A_log[(int64_t)c * N + n]) * (sizeof(T) == 4 ? 1.f : 1.4426950408889634f) : 0.f;
   }
   const float D = live ? p.d.D[c] : 0.f;
   const int off_b = (p.d.dt_rank + 7) / 8 * 8;
@@ -697,7 +700,8 @@ __global__ void __launch_bounds__(128) mamba1_scan_kernel(const Mamba1Run p) {
         float a = 0.f;
 #pragma unroll
         for (int i = 0; i < NPT; ++i) {
-          S[i] = fmaf(exp2f(dt * A[i]), S[i], dx * s_b[t][ln * NPT + i]);
+          if constexpr (sizeof(T) == 4) S[i] += fmaf(expm1f(dt * A[i]), S[i], dx * s_b[t][ln * NPT + i]);
+          else S[i] = fmaf(exp2f(dt * A[i]), S[i], dx * s_b[t][ln * NPT + i]);
           a = fmaf(S[i], s_c[t][ln * NPT + i], a);
         }
         y[u] = a;

@@ -34,7 +34,8 @@ int launch_attn_prep(const AttnPrep& p, int dtype, cudaStream_t st);
 // row or null.  State of a slot: [heads][dk][dv] fp32 at state + slot·slot_stride; a sequence whose first row has
 // position 0 starts from zero.
 constexpr int kScanMaxDim = 512;
-//   read_old (no removal):  o_j = s·r + bonus·v_j with the s from BEFORE the update; bonus: [heads] per row
+//   read_old (no removal):  o_j = s·r + bonus·v_j with the s from BEFORE the update; bonus: [heads] per row; d holds the decay
+//   minus one
 struct LinScan {
   int heads = 0, dk = 0, dv = 0, share = 1, d_scalar = 0;
   int read_old = 0;
@@ -128,7 +129,7 @@ struct WkvRun {
   float eps = 1e-5f, scale = 1.f;   // scale: a factor of the mixer's output (fp32, before it is rounded)
   const void* p4 = nullptr;      // [4][n_tok][heads·dim] T: r | k | v | gate logits
   const float* wl = nullptr;     // [n_tok, heads·dim] fp32: w2·tanh(bottleneck) + w0
-  float* f = nullptr;            // [n_tok, wkv_row_floats] fp32 workspace: decay | k | r | v | bonus
+  float* f = nullptr;            // [n_tok, wkv_row_floats] fp32 workspace: decay − 1 | k | r | v | bonus
   LinScan scan{};                // state, slots, positions, sequences, o
   void* mid = nullptr;           // [n_tok, ld_mid] T, the mixer's columns from column 0 on; columns [heads·dim, n_pad) get zeros
   int64_t ld_mid = 0;

@@ -891,25 +891,41 @@ static int stack_run_sandwich(StackEngine* s, int r, float* x, int n_tok, cudaSt
   return stack_norm_add_next(s, x, s->y, false, L.ff_post_norm, next_run_w, n_tok, st);
 }
 
-// Attention with pooled blocks over the step's rows: few rows split their key lists over CTAs; many go whole, in portions the
-// score workspace holds.
+// Attention with pooled blocks over the step's rows.  bf16 engines send every sequence that brings kTcRows rows or more to the
+// tensor-core kernels; what is left goes to the general ones: few rows split their key lists over CTAs, many go whole, in
+// portions the score workspace holds.
 static int stack_pool_attention(StackEngine* s, const PoolAttn& p0, cudaStream_t st) {
   const int nk = pool_keys_max(s->d.max_ctx, p0.a.window, p0.d.pool), tiles = (nk + kPoolTile - 1) / kPoolTile;
   const int64_t row = (int64_t)p0.a.heads * nk;
-  const int portion = (int)std::max<int64_t>(1, std::min<int64_t>(p0.n_tok, s->pool_score_floats / row));
   int rc;
-  for (int r0 = 0; r0 < p0.n_tok; r0 += portion) {
+  auto rows_from = [&](int r0, int count) {
     PoolAttn p = p0;
-    p.n_tok = std::min(portion, p0.n_tok - r0);
+    p.n_tok = count;
     p.q = (uint8_t*)p0.q + (size_t)r0 * p0.a.heads * p0.a.dim * s->esz;
     p.mid = (uint8_t*)p0.mid + (size_t)r0 * p0.ld_mid * s->esz;
     p.slot = p0.slot + r0; p.pos = p0.pos + r0;
-    p.scores = s->pool_scores; p.parts = s->pool_parts; p.outs = s->pool_outs;
-    p.nk_max = nk;
-    const int splits = std::max(1, std::min({kPoolMaxSplits, tiles, kPoolSplitCtas / p.n_tok}));
-    p.keys_per_split = (tiles + splits - 1) / splits * kPoolTile;
-    p.nsplit = (nk + p.keys_per_split - 1) / p.keys_per_split;
-    if ((rc = launch_pool_attention(p, s->dtype, st)) != B200_OK) return rc;
+    return p;
+  };
+  auto general = [&](int first, int count) {
+    const int portion = (int)std::max<int64_t>(1, std::min<int64_t>(count, s->pool_score_floats / row));
+    for (int r0 = first; r0 < first + count; r0 += portion) {
+      PoolAttn p = rows_from(r0, std::min(portion, first + count - r0));
+      p.scores = s->pool_scores; p.parts = s->pool_parts; p.outs = s->pool_outs;
+      p.nk_max = nk;
+      const int splits = std::max(1, std::min({kPoolMaxSplits, tiles, kPoolSplitCtas / p.n_tok}));
+      p.keys_per_split = (tiles + splits - 1) / splits * kPoolTile;
+      p.nsplit = (nk + p.keys_per_split - 1) / p.keys_per_split;
+      if ((rc = launch_pool_attention(p, s->dtype, st)) != B200_OK) return rc;
+    }
+    return (int)B200_OK;
+  };
+  bool any = false;
+  for (const StackEngine::Seg& g : s->segs) any = any || g.count >= kTcRows;
+  if (!any || !s->fast || !pool_prompt_ok(p0.a)) return general(0, p0.n_tok);
+  for (const StackEngine::Seg& g : s->segs) {
+    rc = g.count < kTcRows ? general(g.row0, g.count)
+                           : launch_pool_prompt(rows_from(g.row0, g.count), g.slot, g.count, g.pos0, s->pool_parts, st);
+    if (rc != B200_OK) return rc;
   }
   return B200_OK;
 }

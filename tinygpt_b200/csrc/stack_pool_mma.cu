@@ -1,0 +1,490 @@
+// stack_pool_mma.cu — prompts of the pooled-block attention on the tensor cores (mma.sync m16n8k16 bf16, fp32 accumulate), for
+// ONE sequence's rows of a step.  Mixing the heads' softmax weights needs every head's finished weights for the same
+// (query, key), so the attention runs in two kernels:
+//   pool_stats_kernel   one CTA per (64 query rows, head): the capped scores of all visible keys, online → the row's maximum
+//                       and the reciprocal of its denominator (the sink included)
+//   pool_mix_kernel     one CTA per (16 query rows, slice of the value columns), all heads: per tile of 16 keys the scores once
+//                       more, the finished weights, their mix across heads and the weighted values
+// The mix is itself a product, talk [heads × heads] times weights [heads × (query, key) pairs]; the weights enter it as the sum
+// of two bf16 numbers (their rounding and what it left), so that it is exact to about 2^-17, and are rounded to bf16 once
+// behind it, where they meet the values.  The key list is visited as tiles of block rows, then tiles of token rows.
+#include <algorithm>
+
+#include "stack_pool.cuh"
+
+namespace b200 {
+
+namespace {
+
+constexpr float kLog2eM = 1.4426950408889634f;
+
+__device__ __forceinline__ void cp16(void* dst, const void* src, bool live) {   // dead chunks are filled with zeros
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_wait() {
+  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
+}
+__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr)
+               : "memory");
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr)
+               : "memory");
+}
+__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// A raw dot product → the capped score times log2(e).  cap·tanh(z) as cap·(1 − 2 / (1 + e^(2z))): an absolute error of about
+// 1e-7·cap, which is what the softmax sees.
+struct ScoreMap {
+  float in, out;   // capped: 2^(s·in) = e^(2·s·scale/cap), out = cap·log2 e;  uncapped: in = 0, out = scale·log2 e
+};
+__device__ __forceinline__ float map_score(float s, const ScoreMap& m) {
+  if (m.in == 0.f) return s * m.out;
+  const float e = exp2f(fminf(s * m.in, 126.f));
+  return m.out * (1.f - __fdividef(2.f, 1.f + e));
+}
+
+struct PoolMma {
+  PoolAttn p{};                  // q, caches, sizes (the sequence's rows: q / mid point at its first row)
+  const __nv_bfloat16 *k = nullptr, *v = nullptr;   // the sequence's cache rows
+  int count = 0, pos0 = 0;       // rows of the sequence in this step, position of the first
+  ScoreMap map{};
+  float* stats = nullptr;        // [count][heads][2]: maximum (log2 units), 1 / denominator
+  int vcols = 0, stages = 1;     // pool_mix_kernel: value columns per CTA, stages of its key / value ring
+};
+
+// The keys a tile of rows at positions [p0, p1] may see: blocks [0, nb) and tokens [lo, p1].
+struct TileList {
+  int nb, lo, p1, block_tiles, tiles;
+};
+template <int BN>
+__device__ __forceinline__ TileList tile_list(const PoolAttn& p, int p0, int p1) {
+  TileList t;
+  t.nb = pool_nb(p1, p.a.window, p.d.pool);
+  t.lo = pool_lo(p0, p.a.window);
+  t.p1 = p1;
+  t.block_tiles = (t.nb + BN - 1) / BN;
+  t.tiles = t.block_tiles + (p1 - t.lo + BN) / BN;
+  return t;
+}
+// first cache row of tile `it`, and how many of its rows are in the list
+__device__ __forceinline__ int tile_row0(const TileList& t, int it, int bn, int max_ctx, int& n) {
+  if (it < t.block_tiles) {
+    n = t.nb - it * bn;
+    return max_ctx + it * bn;
+  }
+  const int j0 = t.lo + (it - t.block_tiles) * bn;
+  n = t.p1 - j0 + 1;
+  return j0;
+}
+
+// ------------------------------------------------------------------------------------------------------------ statistics
+constexpr int kStM = 64, kStN = 64;
+template <int KS>   // dim / 16
+__global__ void __launch_bounds__(128) pool_stats_kernel(const PoolMma m) {
+  extern __shared__ __align__(128) uint8_t ps_smem[];
+  constexpr int LD = KS * 32 + 16;   // bytes per staged row: an odd number of 16-byte chunks, conflict-free for ldmatrix
+  const PoolAttn& p = m.p;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+  const int h = blockIdx.y, H = p.a.heads, G = p.a.kv_heads, dk = KS * 16, kvh = h / (H / G);
+  const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kStM;   // rows with the most keys first
+  const int rows = min(kStM, m.count - q0);
+  uint8_t* Qs = ps_smem;                  // [64][LD]
+  uint8_t* Ks = Qs + kStM * LD;           // [2][64][LD]
+  const TileList tl = tile_list<kStN>(p, m.pos0 + q0, m.pos0 + q0 + rows - 1);
+  const __nv_bfloat16* qg = static_cast<const __nv_bfloat16*>(p.q) + (int64_t)h * dk;
+  const __nv_bfloat16* kg = m.k + (int64_t)kvh * dk;
+  constexpr int CH = KS * 2;
+  for (int i = tid; i < kStM * CH; i += 128) {
+    const int r = i / CH, c = i % CH;
+    cp16(Qs + r * LD + c * 16, qg + (int64_t)min(q0 + r, m.count - 1) * H * dk + c * 8, r < rows);
+  }
+  auto load = [&](int it) {
+    int n;
+    const int r0 = tile_row0(tl, it, kStN, p.max_ctx, n);
+    uint8_t* dst = Ks + (it & 1) * kStN * LD;
+    for (int i = tid; i < kStN * CH; i += 128) {
+      const int r = i / CH, c = i % CH;
+      cp16(dst + r * LD + c * 16, kg + (int64_t)(r0 + min(r, n - 1)) * G * dk + c * 8, r < n);
+    }
+    cp_commit();
+  };
+  load(0);
+  uint32_t qf[KS][4];
+  const int i0 = m.pos0 + q0 + warp * 16 + g, i1 = i0 + 8;
+  const int lo0 = pool_lo(i0, p.a.window), lo1 = pool_lo(i1, p.a.window);
+  const int nb0 = pool_nb(i0, p.a.window, p.d.pool), nb1 = pool_nb(i1, p.a.window, p.d.pool);
+  float mx0 = -INFINITY, mx1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+  for (int it = 0; it < tl.tiles; ++it) {
+    cp_wait<0>();
+    __syncthreads();   // tile `it` is there, and everyone is done with the buffer the next load writes
+    if (it + 1 < tl.tiles) load(it + 1);
+    if (it == 0) {
+#pragma unroll
+      for (int k = 0; k < KS; ++k)
+        ldsm4(smem_u32(Qs + (warp * 16 + (lane & 15)) * LD + k * 32 + (lane >> 4) * 16), qf[k]);
+    }
+    const uint8_t* K = Ks + (it & 1) * kStN * LD;
+    const bool blk = it < tl.block_tiles;
+    const int j0 = blk ? it * kStN : tl.lo + (it - tl.block_tiles) * kStN;
+    // visible keys of the two rows as ranges of in-tile columns
+    const int a0 = blk ? 0 : lo0 - j0, e0 = blk ? nb0 - j0 : i0 - j0 + 1;
+    const int a1 = blk ? 0 : lo1 - j0, e1 = blk ? nb1 - j0 : i1 - j0 + 1;
+    float s[8][4];
+#pragma unroll
+    for (int nt = 0; nt < 8; nt += 2) {
+#pragma unroll
+      for (int x = 0; x < 4; ++x) s[nt][x] = s[nt + 1][x] = 0.f;
+#pragma unroll
+      for (int k = 0; k < KS; ++k) {
+        uint32_t b[4];   // keys nt·8 … + 7: entries 0-7 and 8-15; keys + 8 … + 15: the same
+        ldsm4(smem_u32(K + (nt * 8 + (lane & 7) + (lane >> 4) * 8) * LD + k * 32 + ((lane >> 3) & 1) * 16), b);
+        mma16816(s[nt], qf[k], b[0], b[1]);
+        mma16816(s[nt + 1], qf[k], b[2], b[3]);
+      }
+    }
+    float t0 = -INFINITY, t1 = -INFINITY;
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const int c = nt * 8 + tq * 2 + x;
+        s[nt][x] = c >= a0 && c < e0 ? map_score(s[nt][x], m.map) : -INFINITY;
+        s[nt][x + 2] = c >= a1 && c < e1 ? map_score(s[nt][x + 2], m.map) : -INFINITY;
+        t0 = fmaxf(t0, s[nt][x]);
+        t1 = fmaxf(t1, s[nt][x + 2]);
+      }
+#pragma unroll
+    for (int o = 1; o < 4; o <<= 1) {
+      t0 = fmaxf(t0, __shfl_xor_sync(0xffffffffu, t0, o));
+      t1 = fmaxf(t1, __shfl_xor_sync(0xffffffffu, t1, o));
+    }
+    const float n0 = fmaxf(mx0, t0), n1 = fmaxf(mx1, t1);
+    const float b0 = n0 == -INFINITY ? 0.f : n0, b1 = n1 == -INFINITY ? 0.f : n1;   // nothing seen yet: 2^(−inf − 0) = 0
+    l0 *= exp2f(mx0 - b0);
+    l1 *= exp2f(mx1 - b1);
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        l0 += exp2f(s[nt][x] - b0);
+        l1 += exp2f(s[nt][x + 2] - b1);
+      }
+    mx0 = n0;
+    mx1 = n1;
+  }
+#pragma unroll
+  for (int o = 1; o < 4; o <<= 1) {
+    l0 += __shfl_xor_sync(0xffffffffu, l0, o);
+    l1 += __shfl_xor_sync(0xffffffffu, l1, o);
+  }
+  if (tq != 0) return;
+  const float sink = p.d.sink != nullptr ? p.d.sink[h] * kLog2eM : -INFINITY;
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    const int r = q0 + warp * 16 + g + 8 * x;
+    if (r >= m.count) continue;
+    const float mx = x ? mx1 : mx0, l = x ? l1 : l0, mm = fmaxf(mx, sink);   // a row always sees itself: mx is finite
+    float* o = m.stats + ((int64_t)r * H + h) * 2;
+    o[0] = mm;
+    o[1] = 1.f / (l * exp2f(mx - mm) + exp2f(sink - mm));
+  }
+}
+
+// ------------------------------------------------------------------------------------------------- mixed weights, values
+// Warp w owns heads w·HPW … w·HPW + HPW − 1 for the scores and the values, and every NW-th group of eight (key, query) pairs
+// for the mix.  Shared layouts (16-bit entries; strides padded so that ldmatrix and the scattered stores hit all banks):
+//   weights  [key 16][query 16][head], high and low halves apart — the mix reads eight pairs × 16 heads as its B operand
+//   mixed    [head][key 16][query 16] — the values read it transposed as their A operand
+template <int HPW> struct MixShape {
+  static constexpr int KH = HPW;                          // head groups of 16 (HPW 1: up to 16 heads, 2: up to 32)
+  static constexpr int PW = KH == 1 ? 12 : 20;            // words per pair: 16·KH heads + 16 bytes
+  static constexpr int JW = 16 * PW + 1;                  // words per key
+  static constexpr int WBYTES = (16 * JW * 4 + 15) / 16 * 16;
+  static constexpr int XW = 196;                          // words per head of the mixed weights: 16 rows of 12 words, + 4
+  static constexpr int XBYTES = 16 * KH * XW * 4;
+  static constexpr int NT = 16 / HPW;                     // most 8-column tiles of a CTA's slice of the values
+};
+__host__ __device__ inline int mix_smem(int H, int G, int dk, int vcols, int stages, int wbytes, int xbytes) {
+  return 16 * (H * dk * 2 + 16) + stages * 16 * ((G * dk * 2 + 16) + (G * vcols * 2 + 16)) + 2 * wbytes + xbytes;
+}
+
+template <int HPW>
+__global__ void __launch_bounds__(512) pool_mix_kernel(const PoolMma m) {
+  extern __shared__ __align__(128) uint8_t pm_smem[];
+  using SH = MixShape<HPW>;
+  const PoolAttn& p = m.p;
+  const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3, nw = nthr >> 5;
+  const int H = p.a.heads, G = p.a.kv_heads, per = H / G, dk = p.a.dim, dv = p.a.vdim, ks = dk / 16;
+  const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * 16, rows = min(16, m.count - q0);
+  const int c0 = blockIdx.y * m.vcols, vc = min(m.vcols, dv - c0), nt_v = vc / 8;
+  const int ldq = H * dk * 2 + 16, ldk = G * dk * 2 + 16, ldv = G * m.vcols * 2 + 16;
+  uint8_t* Qs = pm_smem;
+  uint8_t* Ks = Qs + 16 * ldq;
+  uint8_t* Vs = Ks + m.stages * 16 * ldk;
+  uint32_t* Wh = reinterpret_cast<uint32_t*>(Vs + m.stages * 16 * ldv);
+  uint32_t* Wl = Wh + SH::WBYTES / 4;
+  uint32_t* X = Wl + SH::WBYTES / 4;
+  const TileList tl = tile_list<16>(p, m.pos0 + q0, m.pos0 + q0 + rows - 1);
+  {
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q);
+    const int ch = H * dk / 8;
+    for (int i = tid; i < 16 * ch; i += nthr) {
+      const int r = i / ch, c = i % ch;
+      cp16(Qs + r * ldq + c * 16, q + (int64_t)min(q0 + r, m.count - 1) * H * dk + c * 8, r < rows);
+    }
+  }
+  const int kch = G * dk / 8, vch1 = vc / 8, vch = G * vch1;
+  auto load = [&](int it) {
+    int n;
+    const int r0 = tile_row0(tl, it, 16, p.max_ctx, n), st = it % m.stages;
+    uint8_t* kd = Ks + st * 16 * ldk;
+    uint8_t* vd = Vs + st * 16 * ldv;
+    for (int i = tid; i < 16 * kch; i += nthr) {
+      const int r = i / kch, c = i % kch;
+      cp16(kd + r * ldk + c * 16, m.k + (int64_t)(r0 + min(r, n - 1)) * G * dk + c * 8, r < n);
+    }
+    for (int i = tid; i < 16 * vch; i += nthr) {
+      const int r = i / vch, e = i % vch, gg = e / vch1, c = e % vch1;
+      cp16(vd + r * ldv + gg * m.vcols * 2 + c * 16, m.v + (int64_t)(r0 + min(r, n - 1)) * G * dv + gg * dv + c0 + c * 8, r < n);
+    }
+    cp_commit();
+  };
+  load(0);
+  // heads that do not exist keep zero weights
+  for (int i = tid; i < 2 * SH::WBYTES / 4; i += nthr) Wh[i] = 0;
+  // the mixing matrix as A fragments: rows = mixed head, columns = head
+  uint32_t tf[SH::KH][SH::KH][4];
+  {
+    auto talk = [&](int a, int b) {
+      if (a >= H || b >= H) return 0.f;
+      return p.d.talk != nullptr ? p.d.talk[a * H + b] : a == b ? 1.f : 0.f;
+    };
+#pragma unroll
+    for (int a = 0; a < SH::KH; ++a)
+#pragma unroll
+      for (int b = 0; b < SH::KH; ++b)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          const int r = a * 16 + g + (x & 1) * 8, c = b * 16 + tq * 2 + (x >> 1) * 8;
+          tf[a][b][x] = pack2(talk(r, c), talk(r, c + 1));
+        }
+  }
+  const int i0 = m.pos0 + q0 + g, i1 = i0 + 8;
+  const int lo0 = pool_lo(i0, p.a.window), lo1 = pool_lo(i1, p.a.window);
+  const int nb0 = pool_nb(i0, p.a.window, p.d.pool), nb1 = pool_nb(i1, p.a.window, p.d.pool);
+  float mx[HPW][2], il[HPW][2], o[HPW][SH::NT][4];
+#pragma unroll
+  for (int u = 0; u < HPW; ++u) {
+    const int h = warp * HPW + u;
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int r = q0 + g + 8 * x;
+      const bool live = h < H && r < m.count;
+      mx[u][x] = live ? m.stats[((int64_t)r * H + h) * 2] : 0.f;
+      il[u][x] = live ? m.stats[((int64_t)r * H + h) * 2 + 1] : 0.f;
+    }
+#pragma unroll
+    for (int n = 0; n < SH::NT; ++n)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) o[u][n][x] = 0.f;
+  }
+  __nv_bfloat16* Whb = reinterpret_cast<__nv_bfloat16*>(Wh);
+  __nv_bfloat16* Wlb = reinterpret_cast<__nv_bfloat16*>(Wl);
+  for (int it = 0; it < tl.tiles; ++it) {
+    if (m.stages == 1 && it > 0) {
+      __syncthreads();   // the last tile's values have been read
+      load(it);
+    }
+    cp_wait<0>();
+    __syncthreads();     // tile `it` is there; everyone is done with the ring stage the next load writes
+    if (m.stages > 1 && it + 1 < tl.tiles) load(it + 1);
+    const uint8_t* K = Ks + (it % m.stages) * 16 * ldk;
+    const uint8_t* V = Vs + (it % m.stages) * 16 * ldv;
+    const bool blk = it < tl.block_tiles;
+    const int j0 = blk ? it * 16 : tl.lo + (it - tl.block_tiles) * 16;
+    const int a0 = blk ? 0 : lo0 - j0, e0 = blk ? nb0 - j0 : i0 - j0 + 1;
+    const int a1 = blk ? 0 : lo1 - j0, e1 = blk ? nb1 - j0 : i1 - j0 + 1;
+    // ---- scores → finished weights of this warp's heads
+#pragma unroll
+    for (int u = 0; u < HPW; ++u) {
+      const int h = warp * HPW + u;
+      if (h >= H) break;
+      const int kvh = h / per;
+      float s[2][4];
+#pragma unroll
+      for (int x = 0; x < 4; ++x) s[0][x] = s[1][x] = 0.f;
+      const uint32_t qa = smem_u32(Qs + (lane & 15) * ldq + h * dk * 2 + (lane >> 4) * 16);
+      const uint32_t ka = smem_u32(K + ((lane & 7) + (lane >> 4) * 8) * ldk + kvh * dk * 2 + ((lane >> 3) & 1) * 16);
+#pragma unroll 4
+      for (int k = 0; k < ks; ++k) {
+        uint32_t a[4], b[4];
+        ldsm4(qa + k * 32, a);
+        ldsm4(ka + k * 32, b);
+        mma16816(s[0], a, b[0], b[1]);
+        mma16816(s[1], a, b[2], b[3]);
+      }
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          const int j = nt * 8 + tq * 2 + (x & 1), second = x >> 1;
+          const bool vis = second ? j >= a1 && j < e1 : j >= a0 && j < e0;
+          const float w = vis ? exp2f(map_score(s[nt][x], m.map) - mx[u][second]) * il[u][second] : 0.f;
+          const __nv_bfloat16 hi = __float2bfloat16_rn(w);
+          const int at = (j * SH::JW + (g + 8 * second) * SH::PW) * 2 + h;
+          Whb[at] = hi;
+          Wlb[at] = __float2bfloat16_rn(w - __bfloat162float(hi));
+        }
+    }
+    __syncthreads();
+    // ---- mix: eight pairs (one key, queries half·8 …) at a time
+    for (int nt = warp; nt < 32; nt += nw) {
+      const int j = nt >> 1, iq = (nt & 1) * 8;
+      const int at = j * SH::JW + (iq + g) * SH::PW + tq;
+      float x[SH::KH][4];
+#pragma unroll
+      for (int a = 0; a < SH::KH; ++a)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) x[a][e] = 0.f;
+#pragma unroll
+      for (int b = 0; b < SH::KH; ++b) {
+        const uint32_t h0 = Wh[at + b * 8], h1 = Wh[at + b * 8 + 4], l0 = Wl[at + b * 8], l1 = Wl[at + b * 8 + 4];
+#pragma unroll
+        for (int a = 0; a < SH::KH; ++a) {
+          mma16816(x[a], tf[a][b], h0, h1);
+          mma16816(x[a], tf[a][b], l0, l1);
+        }
+      }
+#pragma unroll
+      for (int a = 0; a < SH::KH; ++a) {
+        uint32_t* d = X + (a * 16 + g) * SH::XW + j * 12 + (iq >> 1) + tq;
+        d[0] = pack2(x[a][0], x[a][1]);
+        d[8 * SH::XW] = pack2(x[a][2], x[a][3]);
+      }
+    }
+    __syncthreads();
+    // ---- values
+#pragma unroll
+    for (int u = 0; u < HPW; ++u) {
+      const int h = warp * HPW + u;
+      if (h >= H) break;
+      const int kvh = h / per;
+      uint32_t a[4];   // stored [key][query]: matrices (keys 0-7, queries 0-7), (keys 0-7, queries 8-15), (keys 8-15, …), …
+      ldsm4_t(smem_u32(X + h * SH::XW + ((lane & 7) + (lane >> 4) * 8) * 12) + ((lane >> 3) & 1) * 16, a);
+      const uint32_t va = smem_u32(V + (lane & 15) * ldv + kvh * m.vcols * 2 + (lane >> 4) * 16);
+#pragma unroll
+      for (int n = 0; n < SH::NT; n += 2) {
+        if (n >= nt_v) break;
+        uint32_t b[4];   // columns n·8 … + 7: keys 0-7 and 8-15; columns + 8 … + 15: the same
+        ldsm4_t(va + n * 16, b);
+        mma16816(o[u][n], a, b[0], b[1]);
+        mma16816(o[u][n + 1], a, b[2], b[3]);
+      }
+    }
+  }
+#pragma unroll
+  for (int u = 0; u < HPW; ++u) {
+    const int h = warp * HPW + u;
+    if (h >= H) break;
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int r = q0 + g + 8 * x;
+      if (r >= m.count) continue;
+      __nv_bfloat16* y = static_cast<__nv_bfloat16*>(p.mid) + (int64_t)r * p.ld_mid + h * dv + c0 + tq * 2;
+#pragma unroll
+      for (int n = 0; n < SH::NT; ++n)
+        if (n < nt_v)
+          *reinterpret_cast<uint32_t*>(y + n * 8) = pack2(o[u][n][2 * x] * p.out_scale, o[u][n][2 * x + 1] * p.out_scale);
+    }
+  }
+}
+
+template <int KS>
+int launch_stats(const PoolMma& m, cudaStream_t st) {
+  constexpr int smem = 3 * 64 * (KS * 32 + 16);
+  if (smem > 48 * 1024) {
+    static bool attr_done = false;
+    if (!attr_done) {
+      B200_CUDA(cudaFuncSetAttribute(pool_stats_kernel<KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+      attr_done = true;
+    }
+  }
+  const dim3 grid((m.count + kStM - 1) / kStM, m.p.a.heads);
+  B200_CUDA(launch_pdl(pool_stats_kernel<KS>, grid, dim3(128), (size_t)smem, st, false, m));
+  return B200_OK;
+}
+
+template <int HPW>
+int launch_mix(PoolMma m, cudaStream_t st) {
+  using SH = MixShape<HPW>;
+  const b200_attn_desc& a = m.p.a;
+  static bool attr_done = false;
+  if (!attr_done) {
+    B200_CUDA(cudaFuncSetAttribute(pool_mix_kernel<HPW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    attr_done = true;
+  }
+  const int splits = (a.vdim + SH::NT * 8 - 1) / (SH::NT * 8);
+  m.vcols = ((a.vdim + splits - 1) / splits + 15) / 16 * 16;
+  m.stages = mix_smem(a.heads, a.kv_heads, a.dim, m.vcols, 2, SH::WBYTES, SH::XBYTES) <= 227 * 1024 ? 2 : 1;
+  const int smem = mix_smem(a.heads, a.kv_heads, a.dim, m.vcols, m.stages, SH::WBYTES, SH::XBYTES);
+  const int warps = std::max(4, (a.heads + HPW - 1) / HPW);
+  const dim3 grid((m.count + 15) / 16, (a.vdim + m.vcols - 1) / m.vcols);
+  B200_CUDA(launch_pdl(pool_mix_kernel<HPW>, grid, dim3(warps * 32), (size_t)smem, st, false, m));
+  return B200_OK;
+}
+
+}  // namespace
+
+bool pool_prompt_ok(const b200_attn_desc& a) {
+  if (a.heads > 32 || a.dim % 16 != 0 || a.dim > 128 || a.vdim % 16 != 0 || a.vdim > 256) return false;
+  const int vmax = a.heads <= 16 ? 128 : 64, splits = (a.vdim + vmax - 1) / vmax, vc = ((a.vdim + splits - 1) / splits + 15) / 16 * 16;
+  const int w = a.heads <= 16 ? MixShape<1>::WBYTES : MixShape<2>::WBYTES, x = a.heads <= 16 ? MixShape<1>::XBYTES : MixShape<2>::XBYTES;
+  return mix_smem(a.heads, a.kv_heads, a.dim, vc, 1, w, x) <= 227 * 1024;
+}
+
+int launch_pool_prompt(const PoolAttn& p, int slot, int count, int pos0, float* stats, cudaStream_t st) {
+  const b200_attn_desc& a = p.a;
+  B200_CHECK_ARG(p.q && p.kcache && p.vcache && p.mid && stats && count > 0 && pos0 >= 0 && pos0 + count <= p.max_ctx, "pool prompt attention: bad arguments");
+  B200_CHECK_ARG(pool_prompt_ok(a) && a.heads % a.kv_heads == 0, "pool prompt attention: head sizes not built");
+  B200_CHECK_ARG(((reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.kcache) | reinterpret_cast<uintptr_t>(p.vcache)) & 15) == 0 &&
+                     p.k_slot_stride % 8 == 0 && p.v_slot_stride % 8 == 0 && p.ld_mid % 2 == 0 && (reinterpret_cast<uintptr_t>(p.mid) & 3) == 0,
+                 "pool prompt attention: operands must be 16-byte aligned");
+  PoolMma m;
+  m.p = p; m.count = count; m.pos0 = pos0; m.stats = stats;
+  m.k = (const __nv_bfloat16*)p.kcache + (int64_t)slot * p.k_slot_stride;
+  m.v = (const __nv_bfloat16*)p.vcache + (int64_t)slot * p.v_slot_stride;
+  if (p.d.softcap > 0.f) {
+    m.map.in = 2.f * a.scale / p.d.softcap * kLog2eM;
+    m.map.out = p.d.softcap * kLog2eM;
+  } else {
+    m.map.out = a.scale * kLog2eM;
+  }
+  int rc = B200_OK;
+  switch (a.dim / 16) {
+    case 1: rc = launch_stats<1>(m, st); break;
+    case 2: rc = launch_stats<2>(m, st); break;
+    case 3: rc = launch_stats<3>(m, st); break;
+    case 4: rc = launch_stats<4>(m, st); break;
+    case 5: rc = launch_stats<5>(m, st); break;
+    case 6: rc = launch_stats<6>(m, st); break;
+    case 7: rc = launch_stats<7>(m, st); break;
+    default: rc = launch_stats<8>(m, st); break;
+  }
+  if (rc != B200_OK) return rc;
+  return a.heads <= 16 ? launch_mix<1>(m, st) : launch_mix<2>(m, st);
+}
+
+}  // namespace b200

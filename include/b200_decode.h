@@ -36,7 +36,7 @@ extern "C" {
  * generalized delta rule, Mamba-2, softmax-routed experts (fields appended to b200_moe_desc and b200_stack_layer),
  * b200_stack_lin_scan, b200_stack_attn_prep;  8: + hyper-connected blocks, Mamba's selective scan, RWKV-style time mixing, the
  * pooled-block attention (fields appended to b200_moe_desc, b200_stack_layer and b200_stack_desc), b200_stack_hyper_step,
- * b200_stack_input_conv, b200_stack_pool_attention, b200_stack_wkv, b200_stack_mamba1.  All additive: callers of an older version
+ * b200_stack_input_conv, b200_stack_pool_attention, b200_stack_bonus_scan, b200_stack_mamba1_scan.  All additive: callers of an older version
  * keep working once they are compiled against this header. */
 #define B200_ABI_VERSION 8
 
@@ -671,6 +671,36 @@ int b200_stack_attn_prep(void* proj, int64_t ld_proj, int64_t off_q, int64_t off
                          int64_t ld_keep, float eps, int dtype, void* stream);
 /* y[r, j] = T( min(g, limit)·sigmoid(1.702·min(g, limit))·(clamp(u, ±limit) + 1) ), g = gu[r, j], u = gu[r, n + j] */
 int b200_stack_glu_clamp(void* y, const void* gu, int64_t rows, int64_t n, float limit, int dtype, void* stream);
+
+/* One pass over `streams` copies x [rows, streams, width] (fp32, in place): x_d <- Σ_s mix[s][d]·x_s + mult·out[d]·y (y fp32
+ * [rows, width]; NULL: the copies stay), then h = T( norm(Σ_s in[s]·x_s)·(offset + norm_w) ). */
+int b200_stack_hyper_step(void* h, float* x, const float* y_or_null, const float* in, const b200_hyper_desc* prev, float mult,
+                          const float* norm_w, float eps, float offset, int64_t rows, int64_t streams, int64_t width, int dtype,
+                          void* stream);
+/* h_t = n_t + Σ_j w[taps − 1 − j]·n_(t−j) over the rows n = hn (fp32 [rows, width]; rows of a sequence side by side, slot / pos per
+ * ROW; zeros before position 0), and with mu [5][width] the blends mix_s = h_t + (h_(t−1) − h_t)·mu_s, mix T [5, rows, width].
+ * state: fp32 [taps][width] per slot, the last rows before this step's, oldest first (read; pos 0 ignores it). */
+int b200_stack_input_conv(void* h, void* mix_or_null, const float* hn, const float* w, const float* mu_or_null, int64_t taps,
+                          const float* state, int64_t slot_stride, const int32_t* slot, const int32_t* pos, int64_t rows,
+                          int64_t width, int dtype, void* stream);
+/* Pooled-block attention of prepared queries q (T [n_tok, heads·dim]) over per-slot caches: max_ctx token rows and behind them
+ * max_ctx / pool block rows (both already written); conv, norm and rotation fields of `pool` are not read.  `splits`: CTAs that
+ * share a row's key list.  out T [n_tok, heads·vdim].  Synchronises (allocates its workspace). */
+int b200_stack_pool_attention(void* out, const void* q, const void* kcache, const void* vcache, int64_t k_slot_stride,
+                              int64_t v_slot_stride, int64_t max_ctx, const int32_t* slot, const int32_t* pos, int64_t n_tok,
+                              const b200_attn_desc* attn, const b200_pool_attn_desc* pool, int64_t splits, int dtype, void* stream);
+/* As b200_stack_lin_scan without a removal, the output read from the state BEFORE the token joins it:
+ *   out_j = s·r + bonus·v_j,  s <- (1 + d)∘s + k·v_j;  d (the decay minus one), k, r [heads·dk], v [heads·dv], bonus [heads] per row. */
+int b200_stack_bonus_scan(float* out, const float* d, const float* k, const float* r, const float* v, const float* bonus, int64_t ld,
+                          int64_t heads, int64_t dk, int64_t dv, float* state, int64_t slot_stride, const int32_t* row0,
+                          const int32_t* count, const int32_t* slot, const int32_t* pos, int64_t n_seq, int64_t n_rows, void* stream);
+/* The selective scan of b200_mamba1_desc from its convolved channels xc (T [rows, inner]), xd (fp32 [rows, ld_xd]: columns
+ * [up8(dt_rank), + 2·state) are B | C), step-size logits dt (fp32 [rows, inner], bias included) and gate logits z (T [rows,
+ * inner]); out T [rows, inner].  State of a slot: [inner][state] fp32.  Only sizes, A_log and D of the descriptor are read. */
+int b200_stack_mamba1_scan(void* out, const void* z, const void* xc, const float* xd, int64_t ld_xd, const float* dt,
+                           const b200_mamba1_desc* desc, float* state, int64_t slot_stride, const int32_t* row0,
+                           const int32_t* count, const int32_t* slot, const int32_t* pos, int64_t n_seq, int64_t n_rows, int dtype,
+                           void* stream);
 
 /* ---- tensor parallel (one process per GPU; the caller exchanges the handles with torch.distributed) ---------- */
 

@@ -191,6 +191,11 @@ PROTOTYPES = {
     "b200_stack_glu_clamp": (I32, [P, P, I64, I64, F, I32, P]),
     "b200_stack_lin_scan": (I32, [P, P, P, P, P, P, P, P, I64, I64, I64, I64, I64, I64, P, I64, P, P, P, P, I64, I64, P]),
     "b200_stack_attn_prep": (I32, [P, I64, I64, I64, I64, P, I64, C.POINTER(AttnDesc), C.POINTER(AttnPrepDesc), P, I64, F, I32, P]),
+    "b200_stack_hyper_step": (I32, [P, P, P, P, C.POINTER(HyperDesc), F, P, F, F, I64, I64, I64, I32, P]),
+    "b200_stack_input_conv": (I32, [P, P, P, P, P, I64, P, I64, P, P, I64, I64, I32, P]),
+    "b200_stack_pool_attention": (I32, [P, P, P, P, I64, I64, I64, P, P, I64, C.POINTER(AttnDesc), C.POINTER(PoolAttnDesc), I64, I32, P]),
+    "b200_stack_bonus_scan": (I32, [P, P, P, P, P, P, I64, I64, I64, I64, P, I64, P, P, P, P, I64, I64, P]),
+    "b200_stack_mamba1_scan": (I32, [P, P, P, P, I64, P, C.POINTER(Mamba1Desc), P, I64, P, P, P, P, I64, I64, I32, P]),
     "b200_tp_window_bytes": (I64, [C.POINTER(ModelDesc)]),
     "b200_tp_window_create": (I32, [I64, C.POINTER(P), C.c_char_p]),
     "b200_tp_window_open": (I32, [C.c_char_p, C.POINTER(P)]),

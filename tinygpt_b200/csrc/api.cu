@@ -1,6 +1,10 @@
 // api.cu — C-ABI entry points for the GEMV and the fused building blocks (declared in include/b200_decode.h).
 #include "gemv.cuh"
+#include <algorithm>
+
+#include "stack_hyper.cuh"
 #include "stack_mix.cuh"
+#include "stack_pool.cuh"
 #include "stack_rec.cuh"
 #include <vector>
 #include "ops.cuh"
@@ -320,6 +324,92 @@ int b200_stack_glu_clamp(void* y, const void* gu, int64_t rows, int64_t n, float
   if (rc != B200_OK) return rc;
   B200_CHECK_ARG(n > 0 && n < (1ll << 30) && rows > 0, "stack_glu_clamp: size out of range");
   return b200::launch_stack_glu_clamp(y, n, gu, 2 * n, rows, (int)n, limit, dtype, (cudaStream_t)stream);
+}
+
+// ---- mechanisms of hyper-connected blocks (stack_hyper.cu, stack_pool.cu, stack_rec.cu)
+int b200_stack_hyper_step(void* h, float* x, const float* y, const float* in, const b200_hyper_desc* prev, float mult,
+                          const float* norm_w, float eps, float offset, int64_t rows, int64_t streams, int64_t width, int dtype,
+                          void* stream) {
+  int rc = b200_device_check();
+  if (rc != B200_OK) return rc;
+  B200_CHECK_ARG(h && rows > 0 && rows < (1 << 24) && width > 0 && width < (1 << 24) && (y == nullptr || prev), "stack_hyper_step: bad arguments");
+  b200::HyperStep p;
+  p.streams = (int)streams; p.width = (int)width; p.n_tok = (int)rows; p.x = x; p.y = y; p.mult = mult; p.in = in;
+  if (prev) p.prev = *prev;
+  p.norm_w = norm_w; p.eps = eps; p.offset = offset; p.h = h;
+  return b200::launch_hyper_step(p, dtype, (cudaStream_t)stream);
+}
+
+int b200_stack_input_conv(void* h, void* mix, const float* hn, const float* w, const float* mu, int64_t taps, const float* state,
+                          int64_t slot_stride, const int32_t* slot, const int32_t* pos, int64_t rows, int64_t width, int dtype,
+                          void* stream) {
+  int rc = b200_device_check();
+  if (rc != B200_OK) return rc;
+  B200_CHECK_ARG(rows > 0 && rows < (1 << 24) && width > 0 && width < (1 << 24), "stack_input_conv: bad arguments");
+  b200::InputConv c;
+  c.taps = (int)taps; c.w = w; c.mu = mu; c.h = h; c.mix = mix; c.state = const_cast<float*>(state); c.slot_stride = slot_stride;
+  return b200::launch_input_conv(c, hn, slot, pos, (int)rows, (int)width, dtype, (cudaStream_t)stream);
+}
+
+int b200_stack_pool_attention(void* out, const void* q, const void* kcache, const void* vcache, int64_t k_slot_stride,
+                              int64_t v_slot_stride, int64_t max_ctx, const int32_t* slot, const int32_t* pos, int64_t n_tok,
+                              const b200_attn_desc* attn, const b200_pool_attn_desc* pool, int64_t splits, int dtype, void* stream) {
+  int rc = b200_device_check();
+  if (rc != B200_OK) return rc;
+  B200_CHECK_ARG(attn && pool && n_tok > 0 && n_tok < (1 << 16) && max_ctx > 0 && max_ctx < (1 << 24) && attn->heads > 0 && attn->vdim > 0 &&
+                     attn->window >= 0 && pool->pool >= 0 && splits >= 1 && splits <= b200::kPoolMaxSplits,
+                 "stack_pool_attention: bad arguments");
+  b200::PoolAttn p;
+  p.a = *attn; p.d = *pool;
+  p.d.conv_w = p.d.q_norm = p.d.k_norm = p.d.rot_table = nullptr;
+  p.d.rot_dims = 0;
+  p.q = const_cast<void*>(q); p.kcache = const_cast<void*>(kcache); p.vcache = const_cast<void*>(vcache);
+  p.k_slot_stride = k_slot_stride; p.v_slot_stride = v_slot_stride; p.max_ctx = (int)max_ctx;
+  p.slot = slot; p.pos = pos; p.n_tok = (int)n_tok;
+  p.nk_max = b200::pool_keys_max((int)max_ctx, attn->window, pool->pool);
+  const int tiles = (p.nk_max + b200::kPoolTile - 1) / b200::kPoolTile, n = (int)std::min<int64_t>(splits, tiles);
+  p.keys_per_split = (tiles + n - 1) / n * b200::kPoolTile;
+  p.nsplit = (p.nk_max + p.keys_per_split - 1) / p.keys_per_split;
+  Scratch sc;
+  p.scores = (float*)sc.take((size_t)n_tok * attn->heads * p.nk_max * 4);
+  p.parts = (float*)sc.take((size_t)n_tok * attn->heads * p.nsplit * 8);
+  p.outs = (float*)sc.take((size_t)n_tok * p.nsplit * attn->heads * attn->vdim * 4);
+  B200_CHECK_ARG(p.scores && p.parts && p.outs, "stack_pool_attention: out of device memory");
+  p.mid = out; p.ld_mid = (int64_t)attn->heads * attn->vdim;
+  return b200::launch_pool_attention(p, dtype, (cudaStream_t)stream);
+}
+
+int b200_stack_bonus_scan(float* out, const float* d, const float* k, const float* r, const float* v, const float* bonus, int64_t ld,
+                          int64_t heads, int64_t dk, int64_t dv, float* state, int64_t slot_stride, const int32_t* row0,
+                          const int32_t* count, const int32_t* slot, const int32_t* pos, int64_t n_seq, int64_t n_rows, void* stream) {
+  int rc = b200_device_check();
+  if (rc != B200_OK) return rc;
+  B200_CHECK_ARG(n_seq > 0 && n_rows >= n_seq && n_rows < (1 << 24) && heads > 0 && heads < (1 << 16) && dk > 0 && dv > 0 && dv < (1 << 20),
+                 "stack_bonus_scan: bad arguments");
+  b200::LinScan s;
+  s.heads = (int)heads; s.dk = (int)dk; s.dv = (int)dv; s.read_old = 1; s.bonus = bonus;
+  s.d = d; s.b = k; s.r = r; s.v = v; s.ld = ld;
+  s.state = state; s.slot_stride = slot_stride;
+  s.seg_row0 = row0; s.seg_count = count; s.slot = slot; s.pos = pos; s.n_seg = (int)n_seq; s.n_tok = (int)n_rows;
+  s.o = out; s.ld_o = heads * dv;
+  return b200::launch_lin_scan(s, (cudaStream_t)stream);
+}
+
+int b200_stack_mamba1_scan(void* out, const void* z, const void* xc, const float* xd, int64_t ld_xd, const float* dt,
+                           const b200_mamba1_desc* desc, float* state, int64_t slot_stride, const int32_t* row0,
+                           const int32_t* count, const int32_t* slot, const int32_t* pos, int64_t n_seq, int64_t n_rows, int dtype,
+                           void* stream) {
+  int rc = b200_device_check();
+  if (rc != B200_OK) return rc;
+  B200_CHECK_ARG(desc && n_seq > 0 && n_rows >= n_seq && n_rows < (1 << 24), "stack_mamba1_scan: bad arguments");
+  b200::Mamba1Run m;
+  m.d = *desc;
+  m.proj = z; m.ld_proj = desc->inner; m.off_z = 0;
+  m.xc = const_cast<void*>(xc); m.xd = xd; m.ld_xd = ld_xd; m.dt = const_cast<float*>(dt);
+  m.state = state; m.slot_stride = slot_stride;
+  m.seg_row0 = row0; m.seg_count = count; m.slot = slot; m.pos = pos; m.n_seg = (int)n_seq; m.n_tok = (int)n_rows;
+  m.mid = out; m.ld_mid = desc->inner;
+  return b200::launch_mamba1_scan(m, dtype, (cudaStream_t)stream);
 }
 
 }  // extern "C"

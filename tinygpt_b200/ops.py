@@ -369,24 +369,102 @@ def stack_mlstm(proj: torch.Tensor, off_q: int, off_k: int, off_v: int, gates: t
 
 
 def stack_moe(h: torch.Tensor, router: torch.Tensor, w_exp_in: torch.Tensor, w_exp_out: torch.Tensor, top: int, limit: float = 0.0,
-              *, softmax: bool = False, weight_output: bool = False, act: str = "glu_clamp", route_scale: float = 1.0):
+              *, softmax: bool = False, chosen_only: bool = False, weight_output: bool = False, act: str = "glu_clamp", route_scale: float = 1.0):
     """Routed experts on h [rows, width]: router [E, width], w_exp_in [E, 2·ff, width] (gate | up; [E, ff, width] under a plain
     activation), w_exp_out [E, width, ff] → (y fp32 [rows, width], chosen int32 [rows, top], weights fp32 [rows, top]).
-    softmax: softmax scores with the chosen ones renormalised and scaled (else sigmoid scores); weight_output: the weight
+    softmax: softmax scores with the chosen ones renormalised and scaled (else sigmoid scores); chosen_only: a softmax over the
+    chosen logits alone; act "glu_…": act(gate·h)·(up·h) without a clamp; weight_output: the weight
     multiplies the expert's output (else its input)."""
     import ctypes as C
     from ._lib import MoeDesc
     h = _chk(h, "stack_moe h", h.dtype)
     E, ff2, W = w_exp_in.shape
-    plain = act != "glu_clamp"
+    plain, gated = not act.startswith("glu_"), act.startswith("glu_") and act != "glu_clamp"
     m = MoeDesc(E, int(top), ff2 if plain else ff2 // 2, 0, float(limit), 0.0, router.data_ptr(), w_exp_in.data_ptr(),
-                w_exp_out.data_ptr(), int(softmax), int(weight_output), _ACTS[act] if plain else 0, 1, float(route_scale))
+                w_exp_out.data_ptr(), 2 if chosen_only else int(softmax), int(weight_output),
+                _ACTS[act[4:]] if gated else _ACTS[act] if plain else 0, 1, float(route_scale), int(gated))
     y = torch.empty(h.shape[0], W, dtype=torch.float32, device=h.device)
     chosen = torch.empty(h.shape[0], top, dtype=torch.int32, device=h.device)
     scores = torch.empty(h.shape[0], top, dtype=torch.float32, device=h.device)
     check(lib().b200_stack_moe(y.data_ptr(), h.data_ptr(), h.shape[0], W, C.byref(m), chosen.data_ptr(), scores.data_ptr(),
                                _sdt(h), _stream()), "b200_stack_moe")
     return y, chosen, scores
+
+
+# ---- mechanisms of hyper-connected blocks (csrc/stack_hyper.cu, stack_pool.cu, stack_rec.cu)
+def stack_hyper_step(x: torch.Tensor, w_in: torch.Tensor, norm_w: torch.Tensor, *, eps: float, y: Optional[torch.Tensor] = None,
+                     w_out: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None, mult: float = 1.0, offset: float = 1.0,
+                     dtype: torch.dtype = torch.float32) -> torch.Tensor:
+    """x fp32 [rows, streams, width], IN PLACE: x_d ← Σ_s mix[s, d] x_s + mult·w_out[d]·y (y given), then → dtype
+    [rows, width]: norm(Σ_s w_in[s] x_s)·(offset + norm_w)."""
+    import ctypes as C
+    from ._lib import HyperDesc
+    rows, streams, width = x.shape
+    h = torch.empty(rows, width, dtype=dtype, device=x.device)
+    d = HyperDesc(None, _ptr(w_out), _ptr(mix))
+    check(lib().b200_stack_hyper_step(h.data_ptr(), x.data_ptr(), _ptr(y), w_in.data_ptr(), C.byref(d), float(mult), norm_w.data_ptr(),
+                                      float(eps), float(offset), rows, streams, width, _sdt(h), _stream()), "b200_stack_hyper_step")
+    return h
+
+
+def stack_input_conv(hn: torch.Tensor, w: torch.Tensor, state: torch.Tensor, slot: torch.Tensor, pos: torch.Tensor, *,
+                     mu: Optional[torch.Tensor] = None, dtype: torch.dtype = torch.float32):
+    """h_t = n_t + Σ_j w[taps−1−j] n_(t−j) over the rows hn (fp32; w [taps, width]) and, with mu [5, width], the blends with the
+    row before → (h [rows, width], mix [5, rows, width] or None).  state fp32 [slots, taps, width] is read only."""
+    rows, width = hn.shape
+    h = torch.empty(rows, width, dtype=dtype, device=hn.device)
+    mix = torch.empty(5, rows, width, dtype=dtype, device=hn.device) if mu is not None else None
+    check(lib().b200_stack_input_conv(h.data_ptr(), _ptr(mix), hn.data_ptr(), w.data_ptr(), _ptr(mu), w.shape[0], state.data_ptr(),
+                                      state.stride(0), slot.data_ptr(), pos.data_ptr(), rows, width, _sdt(h), _stream()),
+          "b200_stack_input_conv")
+    return h, mix
+
+
+def stack_pool_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, max_ctx: int, slot: torch.Tensor,
+                         pos: torch.Tensor, *, heads, kv_heads, dim, vdim, scale, window, pool, softcap: float = 0.0,
+                         sink: Optional[torch.Tensor] = None, talk: Optional[torch.Tensor] = None, splits: int = 1) -> torch.Tensor:
+    """Prepared queries [n_tok, heads·dim] over caches [slots, max_ctx + max_ctx // pool, kv_heads·(dim | vdim)] (token rows, then
+    block rows) → [n_tok, heads·vdim]."""
+    import ctypes as C
+    from ._lib import PoolAttnDesc
+    a = _attn_desc(heads, kv_heads, dim, vdim, scale, window, 0, 0)
+    d = PoolAttnDesc(1, 0, int(pool), float(softcap), None, None, None, None, _ptr(sink), _ptr(talk))
+    out = torch.empty(q.shape[0], heads * vdim, dtype=q.dtype, device=q.device)
+    check(lib().b200_stack_pool_attention(out.data_ptr(), q.data_ptr(), kcache.data_ptr(), vcache.data_ptr(), kcache.stride(0),
+                                          vcache.stride(0), int(max_ctx), slot.data_ptr(), pos.data_ptr(), q.shape[0], C.byref(a),
+                                          C.byref(d), int(splits), _sdt(q), _stream()), "b200_stack_pool_attention")
+    return out
+
+
+def stack_bonus_scan(d: torch.Tensor, k: torch.Tensor, r: torch.Tensor, v: torch.Tensor, bonus: torch.Tensor, state: torch.Tensor,
+                     row0: torch.Tensor, count: torch.Tensor, slot: torch.Tensor, pos: torch.Tensor, *, heads, dk, dv) -> torch.Tensor:
+    """o = Sᵀr + bonus·v with the S from before the token joins it, then S ← (1 + d)∘S + k vᵀ; operands fp32 column slices of one
+    row-major matrix (d [rows, heads·dk] is the decay minus one) → fp32 [rows, heads·dv]."""
+    rows, ld = v.shape[0], v.stride(0)
+    for t in (d, k, r, bonus):
+        if t.dtype != torch.float32 or t.stride(0) != ld or t.stride(1) != 1:
+            raise B200Error("stack_bonus_scan: operands must be fp32 column slices of one row-major matrix")
+    out = torch.zeros(rows, heads * dv, dtype=torch.float32, device=v.device)
+    check(lib().b200_stack_bonus_scan(out.data_ptr(), d.data_ptr(), k.data_ptr(), r.data_ptr(), v.data_ptr(), bonus.data_ptr(), ld, heads,
+                                      dk, dv, state.data_ptr(), state.stride(0), row0.data_ptr(), count.data_ptr(), slot.data_ptr(),
+                                      pos.data_ptr(), row0.shape[0], rows, _stream()), "b200_stack_bonus_scan")
+    return out
+
+
+def stack_mamba1_scan(z: torch.Tensor, xc: torch.Tensor, xd: torch.Tensor, dt: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor,
+                      state: torch.Tensor, row0: torch.Tensor, count: torch.Tensor, slot: torch.Tensor, pos: torch.Tensor, *,
+                      dt_rank: int) -> torch.Tensor:
+    """Selective scan: convolved channels xc and gate logits z [rows, inner], xd fp32 [rows, ·] with B | C from column
+    up8(dt_rank) on, step-size logits dt fp32 [rows, inner], A_log [inner, n], D [inner], state fp32 [slots, inner·n] → z.dtype
+    [rows, inner]."""
+    import ctypes as C
+    from ._lib import Mamba1Desc
+    d = Mamba1Desc(A_log.shape[0], A_log.shape[1], int(dt_rank), 1, None, None, None, None, None, A_log.data_ptr(), D.data_ptr())
+    out = torch.empty_like(z)
+    check(lib().b200_stack_mamba1_scan(out.data_ptr(), z.data_ptr(), xc.data_ptr(), xd.data_ptr(), xd.stride(0), dt.data_ptr(), C.byref(d),
+                                       state.data_ptr(), state.stride(0), row0.data_ptr(), count.data_ptr(), slot.data_ptr(),
+                                       pos.data_ptr(), row0.shape[0], z.shape[0], _sdt(z), _stream()), "b200_stack_mamba1_scan")
+    return out
 
 
 # ---- mechanisms of post-norm blocks (csrc/stack_rec.cu)

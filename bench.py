@@ -690,7 +690,17 @@ def main():
                          "with shared keys / values, latent attention with a query latent, gated delta rule, dense feed-forwards) "
                          "beside the Silatar design with dense feed-forwards of equal width, vocabulary and layer runs (sizes of "
                          "tinygpt_b200/stack_bench.py, or all)")
+    ap.add_argument("--bibezen-compare", nargs="?", const="all", default=None, metavar="SIZES",
+                    help="instead of the headline run: prefill / decode throughput of the Bibezen layer-stack design (hyper-connected "
+                         "blocks, selective scan, time mixing, pooled-block attention with mixed heads, SwiGLU experts) beside the "
+                         "Tekosun design of equal width, vocabulary, layers and expert parameters (sizes of "
+                         "tinygpt_b200/stack_bench.py, or all)")
     args = ap.parse_args()
+    if args.bibezen_compare is not None:
+        from tinygpt_b200 import build, stack_bench
+        build.build()
+        stack_bench.main_bibezen(args.bibezen_compare, steps=max(1, min(args.steps, 10)), warmup=max(3, args.warmup))
+        return
     if args.tarudra_compare is not None:
         from tinygpt_b200 import build, stack_bench
         build.build()

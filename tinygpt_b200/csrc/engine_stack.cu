@@ -919,14 +919,12 @@ static int stack_pool_attention(StackEngine* s, const PoolAttn& p0, cudaStream_t
     }
     return (int)B200_OK;
   };
-  bool any = false;
-  for (const StackEngine::Seg& g : s->segs) any = any || g.count >= kTcRows;
-  if (!any || !s->fast || !pool_prompt_ok(p0.a)) return general(0, p0.n_tok);
-  for (const StackEngine::Seg& g : s->segs) {
-    rc = g.count < kTcRows ? general(g.row0, g.count)
-                           : launch_pool_prompt(rows_from(g.row0, g.count), g.slot, g.count, g.pos0, s->pool_parts, st);
-    if (rc != B200_OK) return rc;
-  }
+  int most = 0;
+  for (const StackEngine::Seg& g : s->segs) most = std::max(most, g.count);
+  if (most < kTcRows || !s->fast || !pool_prompt_ok(p0.a)) return general(0, p0.n_tok);
+  if ((rc = launch_pool_prompt(p0, s->m_seg_row0, s->m_seg_count, (int)s->segs.size(), most, kTcRows, s->pool_parts, st)) != B200_OK) return rc;
+  for (const StackEngine::Seg& g : s->segs)
+    if (g.count < kTcRows && (rc = general(g.row0, g.count)) != B200_OK) return rc;
   return B200_OK;
 }
 

@@ -66,9 +66,59 @@ __device__ __forceinline__ void conv_channel(const InputConv& c, int64_t t, int6
     static_cast<T*>(c.mix)[(s * n_tok + t) * width + i] = cvt<T>(fmaf(hp - h, c.mu[(int64_t)s * width + i], h));
 }
 
+// The same for V neighbouring channels and compile-time taps, from a window n[0 … TAPS] of rows (n[j] = the row j positions back):
+// the row h leaves with is handed out, hp is the row before's (only read with mu).
+template <int TAPS, int V>
+__device__ __forceinline__ void conv_window(const float (&n)[TAPS + 1][V], const float (&w)[TAPS][V], int from, float (&h)[V]) {
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    float a = n[from][k];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+      if (from + j <= TAPS) a = fmaf(w[TAPS - 1 - j][k], n[from + j][k], a);
+    h[k] = a;
+  }
+}
+template <typename T, int V>
+__device__ __forceinline__ void store_conv(const InputConv& c, int64_t t, int64_t n_tok, int width, int i, const float (&h)[V],
+                                           const float (&hp)[V], const float (&mu)[kShiftMixes][V]) {
+  if (c.h != nullptr) Vec<V>::store(static_cast<T*>(c.h) + t * width + i, h);
+  if (c.mu == nullptr) return;
+#pragma unroll
+  for (int s = 0; s < kShiftMixes; ++s) {
+    float m[V];
+#pragma unroll
+    for (int k = 0; k < V; ++k) m[k] = fmaf(hp[k] - h[k], mu[s][k], h[k]);
+    Vec<V>::store(static_cast<T*>(c.mix) + (s * n_tok + t) * width + i, m);
+  }
+}
+// the taps and blend weights of V channels
+template <int TAPS, int V>
+__device__ __forceinline__ void load_conv(const InputConv& c, int width, int i, float (&w)[TAPS][V], float (&mu)[kShiftMixes][V]) {
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) {
+    if (c.w != nullptr) {
+      Vec<V>::load(c.w + (int64_t)j * width + i, w[j]);
+    } else {
+#pragma unroll
+      for (int k = 0; k < V; ++k) w[j][k] = 0.f;
+    }
+  }
+#pragma unroll
+  for (int s = 0; s < kShiftMixes; ++s) {
+    if (c.mu != nullptr) {
+      Vec<V>::load(c.mu + (int64_t)s * width + i, mu[s]);
+    } else {
+#pragma unroll
+      for (int k = 0; k < V; ++k) mu[s][k] = 0.f;
+    }
+  }
+}
+
 // One CTA per row; the row's u sits in shared memory between the sum of squares and the norm (a thread comes back to its own
-// entries, so nothing but the sum crosses threads).
-template <typename T, int S, int V>
+// entries, so nothing but the sum crosses threads).  CT > 0: the convolution's taps, known at compile time (0: any number, or no
+// convolution).
+template <typename T, int S, int V, int CT>
 __global__ void __launch_bounds__(512) hyper_step_kernel(const HyperStep p) {
   pdl_trigger();
   extern __shared__ float u[];
@@ -144,6 +194,29 @@ __global__ void __launch_bounds__(512) hyper_step_kernel(const HyperStep p) {
     if (p.hn != nullptr) Vec<V>::store(p.hn + row + i, n);
     if (!p.conv) continue;
     // the row is its sequence's only new one: earlier rows come from the slot, which moves on at once
+    if constexpr (CT > 0) {
+      float* st = p.c.state + (int64_t)p.slot[t] * p.c.slot_stride + i;
+      const int ps = p.pos[t];
+      float win[CT + 1][V], w[CT][V], mu[kShiftMixes][V], h[V], hp[V];
+#pragma unroll
+      for (int j = 1; j <= CT; ++j) {
+        if (ps - j >= 0) {
+          Vec<V>::load(st + (int64_t)(CT - j) * W, win[j]);
+        } else {
+#pragma unroll
+          for (int k = 0; k < V; ++k) win[j][k] = 0.f;
+        }
+      }
+      load_conv<CT, V>(p.c, W, i, w, mu);
+#pragma unroll
+      for (int k = 0; k < V; ++k) win[0][k] = n[k];
+      conv_window<CT, V>(win, w, 0, h);
+      conv_window<CT, V>(win, w, 1, hp);
+      store_conv<T, V>(p.c, t, p.n_tok, W, i, h, hp, mu);
+#pragma unroll
+      for (int e = 0; e < CT; ++e) Vec<V>::store(st + (int64_t)e * W, win[CT - 1 - e]);
+      continue;
+    }
     float* st = p.c.state + (int64_t)p.slot[t] * p.c.slot_stride;
     const int taps = p.c.taps, ps = p.pos[t];
 #pragma unroll
@@ -191,6 +264,51 @@ __global__ void __launch_bounds__(256) input_conv_kernel(const InputConv c, cons
   conv_channel<T>(c, t, n_tok, width, i, back);
 }
 
+// The same for kConvStrip rows per CTA and V neighbouring channels per thread: while a sequence goes on, the window slides through
+// registers and a row's h is the next row's hp.
+constexpr int kConvStrip = 8;
+template <typename T, int TAPS, int V>
+__global__ void __launch_bounds__(128) input_conv_strip_kernel(const InputConv c, const float* __restrict__ hn, const int32_t* __restrict__ slot,
+                                                               const int32_t* __restrict__ pos, int n_tok, int width) {
+  pdl_trigger();
+  const int t0 = blockIdx.x * kConvStrip, i = (blockIdx.y * 128 + threadIdx.x) * V;
+  const bool live = i < width;
+  float w[TAPS][V], mu[kShiftMixes][V];
+  if (live) load_conv<TAPS, V>(c, width, i, w, mu);
+  pdl_wait();
+  if (!live) return;
+  float win[TAPS + 1][V], h[V], hp[V];
+  const int t1 = min(t0 + kConvStrip, n_tok);
+  for (int t = t0; t < t1; ++t) {
+    if (t == t0 || !row_same_seq(slot, pos, t, 1)) {   // a window of its own: the step's rows in front, then the slot's
+      const int front = rows_in_front(slot, pos, t, TAPS), ps = pos[t];
+      const float* st = c.state + (int64_t)slot[t] * c.slot_stride + i;
+#pragma unroll
+      for (int j = 1; j <= TAPS; ++j) {
+        if (j <= front) {
+          Vec<V>::load(hn + (int64_t)(t - j) * width + i, win[j]);
+        } else if (ps - j >= 0) {
+          Vec<V>::load(st + (int64_t)(TAPS - (j - front)) * width, win[j]);
+        } else {
+#pragma unroll
+          for (int k = 0; k < V; ++k) win[j][k] = 0.f;
+        }
+      }
+      conv_window<TAPS, V>(win, w, 1, hp);
+    } else {
+#pragma unroll
+      for (int j = TAPS; j > 0; --j)
+#pragma unroll
+        for (int k = 0; k < V; ++k) win[j][k] = win[j - 1][k];
+#pragma unroll
+      for (int k = 0; k < V; ++k) hp[k] = h[k];
+    }
+    Vec<V>::load(hn + (int64_t)t * width + i, win[0]);
+    conv_window<TAPS, V>(win, w, 0, h);
+    store_conv<T, V>(c, t, n_tok, width, i, h, hp, mu);
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) shift_state_kernel(const ShiftState p) {
   pdl_trigger();
@@ -218,6 +336,12 @@ __global__ void __launch_bounds__(256) shift_state_kernel(const ShiftState p) {
 #define HYPER_DTYPE_CHECK(dtype) \
   B200_CHECK_ARG((dtype) == B200_BF16 || (dtype) == B200_F32, "stack op: unknown dtype %d", (int)(dtype))
 
+// four neighbouring channels at a time (the caller checks that the width is a multiple of four)
+static bool conv_vec_ok(const InputConv& c) {
+  auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  return al(c.w) && al(c.mu) && al(c.h) && al(c.mix) && al(c.state) && c.slot_stride % 4 == 0;   // null pointers are aligned
+}
+
 int launch_hyper_step(const HyperStep& p, int dtype, cudaStream_t st) {
   HYPER_DTYPE_CHECK(dtype);
   B200_CHECK_ARG(p.x && p.n_tok > 0 && p.width > 0 && p.streams >= 1 && p.streams <= kMaxStreams,
@@ -228,33 +352,39 @@ int launch_hyper_step(const HyperStep& p, int dtype, cudaStream_t st) {
   B200_CHECK_ARG(smem <= 200 * 1024, "hyper step: rows wider than 51200 are not built");
   auto al = [](const void* q, size_t a) { return (reinterpret_cast<uintptr_t>(q) % a) == 0; };
   const bool vec = p.width % 4 == 0 && al(p.x, 16) && (p.y == nullptr || al(p.y, 16)) && (p.h == nullptr || al(p.h, 16)) &&
-                   (p.hn == nullptr || al(p.hn, 16)) && (p.norm_w == nullptr || al(p.norm_w, 16)) && !p.conv;
+                   (p.hn == nullptr || al(p.hn, 16)) && (p.norm_w == nullptr || al(p.norm_w, 16)) &&
+                   (!p.conv || (conv_vec_ok(p.c) && p.c.taps <= 4));
   // few rows: as many threads as there are entries, one round of loads; many rows: 256 threads
   const int items = vec ? p.width / 4 : p.width;
   const int threads = p.n_tok <= 148 && items > 256 ? 512 : 256;
-#define B200_HS(T, S, V)                                                                                            \
+#define B200_HS(T, S, V, CT)                                                                                            \
   do {                                                                                                              \
     static bool attr_done = false;                                                                                  \
     if (smem > 40 * 1024 && !attr_done) {                                                                           \
-      B200_CUDA(cudaFuncSetAttribute(hyper_step_kernel<T, S, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); \
+      B200_CUDA(cudaFuncSetAttribute(hyper_step_kernel<T, S, V, CT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); \
       attr_done = true;                                                                                             \
     }                                                                                                               \
-    B200_CUDA(launch_pdl(hyper_step_kernel<T, S, V>, dim3(p.n_tok), dim3(threads), smem, st, stack_pdl(), p));       \
+    B200_CUDA(launch_pdl(hyper_step_kernel<T, S, V, CT>, dim3(p.n_tok), dim3(threads), smem, st, stack_pdl(), p));       \
   } while (0)
-#define B200_HS_S(T, V)                        \
-  do {                                         \
-    if (p.streams == 1) B200_HS(T, 1, V);      \
-    else if (p.streams == 2) B200_HS(T, 2, V); \
-    else if (p.streams <= 4) B200_HS(T, 4, V); \
-    else B200_HS(T, 8, V);                     \
+#define B200_HS_S(T, V, CT)                        \
+  do {                                             \
+    if (p.streams == 1) B200_HS(T, 1, V, CT);      \
+    else if (p.streams == 2) B200_HS(T, 2, V, CT); \
+    else if (p.streams <= 4) B200_HS(T, 4, V, CT); \
+    else B200_HS(T, 8, V, CT);                     \
   } while (0)
-  if (dtype == B200_F32) {
-    if (vec) B200_HS_S(float, 4);
-    else B200_HS_S(float, 1);
-  } else {
-    if (vec) B200_HS_S(__nv_bfloat16, 4);
-    else B200_HS_S(__nv_bfloat16, 1);
-  }
+#define B200_HS_T(T)                                \
+  do {                                              \
+    if (!vec) B200_HS_S(T, 1, 0);                   \
+    else if (!p.conv) B200_HS_S(T, 4, 0);           \
+    else if (p.c.taps == 1) B200_HS_S(T, 4, 1);     \
+    else if (p.c.taps == 2) B200_HS_S(T, 4, 2);     \
+    else if (p.c.taps == 3) B200_HS_S(T, 4, 3);     \
+    else B200_HS_S(T, 4, 4);                        \
+  } while (0)
+  if (dtype == B200_F32) B200_HS_T(float);
+  else B200_HS_T(__nv_bfloat16);
+#undef B200_HS_T
 #undef B200_HS_S
 #undef B200_HS
   return B200_OK;
@@ -279,6 +409,22 @@ int launch_input_conv(const InputConv& c, const float* hn, const int32_t* slot, 
   B200_CHECK_ARG(hn && slot && pos && c.state && n_tok > 0 && width > 0 && c.taps >= 1 && c.taps <= kConvMaxTaps && (c.h || c.mix) &&
                      (c.mu == nullptr || c.mix),
                  "input convolution: bad arguments (1 … %d taps)", kConvMaxTaps);
+  if (width % 4 == 0 && c.taps <= 4 && conv_vec_ok(c) && (reinterpret_cast<uintptr_t>(hn) & 15) == 0) {
+    const dim3 grid((n_tok + kConvStrip - 1) / kConvStrip, (width / 4 + 127) / 128);
+#define B200_IC(T, TAPS) B200_CUDA(launch_pdl(input_conv_strip_kernel<T, TAPS, 4>, grid, dim3(128), 0, st, stack_pdl(), c, hn, slot, pos, n_tok, width))
+#define B200_IC_T(T)                    \
+  do {                                  \
+    if (c.taps == 1) B200_IC(T, 1);     \
+    else if (c.taps == 2) B200_IC(T, 2); \
+    else if (c.taps == 3) B200_IC(T, 3); \
+    else B200_IC(T, 4);                 \
+  } while (0)
+    if (dtype == B200_F32) B200_IC_T(float);
+    else B200_IC_T(__nv_bfloat16);
+#undef B200_IC_T
+#undef B200_IC
+    return B200_OK;
+  }
   const dim3 grid(n_tok, (width + 255) / 256);
   if (dtype == B200_F32) B200_CUDA(launch_pdl(input_conv_kernel<float>, grid, dim3(256), 0, st, stack_pdl(), c, hn, slot, pos, n_tok, width));
   else B200_CUDA(launch_pdl(input_conv_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, stack_pdl(), c, hn, slot, pos, n_tok, width));

@@ -154,6 +154,34 @@ __global__ void __launch_bounds__(256) stack_glu_kernel(T* __restrict__ y, int64
   }
 }
 
+__device__ __forceinline__ void load_run8(const __nv_bfloat16* p, float (&v)[8]) { unpack8(*reinterpret_cast<const uint4*>(p), v); }
+__device__ __forceinline__ void load_run8(const float* p, float (&v)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void store_run8(__nv_bfloat16* p, const float (&v)[8]) {
+  *reinterpret_cast<uint4*>(p) = make_uint4(pack2(v[0], v[1]), pack2(v[2], v[3]), pack2(v[4], v[5]), pack2(v[6], v[7]));
+}
+__device__ __forceinline__ void store_run8(float* p, const float (&v)[8]) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+// silu, eight entries per thread (rows and n on multiples of eight)
+template <typename T>
+__global__ void __launch_bounds__(256) stack_swiglu8_kernel(T* __restrict__ y, int64_t ld_y, const T* __restrict__ gu, int64_t ld_gu, int n) {
+  pdl_trigger();
+  pdl_wait();
+  const int64_t r = blockIdx.x;
+  const int j = (blockIdx.y * 256 + threadIdx.x) * 8;
+  if (j >= n) return;
+  float g[8], u[8];
+  load_run8(gu + r * ld_gu + j, g);
+  load_run8(gu + r * ld_gu + n + j, u);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) g[i] = g[i] / (1.f + expf(-g[i])) * u[i];
+  store_run8(y + r * ld_y + j, g);
+}
+
 __global__ void __launch_bounds__(256) stack_softcap_kernel(float* __restrict__ lg, __nv_bfloat16* __restrict__ lb,
                                                             int64_t total, float cap) {
   pdl_trigger();
@@ -352,32 +380,72 @@ template <> __device__ __forceinline__ void load8<float>(const float* p, float (
   v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
 }
 
-// One warp per output row n of item blockIdx.y.  VEC: 16-byte (bf16) / 32-byte (fp32) pieces of the matrix row and of
-// the M activation rows, lane l takes pieces l, l + 32, …; otherwise element by element.
-template <typename T, bool VEC>
+// eight consecutive elements as they lie in memory
+template <typename T> struct Raw8;
+template <> struct Raw8<__nv_bfloat16> {
+  uint4 a;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { a = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void clear() { a = make_uint4(0, 0, 0, 0); }
+  __device__ __forceinline__ void get(float (&v)[8]) const { unpack8(a, v); }
+};
+template <> struct Raw8<float> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) {
+    a = *reinterpret_cast<const float4*>(p);
+    b = *reinterpret_cast<const float4*>(p + 4);
+  }
+  __device__ __forceinline__ void clear() { a = b = make_float4(0.f, 0.f, 0.f, 0.f); }
+  __device__ __forceinline__ void get(float (&v)[8]) const {
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+  }
+};
+
+// One warp per output row n of item blockIdx.y, up to MB activation rows.  VEC: 16-byte (bf16) / 32-byte (fp32) pieces of the
+// matrix row and of the activation rows, lane l takes pieces l, l + 32, …, kPieces of the matrix row requested together — the
+// first ones ahead of the dependency wait where the matrix is a constant of the model; otherwise element by element.
+template <typename T, bool VEC, int MB>
 __global__ void __launch_bounds__(256) small_gemv_kernel(const SmallGemv g) {
   pdl_trigger();
-  pdl_wait();
+  constexpr int kPieces = MB == 1 ? 8 : 4;
   const int n = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, z = blockIdx.y;
+  const bool ahead = VEC && g.w_const && g.item_mat == nullptr && n < g.N;
+  Raw8<T> wq[kPieces];
+  const int pieces = g.K >> 3;
+  auto fetch = [&](const T* wr, int p0) {
+#pragma unroll
+    for (int u = 0; u < kPieces; ++u) {
+      const int p = p0 + u * 32 + lane;
+      if (p < pieces) wq[u].load(wr + p * 8);
+      else wq[u].clear();
+    }
+  };
+  if (ahead) fetch(static_cast<const T*>(g.w) + (int64_t)z * g.sw + (int64_t)n * g.K, 0);
+  pdl_wait();
   if (n >= g.N) return;
   const int64_t mat = g.item_mat != nullptr ? g.item_mat[z] : z;
   const T* wr = static_cast<const T*>(g.w) + mat * g.sw + (int64_t)n * g.K;
   const T* a = static_cast<const T*>(g.a) + (int64_t)(z / g.item_div) * g.sa;
   const int M = g.m_total > 0 ? min(g.M, g.m_total - z * g.M) : g.M;
-  float acc[kSmallRows];
+  float acc[MB];
 #pragma unroll
-  for (int m = 0; m < kSmallRows; ++m) acc[m] = 0.f;
+  for (int m = 0; m < MB; ++m) acc[m] = 0.f;
   if constexpr (VEC) {
-    for (int k = lane * 8; k < g.K; k += 256) {
-      float wv[8];
-      load8<T>(wr + k, wv);
+    for (int p0 = 0; p0 < pieces; p0 += 32 * kPieces) {
+      if (p0 > 0 || !ahead) fetch(wr, p0);
 #pragma unroll
-      for (int m = 0; m < kSmallRows; ++m) {
-        if (m < M) {
-          float av[8];
-          load8<T>(a + (int64_t)m * g.lda + k, av);
+      for (int u = 0; u < kPieces; ++u) {
+        const int p = p0 + u * 32 + lane;
+        if (p >= pieces) break;
+        float wv[8];
+        wq[u].get(wv);
 #pragma unroll
-          for (int i = 0; i < 8; ++i) acc[m] = fmaf(wv[i], av[i], acc[m]);
+        for (int m = 0; m < MB; ++m) {
+          if (m < M) {
+            float av[8];
+            load8<T>(a + (int64_t)m * g.lda + p * 8, av);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) acc[m] = fmaf(wv[i], av[i], acc[m]);
+          }
         }
       }
     }
@@ -385,12 +453,12 @@ __global__ void __launch_bounds__(256) small_gemv_kernel(const SmallGemv g) {
     for (int k = lane; k < g.K; k += 32) {
       const float wv = ldf<T>(wr + k);
 #pragma unroll
-      for (int m = 0; m < kSmallRows; ++m)
+      for (int m = 0; m < MB; ++m)
         if (m < M) acc[m] = fmaf(wv, ldf<T>(a + (int64_t)m * g.lda + k), acc[m]);
     }
   }
 #pragma unroll
-  for (int m = 0; m < kSmallRows; ++m) {
+  for (int m = 0; m < MB; ++m) {
     if (m >= M) break;
     float v = warp_sum(acc[m]);
     if (lane == 0) {
@@ -854,6 +922,12 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const MoeRun p) {
   const float w = p.m.weight_output ? 1.f : p.sel_w[pair];
   const T* src = static_cast<const T*>(p.h) + (int64_t)t * p.width;
   T* dst = static_cast<T*>(p.a_perm) + (int64_t)p.pair_slot[pair] * p.width;
+  constexpr int kRun = 16 / sizeof(T);
+  if (p.m.weight_output && p.width % kRun == 0 && ((reinterpret_cast<uintptr_t>(p.h) | reinterpret_cast<uintptr_t>(p.a_perm)) & 15) == 0) {
+    for (int i = threadIdx.x; i < p.width / kRun; i += blockDim.x)   // plain copies
+      reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
+    return;
+  }
   for (int i = threadIdx.x; i < p.width; i += blockDim.x) dst[i] = cvt<T>(w * ldf<T>(src + i));
 }
 
@@ -878,6 +952,38 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const MoeRun p) {
     v += gate * (p.shared_f32 ? static_cast<const float*>(p.shared)[o] : ldf<T>(static_cast<const T*>(p.shared) + o));
   }
   p.y[(int64_t)t * p.width + i] = v;
+}
+
+// The same, four neighbouring columns per thread, without a gate on the shared expert.
+__global__ void __launch_bounds__(256) moe_combine4_kernel(const MoeRun p) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, top = p.m.top, i = (blockIdx.y * 256 + threadIdx.x) * 4;
+  if (i >= p.width) return;
+  const int32_t* slots = p.pair_slot + (int64_t)t * top;
+  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int k = 0; k < top; ++k) {
+    const int64_t o = (int64_t)slots[k] * p.width + i;
+    float4 ov;
+    if (p.tc) {
+      const uint2 b = *reinterpret_cast<const uint2*>(p.outp_bf + o);
+      ov = make_float4(bf16_lo(b.x), bf16_hi(b.x), bf16_lo(b.y), bf16_hi(b.y));
+    } else {
+      ov = *reinterpret_cast<const float4*>(p.outp + o);
+    }
+    if (p.m.weight_output) {
+      const float w = p.sel_w[(int64_t)t * top + k];
+      v = make_float4(fmaf(w, ov.x, v.x), fmaf(w, ov.y, v.y), fmaf(w, ov.z, v.z), fmaf(w, ov.w, v.w));
+    } else {
+      v = make_float4(v.x + ov.x, v.y + ov.y, v.z + ov.z, v.w + ov.w);
+    }
+  }
+  const int64_t o = (int64_t)t * p.width + i;
+  if (p.shared != nullptr) {
+    const float4 s = *reinterpret_cast<const float4*>(static_cast<const float*>(p.shared) + o);
+    v = make_float4(v.x + s.x, v.y + s.y, v.z + s.z, v.w + s.w);
+  }
+  *reinterpret_cast<float4*>(p.y + o) = v;
 }
 
 }  // namespace
@@ -956,6 +1062,16 @@ int launch_stack_glu(void* y, int64_t ld_y, const void* gu, int64_t ld_gu, int64
   MIX_DTYPE_CHECK(dtype);
   B200_CHECK_ARG(y && gu && rows > 0 && n > 0 && act >= B200_ACT_GELU_TANH && act <= B200_ACT_TANH, "stack glu: bad arguments");
   const int64_t total = rows * n;
+  if (act == B200_ACT_SILU && n % 8 == 0 && ld_y % 8 == 0 && ld_gu % 8 == 0 && (reinterpret_cast<uintptr_t>(y) & 15) == 0 &&
+      (reinterpret_cast<uintptr_t>(gu) & 15) == 0) {
+    const dim3 vg((unsigned)rows, (n / 8 + 255) / 256);
+    if (dtype == B200_F32)
+      B200_CUDA(launch_pdl(stack_swiglu8_kernel<float>, vg, dim3(256), 0, st, stack_pdl(), (float*)y, ld_y, (const float*)gu, ld_gu, n));
+    else
+      B200_CUDA(launch_pdl(stack_swiglu8_kernel<__nv_bfloat16>, vg, dim3(256), 0, st, stack_pdl(), (__nv_bfloat16*)y, ld_y,
+                           (const __nv_bfloat16*)gu, ld_gu, n));
+    return B200_OK;
+  }
   if (dtype == B200_F32)
     B200_CUDA(launch_pdl(stack_glu_kernel<float>, dim3(grid_cap(total, 256)), dim3(256), 0, st, stack_pdl(), (float*)y, ld_y,
                          (const float*)gu, ld_gu, n, act, total));
@@ -981,13 +1097,21 @@ int launch_small_gemv(const SmallGemv& g, int dtype, cudaStream_t st) {
   const bool vec = g.K % 8 == 0 && (reinterpret_cast<uintptr_t>(g.a) % al) == 0 && (reinterpret_cast<uintptr_t>(g.w) % al) == 0 &&
                    (g.lda * esz) % al == 0 && (g.sa * esz) % al == 0 && (g.sw * esz) % al == 0;
   const dim3 grid((g.N + 7) / 8, g.items);
+#define B200_SG(T, VEC)                                                                                                      \
+  do {                                                                                                                       \
+    if (g.M == 1) B200_CUDA(launch_pdl(small_gemv_kernel<T, VEC, 1>, grid, dim3(256), 0, st, stack_pdl(), g));                \
+    else if (g.M <= 2) B200_CUDA(launch_pdl(small_gemv_kernel<T, VEC, 2>, grid, dim3(256), 0, st, stack_pdl(), g));           \
+    else if (g.M <= 4) B200_CUDA(launch_pdl(small_gemv_kernel<T, VEC, 4>, grid, dim3(256), 0, st, stack_pdl(), g));           \
+    else B200_CUDA(launch_pdl(small_gemv_kernel<T, VEC, kSmallRows>, grid, dim3(256), 0, st, stack_pdl(), g));                \
+  } while (0)
   if (dtype == B200_F32) {
-    if (vec) B200_CUDA(launch_pdl(small_gemv_kernel<float, true>, grid, dim3(256), 0, st, stack_pdl(), g));
-    else B200_CUDA(launch_pdl(small_gemv_kernel<float, false>, grid, dim3(256), 0, st, stack_pdl(), g));
+    if (vec) B200_SG(float, true);
+    else B200_SG(float, false);
   } else {
-    if (vec) B200_CUDA(launch_pdl(small_gemv_kernel<__nv_bfloat16, true>, grid, dim3(256), 0, st, stack_pdl(), g));
-    else B200_CUDA(launch_pdl(small_gemv_kernel<__nv_bfloat16, false>, grid, dim3(256), 0, st, stack_pdl(), g));
+    if (vec) B200_SG(__nv_bfloat16, true);
+    else B200_SG(__nv_bfloat16, false);
   }
+#undef B200_SG
   return B200_OK;
 }
 
@@ -998,7 +1122,7 @@ int launch_skinny_f32(float* C, const void* A, const void* W, const float* bias,
   g.w = A; g.sw = 0;
   g.c = C; g.ldc = 1; g.sc = kSmallRows; g.nc = n; g.c_f32 = true;
   g.M = kSmallRows; g.m_total = n; g.N = rows; g.K = K; g.items = (n + kSmallRows - 1) / kSmallRows;
-  g.bias_m = bias;
+  g.bias_m = bias; g.w_const = false;   // the "matrix" is what the step before has just written
   return launch_small_gemv(g, dtype, st);
 }
 
@@ -1285,6 +1409,11 @@ int run_moe(const MoeRun& p, int dtype, cudaStream_t st) {
   d.tile_group = g.tile_group; d.tile_row0 = g.tile_row0; d.group_end = g.group_end; d.n_tiles = n_tiles;
   if ((rc = launch_stack_gemm(d, dtype, st)) != B200_OK) return rc;
   }
+  }
+  auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  if (p.width % 4 == 0 && (p.shared == nullptr || (m.shared_plain && p.shared_f32)) && al16(p.outp) && al16(p.outp_bf) && al16(p.shared) && al16(p.y)) {
+    B200_CUDA(launch_pdl(moe_combine4_kernel, dim3(p.n_tok, (p.width / 4 + 255) / 256), dim3(256), 0, st, stack_pdl(), p));
+    return B200_OK;
   }
   const dim3 cg(p.n_tok, (p.width + 255) / 256);
   if (dtype == B200_F32) B200_CUDA(launch_pdl(moe_combine_kernel<float>, cg, dim3(256), 0, st, stack_pdl(), p));

@@ -50,6 +50,7 @@ struct SmallGemv {
   int64_t nc = 1;                // stride of the output row index n inside c
   int m_total = 0;               // > 0: item z has min(M, m_total − z·M) rows (the last item may be short)
   const float* bias_m = nullptr; // [m_total]: bias of row z·M + m
+  bool w_const = true;           // w is a weight of the model: readable ahead of the kernel before this one
   int act = -1;                  // B200_ACT_RELU2 / _TANH / _SILU: applied to the fp32 sum (+ bias) before it is stored
 };
 int launch_small_gemv(const SmallGemv& g, int dtype, cudaStream_t st);

@@ -17,6 +17,45 @@ template <typename T> __device__ __forceinline__ T cvt(float v);
 template <> __device__ __forceinline__ float cvt<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 cvt<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
+// One warp: the norm of one head's convolved channels x (query head g·per + hh, or hh == per: key head g), the turn of its first
+// rot_dims entries, and the row it leaves: q, or the cache row.  A key's entries stay in x as the cache holds them.
+template <typename T>
+__device__ __forceinline__ void finish_head(const PoolAttn& p, int t, int ps, int g, int hh, float* x, T* kc, int lane) {
+  const int H = p.a.heads, G = p.a.kv_heads, dk = p.a.dim, per = H / G, half = p.d.rot_dims / 2;
+  const float* tab = half > 0 ? p.d.rot_table + (int64_t)ps * half * 2 : nullptr;
+  const float* w = hh < per ? p.d.q_norm : p.d.k_norm;
+  float inv = 1.f;
+  if (p.d.q_norm != nullptr) {
+    float ss = 0.f;
+    for (int i = lane; i < dk; i += 32) ss += x[i] * x[i];
+    inv = 1.f / sqrtf(warp_sum(ss) / (float)dk + p.eps);
+  }
+  T* dst = hh < per ? static_cast<T*>(p.q) + ((int64_t)t * H + g * per + hh) * dk : kc + ((int64_t)ps * G + g) * dk;
+  for (int i = lane; i < dk - half; i += 32) {   // half pairs, then the entries that do not turn
+    if (i < half) {
+      float u = x[i] * inv, v = x[i + half] * inv;
+      if (p.d.q_norm != nullptr) {
+        u *= w[i];
+        v *= w[i + half];
+      }
+      const float c = tab[2 * i], s = tab[2 * i + 1];
+      const T a = cvt<T>(u * c - v * s), b = cvt<T>(v * c + u * s);
+      dst[i] = a;
+      dst[i + half] = b;
+      if (hh == per) {
+        x[i] = ldf<T>(&a);
+        x[i + half] = ldf<T>(&b);
+      }
+    } else {
+      float u = x[i + half] * inv;
+      if (p.d.q_norm != nullptr) u *= w[i + half];
+      const T a = cvt<T>(u);
+      dst[i + half] = a;
+      if (hh == per) x[i + half] = ldf<T>(&a);
+    }
+  }
+}
+
 // One CTA per (token, key/value head g): the channels of the query heads that read g, of key head g and of value head g.  The
 // convolution of every channel goes to shared memory; then one warp per query / key head takes the head's norm and turns
 // its first rot_dims entries.  Queries leave for q, keys and values for the slot's cache rows.
@@ -50,44 +89,9 @@ __global__ void __launch_bounds__(256) pool_prep_kernel(const PoolAttn p) {
     sm[e] = acc;
   }
   __syncthreads();
-  const int half = p.d.rot_dims / 2;
-  const float* tab = half > 0 ? p.d.rot_table + (int64_t)ps * half * 2 : nullptr;
   T* kc = static_cast<T*>(p.kcache) + (int64_t)p.slot[t] * p.k_slot_stride;
   T* vc = static_cast<T*>(p.vcache) + (int64_t)p.slot[t] * p.v_slot_stride;
-  for (int hh = warp; hh <= per; hh += 8) {   // hh < per: query head g·per + hh; per: the key head
-    float* x = sm + hh * dk;
-    const float* w = hh < per ? p.d.q_norm : p.d.k_norm;
-    float inv = 1.f;
-    if (p.d.q_norm != nullptr) {
-      float ss = 0.f;
-      for (int i = lane; i < dk; i += 32) ss += x[i] * x[i];
-      inv = 1.f / sqrtf(warp_sum(ss) / (float)dk + p.eps);
-    }
-    T* dst = hh < per ? static_cast<T*>(p.q) + ((int64_t)t * H + g * per + hh) * dk : kc + ((int64_t)ps * G + g) * dk;
-    for (int i = lane; i < dk - half; i += 32) {   // half pairs, then the entries that do not turn
-      if (i < half) {
-        float u = x[i] * inv, v = x[i + half] * inv;
-        if (p.d.q_norm != nullptr) {
-          u *= w[i];
-          v *= w[i + half];
-        }
-        const float c = tab[2 * i], s = tab[2 * i + 1];
-        const T a = cvt<T>(u * c - v * s), b = cvt<T>(v * c + u * s);
-        dst[i] = a;
-        dst[i + half] = b;
-        if (hh == per) {   // what the block mean below reads: the key as the cache holds it
-          x[i] = ldf<T>(&a);
-          x[i + half] = ldf<T>(&b);
-        }
-      } else {
-        float u = x[i + half] * inv;
-        if (p.d.q_norm != nullptr) u *= w[i + half];
-        const T a = cvt<T>(u);
-        dst[i + half] = a;
-        if (hh == per) x[i + half] = ldf<T>(&a);
-      }
-    }
-  }
+  for (int hh = warp; hh <= per; hh += 8) finish_head<T>(p, t, ps, g, hh, sm + hh * dk, kc, lane);
   float* v = sm + nq + dk;
   for (int i = tid; i < dv; i += 256) {
     const T a = cvt<T>(v[i]);
@@ -109,6 +113,53 @@ __global__ void __launch_bounds__(256) pool_prep_kernel(const PoolAttn p) {
   }
 }
 
+// Prompts: kPrepStrip tokens per CTA; while a sequence goes on, a channel's window slides through registers.
+constexpr int kPrepStrip = 8;
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256) pool_prep_strip_kernel(const PoolAttn p) {
+  pdl_trigger();
+  extern __shared__ float sm[];   // [kPrepStrip][per·dk: q | dk: k | dv: v]
+  const int t0 = blockIdx.x * kPrepStrip, g = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int H = p.a.heads, G = p.a.kv_heads, dk = p.a.dim, dv = p.a.vdim, per = H / G;
+  const int nq = per * dk, mine = nq + dk + dv, n = min(kPrepStrip, p.n_tok - t0);
+  pdl_wait();
+  for (int e = tid; e < mine; e += 256) {
+    const int col = e < nq ? p.off_q + g * nq + e : e < nq + dk ? p.off_k + g * dk + (e - nq) : p.off_v + g * dv + (e - nq - dk);
+    const T* x = static_cast<const T*>(p.proj) + (int64_t)t0 * p.ld_proj + col;
+    float w[TAPS], win[TAPS];   // win[j]: the row j positions back
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j] = p.d.conv_w[(int64_t)j * p.ld_proj + col];
+    for (int r = 0; r < n; ++r) {
+      const int t = t0 + r;
+      if (r == 0 || !row_same_seq(p.slot, p.pos, t, 1)) {
+        const int front = rows_in_front(p.slot, p.pos, t, TAPS - 1), ps = p.pos[t];
+        const float* cs = p.conv_state + (int64_t)p.slot[t] * p.conv_slot_stride + col;
+#pragma unroll
+        for (int j = 1; j < TAPS; ++j)
+          win[j] = j <= front ? ldf<T>(x + (int64_t)(r - j) * p.ld_proj) : ps - j >= 0 ? cs[(int64_t)(TAPS - 1 - (j - front)) * p.ld_proj] : 0.f;
+      } else {
+#pragma unroll
+        for (int j = TAPS - 1; j > 0; --j) win[j] = win[j - 1];
+      }
+      win[0] = ldf<T>(x + (int64_t)r * p.ld_proj);
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) acc = fmaf(w[TAPS - 1 - j], win[j], acc);
+      sm[r * mine + e] = acc;
+    }
+  }
+  __syncthreads();
+  for (int u = warp; u < n * (per + 1); u += 8) {
+    const int r = u / (per + 1), hh = u % (per + 1), t = t0 + r;
+    finish_head<T>(p, t, p.pos[t], g, hh, sm + r * mine + hh * dk, static_cast<T*>(p.kcache) + (int64_t)p.slot[t] * p.k_slot_stride, lane);
+  }
+  for (int r = warp; r < n; r += 8) {
+    const int t = t0 + r;
+    T* vd = static_cast<T*>(p.vcache) + (int64_t)p.slot[t] * p.v_slot_stride + ((int64_t)p.pos[t] * G + g) * dv;
+    for (int i = lane; i < dv; i += 32) vd[i] = cvt<T>(sm[r * mine + nq + dk + i]);
+  }
+}
+
 // Rows whose position ends a block: the means of the block's cached keys and values (rows of this step or of earlier ones).
 template <typename T>
 __global__ void __launch_bounds__(256) pool_blocks_kernel(const PoolAttn p) {
@@ -116,18 +167,15 @@ __global__ void __launch_bounds__(256) pool_blocks_kernel(const PoolAttn p) {
   pdl_wait();
   const int t = blockIdx.x, P = p.d.pool, ps = p.pos[t];
   if ((ps + 1) % P != 0) return;
-  const int b = ps / P, nk = p.a.kv_heads * p.a.dim, nv = p.a.kv_heads * p.a.vdim;
-  T* kc = static_cast<T*>(p.kcache) + (int64_t)p.slot[t] * p.k_slot_stride;
-  T* vc = static_cast<T*>(p.vcache) + (int64_t)p.slot[t] * p.v_slot_stride;
-  const float inv = 1.f / (float)P;
-  for (int e = threadIdx.x; e < nk + nv; e += 256) {
-    const bool key = e < nk;
-    const int n = key ? nk : nv, i = key ? e : e - nk;
-    T* c = key ? kc : vc;
-    float s = 0.f;
-    for (int j = 0; j < P; ++j) s += ldf<T>(c + (int64_t)(b * P + j) * n + i);
-    c[(int64_t)(p.max_ctx + b) * n + i] = cvt<T>(s * inv);
-  }
+  const int b = ps / P, nk = p.a.kv_heads * p.a.dim, nv = p.a.kv_heads * p.a.vdim, e = blockIdx.y * 256 + threadIdx.x;
+  if (e >= nk + nv) return;
+  const bool key = e < nk;
+  const int n = key ? nk : nv, i = key ? e : e - nk;
+  T* c = key ? static_cast<T*>(p.kcache) + (int64_t)p.slot[t] * p.k_slot_stride : static_cast<T*>(p.vcache) + (int64_t)p.slot[t] * p.v_slot_stride;
+  float s = 0.f;
+#pragma unroll 8
+  for (int j = 0; j < P; ++j) s += ldf<T>(c + (int64_t)(b * P + j) * n + i);
+  c[(int64_t)(p.max_ctx + b) * n + i] = cvt<T>(s * (1.f / (float)P));
 }
 
 __device__ __forceinline__ float capped(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
@@ -367,6 +415,22 @@ int launch_pool_prep(const PoolAttn& p, int dtype, cudaStream_t st) {
                  "pool attention: 1 … %d convolution taps with a state", kConvMaxTaps);
   const size_t smem = (size_t)((p.a.heads / p.a.kv_heads + 1) * p.a.dim + p.a.vdim) * 4;
   B200_CHECK_ARG(smem <= 48 * 1024, "pool attention: the heads that share one key/value head exceed 12288 channels");
+  if (!p.single && p.n_tok > kPrepStrip && p.d.conv_w != nullptr && p.d.taps <= 4 && kPrepStrip * smem <= 48 * 1024) {
+    const dim3 sg((p.n_tok + kPrepStrip - 1) / kPrepStrip, p.a.kv_heads);
+#define B200_PP(T, TAPS) B200_CUDA(launch_pdl(pool_prep_strip_kernel<T, TAPS>, sg, dim3(256), kPrepStrip * smem, st, stack_pdl(), p))
+#define B200_PP_T(T)                    \
+  do {                                  \
+    if (p.d.taps == 1) B200_PP(T, 1);   \
+    else if (p.d.taps == 2) B200_PP(T, 2); \
+    else if (p.d.taps == 3) B200_PP(T, 3); \
+    else B200_PP(T, 4);                 \
+  } while (0)
+    if (dtype == B200_F32) B200_PP_T(float);
+    else B200_PP_T(__nv_bfloat16);
+#undef B200_PP_T
+#undef B200_PP
+    return B200_OK;
+  }
   const dim3 grid(p.n_tok, p.a.kv_heads);
   if (dtype == B200_F32) B200_CUDA(launch_pdl(pool_prep_kernel<float>, grid, dim3(256), smem, st, stack_pdl(), p));
   else B200_CUDA(launch_pdl(pool_prep_kernel<__nv_bfloat16>, grid, dim3(256), smem, st, stack_pdl(), p));
@@ -378,8 +442,9 @@ int launch_pool_blocks(const PoolAttn& p, int dtype, cudaStream_t st) {
   int rc = check_pool(p);
   if (rc != B200_OK) return rc;
   if (p.d.pool <= 0) return B200_OK;
-  if (dtype == B200_F32) B200_CUDA(launch_pdl(pool_blocks_kernel<float>, dim3(p.n_tok), dim3(256), 0, st, stack_pdl(), p));
-  else B200_CUDA(launch_pdl(pool_blocks_kernel<__nv_bfloat16>, dim3(p.n_tok), dim3(256), 0, st, stack_pdl(), p));
+  const dim3 bg(p.n_tok, (p.a.kv_heads * (p.a.dim + p.a.vdim) + 255) / 256);
+  if (dtype == B200_F32) B200_CUDA(launch_pdl(pool_blocks_kernel<float>, bg, dim3(256), 0, st, stack_pdl(), p));
+  else B200_CUDA(launch_pdl(pool_blocks_kernel<__nv_bfloat16>, bg, dim3(256), 0, st, stack_pdl(), p));
   return B200_OK;
 }
 

@@ -54,11 +54,13 @@ inline int pool_keys_max(int ctx, int window, int pool) {
 int launch_pool_prep(const PoolAttn& p, int dtype, cudaStream_t st);      // queries, cache rows, (single: blocks, state)
 int launch_pool_blocks(const PoolAttn& p, int dtype, cudaStream_t st);    // the blocks that end in this step's rows
 int launch_pool_attention(const PoolAttn& p, int dtype, cudaStream_t st); // any shape
-// bf16 prompts on the tensor cores (stack_pool_mma.cu), `count` rows of the sequence in `slot` from position pos0 on (q and mid at
-// its first row); stats: fp32 [count][heads][2].  pool_prompt_ok: head sizes that are multiples of 16 (dim <= 128, vdim <= 256),
-// up to 32 heads, and queries and one key / value tile of all heads fit one CTA's shared memory.
+// bf16 prompts on the tensor cores (stack_pool_mma.cu): the sequences [seg_row0, + seg_count) of the step (device arrays) that bring
+// min_rows rows or more, max_count the most any of them brings; stats: fp32 [n_tok][heads][2].  pool_prompt_ok: head sizes that
+// are multiples of 16 (dim <= 128, vdim <= 256), up to 32 heads, and the queries and one key / value tile of all heads fit one
+// CTA's shared memory.
 bool pool_prompt_ok(const b200_attn_desc& a);
-int launch_pool_prompt(const PoolAttn& p, int slot, int count, int pos0, float* stats, cudaStream_t st);
+int launch_pool_prompt(const PoolAttn& p, const int32_t* seg_row0, const int32_t* seg_count, int n_seg, int max_count, int min_rows,
+                       float* stats, cudaStream_t st);
 
 #ifdef __CUDACC__
 __device__ __forceinline__ int pool_lo(int i, int window) { return window > 0 ? max(0, i - window + 1) : 0; }

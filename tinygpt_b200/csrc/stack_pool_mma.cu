@@ -1,5 +1,5 @@
 // stack_pool_mma.cu — prompts of the pooled-block attention on the tensor cores (mma.sync m16n8k16 bf16, fp32 accumulate), for
-// ONE sequence's rows of a step.  Mixing the heads' softmax weights needs every head's finished weights for the same
+// all sequences of a step that bring enough rows (one grid layer each).  Mixing the heads' softmax weights needs every head's finished weights for the same
 // (query, key), so the attention runs in two kernels:
 //   pool_stats_kernel   one CTA per (64 query rows, head): the capped scores of all visible keys, online → the row's maximum
 //                       and the reciprocal of its denominator (the sink included)
@@ -45,6 +45,17 @@ __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], 
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
+__device__ __forceinline__ float ex2(float x) {   // relative error about 2^-22; 2^(−inf) = 0
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 // A raw dot product → the capped score times log2(e).  cap·tanh(z) as cap·(1 − 2 / (1 + e^(2z))): an absolute error of about
 // 1e-7·cap, which is what the softmax sees.
 struct ScoreMap {
@@ -52,18 +63,33 @@ struct ScoreMap {
 };
 __device__ __forceinline__ float map_score(float s, const ScoreMap& m) {
   if (m.in == 0.f) return s * m.out;
-  const float e = exp2f(fminf(s * m.in, 126.f));
-  return m.out * (1.f - __fdividef(2.f, 1.f + e));
+  const float e = ex2(fminf(s * m.in, 126.f));
+  return fmaf(-2.f * m.out, rcp(1.f + e), m.out);
 }
 
 struct PoolMma {
-  PoolAttn p{};                  // q, caches, sizes (the sequence's rows: q / mid point at its first row)
-  const __nv_bfloat16 *k = nullptr, *v = nullptr;   // the sequence's cache rows
-  int count = 0, pos0 = 0;       // rows of the sequence in this step, position of the first
+  PoolAttn p{};                  // the step's rows
+  const int32_t *seg_row0 = nullptr, *seg_count = nullptr;
+  int min_rows = 1;              // sequences with fewer rows are left to other kernels
   ScoreMap map{};
-  float* stats = nullptr;        // [count][heads][2]: maximum (log2 units), 1 / denominator
+  float* stats = nullptr;        // [n_tok][heads][2]: maximum (log2 units), 1 / denominator
   int vcols = 0, stages = 1;     // pool_mix_kernel: value columns per CTA, stages of its key / value ring
 };
+// one sequence's rows and cache
+struct SeqView {
+  int row0, count, pos0;
+  const __nv_bfloat16 *k, *v;
+};
+__device__ __forceinline__ SeqView seq_view(const PoolMma& m, int seg) {
+  SeqView s;
+  s.row0 = m.seg_row0[seg];
+  s.count = m.seg_count[seg];
+  s.pos0 = m.p.pos[s.row0];
+  const int64_t slot = m.p.slot[s.row0];
+  s.k = static_cast<const __nv_bfloat16*>(m.p.kcache) + slot * m.p.k_slot_stride;
+  s.v = static_cast<const __nv_bfloat16*>(m.p.vcache) + slot * m.p.v_slot_stride;
+  return s;
+}
 
 // The keys a tile of rows at positions [p0, p1] may see: blocks [0, nb) and tokens [lo, p1].
 struct TileList {
@@ -99,17 +125,19 @@ __global__ void __launch_bounds__(128) pool_stats_kernel(const PoolMma m) {
   const PoolAttn& p = m.p;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
   const int h = blockIdx.y, H = p.a.heads, G = p.a.kv_heads, dk = KS * 16, kvh = h / (H / G);
+  const SeqView sv = seq_view(m, blockIdx.z);
   const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kStM;   // rows with the most keys first
-  const int rows = min(kStM, m.count - q0);
+  if (q0 >= sv.count || sv.count < m.min_rows) return;
+  const int rows = min(kStM, sv.count - q0);
   uint8_t* Qs = ps_smem;                  // [64][LD]
   uint8_t* Ks = Qs + kStM * LD;           // [2][64][LD]
-  const TileList tl = tile_list<kStN>(p, m.pos0 + q0, m.pos0 + q0 + rows - 1);
-  const __nv_bfloat16* qg = static_cast<const __nv_bfloat16*>(p.q) + (int64_t)h * dk;
-  const __nv_bfloat16* kg = m.k + (int64_t)kvh * dk;
+  const TileList tl = tile_list<kStN>(p, sv.pos0 + q0, sv.pos0 + q0 + rows - 1);
+  const __nv_bfloat16* qg = static_cast<const __nv_bfloat16*>(p.q) + (int64_t)sv.row0 * H * dk + (int64_t)h * dk;
+  const __nv_bfloat16* kg = sv.k + (int64_t)kvh * dk;
   constexpr int CH = KS * 2;
   for (int i = tid; i < kStM * CH; i += 128) {
     const int r = i / CH, c = i % CH;
-    cp16(Qs + r * LD + c * 16, qg + (int64_t)min(q0 + r, m.count - 1) * H * dk + c * 8, r < rows);
+    cp16(Qs + r * LD + c * 16, qg + (int64_t)min(q0 + r, sv.count - 1) * H * dk + c * 8, r < rows);
   }
   auto load = [&](int it) {
     int n;
@@ -123,7 +151,7 @@ __global__ void __launch_bounds__(128) pool_stats_kernel(const PoolMma m) {
   };
   load(0);
   uint32_t qf[KS][4];
-  const int i0 = m.pos0 + q0 + warp * 16 + g, i1 = i0 + 8;
+  const int i0 = sv.pos0 + q0 + warp * 16 + g, i1 = i0 + 8;
   const int lo0 = pool_lo(i0, p.a.window), lo1 = pool_lo(i1, p.a.window);
   const int nb0 = pool_nb(i0, p.a.window, p.d.pool), nb1 = pool_nb(i1, p.a.window, p.d.pool);
   float mx0 = -INFINITY, mx1 = -INFINITY, l0 = 0.f, l1 = 0.f;
@@ -173,14 +201,14 @@ __global__ void __launch_bounds__(128) pool_stats_kernel(const PoolMma m) {
     }
     const float n0 = fmaxf(mx0, t0), n1 = fmaxf(mx1, t1);
     const float b0 = n0 == -INFINITY ? 0.f : n0, b1 = n1 == -INFINITY ? 0.f : n1;   // nothing seen yet: 2^(−inf − 0) = 0
-    l0 *= exp2f(mx0 - b0);
-    l1 *= exp2f(mx1 - b1);
+    l0 *= ex2(mx0 - b0);
+    l1 *= ex2(mx1 - b1);
 #pragma unroll
     for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
-        l0 += exp2f(s[nt][x] - b0);
-        l1 += exp2f(s[nt][x + 2] - b1);
+        l0 += ex2(s[nt][x] - b0);
+        l1 += ex2(s[nt][x + 2] - b1);
       }
     mx0 = n0;
     mx1 = n1;
@@ -195,11 +223,11 @@ __global__ void __launch_bounds__(128) pool_stats_kernel(const PoolMma m) {
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
     const int r = q0 + warp * 16 + g + 8 * x;
-    if (r >= m.count) continue;
+    if (r >= sv.count) continue;
     const float mx = x ? mx1 : mx0, l = x ? l1 : l0, mm = fmaxf(mx, sink);   // a row always sees itself: mx is finite
-    float* o = m.stats + ((int64_t)r * H + h) * 2;
+    float* o = m.stats + ((int64_t)(sv.row0 + r) * H + h) * 2;
     o[0] = mm;
-    o[1] = 1.f / (l * exp2f(mx - mm) + exp2f(sink - mm));
+    o[1] = 1.f / (l * ex2(mx - mm) + ex2(sink - mm));
   }
 }
 
@@ -228,7 +256,9 @@ __global__ void __launch_bounds__(512) pool_mix_kernel(const PoolMma m) {
   const PoolAttn& p = m.p;
   const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3, nw = nthr >> 5;
   const int H = p.a.heads, G = p.a.kv_heads, per = H / G, dk = p.a.dim, dv = p.a.vdim, ks = dk / 16;
-  const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * 16, rows = min(16, m.count - q0);
+  const SeqView sv = seq_view(m, blockIdx.z);
+  const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * 16, rows = min(16, sv.count - q0);
+  if (rows <= 0 || sv.count < m.min_rows) return;
   const int c0 = blockIdx.y * m.vcols, vc = min(m.vcols, dv - c0), nt_v = vc / 8;
   const int ldq = H * dk * 2 + 16, ldk = G * dk * 2 + 16, ldv = G * m.vcols * 2 + 16;
   uint8_t* Qs = pm_smem;
@@ -237,28 +267,33 @@ __global__ void __launch_bounds__(512) pool_mix_kernel(const PoolMma m) {
   uint32_t* Wh = reinterpret_cast<uint32_t*>(Vs + m.stages * 16 * ldv);
   uint32_t* Wl = Wh + SH::WBYTES / 4;
   uint32_t* X = Wl + SH::WBYTES / 4;
-  const TileList tl = tile_list<16>(p, m.pos0 + q0, m.pos0 + q0 + rows - 1);
+  const TileList tl = tile_list<16>(p, sv.pos0 + q0, sv.pos0 + q0 + rows - 1);
   {
-    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q);
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q) + (int64_t)sv.row0 * H * dk;
     const int ch = H * dk / 8;
     for (int i = tid; i < 16 * ch; i += nthr) {
       const int r = i / ch, c = i % ch;
-      cp16(Qs + r * ldq + c * 16, q + (int64_t)min(q0 + r, m.count - 1) * H * dk + c * 8, r < rows);
+      cp16(Qs + r * ldq + c * 16, q + (int64_t)min(q0 + r, sv.count - 1) * H * dk + c * 8, r < rows);
     }
   }
-  const int kch = G * dk / 8, vch1 = vc / 8, vch = G * vch1;
+  // a warp copies whole rows, so that no index is divided per chunk; the columns of a slice of the values lie vch1 chunks per
+  // key/value head apart (the reciprocal is exact for the few hundred chunks of a row)
+  const int kch = G * dk / 8, vch1 = vc / 8, vch = G * vch1, vmagic = (65536 + vch1 - 1) / vch1;
   auto load = [&](int it) {
     int n;
     const int r0 = tile_row0(tl, it, 16, p.max_ctx, n), st = it % m.stages;
-    uint8_t* kd = Ks + st * 16 * ldk;
-    uint8_t* vd = Vs + st * 16 * ldv;
-    for (int i = tid; i < 16 * kch; i += nthr) {
-      const int r = i / kch, c = i % kch;
-      cp16(kd + r * ldk + c * 16, m.k + (int64_t)(r0 + min(r, n - 1)) * G * dk + c * 8, r < n);
-    }
-    for (int i = tid; i < 16 * vch; i += nthr) {
-      const int r = i / vch, e = i % vch, gg = e / vch1, c = e % vch1;
-      cp16(vd + r * ldv + gg * m.vcols * 2 + c * 16, m.v + (int64_t)(r0 + min(r, n - 1)) * G * dv + gg * dv + c0 + c * 8, r < n);
+    for (int r = warp; r < 16; r += nw) {
+      const bool live = r < n;
+      const int64_t row = r0 + min(r, n - 1);
+      uint8_t* kd = Ks + (st * 16 + r) * ldk;
+      uint8_t* vd = Vs + (st * 16 + r) * ldv;
+      const __nv_bfloat16* kr = sv.k + row * G * dk;
+      const __nv_bfloat16* vr = sv.v + row * G * dv + c0;
+      for (int c = lane; c < kch; c += 32) cp16(kd + c * 16, kr + c * 8, live);
+      for (int e = lane; e < vch; e += 32) {
+        const int gg = (e * vmagic) >> 16, c = e - gg * vch1;
+        cp16(vd + gg * m.vcols * 2 + c * 16, vr + gg * dv + c * 8, live);
+      }
     }
     cp_commit();
   };
@@ -282,7 +317,7 @@ __global__ void __launch_bounds__(512) pool_mix_kernel(const PoolMma m) {
           tf[a][b][x] = pack2(talk(r, c), talk(r, c + 1));
         }
   }
-  const int i0 = m.pos0 + q0 + g, i1 = i0 + 8;
+  const int i0 = sv.pos0 + q0 + g, i1 = i0 + 8;
   const int lo0 = pool_lo(i0, p.a.window), lo1 = pool_lo(i1, p.a.window);
   const int nb0 = pool_nb(i0, p.a.window, p.d.pool), nb1 = pool_nb(i1, p.a.window, p.d.pool);
   float mx[HPW][2], il[HPW][2], o[HPW][SH::NT][4];
@@ -292,9 +327,9 @@ __global__ void __launch_bounds__(512) pool_mix_kernel(const PoolMma m) {
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
       const int r = q0 + g + 8 * x;
-      const bool live = h < H && r < m.count;
-      mx[u][x] = live ? m.stats[((int64_t)r * H + h) * 2] : 0.f;
-      il[u][x] = live ? m.stats[((int64_t)r * H + h) * 2 + 1] : 0.f;
+      const bool live = h < H && r < sv.count;
+      mx[u][x] = live ? m.stats[((int64_t)(sv.row0 + r) * H + h) * 2] : 0.f;
+      il[u][x] = live ? m.stats[((int64_t)(sv.row0 + r) * H + h) * 2 + 1] : 0.f;
     }
 #pragma unroll
     for (int n = 0; n < SH::NT; ++n)
@@ -317,6 +352,10 @@ __global__ void __launch_bounds__(512) pool_mix_kernel(const PoolMma m) {
     const int j0 = blk ? it * 16 : tl.lo + (it - tl.block_tiles) * 16;
     const int a0 = blk ? 0 : lo0 - j0, e0 = blk ? nb0 - j0 : i0 - j0 + 1;
     const int a1 = blk ? 0 : lo1 - j0, e1 = blk ? nb1 - j0 : i1 - j0 + 1;
+    // tiles every row sees whole need no mask: keys from the last row's window edge to the first row's position, or blocks the
+    // first row sees
+    const bool whole = blk ? j0 + 16 <= pool_nb(sv.pos0 + q0, p.a.window, p.d.pool)
+                           : j0 >= pool_lo(sv.pos0 + q0 + 15, p.a.window) && j0 + 15 <= sv.pos0 + q0;
     // ---- scores → finished weights of this warp's heads
 #pragma unroll
     for (int u = 0; u < HPW; ++u) {
@@ -336,17 +375,32 @@ __global__ void __launch_bounds__(512) pool_mix_kernel(const PoolMma m) {
         mma16816(s[0], a, b[0], b[1]);
         mma16816(s[1], a, b[2], b[3]);
       }
+      if (!whole) {   // hidden keys: a score of −inf
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+          for (int x = 0; x < 4; ++x) {
+            const int j = nt * 8 + tq * 2 + (x & 1);
+            const bool vis = (x >> 1) ? j >= a1 && j < e1 : j >= a0 && j < e0;
+            s[nt][x] = vis ? map_score(s[nt][x], m.map) : -INFINITY;
+          }
+      } else {
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+          for (int x = 0; x < 4; ++x) s[nt][x] = map_score(s[nt][x], m.map);
+      }
+      __nv_bfloat16* wh = Whb + (tq * 2 * SH::JW + g * SH::PW) * 2 + h;
+      __nv_bfloat16* wl = Wlb + (tq * 2 * SH::JW + g * SH::PW) * 2 + h;
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
-          const int j = nt * 8 + tq * 2 + (x & 1), second = x >> 1;
-          const bool vis = second ? j >= a1 && j < e1 : j >= a0 && j < e0;
-          const float w = vis ? exp2f(map_score(s[nt][x], m.map) - mx[u][second]) * il[u][second] : 0.f;
+          const float w = ex2(s[nt][x] - mx[u][x >> 1]) * il[u][x >> 1];
           const __nv_bfloat16 hi = __float2bfloat16_rn(w);
-          const int at = (j * SH::JW + (g + 8 * second) * SH::PW) * 2 + h;
-          Whb[at] = hi;
-          Wlb[at] = __float2bfloat16_rn(w - __bfloat162float(hi));
+          const int at = ((nt * 8 + (x & 1)) * SH::JW + (x >> 1) * 8 * SH::PW) * 2;   // a constant
+          wh[at] = hi;
+          wl[at] = __float2bfloat16_rn(w - __bfloat162float(hi));
         }
     }
     __syncthreads();
@@ -402,8 +456,8 @@ __global__ void __launch_bounds__(512) pool_mix_kernel(const PoolMma m) {
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
       const int r = q0 + g + 8 * x;
-      if (r >= m.count) continue;
-      __nv_bfloat16* y = static_cast<__nv_bfloat16*>(p.mid) + (int64_t)r * p.ld_mid + h * dv + c0 + tq * 2;
+      if (r >= sv.count) continue;
+      __nv_bfloat16* y = static_cast<__nv_bfloat16*>(p.mid) + (int64_t)(sv.row0 + r) * p.ld_mid + h * dv + c0 + tq * 2;
 #pragma unroll
       for (int n = 0; n < SH::NT; ++n)
         if (n < nt_v)
@@ -413,7 +467,7 @@ __global__ void __launch_bounds__(512) pool_mix_kernel(const PoolMma m) {
 }
 
 template <int KS>
-int launch_stats(const PoolMma& m, cudaStream_t st) {
+int launch_stats(const PoolMma& m, int n_seg, int max_count, cudaStream_t st) {
   constexpr int smem = 3 * 64 * (KS * 32 + 16);
   if (smem > 48 * 1024) {
     static bool attr_done = false;
@@ -422,13 +476,13 @@ int launch_stats(const PoolMma& m, cudaStream_t st) {
       attr_done = true;
     }
   }
-  const dim3 grid((m.count + kStM - 1) / kStM, m.p.a.heads);
+  const dim3 grid((max_count + kStM - 1) / kStM, m.p.a.heads, n_seg);
   B200_CUDA(launch_pdl(pool_stats_kernel<KS>, grid, dim3(128), (size_t)smem, st, false, m));
   return B200_OK;
 }
 
 template <int HPW>
-int launch_mix(PoolMma m, cudaStream_t st) {
+int launch_mix(PoolMma m, int n_seg, int max_count, cudaStream_t st) {
   using SH = MixShape<HPW>;
   const b200_attn_desc& a = m.p.a;
   static bool attr_done = false;
@@ -441,7 +495,7 @@ int launch_mix(PoolMma m, cudaStream_t st) {
   m.stages = mix_smem(a.heads, a.kv_heads, a.dim, m.vcols, 2, SH::WBYTES, SH::XBYTES) <= 227 * 1024 ? 2 : 1;
   const int smem = mix_smem(a.heads, a.kv_heads, a.dim, m.vcols, m.stages, SH::WBYTES, SH::XBYTES);
   const int warps = std::max(4, (a.heads + HPW - 1) / HPW);
-  const dim3 grid((m.count + 15) / 16, (a.vdim + m.vcols - 1) / m.vcols);
+  const dim3 grid((max_count + 15) / 16, (a.vdim + m.vcols - 1) / m.vcols, n_seg);
   B200_CUDA(launch_pdl(pool_mix_kernel<HPW>, grid, dim3(warps * 32), (size_t)smem, st, false, m));
   return B200_OK;
 }
@@ -455,17 +509,17 @@ bool pool_prompt_ok(const b200_attn_desc& a) {
   return mix_smem(a.heads, a.kv_heads, a.dim, vc, 1, w, x) <= 227 * 1024;
 }
 
-int launch_pool_prompt(const PoolAttn& p, int slot, int count, int pos0, float* stats, cudaStream_t st) {
+int launch_pool_prompt(const PoolAttn& p, const int32_t* seg_row0, const int32_t* seg_count, int n_seg, int max_count, int min_rows, float* stats,
+                       cudaStream_t st) {
   const b200_attn_desc& a = p.a;
-  B200_CHECK_ARG(p.q && p.kcache && p.vcache && p.mid && stats && count > 0 && pos0 >= 0 && pos0 + count <= p.max_ctx, "pool prompt attention: bad arguments");
+  B200_CHECK_ARG(p.q && p.kcache && p.vcache && p.mid && stats && seg_row0 && seg_count && p.slot && p.pos && n_seg > 0 && max_count > 0,
+                 "pool prompt attention: bad arguments");
   B200_CHECK_ARG(pool_prompt_ok(a) && a.heads % a.kv_heads == 0, "pool prompt attention: head sizes not built");
   B200_CHECK_ARG(((reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.kcache) | reinterpret_cast<uintptr_t>(p.vcache)) & 15) == 0 &&
                      p.k_slot_stride % 8 == 0 && p.v_slot_stride % 8 == 0 && p.ld_mid % 2 == 0 && (reinterpret_cast<uintptr_t>(p.mid) & 3) == 0,
                  "pool prompt attention: operands must be 16-byte aligned");
   PoolMma m;
-  m.p = p; m.count = count; m.pos0 = pos0; m.stats = stats;
-  m.k = (const __nv_bfloat16*)p.kcache + (int64_t)slot * p.k_slot_stride;
-  m.v = (const __nv_bfloat16*)p.vcache + (int64_t)slot * p.v_slot_stride;
+  m.p = p; m.seg_row0 = seg_row0; m.seg_count = seg_count; m.min_rows = min_rows; m.stats = stats;
   if (p.d.softcap > 0.f) {
     m.map.in = 2.f * a.scale / p.d.softcap * kLog2eM;
     m.map.out = p.d.softcap * kLog2eM;
@@ -474,17 +528,17 @@ int launch_pool_prompt(const PoolAttn& p, int slot, int count, int pos0, float* 
   }
   int rc = B200_OK;
   switch (a.dim / 16) {
-    case 1: rc = launch_stats<1>(m, st); break;
-    case 2: rc = launch_stats<2>(m, st); break;
-    case 3: rc = launch_stats<3>(m, st); break;
-    case 4: rc = launch_stats<4>(m, st); break;
-    case 5: rc = launch_stats<5>(m, st); break;
-    case 6: rc = launch_stats<6>(m, st); break;
-    case 7: rc = launch_stats<7>(m, st); break;
-    default: rc = launch_stats<8>(m, st); break;
+    case 1: rc = launch_stats<1>(m, n_seg, max_count, st); break;
+    case 2: rc = launch_stats<2>(m, n_seg, max_count, st); break;
+    case 3: rc = launch_stats<3>(m, n_seg, max_count, st); break;
+    case 4: rc = launch_stats<4>(m, n_seg, max_count, st); break;
+    case 5: rc = launch_stats<5>(m, n_seg, max_count, st); break;
+    case 6: rc = launch_stats<6>(m, n_seg, max_count, st); break;
+    case 7: rc = launch_stats<7>(m, n_seg, max_count, st); break;
+    default: rc = launch_stats<8>(m, n_seg, max_count, st); break;
   }
   if (rc != B200_OK) return rc;
-  return a.heads <= 16 ? launch_mix<1>(m, st) : launch_mix<2>(m, st);
+  return a.heads <= 16 ? launch_mix<1>(m, n_seg, max_count, st) : launch_mix<2>(m, n_seg, max_count, st);
 }
 
 }  // namespace b200

@@ -605,6 +605,49 @@ __global__ void __launch_bounds__(128) mamba1_conv_kernel(const Mamba1Run p) {
     }
 }
 
+// Prompts: kM1Strip rows and two neighbouring channels per thread; while a sequence goes on, the window slides through registers.
+constexpr int kM1Strip = 16;
+__device__ __forceinline__ float2 ld2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 ld2(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+__device__ __forceinline__ void st2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void st2(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) mamba1_conv_strip_kernel(const Mamba1Run p) {
+  pdl_trigger();
+  const int t0 = blockIdx.x * kM1Strip, c = (blockIdx.y * 128 + threadIdx.x) * 2, inner = p.d.inner;
+  const bool mine = c < inner;
+  float2 w[TAPS], win[TAPS], bias = make_float2(0.f, 0.f);
+  if (mine) {
+    bias = ld2(p.d.conv_b + c);
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j] = ld2(p.d.conv_w + (int64_t)j * inner + c);
+  }
+  pdl_wait();
+  if (!mine) return;
+  const T* x = static_cast<const T*>(p.proj) + p.off_x + c;
+  const int t1 = min(t0 + kM1Strip, p.n_tok);
+  for (int t = t0; t < t1; ++t) {
+    if (t == t0 || !row_same_seq(p.slot, p.pos, t, 1)) {
+      const int front = rows_in_front(p.slot, p.pos, t, TAPS - 1), ps = p.pos[t];
+      const float* cs = p.conv_state + (int64_t)p.slot[t] * p.slot_stride + c;
+#pragma unroll
+      for (int j = 1; j < TAPS; ++j)
+        win[j] = j <= front ? ld2(x + (int64_t)(t - j) * p.ld_proj) : ps - j >= 0 ? ld2(cs + (int64_t)(TAPS - 1 - (j - front)) * inner) : make_float2(0.f, 0.f);
+    } else {
+#pragma unroll
+      for (int j = TAPS - 1; j > 0; --j) win[j] = win[j - 1];
+    }
+    win[0] = ld2(x + (int64_t)t * p.ld_proj);
+    float2 a = bias;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      a.x = fmaf(w[TAPS - 1 - j].x, win[j].x, a.x);
+      a.y = fmaf(w[TAPS - 1 - j].y, win[j].y, a.y);
+    }
+    st2(static_cast<T*>(p.xc) + (int64_t)t * inner + c, siluf(a.x), siluf(a.y));
+  }
+}
+
 // One warp per (row, channel): dt logit = Σ_r w_dt[c][r]·T(dt_r) + dt_b
 template <typename T>
 __global__ void __launch_bounds__(256) mamba1_dt_kernel(const Mamba1Run p) {
@@ -621,22 +664,43 @@ __global__ void __launch_bounds__(256) mamba1_dt_kernel(const Mamba1Run p) {
   if (lane == 0) p.dt[(int64_t)t * p.d.inner + c] = a + p.d.dt_b[c];
 }
 
-// LPC lanes share a channel, NPT state entries each; 128 threads = 128 / LPC channels per CTA.  The CTA walks its sequence CH
+// 2^x and the two gates by the hardware's approximate exponential, logarithm and reciprocal (relative errors of about 2^-22; bf16
+// engines), or as CUDA's functions (fp32 engines).
+__device__ __forceinline__ float ex2_fast(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+template <typename T> __device__ __forceinline__ float gate_softplus(float z) { return softplusf(z); }
+template <> __device__ __forceinline__ float gate_softplus<__nv_bfloat16>(float z) {
+  const float e = ex2_fast(-fabsf(z) * 1.4426950408889634f);   // log(1 + e): its series where the sum would lose e's digits
+  return fmaxf(z, 0.f) + (e < 0.01f ? e * (1.f - e * (0.5f - 0.33333333f * e)) : __logf(1.f + e));
+}
+template <typename T> __device__ __forceinline__ float gate_silu(float z) { return siluf(z); }
+template <> __device__ __forceinline__ float gate_silu<__nv_bfloat16>(float z) {
+  return __fdividef(z, 1.f + ex2_fast(fminf(-z * 1.4426950408889634f, 80.f)));
+}
+
+// LPC lanes share a channel, NPT state entries each; 256 threads = 256 / LPC channels per CTA.  The CTA walks its sequence CH
 // tokens at a time: the chunk's B and C rows (fp32) and its channels' step sizes, inputs and gates sit in shared memory,
 // while the next chunk's values are already on their way into registers.  The state is in registers for the whole walk; a
 // token costs a thread NPT exponentials and 3·NPT multiply-adds, and the lanes' partial sums of four tokens meet side by
-// side, off the state's chain.  The decay is 2^(dt·A·log2 e); fp32 engines take exp(dt·A) − 1 instead, so that thousands of
-// decays close to one do not add up a rounding of their own.  Entries past the state's size hold zeros (decay 1, B = C = 0).
+// side, off the state's chain, each pair of lanes keeping half of the tokens.  The decay is 2^(dt·A·log2 e); fp32 engines take
+// exp(dt·A) − 1 instead, so that thousands of decays close to one do not add up a rounding of their own.  Entries past the
+// state's size hold zeros (decay 1, B = C = 0).  A chunk's outputs leave together.
 template <typename T, int LPC, int NPT>
-__global__ void __launch_bounds__(128) mamba1_scan_kernel(const Mamba1Run p) {
+__global__ void __launch_bounds__(256) mamba1_scan_kernel(const Mamba1Run p) {
   pdl_trigger();
   pdl_wait();
-  constexpr int NS = LPC * NPT, CPB = 128 / LPC;
+  constexpr int NS = LPC * NPT, CPB = 256 / LPC;
   constexpr int CH = NS <= 32 ? 32 : NS <= 64 ? 16 : 8;         // tokens per chunk
-  constexpr int NBC = CH * 2 * NS / 128;                        // staged B | C entries per thread
-  constexpr int NX = (CH * CPB + 127) / 128;                    // staged (token, channel) triples per thread
+  constexpr int NBC = CH * 2 * NS / 256;                        // staged B | C entries per thread
+  constexpr int NX = (CH * CPB + 255) / 256;                    // staged (token, channel) triples per thread
+  static_assert(LPC >= 4 && CH * 2 * NS % 256 == 0, "mamba1 scan tiling");
   __shared__ float s_b[CH][NS], s_c[CH][NS];
-  __shared__ float s_dt[CH][CPB], s_x[CH][CPB], s_z[CH][CPB];
+  __shared__ float2 s_d[CH][CPB];                               // step size, step size · input
+  __shared__ float2 s_o[CH][CPB];                               // D · input, gate
+  __shared__ float s_y[CH][CPB];
   const int seg = blockIdx.x, tid = threadIdx.x, ch = tid / LPC, ln = tid % LPC;
   const int c0 = blockIdx.y * CPB, c = c0 + ch, inner = p.d.inner, N = p.d.state;
   const int r0 = p.seg_row0 != nullptr ? p.seg_row0[seg] : seg;
@@ -650,77 +714,95 @@ __global__ void __launch_bounds__(128) mamba1_scan_kernel(const Mamba1Run p) {
     S[i] = live && n < N && !fresh ? st[n] : 0.f;
     A[i] = live && n < N ? -expf(p.d.A_log[(int64_t)c * N + n]) * (sizeof(T) == 4 ? 1.f : 1.4426950408889634f) : 0.f;
   }
-  const float D = live ? p.d.D[c] : 0.f;
   const int off_b = (p.d.dt_rank + 7) / 8 * 8;
   float r_bc[NBC], r_dt[NX], r_x[NX], r_z[NX];
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int i = 0; i < NBC; ++i) {
-      const int e = tid + 128 * i, t = e / (2 * NS), w = (e / NS) & 1, n = e % NS;
+      const int e = tid + 256 * i, t = e / (2 * NS), w = (e / NS) & 1, n = e % NS;
       r_bc[i] = t0 + t < cnt && n < N ? p.xd[(int64_t)(r0 + t0 + t) * p.ld_xd + off_b + w * N + n] : 0.f;
     }
 #pragma unroll
     for (int i = 0; i < NX; ++i) {
-      const int e = tid + 128 * i, t = e / CPB, cc = c0 + e % CPB;
-      r_dt[i] = r_x[i] = r_z[i] = 0.f;
+      const int e = tid + 256 * i, t = e / CPB, cc = c0 + e % CPB;
+      r_dt[i] = -INFINITY;   // rows past the end: step size softplus(−inf) = 0, the state stays
+      r_x[i] = r_z[i] = 0.f;
       if (e < CH * CPB && t0 + t < cnt && cc < inner) {
         const int64_t row = r0 + t0 + t;
-        r_dt[i] = softplusf(p.dt[row * inner + cc]);
+        r_dt[i] = p.dt[row * inner + cc];
         r_x[i] = ldf<T>(static_cast<const T*>(p.xc) + row * inner + cc);
-        r_z[i] = siluf(ldf<T>(static_cast<const T*>(p.proj) + row * p.ld_proj + p.off_z + cc));
+        r_z[i] = ldf<T>(static_cast<const T*>(p.proj) + row * p.ld_proj + p.off_z + cc);
       }
     }
   };
+  auto flush = [&](int t0) {   // the outputs of the chunk that starts at t0
+#pragma unroll
+    for (int i = 0; i < NX; ++i) {
+      const int e = tid + 256 * i, t = e / CPB, cc = e % CPB;
+      if (e < CH * CPB && t0 + t < cnt && c0 + cc < inner) {
+        const float2 o = s_o[t][cc];
+        static_cast<T*>(p.mid)[(int64_t)(r0 + t0 + t) * p.ld_mid + c0 + cc] = cvt<T>((s_y[t][cc] + o.x) * o.y);
+      }
+    }
+  };
+  float D[NX];
+#pragma unroll
+  for (int i = 0; i < NX; ++i) {
+    const int cc = c0 + (tid + 256 * i) % CPB;
+    D[i] = cc < inner ? p.d.D[cc] : 0.f;
+  }
+  const bool hi1 = (ln & (LPC / 2)) != 0, hi2 = (ln & (LPC / 4)) != 0, owner = (ln & (LPC / 4 - 1)) == 0;
+  const int own = (hi1 ? 2 : 0) + (hi2 ? 1 : 0);   // which of four tokens this lane ends up with
   fetch(0);
   for (int t0 = 0; t0 < cnt; t0 += CH) {
-    const int n_t = min(CH, cnt - t0);
+    __syncthreads();
+    if (t0 > 0) flush(t0 - CH);
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < NBC; ++i) {
-      const int e = tid + 128 * i, t = e / (2 * NS), w = (e / NS) & 1, n = e % NS;
+      const int e = tid + 256 * i, t = e / (2 * NS), w = (e / NS) & 1, n = e % NS;
       (w ? s_c : s_b)[t][n] = r_bc[i];
     }
 #pragma unroll
     for (int i = 0; i < NX; ++i) {
-      const int e = tid + 128 * i;
+      const int e = tid + 256 * i;
       if (e < CH * CPB) {
-        (&s_dt[0][0])[e] = r_dt[i];
-        (&s_x[0][0])[e] = r_x[i];
-        (&s_z[0][0])[e] = r_z[i];
+        const float dt = r_dt[i] == -INFINITY ? 0.f : gate_softplus<T>(r_dt[i]);
+        (&s_d[0][0])[e] = make_float2(dt, dt * r_x[i]);
+        (&s_o[0][0])[e] = make_float2(D[i] * r_x[i], gate_silu<T>(r_z[i]));
       }
     }
     __syncthreads();
     if (t0 + CH < cnt) fetch(t0 + CH);
-    for (int t4 = 0; t4 < n_t; t4 += 4) {   // rows past the end hold dt = 0, x = 0: the state stays (2^0·S + 0)
+    const int n4 = min(CH, (cnt - t0 + 3) / 4 * 4);
+    for (int t4 = 0; t4 < n4; t4 += 4) {
       float y[4];
 #pragma unroll
       for (int u = 0; u < 4; ++u) {
         const int t = t4 + u;
-        const float dt = s_dt[t][ch], dx = dt * s_x[t][ch];
+        const float2 d = s_d[t][ch];
         float a = 0.f;
 #pragma unroll
         for (int i = 0; i < NPT; ++i) {
-          if constexpr (sizeof(T) == 4) S[i] += fmaf(expm1f(dt * A[i]), S[i], dx * s_b[t][ln * NPT + i]);
-          else S[i] = fmaf(exp2f(dt * A[i]), S[i], dx * s_b[t][ln * NPT + i]);
+          const float b = s_b[t][ln * NPT + i];
+          if constexpr (sizeof(T) == 4) S[i] += fmaf(expm1f(d.x * A[i]), S[i], d.y * b);
+          else S[i] = fmaf(ex2_fast(d.x * A[i]), S[i], d.y * b);
           a = fmaf(S[i], s_c[t][ln * NPT + i], a);
         }
         y[u] = a;
       }
+      float a0 = hi1 ? y[2] : y[0], a1 = hi1 ? y[3] : y[1];
+      a0 += __shfl_xor_sync(0xffffffffu, hi1 ? y[0] : y[2], LPC / 2);
+      a1 += __shfl_xor_sync(0xffffffffu, hi1 ? y[1] : y[3], LPC / 2);
+      float a = hi2 ? a1 : a0;
+      a += __shfl_xor_sync(0xffffffffu, hi2 ? a0 : a1, LPC / 4);
 #pragma unroll
-      for (int o = LPC / 2; o > 0; o >>= 1) {
-#pragma unroll
-        for (int u = 0; u < 4; ++u) y[u] += __shfl_xor_sync(0xffffffffu, y[u], o);
-      }
-#pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        const int t = t4 + u;
-        if (ln == (u & (LPC - 1)) && t < n_t && live) {
-          const float v = fmaf(D, s_x[t][ch], y[u]) * s_z[t][ch];
-          static_cast<T*>(p.mid)[(int64_t)(r0 + t0 + t) * p.ld_mid + c] = cvt<T>(v);
-        }
-      }
+      for (int o = LPC / 8; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
+      if (owner) s_y[t4 + own][ch] = a;
     }
   }
+  __syncthreads();
+  flush((cnt - 1) / CH * CH);
   if (!live) return;
 #pragma unroll
   for (int i = 0; i < NPT; ++i) {
@@ -945,6 +1027,24 @@ int launch_mamba1_conv(const Mamba1Run& p, int dtype, cudaStream_t st) {
   B200_CHECK_ARG(p.proj && p.xc && p.slot && p.pos && p.n_tok > 0 && d.inner > 0 && d.conv_w && d.conv_b && d.taps >= 1 && d.taps <= kMambaMaxTaps,
                  "mamba1 convolution: bad arguments (1 … %d taps)", kMambaMaxTaps);
   B200_CHECK_ARG(d.taps == 1 || p.conv_state, "mamba1 convolution: null state");
+  if (!p.advance && p.n_tok > kM1Strip && d.taps <= 4 && d.inner % 2 == 0 && p.ld_proj % 2 == 0 && p.off_x % 2 == 0 && p.slot_stride % 2 == 0 &&
+      ((reinterpret_cast<uintptr_t>(p.proj) | reinterpret_cast<uintptr_t>(p.xc) | reinterpret_cast<uintptr_t>(p.conv_state) |
+        reinterpret_cast<uintptr_t>(d.conv_w) | reinterpret_cast<uintptr_t>(d.conv_b)) & 7) == 0) {
+    const dim3 sg((p.n_tok + kM1Strip - 1) / kM1Strip, (d.inner / 2 + 127) / 128);
+#define B200_MC(T, TAPS) B200_CUDA(launch_pdl(mamba1_conv_strip_kernel<T, TAPS>, sg, dim3(128), 0, st, stack_pdl(), p))
+#define B200_MC_T(T)                    \
+  do {                                  \
+    if (d.taps == 1) B200_MC(T, 1);     \
+    else if (d.taps == 2) B200_MC(T, 2); \
+    else if (d.taps == 3) B200_MC(T, 3); \
+    else B200_MC(T, 4);                 \
+  } while (0)
+    if (dtype == B200_F32) B200_MC_T(float);
+    else B200_MC_T(__nv_bfloat16);
+#undef B200_MC_T
+#undef B200_MC
+    return B200_OK;
+  }
   const dim3 grid(p.n_tok, (d.inner + 127) / 128);
   if (dtype == B200_F32) B200_CUDA(launch_pdl(mamba1_conv_kernel<float>, grid, dim3(128), 0, st, stack_pdl(), p));
   else B200_CUDA(launch_pdl(mamba1_conv_kernel<__nv_bfloat16>, grid, dim3(128), 0, st, stack_pdl(), p));
@@ -966,9 +1066,9 @@ int launch_mamba1_scan(const Mamba1Run& p, int dtype, cudaStream_t st) {
   B200_CHECK_ARG(p.xd && p.dt && p.xc && p.proj && p.state && p.mid && p.slot && p.pos && p.n_seg > 0 && p.n_tok > 0 && d.A_log && d.D,
                  "mamba1 scan: null argument");
   B200_CHECK_ARG(d.inner > 0 && d.state > 0 && d.state <= kMamba1MaxState, "mamba1 scan: state 1 … %d", kMamba1MaxState);
-#define B200_M1(LPC, NPT)                                                                                                  do {                                                                                                                       const dim3 grid(p.n_seg, (d.inner + 128 / LPC - 1) / (128 / LPC));                                                       if (dtype == B200_F32) B200_CUDA(launch_pdl(mamba1_scan_kernel<float, LPC, NPT>, grid, dim3(128), 0, st, stack_pdl(), p));     else B200_CUDA(launch_pdl(mamba1_scan_kernel<__nv_bfloat16, LPC, NPT>, grid, dim3(128), 0, st, stack_pdl(), p));       } while (0)
-  if (d.state <= 8) B200_M1(2, 4);
-  else if (d.state <= 16) B200_M1(4, 4);
+#define B200_M1(LPC, NPT)                                                                                                  do {                                                                                                                       const dim3 grid(p.n_seg, (d.inner + 256 / LPC - 1) / (256 / LPC));                                                       if (dtype == B200_F32) B200_CUDA(launch_pdl(mamba1_scan_kernel<float, LPC, NPT>, grid, dim3(256), 0, st, stack_pdl(), p));     else B200_CUDA(launch_pdl(mamba1_scan_kernel<__nv_bfloat16, LPC, NPT>, grid, dim3(256), 0, st, stack_pdl(), p));       } while (0)
+  if (d.state <= 8) B200_M1(4, 2);
+  else if (d.state <= 16) B200_M1(8, 2);
   else if (d.state <= 32) B200_M1(8, 4);
   else if (d.state <= 64) B200_M1(16, 4);
   else if (d.state <= 128) B200_M1(32, 4);

@@ -10,6 +10,7 @@ written between timed iterations.
 """
 from __future__ import annotations
 
+import dataclasses
 import json
 from typing import Dict, List
 
@@ -381,6 +382,123 @@ def compare_tarudra(sizes: List[str], steps: int = 5, warmup: int = 3, prompt_le
 def main_tarudra(sizes: str, steps: int, warmup: int) -> None:
     names = [s for s in sizes.split(",") if s] if sizes and sizes != "all" else list(TARUDRA_SIZES)
     print(json.dumps(compare_tarudra(names, steps=steps, warmup=warmup)), flush=True)
+
+
+# Bibezen sizes: six layers [selective scan, attention + time mixing, time mixing] twice, every one with routed experts (32
+# experts, top 4, a shared expert).  The model beside it is the Tekosun design — the framework's other design with a selective
+# state-space mixer, a decaying matrix memory, a windowed attention behind query / key norms and rotate-half positions, and
+# softmax-routed experts — at the same width, vocabulary and number of layers, its two-matrix experts half again as wide (equal
+# expert parameters).
+BIBEZEN_SIZES = {
+    "z2048": dict(width=2048, vocab=65536, streams=4, taps=4, heads=16, kv_heads=8, dim=128, vdim=128, window=1024, pool=16, conv=4,
+                  rot_dims=64, right_heads=16, w_heads=32, w_dim=64, rank=64, inner=4096, state=16, dt_rank=128, experts=32, top=4,
+                  expert_ff=1024, shared_ff=1024, beside="t2048"),
+    "z3072": dict(width=3072, vocab=65536, streams=4, taps=4, heads=24, kv_heads=8, dim=128, vdim=128, window=1024, pool=16, conv=4,
+                  rot_dims=64, right_heads=24, w_heads=48, w_dim=64, rank=96, inner=6144, state=16, dt_rank=192, experts=32, top=4,
+                  expert_ff=1536, shared_ff=1536, beside="t3072"),
+}
+
+
+def bibezen_spec(name: str, max_ctx: int, max_slots: int = 8) -> models.StackSpec:
+    z = BIBEZEN_SIZES[name]
+    pool = models.PoolAttnSpec(z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["dim"] ** -0.5, z["conv"], z["window"], z["pool"],
+                               models.HalfRotarySpec(dims=z["rot_dims"], base=5e5), 30.0)
+    moe = models.MoeSpec(z["experts"], z["top"], z["expert_ff"], shared_ff=z["shared_ff"], router="softmax_chosen", weight_output=True,
+                         act="glu_silu", shared_plain=True)
+    L = models.StackLayerSpec
+    kw = dict(ff_kind="moe", moe=moe, canon=z["taps"])
+    m = L(mixer="mamba1", mamba1=models.Mamba1Spec(z["inner"], z["state"], z["dt_rank"], z["conv"]), **kw)
+    a = L(mixer="parallel", pool=pool, wkv=models.WkvSpec(z["right_heads"], z["w_dim"], z["rank"]), left_scale=0.7, right_scale=0.5, **kw)
+    w = L(mixer="wkv", wkv=models.WkvSpec(z["w_heads"], z["w_dim"], z["rank"]), **kw)
+    return models.StackSpec(name="bibezen-" + name, architecture="Bibezen", width=z["width"], vocab=z["vocab"], layers=(m, a, w, m, a, w),
+                            embed_scale=8.0, residual_mult=0.7, norm_eps=1e-6, norm_offset=1.0, block="hyper", norm_kind="rms",
+                            loop_mix=False, streams=z["streams"], max_ctx=max_ctx, max_slots=max_slots)
+
+
+def tekosun_beside(name: str, max_ctx: int, max_slots: int = 8) -> models.StackSpec:
+    spec = tekosun_spec(BIBEZEN_SIZES[name]["beside"], max_ctx, max_slots)
+
+    def wider(m: models.MoeSpec) -> models.MoeSpec:
+        return dataclasses.replace(m, expert_ff=m.expert_ff * 3 // 2, shared_ff=m.shared_ff * 3 // 2)
+
+    return dataclasses.replace(spec, layers=tuple(dataclasses.replace(L, moe=wider(L.moe)) for L in spec.layers))
+
+
+def device_bibezen_weights(spec: models.StackSpec, device, seed: int = 0) -> Dict[str, torch.Tensor]:
+    """Random Bibezen weights straight in the engine's layout on the device."""
+    g = torch.Generator(device=device).manual_seed(seed)
+    W, S = spec.width, spec.streams
+
+    def mat(*shape):
+        return (torch.randn(*shape, generator=g, device=device, dtype=torch.float32) * (shape[-1] ** -0.5)).to(torch.bfloat16)
+
+    def vec(n, centre=1.0, spread=0.05):
+        return centre + torch.randn(n, generator=g, device=device, dtype=torch.float32) * spread
+
+    w = {"embed": mat(spec.vocab, W), "final_norm": vec(W, 0.0)}
+    w["head"] = w["embed"]
+    for i, L in enumerate(spec.layers):
+        lay, p = spec.mix_layout(i), f"l{i}."
+        w[p + "norm"], w[p + "ff_norm"], w[p + "canon_w"] = vec(W, 0.0), vec(W, 0.0), vec(L.canon * W, 0.0, 0.2)
+        for h in ("hc1.", "hc2."):
+            w[p + h + "in"], w[p + h + "out"] = vec(S, 1.0 / S), vec(S)
+            w[p + h + "mix"] = (torch.eye(S, device=device).reshape(-1) * 0.9 + vec(S * S, 0.0)).contiguous()
+        w[p + "w_out"] = mat(W, lay.k_out)
+        if lay.n_in > 0:
+            w[p + "w_in"] = mat(lay.n_in, W)
+        if L.mamba1 is not None:
+            a = L.mamba1
+            w[p + "conv_w"], w[p + "conv_b"] = vec(a.conv * a.inner, 0.0, 0.4), vec(a.inner, 0.0, 0.2)
+            w[p + "w_x"], w[p + "w_dt"] = mat(models._up8(models._up8(a.dt_rank) + 2 * a.state), a.inner), mat(a.inner, models._up8(a.dt_rank))
+            w[p + "dt_b"], w[p + "A_log"], w[p + "D"] = vec(a.inner, -1.0, 0.5), vec(a.inner * a.state, 0.0, 0.5), vec(a.inner)
+        if L.wkv is not None:
+            a = L.wkv
+            n, rk = a.heads * a.dim, models._up8(a.rank)
+            w[p + "mu"], w[p + "w_rkvg"] = vec(5 * W, 0.5, 0.2), mat(4, n, W)
+            w[p + "w1"], w[p + "w2"], w[p + "w0"] = mat(rk, W), mat(n, rk), vec(n, -1.0, 0.5)
+            w[p + "u"], w[p + "head_norm"] = vec(n, 0.0, 0.5), vec(n)
+        if L.pool is not None:
+            a = L.pool
+            w[p + "b_in"], w[p + "left.conv_w"] = vec(lay.n_in, 0.0, 0.2), vec(a.conv * lay.n_in, 0.0, 0.4)
+            w[p + "left.q_norm"], w[p + "left.k_norm"], w[p + "left.sink"] = vec(a.dim), vec(a.dim), vec(a.heads, 0.0, 0.5)
+            w[p + "left.talk"] = (torch.eye(a.heads, device=device).reshape(-1) + vec(a.heads * a.heads, 0.0, 0.1)).contiguous()
+        m = L.moe
+        w[p + "router"] = mat(m.experts, W)
+        w[p + "w_exp_in"], w[p + "w_exp_out"] = mat(m.experts, 2 * m.expert_ff, W), mat(m.experts, W, m.expert_ff)
+        w[p + "w_ff_in"], w[p + "w_ff_out"] = mat(models._up8(2 * m.shared_ff), W), mat(W, m.shared_ff)
+    return w
+
+
+def compare_bibezen(sizes: List[str], steps: int = 5, warmup: int = 3, prompt_len: int = 2048, n_decode: int = 32) -> dict:
+    dev = torch.device("cuda:0")
+    torch.cuda.set_device(dev)
+    timer = _Timer(dev)
+    max_ctx = prompt_len + n_decode + 8
+    rows = {}
+    for name in sizes:
+        def one(spec, weights):
+            eng = engine.DecodeEngine(spec, weights)
+            k = _measure(eng, True, prompt_len, n_decode, timer, steps, warmup, spec.vocab)
+            k["bytes_per_decode_token"] = eng.bytes_per_token(prompt_len)
+            k["launches_per_decode_token"] = eng.launches_per_token
+            k["matrix_params_per_token"] = spec.weight_params()
+            eng.close()
+            del eng
+            torch.cuda.empty_cache()
+            return k
+        bspec = bibezen_spec(name, max_ctx)
+        k = one(bspec, device_bibezen_weights(bspec, dev))
+        tspec = tekosun_beside(name, max_ctx)
+        l = one(tspec, device_tekosun_weights(tspec, dev))
+        rows[name] = {"bibezen": k, "tekosun": l, "ratio": {m: round(k[m] / l[m], 3) for m in k if m.endswith("tok_s")}}
+    return {"metric": "bibezen_compare", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic", "prompt_len": prompt_len,
+            "decode_steps": n_decode, "steps": steps, "warmup": warmup, "l2": "flushed between timed iterations",
+            "sizes": rows}
+
+
+def main_bibezen(sizes: str, steps: int, warmup: int) -> None:
+    names = [s for s in sizes.split(",") if s] if sizes and sizes != "all" else list(BIBEZEN_SIZES)
+    print(json.dumps(compare_bibezen(names, steps=steps, warmup=warmup)), flush=True)
 
 
 class _Timer:

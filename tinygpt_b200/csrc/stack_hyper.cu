@@ -279,8 +279,10 @@ __global__ void __launch_bounds__(128) input_conv_strip_kernel(const InputConv c
   if (!live) return;
   float win[TAPS + 1][V], h[V], hp[V];
   const int t1 = min(t0 + kConvStrip, n_tok);
+  const bool one = rows_one_seq(slot, pos, t0, t1);
+#pragma unroll 2
   for (int t = t0; t < t1; ++t) {
-    if (t == t0 || !row_same_seq(slot, pos, t, 1)) {   // a window of its own: the step's rows in front, then the slot's
+    if (t == t0 || (!one && !row_same_seq(slot, pos, t, 1))) {   // a window of its own: the step's rows in front, then the slot's
       const int front = rows_in_front(slot, pos, t, TAPS), ps = pos[t];
       const float* st = c.state + (int64_t)slot[t] * c.slot_stride + i;
 #pragma unroll

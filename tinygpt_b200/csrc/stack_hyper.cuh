@@ -85,6 +85,10 @@ int launch_shift_state(const ShiftState& p, int dtype, cudaStream_t st);
 __device__ __forceinline__ bool row_same_seq(const int32_t* slot, const int32_t* pos, int t, int j) {
   return t - j >= 0 && slot[t - j] == slot[t] && pos[t - j] == pos[t] - j;
 }
+// rows [t0, t1) are one sequence's, in order (a sequence's rows lie side by side in a step, so the ends tell)
+__device__ __forceinline__ bool rows_one_seq(const int32_t* slot, const int32_t* pos, int t0, int t1) {
+  return slot[t0] == slot[t1 - 1] && pos[t1 - 1] - pos[t0] == t1 - 1 - t0;
+}
 // rows of this sequence in front of row t, counted up to `most`
 __device__ __forceinline__ int rows_in_front(const int32_t* slot, const int32_t* pos, int t, int most) {
   int n = 0;

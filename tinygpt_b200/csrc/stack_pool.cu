@@ -123,6 +123,7 @@ __global__ void __launch_bounds__(256) pool_prep_strip_kernel(const PoolAttn p) 
   const int H = p.a.heads, G = p.a.kv_heads, dk = p.a.dim, dv = p.a.vdim, per = H / G;
   const int nq = per * dk, mine = nq + dk + dv, n = min(kPrepStrip, p.n_tok - t0);
   pdl_wait();
+  const bool one = rows_one_seq(p.slot, p.pos, t0, t0 + n);
   for (int e = tid; e < mine; e += 256) {
     const int col = e < nq ? p.off_q + g * nq + e : e < nq + dk ? p.off_k + g * dk + (e - nq) : p.off_v + g * dv + (e - nq - dk);
     const T* x = static_cast<const T*>(p.proj) + (int64_t)t0 * p.ld_proj + col;
@@ -131,7 +132,7 @@ __global__ void __launch_bounds__(256) pool_prep_strip_kernel(const PoolAttn p) 
     for (int j = 0; j < TAPS; ++j) w[j] = p.d.conv_w[(int64_t)j * p.ld_proj + col];
     for (int r = 0; r < n; ++r) {
       const int t = t0 + r;
-      if (r == 0 || !row_same_seq(p.slot, p.pos, t, 1)) {
+      if (r == 0 || (!one && !row_same_seq(p.slot, p.pos, t, 1))) {
         const int front = rows_in_front(p.slot, p.pos, t, TAPS - 1), ps = p.pos[t];
         const float* cs = p.conv_state + (int64_t)p.slot[t] * p.conv_slot_stride + col;
 #pragma unroll

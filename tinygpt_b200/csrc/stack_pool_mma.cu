@@ -73,7 +73,7 @@ struct PoolMma {
   int min_rows = 1;              // sequences with fewer rows are left to other kernels
   ScoreMap map{};
   float* stats = nullptr;        // [n_tok][heads][2]: maximum (log2 units), 1 / denominator
-  int vcols = 0, stages = 1;     // pool_mix_kernel: value columns per CTA, stages of its key / value ring
+  int vcols = 0, kstages = 1;    // pool_mix_kernel: value columns per CTA, key tiles in shared memory
 };
 // one sequence's rows and cache
 struct SeqView {
@@ -233,40 +233,45 @@ __global__ void __launch_bounds__(128) pool_stats_kernel(const PoolMma m) {
 
 // ------------------------------------------------------------------------------------------------- mixed weights, values
 // Warp w owns heads w·HPW … w·HPW + HPW − 1 for the scores and the values, and every NW-th group of eight (key, query) pairs
-// for the mix.  Shared layouts (16-bit entries; strides padded so that ldmatrix and the scattered stores hit all banks):
-//   weights  [key 16][query 16][head], high and low halves apart — the mix reads eight pairs × 16 heads as its B operand
+// for the mix.  HPW 1: up to 16 heads; 2: up to 32, and half as many value columns per CTA.  Shared layouts (16-bit entries;
+// strides padded so that ldmatrix and the scattered stores meet few bank conflicts):
+//   weights  [key 16][query 16][head] words {low part, high part} — the mix reads eight pairs × eight heads as its B operand of
+//            sixteen columns, against a mixing matrix that has every column twice
 //   mixed    [head][key 16][query 16] — the values read it transposed as their A operand
+// The tiles run through two phases: the scores and weights of tile t + 1 beside the values of tile t, then the mix of tile
+// t + 1.  Keys and values of later tiles are on their way meanwhile.
 template <int HPW> struct MixShape {
-  static constexpr int KH = HPW;                          // head groups of 16 (HPW 1: up to 16 heads, 2: up to 32)
-  static constexpr int PW = KH == 1 ? 12 : 20;            // words per pair: 16·KH heads + 16 bytes
+  static constexpr int KH = HPW;                          // head groups of 16
+  static constexpr int PW = 16 * KH + 4;                  // words per pair
   static constexpr int JW = 16 * PW + 1;                  // words per key
   static constexpr int WBYTES = (16 * JW * 4 + 15) / 16 * 16;
   static constexpr int XW = 196;                          // words per head of the mixed weights: 16 rows of 12 words, + 4
   static constexpr int XBYTES = 16 * KH * XW * 4;
   static constexpr int NT = 16 / HPW;                     // most 8-column tiles of a CTA's slice of the values
 };
-__host__ __device__ inline int mix_smem(int H, int G, int dk, int vcols, int stages, int wbytes, int xbytes) {
-  return 16 * (H * dk * 2 + 16) + stages * 16 * ((G * dk * 2 + 16) + (G * vcols * 2 + 16)) + 2 * wbytes + xbytes;
+__host__ __device__ inline int mix_smem(int H, int G, int dk, int vcols, int kstages, int wbytes, int xbytes) {
+  return 16 * (H * dk * 2 + 16) + 16 * (kstages * (G * dk * 2 + 16) + 2 * (G * vcols * 2 + 16)) + wbytes + xbytes;
 }
 
-template <int HPW>
-__global__ void __launch_bounds__(512) pool_mix_kernel(const PoolMma m) {
+// KS: dim / 16 and the CTA's whole NT column tiles, known at compile time; 0: any size.
+template <int HPW, int KS>
+__global__ void __launch_bounds__(512, 1) pool_mix_kernel(const PoolMma m) {
   extern __shared__ __align__(128) uint8_t pm_smem[];
   using SH = MixShape<HPW>;
+  constexpr int KH = SH::KH;
   const PoolAttn& p = m.p;
   const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3, nw = nthr >> 5;
-  const int H = p.a.heads, G = p.a.kv_heads, per = H / G, dk = p.a.dim, dv = p.a.vdim, ks = dk / 16;
+  const int H = p.a.heads, G = p.a.kv_heads, per = H / G, dk = p.a.dim, dv = p.a.vdim, ks = KS > 0 ? KS : dk / 16;
   const SeqView sv = seq_view(m, blockIdx.z);
   const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * 16, rows = min(16, sv.count - q0);
   if (rows <= 0 || sv.count < m.min_rows) return;
-  const int c0 = blockIdx.y * m.vcols, vc = min(m.vcols, dv - c0), nt_v = vc / 8;
+  const int c0 = blockIdx.y * m.vcols, vc = min(m.vcols, dv - c0), nt_v = KS > 0 ? SH::NT : vc / 8;
   const int ldq = H * dk * 2 + 16, ldk = G * dk * 2 + 16, ldv = G * m.vcols * 2 + 16;
   uint8_t* Qs = pm_smem;
   uint8_t* Ks = Qs + 16 * ldq;
-  uint8_t* Vs = Ks + m.stages * 16 * ldk;
-  uint32_t* Wh = reinterpret_cast<uint32_t*>(Vs + m.stages * 16 * ldv);
-  uint32_t* Wl = Wh + SH::WBYTES / 4;
-  uint32_t* X = Wl + SH::WBYTES / 4;
+  uint8_t* Vs = Ks + m.kstages * 16 * ldk;
+  uint32_t* W = reinterpret_cast<uint32_t*>(Vs + 2 * 16 * ldv);
+  uint32_t* X = W + SH::WBYTES / 4;
   const TileList tl = tile_list<16>(p, sv.pos0 + q0, sv.pos0 + q0 + rows - 1);
   {
     const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q) + (int64_t)sv.row0 * H * dk;
@@ -279,47 +284,66 @@ __global__ void __launch_bounds__(512) pool_mix_kernel(const PoolMma m) {
   // a warp copies whole rows, so that no index is divided per chunk; the columns of a slice of the values lie vch1 chunks per
   // key/value head apart (the reciprocal is exact for the few hundred chunks of a row)
   const int kch = G * dk / 8, vch1 = vc / 8, vch = G * vch1, vmagic = (65536 + vch1 - 1) / vch1;
-  auto load = [&](int it) {
+  auto k_buf = [&](int it) { return Ks + (m.kstages == 2 ? it & 1 : 0) * 16 * ldk; };
+  auto v_buf = [&](int it) { return Vs + (it & 1) * 16 * ldv; };
+  const int64_t krow = (int64_t)G * dk, vrow = (int64_t)G * dv;
+  const __nv_bfloat16* k_src = sv.k + lane * 8;
+  const __nv_bfloat16* v_src = sv.v + c0;
+  const bool v_whole = vc == dv;   // the slice is the whole row: one run of chunks
+  auto load_k = [&](int it) {
+    if (it >= tl.tiles) return;
     int n;
-    const int r0 = tile_row0(tl, it, 16, p.max_ctx, n), st = it % m.stages;
+    const int r0 = tile_row0(tl, it, 16, p.max_ctx, n);
+    uint8_t* d = k_buf(it) + lane * 16;
     for (int r = warp; r < 16; r += nw) {
-      const bool live = r < n;
-      const int64_t row = r0 + min(r, n - 1);
-      uint8_t* kd = Ks + (st * 16 + r) * ldk;
-      uint8_t* vd = Vs + (st * 16 + r) * ldv;
-      const __nv_bfloat16* kr = sv.k + row * G * dk;
-      const __nv_bfloat16* vr = sv.v + row * G * dv + c0;
-      for (int c = lane; c < kch; c += 32) cp16(kd + c * 16, kr + c * 8, live);
+      const __nv_bfloat16* kr = k_src + (int64_t)(r0 + min(r, n - 1)) * krow;
+#pragma unroll 4
+      for (int c = 0; c + lane < kch; c += 32) cp16(d + r * ldk + c * 16, kr + c * 8, r < n);
+    }
+  };
+  auto load_v = [&](int it) {
+    if (it >= tl.tiles) return;
+    int n;
+    const int r0 = tile_row0(tl, it, 16, p.max_ctx, n);
+    uint8_t* d = v_buf(it);
+    for (int r = warp; r < 16; r += nw) {
+      const __nv_bfloat16* vr = v_src + (int64_t)(r0 + min(r, n - 1)) * vrow;
+      if (v_whole) {
+#pragma unroll 4
+        for (int e = lane; e < vch; e += 32) cp16(d + r * ldv + e * 16, vr + e * 8, r < n);
+        continue;
+      }
       for (int e = lane; e < vch; e += 32) {
         const int gg = (e * vmagic) >> 16, c = e - gg * vch1;
-        cp16(vd + gg * m.vcols * 2 + c * 16, vr + gg * dv + c * 8, live);
+        cp16(d + r * ldv + gg * m.vcols * 2 + c * 16, vr + gg * dv + c * 8, r < n);
       }
     }
-    cp_commit();
   };
-  load(0);
+  load_k(0);
+  load_v(0);
+  if (m.kstages == 2) load_k(1);
+  cp_commit();
   // heads that do not exist keep zero weights
-  for (int i = tid; i < 2 * SH::WBYTES / 4; i += nthr) Wh[i] = 0;
-  // the mixing matrix as A fragments: rows = mixed head, columns = head
-  uint32_t tf[SH::KH][SH::KH][4];
+  for (int i = tid; i < SH::WBYTES / 4; i += nthr) W[i] = 0;
+  // the mixing matrix as A fragments: rows = mixed head, columns 2h and 2h + 1 = head h
+  uint32_t tf[KH][2 * KH][4];
   {
     auto talk = [&](int a, int b) {
       if (a >= H || b >= H) return 0.f;
       return p.d.talk != nullptr ? p.d.talk[a * H + b] : a == b ? 1.f : 0.f;
     };
 #pragma unroll
-    for (int a = 0; a < SH::KH; ++a)
+    for (int a = 0; a < KH; ++a)
 #pragma unroll
-      for (int b = 0; b < SH::KH; ++b)
+      for (int b = 0; b < 2 * KH; ++b)
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
-          const int r = a * 16 + g + (x & 1) * 8, c = b * 16 + tq * 2 + (x >> 1) * 8;
-          tf[a][b][x] = pack2(talk(r, c), talk(r, c + 1));
+          const float v = talk(a * 16 + g + (x & 1) * 8, b * 8 + tq + (x >> 1) * 4);
+          tf[a][b][x] = pack2(v, v);
         }
   }
-  const int i0 = sv.pos0 + q0 + g, i1 = i0 + 8;
-  const int lo0 = pool_lo(i0, p.a.window), lo1 = pool_lo(i1, p.a.window);
-  const int nb0 = pool_nb(i0, p.a.window, p.d.pool), nb1 = pool_nb(i1, p.a.window, p.d.pool);
+  const int i0 = sv.pos0 + q0 + g, i1 = i0 + 8, nb0 = pool_nb(i0, p.a.window, p.d.pool), nb1 = pool_nb(i1, p.a.window, p.d.pool);
+  const int nb_first = pool_nb(sv.pos0 + q0, p.a.window, p.d.pool), lo_last = pool_lo(sv.pos0 + q0 + 15, p.a.window);
   float mx[HPW][2], il[HPW][2], o[HPW][SH::NT][4];
 #pragma unroll
   for (int u = 0; u < HPW; ++u) {
@@ -336,118 +360,134 @@ __global__ void __launch_bounds__(512) pool_mix_kernel(const PoolMma m) {
 #pragma unroll
       for (int x = 0; x < 4; ++x) o[u][n][x] = 0.f;
   }
-  __nv_bfloat16* Whb = reinterpret_cast<__nv_bfloat16*>(Wh);
-  __nv_bfloat16* Wlb = reinterpret_cast<__nv_bfloat16*>(Wl);
-  for (int it = 0; it < tl.tiles; ++it) {
-    if (m.stages == 1 && it > 0) {
-      __syncthreads();   // the last tile's values have been read
-      load(it);
+  float s[HPW][2][4];
+  // raw scores of tile `it`, this warp's heads
+  auto scores = [&](int it) {
+    const uint8_t* K = k_buf(it);
+#pragma unroll
+    for (int u = 0; u < HPW; ++u) {
+      const int h = warp * HPW + u;
+#pragma unroll
+      for (int x = 0; x < 4; ++x) s[u][0][x] = s[u][1][x] = 0.f;
+      if (h >= H) break;
+      const uint32_t qa = smem_u32(Qs + (lane & 15) * ldq + h * dk * 2 + (lane >> 4) * 16);
+      const uint32_t ka = smem_u32(K + ((lane & 7) + (lane >> 4) * 8) * ldk + (h / per) * dk * 2 + ((lane >> 3) & 1) * 16);
+#pragma unroll(KS > 0 ? KS : 2)
+      for (int k = 0; k < ks; ++k) {
+        uint32_t a[4], b[4];   // b: keys 0-7, entries 0-7 and 8-15; keys 8-15, the same
+        ldsm4(qa + k * 32, a);
+        ldsm4(ka + k * 32, b);
+        mma16816(s[u][0], a, b[0], b[1]);
+        mma16816(s[u][1], a, b[2], b[3]);
+      }
     }
-    cp_wait<0>();
-    __syncthreads();     // tile `it` is there; everyone is done with the ring stage the next load writes
-    if (m.stages > 1 && it + 1 < tl.tiles) load(it + 1);
-    const uint8_t* K = Ks + (it % m.stages) * 16 * ldk;
-    const uint8_t* V = Vs + (it % m.stages) * 16 * ldv;
+  };
+  // … → finished weights in W
+  uint32_t* Wt = W + tq * 2 * SH::JW + g * SH::PW;
+  auto weights = [&](int it) {
     const bool blk = it < tl.block_tiles;
     const int j0 = blk ? it * 16 : tl.lo + (it - tl.block_tiles) * 16;
-    const int a0 = blk ? 0 : lo0 - j0, e0 = blk ? nb0 - j0 : i0 - j0 + 1;
-    const int a1 = blk ? 0 : lo1 - j0, e1 = blk ? nb1 - j0 : i1 - j0 + 1;
     // tiles every row sees whole need no mask: keys from the last row's window edge to the first row's position, or blocks the
     // first row sees
-    const bool whole = blk ? j0 + 16 <= pool_nb(sv.pos0 + q0, p.a.window, p.d.pool)
-                           : j0 >= pool_lo(sv.pos0 + q0 + 15, p.a.window) && j0 + 15 <= sv.pos0 + q0;
-    // ---- scores → finished weights of this warp's heads
+    const bool whole = blk ? j0 + 16 <= nb_first : j0 >= lo_last && j0 + 15 <= sv.pos0 + q0;
+    int a0 = 0, e0 = 16, a1 = 0, e1 = 16;   // visible keys of the two rows as ranges of in-tile columns
+    if (!whole) {
+      a0 = blk ? 0 : pool_lo(i0, p.a.window) - j0;
+      a1 = blk ? 0 : pool_lo(i1, p.a.window) - j0;
+      e0 = (blk ? nb0 : i0 + 1) - j0;
+      e1 = (blk ? nb1 : i1 + 1) - j0;
+    }
 #pragma unroll
     for (int u = 0; u < HPW; ++u) {
       const int h = warp * HPW + u;
       if (h >= H) break;
-      const int kvh = h / per;
-      float s[2][4];
-#pragma unroll
-      for (int x = 0; x < 4; ++x) s[0][x] = s[1][x] = 0.f;
-      const uint32_t qa = smem_u32(Qs + (lane & 15) * ldq + h * dk * 2 + (lane >> 4) * 16);
-      const uint32_t ka = smem_u32(K + ((lane & 7) + (lane >> 4) * 8) * ldk + kvh * dk * 2 + ((lane >> 3) & 1) * 16);
-#pragma unroll 4
-      for (int k = 0; k < ks; ++k) {
-        uint32_t a[4], b[4];
-        ldsm4(qa + k * 32, a);
-        ldsm4(ka + k * 32, b);
-        mma16816(s[0], a, b[0], b[1]);
-        mma16816(s[1], a, b[2], b[3]);
-      }
-      if (!whole) {   // hidden keys: a score of −inf
-#pragma unroll
-        for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-          for (int x = 0; x < 4; ++x) {
-            const int j = nt * 8 + tq * 2 + (x & 1);
-            const bool vis = (x >> 1) ? j >= a1 && j < e1 : j >= a0 && j < e0;
-            s[nt][x] = vis ? map_score(s[nt][x], m.map) : -INFINITY;
-          }
-      } else {
-#pragma unroll
-        for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-          for (int x = 0; x < 4; ++x) s[nt][x] = map_score(s[nt][x], m.map);
-      }
-      __nv_bfloat16* wh = Whb + (tq * 2 * SH::JW + g * SH::PW) * 2 + h;
-      __nv_bfloat16* wl = Wlb + (tq * 2 * SH::JW + g * SH::PW) * 2 + h;
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
-          const float w = ex2(s[nt][x] - mx[u][x >> 1]) * il[u][x >> 1];
-          const __nv_bfloat16 hi = __float2bfloat16_rn(w);
-          const int at = ((nt * 8 + (x & 1)) * SH::JW + (x >> 1) * 8 * SH::PW) * 2;   // a constant
-          wh[at] = hi;
-          wl[at] = __float2bfloat16_rn(w - __bfloat162float(hi));
+          float w = ex2(map_score(s[u][nt][x], m.map) - mx[u][x >> 1]) * il[u][x >> 1];
+          if (!whole) {
+            const int j = nt * 8 + tq * 2 + (x & 1);
+            if (!((x >> 1) ? j >= a1 && j < e1 : j >= a0 && j < e0)) w = 0.f;
+          }
+          const float hi = __uint_as_float(__float_as_uint(w) & 0xffff0000u);   // the upper half is a bf16 number as it is
+          Wt[(nt * 8 + (x & 1)) * SH::JW + (x >> 1) * 8 * SH::PW + h] = pack2(w - hi, hi);
         }
     }
-    __syncthreads();
-    // ---- mix: eight pairs (one key, queries half·8 …) at a time
-    for (int nt = warp; nt < 32; nt += nw) {
-      const int j = nt >> 1, iq = (nt & 1) * 8;
-      const int at = j * SH::JW + (iq + g) * SH::PW + tq;
-      float x[SH::KH][4];
+  };
+  // W → mixed weights in X, eight pairs (one key, queries iq …) at a time
+  auto mixed = [&]() {
+    const int iq = (warp & 1) * 8;   // the number of warps is even
+    const uint32_t* w = W + (warp >> 1) * SH::JW + (iq + g) * SH::PW + tq;
+    uint32_t* d = X + g * SH::XW + (warp >> 1) * 12 + (iq >> 1) + tq;
+    for (int nt = warp; nt < 32; nt += nw, w += (nw >> 1) * SH::JW, d += (nw >> 1) * 12) {
+      float x[KH][4];
 #pragma unroll
-      for (int a = 0; a < SH::KH; ++a)
+      for (int a = 0; a < KH; ++a)
 #pragma unroll
         for (int e = 0; e < 4; ++e) x[a][e] = 0.f;
 #pragma unroll
-      for (int b = 0; b < SH::KH; ++b) {
-        const uint32_t h0 = Wh[at + b * 8], h1 = Wh[at + b * 8 + 4], l0 = Wl[at + b * 8], l1 = Wl[at + b * 8 + 4];
+      for (int b = 0; b < 2 * KH; ++b) {
+        const uint32_t w0 = w[b * 8], w1 = w[b * 8 + 4];
 #pragma unroll
-        for (int a = 0; a < SH::KH; ++a) {
-          mma16816(x[a], tf[a][b], h0, h1);
-          mma16816(x[a], tf[a][b], l0, l1);
-        }
+        for (int a = 0; a < KH; ++a) mma16816(x[a], tf[a][b], w0, w1);
       }
 #pragma unroll
-      for (int a = 0; a < SH::KH; ++a) {
-        uint32_t* d = X + (a * 16 + g) * SH::XW + j * 12 + (iq >> 1) + tq;
-        d[0] = pack2(x[a][0], x[a][1]);
-        d[8 * SH::XW] = pack2(x[a][2], x[a][3]);
+      for (int a = 0; a < KH; ++a) {
+        d[a * 16 * SH::XW] = pack2(x[a][0], x[a][1]);
+        d[(a * 16 + 8) * SH::XW] = pack2(x[a][2], x[a][3]);
       }
     }
-    __syncthreads();
-    // ---- values
+  };
+  // mixed weights of tile `it` times its values
+  auto values = [&](int it) {
+    const uint8_t* V = v_buf(it);
 #pragma unroll
     for (int u = 0; u < HPW; ++u) {
       const int h = warp * HPW + u;
       if (h >= H) break;
-      const int kvh = h / per;
       uint32_t a[4];   // stored [key][query]: matrices (keys 0-7, queries 0-7), (keys 0-7, queries 8-15), (keys 8-15, …), …
       ldsm4_t(smem_u32(X + h * SH::XW + ((lane & 7) + (lane >> 4) * 8) * 12) + ((lane >> 3) & 1) * 16, a);
-      const uint32_t va = smem_u32(V + (lane & 15) * ldv + kvh * m.vcols * 2 + (lane >> 4) * 16);
+      const uint32_t va = smem_u32(V + (lane & 15) * ldv + (h / per) * m.vcols * 2 + (lane >> 4) * 16);
 #pragma unroll
       for (int n = 0; n < SH::NT; n += 2) {
-        if (n >= nt_v) break;
+        if (KS == 0 && n >= nt_v) break;
         uint32_t b[4];   // columns n·8 … + 7: keys 0-7 and 8-15; columns + 8 … + 15: the same
         ldsm4_t(va + n * 16, b);
         mma16816(o[u][n], a, b[0], b[1]);
         mma16816(o[u][n + 1], a, b[2], b[3]);
       }
     }
+  };
+  cp_wait<0>();
+  __syncthreads();
+  scores(0);
+  weights(0);
+  __syncthreads();
+  if (m.kstages == 1) {
+    load_k(1);
+    cp_commit();
+  }
+  mixed();
+  cp_wait<0>();
+  __syncthreads();
+  for (int it = 0; it < tl.tiles; ++it) {
+    const bool more = it + 1 < tl.tiles;
+    load_v(it + 1);
+    if (m.kstages == 2) load_k(it + 2);
+    cp_commit();
+    if (more) scores(it + 1);
+    values(it);
+    if (!more) break;
+    weights(it + 1);
+    __syncthreads();   // every weight of tile it + 1 is in W; tile it's values and mixed weights have been read
+    if (m.kstages == 1) {
+      load_k(it + 2);
+      cp_commit();
+    }
+    mixed();
+    cp_wait<0>();
+    __syncthreads();   // mixed weights, and the next keys and values
   }
 #pragma unroll
   for (int u = 0; u < HPW; ++u) {
@@ -481,22 +521,22 @@ int launch_stats(const PoolMma& m, int n_seg, int max_count, cudaStream_t st) {
   return B200_OK;
 }
 
-template <int HPW>
+template <int HPW, int KS>
 int launch_mix(PoolMma m, int n_seg, int max_count, cudaStream_t st) {
   using SH = MixShape<HPW>;
   const b200_attn_desc& a = m.p.a;
   static bool attr_done = false;
   if (!attr_done) {
-    B200_CUDA(cudaFuncSetAttribute(pool_mix_kernel<HPW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    B200_CUDA(cudaFuncSetAttribute(pool_mix_kernel<HPW, KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     attr_done = true;
   }
   const int splits = (a.vdim + SH::NT * 8 - 1) / (SH::NT * 8);
   m.vcols = ((a.vdim + splits - 1) / splits + 15) / 16 * 16;
-  m.stages = mix_smem(a.heads, a.kv_heads, a.dim, m.vcols, 2, SH::WBYTES, SH::XBYTES) <= 227 * 1024 ? 2 : 1;
-  const int smem = mix_smem(a.heads, a.kv_heads, a.dim, m.vcols, m.stages, SH::WBYTES, SH::XBYTES);
-  const int warps = std::max(4, (a.heads + HPW - 1) / HPW);
+  m.kstages = mix_smem(a.heads, a.kv_heads, a.dim, m.vcols, 2, SH::WBYTES, SH::XBYTES) <= 227 * 1024 ? 2 : 1;
+  const int smem = mix_smem(a.heads, a.kv_heads, a.dim, m.vcols, m.kstages, SH::WBYTES, SH::XBYTES);
+  const int warps = std::max(4, ((a.heads + HPW - 1) / HPW + 1) / 2 * 2);
   const dim3 grid((max_count + 15) / 16, (a.vdim + m.vcols - 1) / m.vcols, n_seg);
-  B200_CUDA(launch_pdl(pool_mix_kernel<HPW>, grid, dim3(warps * 32), (size_t)smem, st, false, m));
+  B200_CUDA(launch_pdl(pool_mix_kernel<HPW, KS>, grid, dim3(warps * 32), (size_t)smem, st, false, m));
   return B200_OK;
 }
 
@@ -538,7 +578,9 @@ int launch_pool_prompt(const PoolAttn& p, const int32_t* seg_row0, const int32_t
     default: rc = launch_stats<8>(m, n_seg, max_count, st); break;
   }
   if (rc != B200_OK) return rc;
-  return a.heads <= 16 ? launch_mix<1>(m, n_seg, max_count, st) : launch_mix<2>(m, n_seg, max_count, st);
+  const bool k8 = a.dim == 128 && a.vdim == 128;
+  if (a.heads <= 16) return k8 ? launch_mix<1, 8>(m, n_seg, max_count, st) : launch_mix<1, 0>(m, n_seg, max_count, st);
+  return k8 ? launch_mix<2, 8>(m, n_seg, max_count, st) : launch_mix<2, 0>(m, n_seg, max_count, st);
 }
 
 }  // namespace b200

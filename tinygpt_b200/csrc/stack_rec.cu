@@ -626,8 +626,10 @@ __global__ void __launch_bounds__(128) mamba1_conv_strip_kernel(const Mamba1Run 
   if (!mine) return;
   const T* x = static_cast<const T*>(p.proj) + p.off_x + c;
   const int t1 = min(t0 + kM1Strip, p.n_tok);
+  const bool one = rows_one_seq(p.slot, p.pos, t0, t1);
+#pragma unroll 4
   for (int t = t0; t < t1; ++t) {
-    if (t == t0 || !row_same_seq(p.slot, p.pos, t, 1)) {
+    if (t == t0 || (!one && !row_same_seq(p.slot, p.pos, t, 1))) {
       const int front = rows_in_front(p.slot, p.pos, t, TAPS - 1), ps = p.pos[t];
       const float* cs = p.conv_state + (int64_t)p.slot[t] * p.slot_stride + c;
 #pragma unroll
@@ -715,7 +717,8 @@ __global__ void __launch_bounds__(256) mamba1_scan_kernel(const Mamba1Run p) {
     A[i] = live && n < N ? -expf(p.d.A_log[(int64_t)c * N + n]) * (sizeof(T) == 4 ? 1.f : 1.4426950408889634f) : 0.f;
   }
   const int off_b = (p.d.dt_rank + 7) / 8 * 8;
-  float r_bc[NBC], r_dt[NX], r_x[NX], r_z[NX];
+  float r_bc[NBC], r_dt[NX];
+  T r_x[NX], r_z[NX];   // as they lie in memory: widening them here would wait for the loads
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int i = 0; i < NBC; ++i) {
@@ -726,12 +729,12 @@ __global__ void __launch_bounds__(256) mamba1_scan_kernel(const Mamba1Run p) {
     for (int i = 0; i < NX; ++i) {
       const int e = tid + 256 * i, t = e / CPB, cc = c0 + e % CPB;
       r_dt[i] = -INFINITY;   // rows past the end: step size softplus(−inf) = 0, the state stays
-      r_x[i] = r_z[i] = 0.f;
+      r_x[i] = r_z[i] = cvt<T>(0.f);
       if (e < CH * CPB && t0 + t < cnt && cc < inner) {
         const int64_t row = r0 + t0 + t;
         r_dt[i] = p.dt[row * inner + cc];
-        r_x[i] = ldf<T>(static_cast<const T*>(p.xc) + row * inner + cc);
-        r_z[i] = ldf<T>(static_cast<const T*>(p.proj) + row * p.ld_proj + p.off_z + cc);
+        r_x[i] = static_cast<const T*>(p.xc)[row * inner + cc];
+        r_z[i] = static_cast<const T*>(p.proj)[row * p.ld_proj + p.off_z + cc];
       }
     }
   };
@@ -767,9 +770,9 @@ __global__ void __launch_bounds__(256) mamba1_scan_kernel(const Mamba1Run p) {
     for (int i = 0; i < NX; ++i) {
       const int e = tid + 256 * i;
       if (e < CH * CPB) {
-        const float dt = r_dt[i] == -INFINITY ? 0.f : gate_softplus<T>(r_dt[i]);
-        (&s_d[0][0])[e] = make_float2(dt, dt * r_x[i]);
-        (&s_o[0][0])[e] = make_float2(D[i] * r_x[i], gate_silu<T>(r_z[i]));
+        const float dt = r_dt[i] == -INFINITY ? 0.f : gate_softplus<T>(r_dt[i]), x = ldf<T>(&r_x[i]);
+        (&s_d[0][0])[e] = make_float2(dt, dt * x);
+        (&s_o[0][0])[e] = make_float2(D[i] * x, gate_silu<T>(ldf<T>(&r_z[i])));
       }
     }
     __syncthreads();

@@ -1064,6 +1064,8 @@ static int stack_run_hyper(StackEngine* s, int r, float* x, int n_tok, cudaStrea
     p.slot = s->m_slot; p.pos = s->m_pos; p.n_tok = n_tok;
     p.mid = s->mid; p.ld_mid = L.k_out; p.n_pad = right_off; p.out_scale = L.left_scale;
     if ((rc = launch_pool_prep(p, dt, st)) != B200_OK) return rc;
+    p.seg_row0 = s->m_seg_row0; p.seg_count = s->m_seg_count; p.n_seg = (int)s->segs.size();
+    for (const StackEngine::Seg& g : s->segs) p.max_count = std::max(p.max_count, g.count);
     if (!single && (rc = launch_pool_blocks(p, dt, st)) != B200_OK) return rc;
     if (L.pool.conv_w != nullptr) keep_rows(s->proj, false, L.n_in, L.n_in, L.pool.taps - 1, state + hs.pool_conv);
     if ((rc = stack_pool_attention(s, p, st)) != B200_OK) return rc;

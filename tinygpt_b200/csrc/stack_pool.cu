@@ -161,14 +161,15 @@ __global__ void __launch_bounds__(256) pool_prep_strip_kernel(const PoolAttn p) 
   }
 }
 
-// Rows whose position ends a block: the means of the block's cached keys and values (rows of this step or of earlier ones).
+// The blocks whose last position is among a sequence's rows of this step: the means of their cached keys and values (rows of
+// this step or of earlier ones).
 template <typename T>
 __global__ void __launch_bounds__(256) pool_blocks_kernel(const PoolAttn p) {
   pdl_trigger();
   pdl_wait();
-  const int t = blockIdx.x, P = p.d.pool, ps = p.pos[t];
-  if ((ps + 1) % P != 0) return;
-  const int b = ps / P, nk = p.a.kv_heads * p.a.dim, nv = p.a.kv_heads * p.a.vdim, e = blockIdx.y * 256 + threadIdx.x;
+  const int t = p.seg_row0[blockIdx.z], P = p.d.pool, ps = p.pos[t], b = ps / P + blockIdx.x;
+  if (b >= (ps + p.seg_count[blockIdx.z]) / P) return;
+  const int nk = p.a.kv_heads * p.a.dim, nv = p.a.kv_heads * p.a.vdim, e = blockIdx.y * 256 + threadIdx.x;
   if (e >= nk + nv) return;
   const bool key = e < nk;
   const int n = key ? nk : nv, i = key ? e : e - nk;
@@ -443,7 +444,8 @@ int launch_pool_blocks(const PoolAttn& p, int dtype, cudaStream_t st) {
   int rc = check_pool(p);
   if (rc != B200_OK) return rc;
   if (p.d.pool <= 0) return B200_OK;
-  const dim3 bg(p.n_tok, (p.a.kv_heads * (p.a.dim + p.a.vdim) + 255) / 256);
+  B200_CHECK_ARG(p.seg_row0 && p.seg_count && p.n_seg > 0 && p.max_count > 0, "pool blocks: null sequences");
+  const dim3 bg(p.max_count / p.d.pool + 1, (p.a.kv_heads * (p.a.dim + p.a.vdim) + 255) / 256, p.n_seg);
   if (dtype == B200_F32) B200_CUDA(launch_pdl(pool_blocks_kernel<float>, bg, dim3(256), 0, st, stack_pdl(), p));
   else B200_CUDA(launch_pdl(pool_blocks_kernel<__nv_bfloat16>, bg, dim3(256), 0, st, stack_pdl(), p));
   return B200_OK;

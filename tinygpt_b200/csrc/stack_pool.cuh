@@ -14,7 +14,6 @@ namespace b200 {
 
 constexpr int kPoolMaxSplits = 64;
 constexpr int kPoolTile = 32;          // keys per tile of the general kernels
-constexpr int kPoolSplitRows = 8;      // most rows a split-key launch serves
 
 struct PoolAttn {
   b200_attn_desc a{};
@@ -35,6 +34,9 @@ struct PoolAttn {
   const int32_t* slot = nullptr;
   const int32_t* pos = nullptr;
   int n_tok = 0;
+  // the step's sequences (launch_pool_blocks): first row and row count of each, the most rows any of them brings
+  const int32_t *seg_row0 = nullptr, *seg_count = nullptr;
+  int n_seg = 0, max_count = 0;
   // attention workspaces: scores [n_tok][heads][nk_max], softmax parts [n_tok][heads][nsplit][2], outputs
   // [n_tok][nsplit][heads·vdim] (nsplit > 1), all fp32; nk_max >= every row's key list, nsplit · keys_per_split >= nk_max
   float *scores = nullptr, *parts = nullptr, *outs = nullptr;

@@ -579,7 +579,7 @@ def fast_config():
     """Sizes that reach the bf16 engines' fast paths: tcgen05 products (multiples of 8, 64 and up) also for the bottlenecks and
     the experts, the tensor-core prompt attention (head sizes on multiples of 16; one and two warps' worth of heads; value
     columns split over CTAs), split-key decode."""
-    return config([(parallel(heads=8, kv_heads=4, dim=48, vdim=80, window=48, pool=8, rot_dims=32, right={"heads": 4, "dim": 32, "rank": 64}), moe(4, 2, 64, 128)),
+    return config([(parallel(heads=10, kv_heads=5, dim=48, vdim=112, window=40, pool=6, conv=4, rot_dims=32, right={"heads": 4, "dim": 32, "rank": 64}), moe(4, 2, 64, 96)),
                    (mamba(inner=256, state=16, dt_rank=64, conv=4), ff(256)), (wkv(heads=2, dim=64, rank=64), moe(4, 2, 64, 64)),
                    (parallel(heads=24, kv_heads=8, dim=16, vdim=96, window=70, pool=16, rot_dims=16, right={"heads": 2, "dim": 64, "rank": 24}), ff(128)),
                    (parallel(heads=4, kv_heads=2, dim=128, vdim=144, window=33, pool=4, rot_dims=128, right={"heads": 2, "dim": 64, "rank": 24}), None)],

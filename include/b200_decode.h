@@ -36,9 +36,11 @@ extern "C" {
  * generalized delta rule, Mamba-2, softmax-routed experts (fields appended to b200_moe_desc and b200_stack_layer),
  * b200_stack_lin_scan, b200_stack_attn_prep;  8: + hyper-connected blocks, Mamba's selective scan, RWKV-style time mixing, the
  * pooled-block attention (fields appended to b200_moe_desc, b200_stack_layer and b200_stack_desc), b200_stack_hyper_step,
- * b200_stack_input_conv, b200_stack_pool_attention, b200_stack_bonus_scan, b200_stack_mamba1_scan.  All additive: callers of an older version
- * keep working once they are compiled against this header. */
-#define B200_ABI_VERSION 8
+ * b200_stack_input_conv, b200_stack_pool_attention, b200_stack_bonus_scan, b200_stack_mamba1_scan;  9: + gated linear attention
+ * (b200_gla_desc), capped scores, distance biases and values that are the keys (fields appended to b200_attn_desc), short
+ * convolutions and per-head norms in front of any attention (fields appended to b200_attn_prep_desc and b200_pool_attn_desc),
+ * gated feed-forwards in sandwich blocks.  All additive: callers of an older version keep working once they are compiled against this header. */
+#define B200_ABI_VERSION 9
 
 typedef enum b200_status {
   B200_OK = 0,
@@ -320,15 +322,18 @@ typedef enum b200_norm_kind { B200_NORM_RMS = 0, B200_NORM_LAYER = 1 } b200_norm
  * per-token preparation of b200_attn_prep_desc (query / key norms, rotary positions, value norm, value mix-in).
  * GATED_DELTA: the gated delta rule — a key × value matrix per head with one decay per head and a removal along the unit
  * key weighted by a per-head write strength, behind short causal convolutions (b200_gdelta_desc).
+ * GLA: gated linear attention — a key × value matrix per head with a decay per key channel (b200_gla_desc); sandwich blocks.
  * In hyper-connected blocks: MAMBA1: a selective scan with a decay per channel and state entry (b200_mamba1_desc).  WKV: time
  * mixing with a decay per key channel and a bonus for the current token (b200_wkv_desc).  POOL_ATTENTION: attention behind
  * short convolutions, with pooled blocks behind its window and mixed heads (b200_pool_attn_desc).  PARALLEL: left_scale ·
  * (a POOL_ATTENTION) + right_scale · (a WKV) over the same input. */
 typedef enum b200_mixer_kind {
   B200_MIX_ATTENTION = 0, B200_MIX_LATENT = 1, B200_MIX_MLSTM = 2, B200_MIX_DELTA = 3, B200_MIX_MAMBA2 = 4,
-  B200_MIX_GATED_DELTA = 5, B200_MIX_MAMBA1 = 6, B200_MIX_WKV = 7, B200_MIX_POOL_ATTENTION = 8, B200_MIX_PARALLEL = 9
+  B200_MIX_GATED_DELTA = 5, B200_MIX_MAMBA1 = 6, B200_MIX_WKV = 7, B200_MIX_POOL_ATTENTION = 8, B200_MIX_PARALLEL = 9,
+  B200_MIX_GLA = 10
 } b200_mixer_kind;
-/* GATED: act(gate)·up → down (merged into w_in / w_out).  DENSE: act(up) → down.  MOE: routed clamped gated experts
+/* GATED: act(gate)·up → down (parallel blocks: merged into w_in / w_out; sandwich blocks: w_ff_in [2·ff, width] = [gate | up],
+ * w_ff_out [width, ff]).  DENSE: act(up) → down.  MOE: routed clamped gated experts
  * (+ optional gated shared expert), b200_moe_desc.  GLU_CLAMP: one clamped gated unit, g = min(gate·h, limit),
  * u = clamp(up·h, ±limit), down·(g·sigmoid(1.702 g)·(u + 1)) (hyper-connected blocks). */
 typedef enum b200_ff_kind { B200_FF_GATED = 0, B200_FF_DENSE = 1, B200_FF_MOE = 2, B200_FF_GLU_CLAMP = 3 } b200_ff_kind;
@@ -343,6 +348,10 @@ typedef struct b200_attn_desc {
   int32_t keep_first;  /* keys j < keep_first stay visible whatever the window */
   int32_t out_gate;    /* 1: head output × sigmoid(gate logit of that head) */
   int32_t sink;        /* 1: the softmax's denominator gains 1 — a sink of score 0 that has no value */
+  float softcap;       /* > 0: score <- softcap·tanh(score / softcap) */
+  const float* slopes; /* [heads] (device) or NULL; then score <- score − slopes[head]·(i − j), the distance of query i to key j */
+  int32_t values_are_keys; /* 1: the value heads are the key heads (vdim = dim): no value rows in w_in, no value cache.  Sandwich
+                        * blocks */
 } b200_attn_desc;
 
 /* Latent attention (sizes heads / dim / vdim / scale / window in b200_attn_desc; kv_heads = 1, no per-head gate).  Per head the
@@ -413,6 +422,11 @@ typedef struct b200_attn_prep_desc {
   const float* rot_table;   /* [max_ctx][rot_dims/2][2] fp32 */
   const float* mix_lambda;  /* [1] */
   int32_t rot_interleaved;  /* 1: pair i is entries (2i, 2i+1) of the head instead of (i, i + rot_dims/2) */
+  /* sandwich blocks: a short convolution in front of norms and rotation, and norms per head */
+  int32_t head_norm;        /* 1: every query / key head is RMS-normed by itself and multiplied by q_norm / k_norm [dim], shared by
+                             * the heads (qk_norm = 0) */
+  int32_t taps;             /* taps of the causal convolution every channel of q, k and v passes (zeros before the sequence) */
+  const float* conv_w;      /* [taps][n_in]: row taps − 1 meets the current token; columns are rows of w_in.  NULL: none */
 } b200_attn_prep_desc;
 
 /* Generalized delta rule (sizes heads / dim / vdim in b200_attn_desc).  w_in rows [r | k | v | out gate: heads·vdim |
@@ -485,6 +499,7 @@ typedef struct b200_pool_attn_desc {
   const float* rot_table;   /* [max_ctx][rot_dims/2][2] fp32 */
   const float* sink;        /* [heads] or NULL */
   const float* talk;        /* [heads][heads] or NULL */
+  int32_t rot_interleaved;  /* 1: entry 2i turns with entry 2i + 1 */
 } b200_pool_attn_desc;
 
 /* RWKV-style time mixing.  Five blends of the mixer's input with the previous token's, mix_s = h + (h' − h)·mu_s for
@@ -517,6 +532,18 @@ typedef struct b200_mamba1_desc {
   const float* A_log;       /* [inner][state] */
   const float* D;           /* [inner] */
 } b200_mamba1_desc;
+
+/* Gated linear attention (heads, dim, vdim in b200_attn_desc).  w_in rows [q: heads·dim | k: heads·dim | v: heads·vdim | out gate:
+ * heads·vdim | decay bottleneck: rank] at off_q / off_k / off_v / off_g / off_up.  Per head and key channel the decay is
+ * alpha = sigmoid(a2·bottleneck + a2_b)^(1/tau);  S <- diag(alpha) S + k vᵀ,  o = Sᵀ(q·dim^(−1/2));  then o / rms(o) per head ·
+ * head_norm · silu(out gate).  The state S (fp32) lives in the slot. */
+typedef struct b200_gla_desc {
+  int32_t rank;
+  float tau;
+  const void* a2;           /* [heads·dim, up8(rank)] (padding columns zero) */
+  const float* a2_b;        /* [heads·dim] */
+  const float* head_norm;   /* [vdim], shared by the heads */
+} b200_gla_desc;
 
 typedef struct b200_stack_layer {
   b200_attn_desc attn;
@@ -565,6 +592,7 @@ typedef struct b200_stack_layer {
   b200_pool_attn_desc pool;
   b200_wkv_desc wkv;
   b200_mamba1_desc mamba1;
+  b200_gla_desc gla;
 } b200_stack_layer;
 
 typedef struct b200_stack_desc {

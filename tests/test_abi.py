@@ -62,7 +62,7 @@ def test_stack_struct_layouts_match_the_compiler(built_lib, tmp_path):
     from tinygpt_b200 import _lib
     src = tmp_path / "sz.c"
     src.write_text('#include <stdio.h>\n#include <stddef.h>\n#include "b200_decode.h"\n'
-                   'int main(void) { printf("%zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu\\n", sizeof(b200_attn_desc), '
+                   'int main(void) { printf("%zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu\\n", sizeof(b200_attn_desc), '
                    'sizeof(b200_stack_layer), sizeof(b200_stack_desc), offsetof(b200_stack_layer, side_norm), '
                    'offsetof(b200_stack_desc, layers_host), offsetof(b200_stack_layer, w_out), sizeof(b200_latent_desc), '
                    'sizeof(b200_mlstm_desc), sizeof(b200_moe_desc), offsetof(b200_stack_layer, moe), '
@@ -72,7 +72,9 @@ def test_stack_struct_layouts_match_the_compiler(built_lib, tmp_path):
                    'offsetof(b200_stack_layer, kv_share), offsetof(b200_latent_desc, out_gate), '
                    'offsetof(b200_attn_prep_desc, rot_interleaved), sizeof(b200_hyper_desc), sizeof(b200_pool_attn_desc), '
                    'sizeof(b200_wkv_desc), sizeof(b200_mamba1_desc), offsetof(b200_stack_layer, canon_w), '
-                   'offsetof(b200_stack_layer, mamba1), offsetof(b200_stack_desc, streams), offsetof(b200_moe_desc, expert_gated)); '
+                   'offsetof(b200_stack_layer, mamba1), offsetof(b200_stack_desc, streams), offsetof(b200_moe_desc, expert_gated), '
+                   'offsetof(b200_attn_desc, slopes), offsetof(b200_attn_desc, values_are_keys), offsetof(b200_attn_prep_desc, conv_w), '
+                   'offsetof(b200_pool_attn_desc, rot_interleaved), sizeof(b200_gla_desc), offsetof(b200_stack_layer, gla)); '
                    'return 0; }\n')
     exe = tmp_path / "sz"
     subprocess.run(["gcc", "-I", str(ROOT / "include"), str(src), "-o", str(exe)], check=True)
@@ -85,7 +87,9 @@ def test_stack_struct_layouts_match_the_compiler(built_lib, tmp_path):
             _lib.StackLayer.gdelta.offset, _lib.StackLayer.kv_share.offset, _lib.LatentDesc.out_gate.offset,
             _lib.AttnPrepDesc.rot_interleaved.offset, C.sizeof(_lib.HyperDesc), C.sizeof(_lib.PoolAttnDesc), C.sizeof(_lib.WkvDesc),
             C.sizeof(_lib.Mamba1Desc), _lib.StackLayer.canon_w.offset, _lib.StackLayer.mamba1.offset, _lib.StackDesc.streams.offset,
-            _lib.MoeDesc.expert_gated.offset]
+            _lib.MoeDesc.expert_gated.offset, _lib.AttnDesc.slopes.offset, _lib.AttnDesc.values_are_keys.offset,
+            _lib.AttnPrepDesc.conv_w.offset, _lib.PoolAttnDesc.rot_interleaved.offset, C.sizeof(_lib.GlaDesc),
+            _lib.StackLayer.gla.offset]
     assert got == want
 
 

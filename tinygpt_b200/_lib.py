@@ -38,7 +38,7 @@ class WeightTable(C.Structure):
 class AttnDesc(C.Structure):
     _fields_ = [("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32),
                 ("scale", C.c_float), ("window", C.c_int32), ("keep_first", C.c_int32), ("out_gate", C.c_int32),
-                ("sink", C.c_int32)]
+                ("sink", C.c_int32), ("softcap", C.c_float), ("slopes", C.c_void_p), ("values_are_keys", C.c_int32)]
 
 
 class LatentDesc(C.Structure):
@@ -63,7 +63,7 @@ class MoeDesc(C.Structure):
 class AttnPrepDesc(C.Structure):
     _fields_ = [("qk_norm", C.c_int32), ("rot_dims", C.c_int32), ("v_norm", C.c_int32), ("v_mix", C.c_int32),
                 ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("rot_table", C.c_void_p), ("mix_lambda", C.c_void_p),
-                ("rot_interleaved", C.c_int32)]
+                ("rot_interleaved", C.c_int32), ("head_norm", C.c_int32), ("taps", C.c_int32), ("conv_w", C.c_void_p)]
 
 
 class DeltaDesc(C.Structure):
@@ -89,7 +89,7 @@ class HyperDesc(C.Structure):
 class PoolAttnDesc(C.Structure):
     _fields_ = [("taps", C.c_int32), ("rot_dims", C.c_int32), ("pool", C.c_int32), ("softcap", C.c_float),
                 ("conv_w", C.c_void_p), ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("rot_table", C.c_void_p),
-                ("sink", C.c_void_p), ("talk", C.c_void_p)]
+                ("sink", C.c_void_p), ("talk", C.c_void_p), ("rot_interleaved", C.c_int32)]
 
 
 class WkvDesc(C.Structure):
@@ -101,6 +101,10 @@ class Mamba1Desc(C.Structure):
     _fields_ = [("inner", C.c_int32), ("state", C.c_int32), ("dt_rank", C.c_int32), ("taps", C.c_int32),
                 ("conv_w", C.c_void_p), ("conv_b", C.c_void_p), ("w_x", C.c_void_p), ("w_dt", C.c_void_p), ("dt_b", C.c_void_p),
                 ("A_log", C.c_void_p), ("D", C.c_void_p)]
+
+
+class GlaDesc(C.Structure):
+    _fields_ = [("rank", C.c_int32), ("tau", C.c_float), ("a2", C.c_void_p), ("a2_b", C.c_void_p), ("head_norm", C.c_void_p)]
 
 
 class StackLayer(C.Structure):
@@ -117,7 +121,8 @@ class StackLayer(C.Structure):
                 ("prep", AttnPrepDesc), ("delta", DeltaDesc), ("mamba", MambaDesc), ("gdelta", GatedDeltaDesc),
                 ("b_out", C.c_void_p), ("kv_share", C.c_int32),
                 ("hc1", HyperDesc), ("hc2", HyperDesc), ("canon_taps", C.c_int32), ("canon_w", C.c_void_p), ("ff_limit", C.c_float),
-                ("left_scale", C.c_float), ("right_scale", C.c_float), ("pool", PoolAttnDesc), ("wkv", WkvDesc), ("mamba1", Mamba1Desc)]
+                ("left_scale", C.c_float), ("right_scale", C.c_float), ("pool", PoolAttnDesc), ("wkv", WkvDesc), ("mamba1", Mamba1Desc),
+                ("gla", GlaDesc)]
 
 
 class StackDesc(C.Structure):

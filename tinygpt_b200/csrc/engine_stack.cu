@@ -35,7 +35,10 @@
 //
 // Sandwich blocks also take the prepared attention (biases, either rotary layout, a sink in the softmax; a layer may read the
 // keys and values an earlier layer cached instead of projecting its own), the latent attention with a query latent, a
-// sliding window and an element-wise output gate, and the gated delta rule behind short convolutions.
+// sliding window and an element-wise output gate, the gated delta rule behind short convolutions, gated linear attention, and
+// gated feed-forwards.  Their attention may pass short convolutions and per-head norms first (the preparation of the pooled-block
+// attention: queries to a buffer of their own, keys and values straight to the cache), cap its scores, take a distance bias off
+// them, and use its keys as values.
 //
 // Per run of a layer (hyper-connected block: `streams` copies of the stream):
 //   one pass per sublayer boundary: x_d <- Σ mix·x_s + m·out_d·y of the sublayer before, u = Σ in_s·x_s, n = norm(u)·(offset + w)
@@ -460,7 +463,7 @@ static int stack_product_head(StackEngine* s, const float* x, const int32_t* row
   return launch_stack_gemm(g, s->dtype, st);
 }
 
-// Attention of a run over the step's rows.  bf16 engines with equal key / value head sizes of 64 or 128 send every
+// Attention of a run over the step's rows.  bf16 engines with equal key / value head sizes of 64, 96 or 128 send every
 // sequence that brings kTcRows rows or more to the tensor-core kernel (prefill_attn.cu), one launch per sequence; what is
 // left (short parts, decode tokens, other head sizes, fp32) goes to the general kernel, with the keys split over CTAs when
 // the step is a handful of rows over a long key list.
@@ -486,7 +489,7 @@ static int stack_attention(StackEngine* s, const StackAttn& a, const b200_stack_
     }
     return launch_stack_attention(q, dt, st);
   };
-  const bool tc = s->fast && d.dim == d.vdim && (d.dim == 64 || d.dim == 128);
+  const bool tc = s->fast && d.dim == d.vdim && prefill_window_ok(d.dim);
   bool any = false;
   for (const StackEngine::Seg& g : s->segs) any = any || g.count >= kTcRows;
   if (!tc || !any) return general(0, a.n_tok);
@@ -500,7 +503,8 @@ static int stack_attention(StackEngine* s, const StackAttn& a, const b200_stack_
                                          d.out_gate ? prow + a.off_g : nullptr, a.ld_proj,
                                          (const __nv_bfloat16*)a.kcache + (size_t)g.slot * a.k_slot_stride,
                                          (const __nv_bfloat16*)a.vcache + (size_t)g.slot * a.v_slot_stride, g.count, d.heads,
-                                         d.kv_heads, d.dim, g.pos0, d.scale, d.window, d.keep_first, st, d.sink)) != B200_OK)
+                                         d.kv_heads, d.dim, g.pos0, d.scale, d.window, d.keep_first, st, d.sink, d.softcap,
+                                         d.slopes)) != B200_OK)
       return rc;
   }
   return B200_OK;
@@ -656,6 +660,9 @@ static int stack_moe_ff(StackEngine* s, const b200_stack_layer& L, const StackEn
   return run_moe(m, dt, st);
 }
 
+// An attention mixer whose q, k and v pass short convolutions or norms per head
+static inline bool stack_head_prep(const b200_stack_layer& L) { return L.prep.head_norm || L.prep.conv_w != nullptr; }
+
 static int stack_run_sandwich(StackEngine* s, int r, float* x, int n_tok, cudaStream_t st) {
   const b200_stack_desc& d = s->d;
   const int li = s->run_layer[r];
@@ -665,7 +672,7 @@ static int stack_run_sandwich(StackEngine* s, int r, float* x, int n_tok, cudaSt
   const size_t esz = s->esz;
   int rc;
   // every sublayer's post-norm hands the next sublayer its normed input in the same pass; only the first run norms alone
-  const bool has_ff = !(L.ff_kind == B200_FF_DENSE && L.ff <= 0);
+  const bool has_ff = !(L.ff_kind != B200_FF_MOE && L.ff <= 0);
   // sandwich blocks norm the stream in front of every sublayer; post-norm blocks hand the sublayer the stream itself —
   // fp32 engines read it in place, bf16 engines its rounded copy in h (left there by the previous post-norm pass)
   const bool pre = d.block == B200_BLOCK_SANDWICH;
@@ -711,9 +718,11 @@ static int stack_run_sandwich(StackEngine* s, int r, float* x, int n_tok, cudaSt
   if (!s->segs.empty()) {
     seq.n_seg = (int)s->segs.size(); seq.seg_row0 = s->m_seg_row0; seq.seg_count = s->m_seg_count;
   }
+  bool single = true;   // every row is its sequence's only new one
+  for (const StackEngine::Seg& g : s->segs) single = single && g.count == 1;
   if (L.mixer == B200_MIX_ATTENTION) {
     const bool shared_kv = s->run_kv_shared[r] != 0;   // the keys and values of these positions are in another run's cache already
-    if (L.prep.qk_norm || L.prep.rot_dims > 0 || L.prep.v_norm || L.prep.v_mix) {
+    if (!stack_head_prep(L) && (L.prep.qk_norm || L.prep.rot_dims > 0 || L.prep.v_norm || L.prep.v_mix)) {
       AttnPrep ap;
       ap.a = L.attn; ap.d = L.prep; ap.eps = d.norm_eps;
       ap.proj = s->proj; ap.ld_proj = L.n_in; ap.off_q = L.off_q; ap.off_k = L.off_k; ap.off_v = L.off_v;
@@ -728,12 +737,40 @@ static int stack_run_sandwich(StackEngine* s, int r, float* x, int n_tok, cudaSt
     a.kcache = s->kbase + s->run_k_off[r] * esz;
     a.vcache = s->vbase + s->run_v_off[r] * esz;
     a.k_slot_stride = (int64_t)s->k_slot; a.v_slot_stride = (int64_t)s->v_slot;
+    if (L.attn.values_are_keys) {
+      a.vcache = a.kcache; a.v_slot_stride = a.k_slot_stride; a.off_v = a.off_k;
+    }
     a.slot = s->m_slot; a.pos = s->m_pos; a.n_tok = n_tok;
     a.out = s->mid; a.ld_out = L.k_out;
-    bool single = true;   // decode steps append K/V inside the attention launch
-    for (const StackEngine::Seg& g : s->segs) single = single && g.count == 1;
-    a.own_from_proj = single && !shared_kv ? 1 : 0;
-    if (!a.own_from_proj && !shared_kv && (rc = launch_stack_kv_store(a, dt, st)) != B200_OK) return rc;
+    const bool head_prep = stack_head_prep(L);
+    if (head_prep) {   // queries go to rows of their own, keys and values straight to the cache
+      PoolAttn p;
+      p.a = L.attn; p.eps = d.norm_eps;
+      p.d.taps = L.prep.taps; p.d.conv_w = L.prep.conv_w;
+      p.d.q_norm = L.prep.head_norm ? L.prep.q_norm : nullptr; p.d.k_norm = L.prep.head_norm ? L.prep.k_norm : nullptr;
+      p.d.rot_dims = L.prep.rot_dims; p.d.rot_table = L.prep.rot_table; p.d.rot_interleaved = L.prep.rot_interleaved;
+      p.proj = s->proj; p.ld_proj = L.n_in; p.off_q = L.off_q; p.off_k = L.off_k; p.off_v = L.off_v;
+      p.q = s->qa; p.q_only = shared_kv ? 1 : 0;
+      p.kcache = a.kcache; p.vcache = a.vcache; p.k_slot_stride = a.k_slot_stride; p.v_slot_stride = a.v_slot_stride; p.max_ctx = d.max_ctx;
+      p.conv_state = s->rstate + s->run_s_off[r]; p.conv_slot_stride = (int64_t)s->s_slot;
+      p.single = single ? 1 : 0;
+      p.slot = s->m_slot; p.pos = s->m_pos; p.n_tok = n_tok;
+      if ((rc = launch_pool_prep(p, dt, st)) != B200_OK) return rc;
+      if (!single && L.prep.conv_w != nullptr && L.prep.taps > 1) {   // the convolutions' last inputs move on
+        ShiftState shift;
+        shift.seg_row0 = s->m_seg_row0; shift.seg_count = s->m_seg_count; shift.slot = s->m_slot; shift.pos = s->m_pos;
+        shift.n_seg = (int)s->segs.size(); shift.slot_stride = (int64_t)s->s_slot;
+        shift.src[shift.n_src++] = ShiftSource{s->proj, false, L.n_in, L.n_in, L.prep.taps - 1, p.conv_state};
+        if ((rc = launch_shift_state(shift, dt, st)) != B200_OK) return rc;
+      }
+      a.proj = s->qa; a.ld_proj = (int64_t)L.attn.heads * L.attn.dim;
+      a.off_q = a.off_k = a.off_v = 0;
+    }
+    // decode steps append K/V inside the attention launch, unless they are in the cache already
+    const bool cached = shared_kv || head_prep;
+    a.own_from_proj = single && !cached ? 1 : 0;
+    a.own_cached = single && cached ? 1 : 0;
+    if (!a.own_from_proj && !cached && (rc = launch_stack_kv_store(a, dt, st)) != B200_OK) return rc;
     if ((rc = stack_attention(s, a, L, st)) != B200_OK) return rc;
   } else if (L.mixer == B200_MIX_GATED_DELTA) {
     const int H = L.attn.heads, G = L.attn.kv_heads;
@@ -749,6 +786,19 @@ static int stack_run_sandwich(StackEngine* s, int r, float* x, int n_tok, cudaSt
     m.scan.o = s->rec_o; m.scan.ld_o = (int64_t)H * L.attn.vdim;
     m.mid = s->mid; m.ld_mid = L.k_out;
     if ((rc = run_gdelta(m, dt, st)) != B200_OK) return rc;
+  } else if (L.mixer == B200_MIX_GLA) {
+    GlaRun m;
+    m.a = L.attn; m.d = L.gla; m.eps = d.norm_eps;
+    m.proj = s->proj; m.ld_proj = L.n_in;
+    m.off_q = L.off_q; m.off_k = L.off_k; m.off_v = L.off_v; m.off_g = L.off_g; m.off_a = L.off_up;
+    m.single = single ? 1 : 0;
+    m.f = s->rec_f;
+    m.scan = seq;
+    m.scan.ld = gla_row_floats(L.attn.heads, L.attn.dim, L.attn.vdim);
+    m.scan.state = s->rstate + s->run_s_off[r]; m.scan.slot_stride = (int64_t)s->s_slot;
+    m.scan.o = s->rec_o; m.scan.ld_o = (int64_t)L.attn.heads * L.attn.vdim;
+    m.mid = s->mid; m.ld_mid = L.k_out;
+    if ((rc = run_gla(m, dt, st)) != B200_OK) return rc;
   } else if (L.mixer == B200_MIX_DELTA) {
     const int H = L.attn.heads, hd = H * L.attn.dim, rk = up8i(L.delta.rank);
     // decay logits: tanh of the bottleneck rows (T), then w2·(…) + w0 in fp32
@@ -884,6 +934,13 @@ static int stack_run_sandwich(StackEngine* s, int r, float* x, int n_tok, cudaSt
     if ((rc = stack_lin(s, hin, L.w_ff_in, nullptr, n_tok, L.ff, W, pl.ok_ff_in ? &pl.ff_in : nullptr, s->proj, nullptr, st)) != B200_OK)
       return rc;
     if ((rc = launch_stack_act_mul(s->mid, L.ff, s->proj, nullptr, L.ff, n_tok, L.ff, L.ff_act, dt, st)) != B200_OK) return rc;
+    return stack_lin_norm_add(s, s->mid, L.w_ff_out, n_tok, L.ff, pl.ok_ff_out ? &pl.ff_out : nullptr, L.ff_post_norm, x,
+                              next_run_w, st);
+  }
+  if (L.ff_kind == B200_FF_GATED) {
+    if ((rc = stack_lin(s, hin, L.w_ff_in, nullptr, n_tok, 2 * L.ff, W, pl.ok_ff_in ? &pl.ff_in : nullptr, s->proj, nullptr, st)) != B200_OK)
+      return rc;
+    if ((rc = launch_stack_glu(s->mid, L.ff, s->proj, 2 * L.ff, n_tok, L.ff, L.ff_act, dt, st)) != B200_OK) return rc;
     return stack_lin_norm_add(s, s->mid, L.w_ff_out, n_tok, L.ff, pl.ok_ff_out ? &pl.ff_out : nullptr, L.ff_post_norm, x,
                               next_run_w, st);
   }
@@ -1483,7 +1540,10 @@ int64_t stack_bytes_per_token(const b200_engine* e, int64_t ctx) {
       if (L.mixer == B200_MIX_ATTENTION) {
         int64_t keys = ctx + 1;
         if (a.window > 0) keys = std::min<int64_t>(keys, (int64_t)a.window + a.keep_first);
-        bytes += (keys + 1) * a.kv_heads * (a.dim + a.vdim) * s->esz;
+        bytes += (keys + 1) * a.kv_heads * (a.dim + (a.values_are_keys ? 0 : a.vdim)) * s->esz;
+        if (L.prep.conv_w != nullptr) bytes += 2ll * (L.prep.taps - 1) * L.n_in * 4;
+      } else if (L.mixer == B200_MIX_GLA) {   // the decay's second stage; the state read and written
+        bytes += (int64_t)a.heads * a.dim * L.gla.rank * s->esz + 2ll * a.heads * a.dim * a.vdim * 4;
       } else if (L.mixer == B200_MIX_GATED_DELTA) {   // the state and the convolutions' inputs read and written
         bytes += 2 * gdelta_state_floats(a.heads, a.kv_heads, a.dim, a.vdim, L.gdelta.taps) * 4;
       } else if (L.mixer == B200_MIX_DELTA) {   // the decay's second stage; the state read and written
@@ -1499,6 +1559,7 @@ int64_t stack_bytes_per_token(const b200_engine* e, int64_t ctx) {
       else                              // the state read and written
         bytes += 2 * mlstm_state_floats(a.heads, a.dim, a.vdim) * 4;
       if (L.ff_kind == B200_FF_DENSE) bytes += 2ll * L.ff * d.width * s->esz;
+      else if (L.ff_kind == B200_FF_GATED) bytes += 3ll * L.ff * d.width * s->esz;
       else if (L.moe.expert_act != 0) bytes += ((int64_t)L.moe.experts + 2ll * L.moe.top * L.moe.expert_ff + 2ll * L.moe.shared_ff) * d.width * s->esz;
       else bytes += ((int64_t)L.moe.experts + 3ll * L.moe.top * L.moe.expert_ff + 3ll * L.moe.shared_ff + 1) * d.width * s->esz;
       continue;
@@ -1540,7 +1601,7 @@ static int stack_check_hyper(StackEngine* s, int l) {
                        (q.q_norm == nullptr) == (q.k_norm == nullptr) &&
                        (q.conv_w == nullptr || (q.taps >= 1 && q.taps <= kConvMaxTaps)),
                    "engine_create_stack: layer %d: attention preparation", l);
-    B200_CHECK_ARG((size_t)((a.heads / a.kv_heads + 1) * a.dim + a.vdim) * 4 <= 48 * 1024 && (size_t)a.heads * a.dim * 4 <= 200 * 1024 &&
+    B200_CHECK_ARG((size_t)(2 * a.dim + a.vdim) * 4 <= 48 * 1024 && !a.slopes && !a.values_are_keys && a.softcap == 0.f && (size_t)a.heads * a.dim * 4 <= 200 * 1024 &&
                        (size_t)(2 * a.heads + 2 * a.heads * (kPoolTile + 1) + a.heads * a.vdim) * 4 <= 200 * 1024,
                    "engine_create_stack: layer %d: heads · head size above one CTA's shared memory", l);
     st.pool_conv = st.total;
@@ -1611,6 +1672,11 @@ static int stack_check_hyper(StackEngine* s, int l) {
   return B200_OK;
 }
 
+// floats of a slot that hold the last inputs of an attention run's convolutions
+static size_t stack_conv_floats(const b200_stack_layer& L) {
+  return L.prep.conv_w != nullptr && L.prep.taps > 1 ? ((size_t)(L.prep.taps - 1) * L.n_in + 3) / 4 * 4 : 0;
+}
+
 static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
   B200_CHECK_ARG(desc && out, "engine_create_stack: null argument");
   *out = nullptr;
@@ -1669,7 +1735,10 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
     const b200_stack_layer& L = s->layers[l];
     const b200_attn_desc& a = L.attn;
     const int W = d.width;
-    B200_CHECK_ARG(L.mixer >= B200_MIX_ATTENTION && L.mixer <= B200_MIX_GATED_DELTA, "engine_create_stack: layer %d: mixer kind %d is not built", l, L.mixer);
+    B200_CHECK_ARG(d.block == B200_BLOCK_SANDWICH || (!a.values_are_keys && !a.slopes && a.softcap == 0.f),
+                   "engine_create_stack: layer %d: capped scores, distance biases and values that are the keys are built for sandwich blocks", l);
+    B200_CHECK_ARG((L.mixer >= B200_MIX_ATTENTION && L.mixer <= B200_MIX_GATED_DELTA) || (L.mixer == B200_MIX_GLA && d.block == B200_BLOCK_SANDWICH),
+                   "engine_create_stack: layer %d: mixer kind %d is not built", l, L.mixer);
     B200_CHECK_ARG(a.heads > 0 && a.dim > 0 && a.vdim > 0, "engine_create_stack: layer %d: bad mixer sizes", l);
     B200_CHECK_ARG((L.norm || d.block == B200_BLOCK_POSTNORM) && L.post_norm && L.w_in && L.w_out && L.n_in > 0 &&
                        L.k_out == a.heads * a.vdim,
@@ -1679,14 +1748,27 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
       B200_CHECK_ARG(a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.window >= 0 && a.keep_first >= 0 && a.vdim <= 256 && a.dim <= 1024,
                      "engine_create_stack: layer %d: bad attention sizes", l);
       B200_CHECK_ARG(L.off_q >= 0 && L.off_q + a.heads * a.dim <= L.n_in &&
-                         (L.kv_share > 0 || (L.off_k + a.kv_heads * a.dim <= L.n_in && L.off_v + a.kv_heads * a.vdim <= L.n_in)) &&
+                         (L.kv_share > 0 || (L.off_k + a.kv_heads * a.dim <= L.n_in && (a.values_are_keys || L.off_v + a.kv_heads * a.vdim <= L.n_in))) &&
                          (!a.out_gate || L.off_g + a.heads <= L.n_in),
                      "engine_create_stack: layer %d: segment offsets do not fit", l);
+      B200_CHECK_ARG(a.softcap >= 0.f && (!a.values_are_keys || a.vdim == a.dim),
+                     "engine_create_stack: layer %d: negative softcap, or values that are keys of another size", l);
+      if (stack_head_prep(L)) {
+        B200_CHECK_ARG(d.block == B200_BLOCK_SANDWICH && !a.out_gate && !a.values_are_keys && !q.qk_norm && !q.v_norm && !q.v_mix,
+                       "engine_create_stack: layer %d: convolutions and per-head norms are built for sandwich blocks without an output gate, norms over "
+                       "whole projections, value norms or values that are the keys", l);
+        B200_CHECK_ARG((q.conv_w == nullptr || (q.taps >= 1 && q.taps <= kConvMaxTaps)) && (!q.head_norm || (q.q_norm && (L.kv_share > 0 || q.k_norm))) &&
+                           (2 * a.dim + a.vdim) * 4 <= 48 * 1024,
+                       "engine_create_stack: layer %d: 1 … %d taps, head norms with their weights", l, kConvMaxTaps);
+        s->qa_max = std::max(s->qa_max, a.heads * a.dim);
+        if (q.conv_w != nullptr && q.taps > 1) s->recurrent = true;   // the last inputs cannot be rewound
+        s->any_rec = true;                                             // the step's sequences travel to the device
+      }
       if (L.kv_share > 0) {   // the source: an earlier attention layer with projections of its own and the same cache rows
         B200_CHECK_ARG(L.kv_share - 1 < l, "engine_create_stack: layer %d reads the keys and values of layer %d, which is not an earlier layer", l, L.kv_share - 1);
         const b200_stack_layer& S = s->layers[L.kv_share - 1];
         B200_CHECK_ARG(S.mixer == B200_MIX_ATTENTION && S.kv_share == 0 && S.attn.kv_heads == a.kv_heads && S.attn.dim == a.dim &&
-                           S.attn.vdim == a.vdim,
+                           S.attn.vdim == a.vdim && S.attn.values_are_keys == a.values_are_keys,
                        "engine_create_stack: layer %d: layer %d is not an attention layer with keys and values of its own and equal sizes", l, L.kv_share - 1);
         B200_CHECK_ARG(!q.v_norm && !q.v_mix, "engine_create_stack: layer %d: a layer without values of its own cannot norm or mix them", l);
       }
@@ -1712,6 +1794,16 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
                      "engine_create_stack: layer %d: segment offsets do not fit", l);
       s->rec_o_max = std::max(s->rec_o_max, a.heads * a.vdim);
       s->rec_f_max = std::max(s->rec_f_max, (int)gdelta_row_floats(a.heads, a.kv_heads, a.dim, a.vdim));
+      s->any_rec = s->recurrent = true;
+    } else if (L.mixer == B200_MIX_GLA) {
+      const b200_gla_desc& q = L.gla;
+      B200_CHECK_ARG(a.dim <= kScanMaxDim && q.rank > 0 && q.rank <= kGlaMaxRank && q.tau > 0.f && q.a2 && q.a2_b && q.head_norm,
+                     "engine_create_stack: layer %d: gated linear attention description (key size up to %d, bottleneck up to %d)", l, kScanMaxDim, kGlaMaxRank);
+      B200_CHECK_ARG(L.off_q >= 0 && L.off_q + a.heads * a.dim <= L.n_in && L.off_k + a.heads * a.dim <= L.n_in &&
+                         L.off_v + a.heads * a.vdim <= L.n_in && L.off_g + a.heads * a.vdim <= L.n_in && L.off_up + q.rank <= L.n_in,
+                     "engine_create_stack: layer %d: segment offsets do not fit", l);
+      s->rec_o_max = std::max(s->rec_o_max, a.heads * a.vdim);
+      s->rec_f_max = std::max(s->rec_f_max, (int)gla_row_floats(a.heads, a.dim, a.vdim));
       s->any_rec = s->recurrent = true;
     } else if (L.mixer == B200_MIX_DELTA) {
       const b200_delta_desc& q = L.delta;
@@ -1778,6 +1870,12 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
       B200_CHECK_ARG(L.ff_act >= B200_ACT_GELU_TANH && L.ff_act <= B200_ACT_TANH, "engine_create_stack: layer %d: activation %d", l,
                      L.ff_act);
       ff_rows = ff_mid = L.ff;
+    } else if (L.ff_kind == B200_FF_GATED && d.block == B200_BLOCK_SANDWICH) {
+      B200_CHECK_ARG(L.ff >= 0 && (L.ff == 0 || (L.ff_norm && L.ff_post_norm && L.w_ff_in && L.w_ff_out)) && L.ff_act >= B200_ACT_GELU_TANH &&
+                         L.ff_act <= B200_ACT_TANH,
+                     "engine_create_stack: layer %d: gated feed-forward", l);
+      ff_rows = 2 * L.ff;
+      ff_mid = L.ff;
     } else {
       const b200_moe_desc& m = L.moe;
       B200_CHECK_ARG(L.ff_kind == B200_FF_MOE, "engine_create_stack: layer %d: feed-forward kind %d is not built for sandwich blocks", l, L.ff_kind);
@@ -1809,7 +1907,8 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
     B200_CHECK_ARG(a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.dim > 0 && a.vdim > 0 && a.window >= 0 &&
                        a.keep_first >= 0,
                    "engine_create_stack: layer %d: bad attention sizes", l);
-    B200_CHECK_ARG(a.vdim <= 256 && a.dim <= 1024, "engine_create_stack: layer %d: head sizes above 1024 / 256 not built", l);
+    B200_CHECK_ARG(a.vdim <= 256 && a.dim <= 1024 && !a.values_are_keys, "engine_create_stack: layer %d: head sizes above 1024 / 256, or values that are "
+                   "the keys, not built", l);
     B200_CHECK_ARG(L.norm && L.w_in && L.w_out && L.n_in > 0 && L.k_out > 0 && L.ff >= 0, "engine_create_stack: layer %d: null weight", l);
     B200_CHECK_ARG(L.off_q >= 0 && L.off_q + a.heads * a.dim <= L.n_in && L.off_k + a.kv_heads * a.dim <= L.n_in &&
                        L.off_v + a.kv_heads * a.vdim <= L.n_in && (!a.out_gate || L.off_g + a.heads <= L.n_in) &&
@@ -1854,9 +1953,13 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
       s->run_k_off[r] = s->run_k_off[src];
       s->run_v_off[r] = s->run_v_off[src];
       s->run_kv_shared[r] = 1;
+      s->s_slot += stack_conv_floats(RL);   // its queries' convolution
     } else if (RL.mixer == B200_MIX_ATTENTION) {
-      s->k_slot += (size_t)d.max_ctx * a.kv_heads * a.dim;
-      s->v_slot += (size_t)d.max_ctx * a.kv_heads * a.vdim;
+      s->k_slot += ((size_t)d.max_ctx * a.kv_heads * a.dim + 7) / 8 * 8;   // every run starts on a 16-byte boundary
+      if (!a.values_are_keys) s->v_slot += ((size_t)d.max_ctx * a.kv_heads * a.vdim + 7) / 8 * 8;
+      s->s_slot += stack_conv_floats(RL);
+    } else if (RL.mixer == B200_MIX_GLA) {   // no rows per position: a fixed-size state
+      s->s_slot += ((size_t)a.heads * a.dim * a.vdim + 3) / 4 * 4;
     } else if (RL.mixer == B200_MIX_GATED_DELTA) {   // a fixed-size state and the convolutions' last inputs
       s->s_slot += (size_t)gdelta_state_floats(a.heads, a.kv_heads, a.dim, a.vdim, RL.gdelta.taps);
     } else if (RL.mixer == B200_MIX_LATENT) {   // one row per position: [latent | rotated shared key part]
@@ -1918,6 +2021,9 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
         sp.ok_uq = plan(&sp.uq, L.lat.uq, (int64_t)L.attn.heads * (L.attn.dim + L.lat.rot_dim), up8i(L.lat.q_rank), EPI_BIAS_F32);
       if (L.ff_kind == B200_FF_DENSE && L.ff > 0) {
         sp.ok_ff_in = plan(&sp.ff_in, L.w_ff_in, L.ff, d.width, EPI_BIAS_F32);
+        sp.ok_ff_out = plan(&sp.ff_out, L.w_ff_out, d.width, L.ff, EPI_BIAS_F32);
+      } else if (L.ff_kind == B200_FF_GATED && L.ff > 0) {
+        sp.ok_ff_in = plan(&sp.ff_in, L.w_ff_in, 2 * (int64_t)L.ff, d.width, EPI_BIAS_F32);
         sp.ok_ff_out = plan(&sp.ff_out, L.w_ff_out, d.width, L.ff, EPI_BIAS_F32);
       } else if (L.ff_kind == B200_FF_MOE && L.moe.shared_ff > 0) {
         sp.ok_ff_in = plan(&sp.ff_in, L.w_ff_in, L.moe.expert_act != 0 ? up8i(L.moe.shared_ff) : up8i(2 * L.moe.shared_ff + 1),

@@ -79,25 +79,68 @@ struct PrefillAttnParams {
   int window, keep_first;
   const __nv_bfloat16* gate;    // per-head gate logits, head h of row r at gate + b*q_bs + r*q_rs + h; null = none
   int sink;                     // 1: the softmax's denominator gains 1 (a key of score 0 that has no value)
+  // SCORE kernels: score = (q·k)·scale, then cap·tanh(score / cap) (cap 0: none), then − slopes[h]·(i − j) (null: none)
+  float scale, cap;
+  const float* slopes;
+  int same;                     // SCORE kernels: the values are the keys (v == k): one tile serves both
 };
 
+// bytes of a tile row in shared memory: whole groups of eight 16-byte chunks
+template <int HD>
+__host__ __device__ constexpr int row_bytes() { return (HD + 63) / 64 * 128; }
 // byte offset of 16-byte chunk c of row r inside a [rows][HD] bf16 tile (chunks XOR-swizzled within groups of 8)
 template <int HD>
 __device__ __forceinline__ uint32_t sw_off(int r, int c) {
-  return (uint32_t)(r * (HD * 2) + ((c ^ (r & 7)) << 4));
+  return (uint32_t)(r * row_bytes<HD>() + ((c ^ (r & 7)) << 4));
 }
 
-template <int HD>
+// cap·tanh(v / cap) of a warp's 16 × 64 scores, fp32.  While every |v / cap| is at most 1/4 (scores far below the cap, the
+// common case) the odd Taylor series up to the eleventh power: the first term left out is below 7·10⁻¹⁰ of the value.  Beyond,
+// 1 − 2 / (1 + e^(2z)).
+__device__ __forceinline__ void cap_scores(float (&s)[8][4], float scale, float cap) {
+  const float f = scale / cap;
+  float zm = 0.f;
+#pragma unroll
+  for (int n = 0; n < 8; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      s[n][e] *= f;
+      zm = fmaxf(zm, fabsf(s[n][e]));
+    }
+  if (__any_sync(0xffffffffu, !(zm <= 0.25f))) {
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[n][e] = cap * (1.f - __fdividef(2.f, 1.f + __expf(2.f * fminf(s[n][e], 40.f))));
+  } else {
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float z = s[n][e], q = z * z;
+        float t = fmaf(q, -1382.f / 155925.f, 62.f / 2835.f);
+        t = fmaf(q, t, -17.f / 315.f);
+        t = fmaf(q, t, 2.f / 15.f);
+        t = fmaf(q, t, -1.f / 3.f);
+        s[n][e] = cap * fmaf(z * q, t, z);
+      }
+  }
+}
+
+template <int HD, bool SCORE>
 __global__ void __launch_bounds__(kPfThreads) attn_prefill_mma_kernel(const PrefillAttnParams p) {
   constexpr int CH = HD / 8;    // 16-byte chunks per row
+  constexpr int TB = kBN * row_bytes<HD>();   // bytes of a key / value tile
   constexpr int KS = HD / 16;   // k-steps of Q·Kᵀ
   constexpr int ND = HD / 8;    // 8-wide output column blocks of O
-  const float kScale = p.scale_log2;
+  const float kScale = SCORE ? kLog2eP : p.scale_log2;   // SCORE: the scores carry their scale already
+  const bool same = SCORE && p.same != 0;
+  const float slope = SCORE && p.slopes != nullptr ? p.slopes[blockIdx.y] : 0.f;
 
   extern __shared__ __align__(128) uint8_t pf_smem[];
   uint8_t* const Qs = pf_smem;                       // [kBM][HD]
-  uint8_t* const Ks = Qs + kBM * HD * 2;             // [2][kBN][HD]
-  uint8_t* const Vs = Ks + 2 * kBN * HD * 2;         // [2][kBN][HD]
+  uint8_t* const Ks = Qs + kBM * row_bytes<HD>();    // [2][kBN][HD]
+  uint8_t* const Vs = same ? Ks : Ks + 2 * TB;       // [2][kBN][HD]
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, tq = lane & 3;
@@ -130,15 +173,15 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_mma_kernel(const Pref
   pf_commit();
   auto load_kv = [&](int t, int buf) {
     const int k0 = t * kBN;
-    uint8_t* kd = Ks + buf * (kBN * HD * 2);
-    uint8_t* vd = Vs + buf * (kBN * HD * 2);
+    uint8_t* kd = Ks + buf * TB;
+    uint8_t* vd = Vs + buf * TB;
     for (int i = tid; i < kBN * CH; i += kPfThreads) {
       const int r = i / CH, c = i % CH;
       const uint32_t off = sw_off<HD>(r, c);
       const int key = k0 + r;
       if (key < nkeys) {
         pf_cp_async16(kd + off, kg + (size_t)key * p.kv_rs + c * 8);
-        pf_cp_async16(vd + off, vg + (size_t)key * p.kv_rs + c * 8);
+        if (!same) pf_cp_async16(vd + off, vg + (size_t)key * p.kv_rs + c * 8);
       } else {  // beyond the last visible key: zeros (masked to -inf in S; P = 0 must not meet a NaN in V)
         *reinterpret_cast<uint4*>(kd + off) = make_uint4(0, 0, 0, 0);
         *reinterpret_cast<uint4*>(vd + off) = make_uint4(0, 0, 0, 0);
@@ -184,7 +227,7 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_mma_kernel(const Pref
     for (int n = 0; n < 8; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) s[n][e] = 0.f;
-    const uint32_t kt_u = ks_u + buf * (kBN * HD * 2);
+    const uint32_t kt_u = ks_u + buf * TB;
 #pragma unroll
     for (int kk = 0; kk < KS; ++kk) {
 #pragma unroll
@@ -198,6 +241,22 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_mma_kernel(const Pref
 
     // ---- causal mask (only tiles that reach past the block's first row can contain masked keys)
     const int kbase = t * kBN;
+    if constexpr (SCORE) {
+      if (p.cap > 0.f) {
+        cap_scores(s, p.scale, p.cap);
+      } else {
+#pragma unroll
+        for (int n = 0; n < 8; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[n][e] *= p.scale;
+      }
+      if (p.slopes != nullptr) {
+#pragma unroll
+        for (int n = 0; n < 8; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[n][e] = fmaf(-slope, (float)(rpos[e >> 1] - (kbase + n * 8 + 2 * tq + (e & 1))), s[n][e]);
+      }
+    }
     if (p.window > 0) {
 #pragma unroll
       for (int n = 0; n < 8; ++n) {
@@ -249,7 +308,7 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_mma_kernel(const Pref
     }
 
     // ---- O += P·V
-    const uint32_t vt_u = vs_u + buf * (kBN * HD * 2);
+    const uint32_t vt_u = vs_u + buf * TB;
 #pragma unroll
     for (int k2 = 0; k2 < 4; ++k2) {
 #pragma unroll
@@ -283,18 +342,19 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_mma_kernel(const Pref
   }
 }
 
-template <int HD>
+template <int HD, bool SCORE = false>
 int launch_pf(const PrefillAttnParams& p, int B, cudaStream_t st) {
-  constexpr int smem = (kBM + 4 * kBN) * HD * 2;
+  constexpr int smem_max = (kBM + 4 * kBN) * row_bytes<HD>();
+  const int smem = SCORE && p.same ? (kBM + 2 * kBN) * row_bytes<HD>() : smem_max;
   static std::once_flag once;   // one per instantiation; the reference's server has a worker thread next to main
   static cudaError_t attr_err = cudaSuccess;
   std::call_once(once, [] {
-    attr_err = cudaFuncSetAttribute(attn_prefill_mma_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    attr_err = cudaFuncSetAttribute(attn_prefill_mma_kernel<HD, SCORE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_max);
   });
   B200_CUDA(attr_err);
   dim3 grid((unsigned)((p.S + kBM - 1) / kBM), (unsigned)p.Hq, (unsigned)B);
   g_launches.fetch_add(1);
-  attn_prefill_mma_kernel<HD><<<grid, kPfThreads, smem, st>>>(p);
+  attn_prefill_mma_kernel<HD, SCORE><<<grid, kPfThreads, smem, st>>>(p);
   B200_CUDA(cudaGetLastError());
   return B200_OK;
 }
@@ -329,10 +389,12 @@ int launch_attn_prefill_mma(void* o, const void* qkv, const void* kcache, const 
 // Layer-stack models: one sequence's rows of a step (positions p0 … p0+S-1) against that sequence's cache, with an
 // explicit score scale, a sliding window with kept first keys and a per-head sigmoid gate on the output.  q (and the
 // gate logits) are column ranges of the merged projection rows (stride q_rs), o a column range of rows of stride o_rs.
+// softcap > 0: capped scores; slopes [Hq]: a distance bias per head; vcache == kcache: the values are the keys.
+bool prefill_window_ok(int hd) { return hd == 64 || hd == 96 || hd == 128; }
 int launch_attn_prefill_window(void* o, int64_t o_rs, const void* q, const void* gate_or_null, int64_t q_rs,
                                const void* kcache, const void* vcache, int S, int Hq, int Hkv, int hd, int p0, float scale,
-                               int window, int keep_first, cudaStream_t st, int sink) {
-  B200_CHECK_ARG(hd == 64 || hd == 128, "prefill attention: head size %d not built", hd);
+                               int window, int keep_first, cudaStream_t st, int sink, float softcap, const float* slopes) {
+  B200_CHECK_ARG(prefill_window_ok(hd), "prefill attention: head size %d not built", hd);
   B200_CHECK_ARG(S > 0 && Hkv > 0 && Hq % Hkv == 0 && Hq < 65536 && p0 >= 0 && window >= 0 && keep_first >= 0,
                  "prefill attention: bad shape");
   B200_CHECK_ARG(((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kcache) | reinterpret_cast<uintptr_t>(vcache)) & 15) == 0 &&
@@ -355,7 +417,13 @@ int launch_attn_prefill_window(void* o, int64_t o_rs, const void* q, const void*
   p.window = window;
   p.keep_first = keep_first;
   p.sink = sink;
-  return hd == 64 ? launch_pf<64>(p, 1, st) : launch_pf<128>(p, 1, st);
+  p.scale = scale;
+  p.cap = softcap;
+  p.slopes = slopes;
+  p.same = kcache == vcache ? 1 : 0;
+  if (softcap > 0.f || slopes != nullptr || p.same)
+    return hd == 64 ? launch_pf<64, true>(p, 1, st) : hd == 96 ? launch_pf<96, true>(p, 1, st) : launch_pf<128, true>(p, 1, st);
+  return hd == 64 ? launch_pf<64>(p, 1, st) : hd == 96 ? launch_pf<96>(p, 1, st) : launch_pf<128>(p, 1, st);
 }
 
 // Boundary B (b200_attn_bf16, causal, Sq == Skv): separate BSHD tensors, the reference's top-left-aligned mask.

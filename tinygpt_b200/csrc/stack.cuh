@@ -83,7 +83,7 @@ struct StackAttn {
   int64_t ld_proj = 0;
   int off_q = 0, off_k = 0, off_v = 0, off_g = 0;
   void* kcache = nullptr;       // this run's rows of slot 0: [max_ctx, kv_heads·dim]; slot s is s·k_slot_stride further
-  void* vcache = nullptr;       // [max_ctx, kv_heads·vdim]
+  void* vcache = nullptr;       // [max_ctx, kv_heads·vdim] (a.values_are_keys: the key cache and its slot stride again)
   int64_t k_slot_stride = 0, v_slot_stride = 0;
   const int32_t* slot = nullptr;
   const int32_t* pos = nullptr;
@@ -98,6 +98,9 @@ struct StackAttn {
   // decode steps (every row the only new row of its sequence): the row's own key / value are read from proj and one
   // CTA per (row, kv head) appends them to the cache in the same launch — no separate kv_store
   int own_from_proj = 0;
+  // 1: the same kind of step, but the rows' own keys and values are in the cache already (an earlier launch of the step put
+  // them there, or they belong to another layer)
+  int own_cached = 0;
   int nsplit = 1, keys_per_split = 0;
 };
 constexpr int kStackSplitRows = 16;    // most rows a split-key attention launch serves

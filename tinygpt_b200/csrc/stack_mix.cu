@@ -64,11 +64,11 @@ __global__ void __launch_bounds__(256) stack_layernorm_kernel(YT* __restrict__ y
 }
 
 // A sublayer's post-norm, the residual sum and the next sublayer's pre-norm in one pass over the row:
-//   x ← x + mult·LN(y)·w_post (fp32, stored),   h ← T(LN(x)·(offset + w_next))
-// One CTA per row; the new x stays in registers between the two norms (dim <= 256·kLn2Regs).
+//   x ← x + mult·norm(y)·w_post (fp32, stored),   h ← T(norm(x)·(offset + w_next))
+// with layer norms or (RMS) RMS norms.  One CTA per row; the new x stays in registers between the two norms (dim <= 256·REGS).
 constexpr int kLn2Regs = 32;
-template <typename YT, typename HT>
-__global__ void __launch_bounds__(256) stack_layernorm2_kernel(float* __restrict__ x, const YT* __restrict__ y,
+template <typename YT, typename HT, bool RMS, int REGS>
+__global__ void __launch_bounds__(256) stack_norm2_kernel(float* __restrict__ x, const YT* __restrict__ y,
                                                                const float* __restrict__ w_post, HT* __restrict__ h,
                                                                const float* __restrict__ w_next, int dim, float eps,
                                                                float offset, float mult) {
@@ -76,17 +76,17 @@ __global__ void __launch_bounds__(256) stack_layernorm2_kernel(float* __restrict
   pdl_wait();
   __shared__ float red[8];
   const int64_t base = (int64_t)blockIdx.x * dim;
-  float v[kLn2Regs];
+  float v[REGS];
   float s = 0.f;
 #pragma unroll
-  for (int u = 0; u < kLn2Regs; ++u) {
+  for (int u = 0; u < REGS; ++u) {
     const int i = threadIdx.x + 256 * u;
     v[u] = i < dim ? ldf<YT>(y + base + i) : 0.f;
     s += v[u];
   }
-  float mean = block_sum(s, red) / (float)dim, q = 0.f;
+  float mean = RMS ? 0.f : block_sum(s, red) / (float)dim, q = 0.f;
 #pragma unroll
-  for (int u = 0; u < kLn2Regs; ++u) {
+  for (int u = 0; u < REGS; ++u) {
     const int i = threadIdx.x + 256 * u;
     const float d = i < dim ? v[u] - mean : 0.f;
     q += d * d;
@@ -94,7 +94,7 @@ __global__ void __launch_bounds__(256) stack_layernorm2_kernel(float* __restrict
   float inv = rsqrtf(block_sum(q, red) / (float)dim + eps);
   s = 0.f;
 #pragma unroll
-  for (int u = 0; u < kLn2Regs; ++u) {
+  for (int u = 0; u < REGS; ++u) {
     const int i = threadIdx.x + 256 * u;
     if (i < dim) {
       v[u] = x[base + i] + mult * (v[u] - mean) * inv * w_post[i];
@@ -104,17 +104,17 @@ __global__ void __launch_bounds__(256) stack_layernorm2_kernel(float* __restrict
       v[u] = 0.f;
     }
   }
-  mean = block_sum(s, red) / (float)dim;
+  mean = RMS ? 0.f : block_sum(s, red) / (float)dim;
   q = 0.f;
 #pragma unroll
-  for (int u = 0; u < kLn2Regs; ++u) {
+  for (int u = 0; u < REGS; ++u) {
     const int i = threadIdx.x + 256 * u;
     const float d = i < dim ? v[u] - mean : 0.f;
     q += d * d;
   }
   inv = rsqrtf(block_sum(q, red) / (float)dim + eps);
 #pragma unroll
-  for (int u = 0; u < kLn2Regs; ++u) {
+  for (int u = 0; u < REGS; ++u) {
     const int i = threadIdx.x + 256 * u;
     if (i < dim) h[base + i] = cvt<HT>((v[u] - mean) * inv * (offset + w_next[i]));
   }
@@ -1027,19 +1027,28 @@ int launch_stack_norm_add_norm(float* x, const void* y, bool y_bf16, const float
                                int64_t rows, int dim, float eps, float offset, float mult, int kind, int dtype, cudaStream_t st) {
   MIX_DTYPE_CHECK(dtype);
   B200_CHECK_ARG(x && y && w_post && h && w_next && rows > 0 && dim > 0, "stack norm_add_norm: bad arguments");
-  if (kind != B200_NORM_LAYER || dim > 256 * kLn2Regs) {   // two launches do the same
+  B200_CHECK_ARG(kind == B200_NORM_RMS || kind == B200_NORM_LAYER, "stack norm_add_norm: unknown kind %d", kind);
+  if (dim > 256 * kLn2Regs) {   // two launches do the same
     int rc = launch_stack_norm_add(x, y, y_bf16, w_post, rows, dim, eps, mult, kind, st);
     if (rc != B200_OK) return rc;
     return launch_stack_norm(h, x, w_next, nullptr, rows, dim, eps, offset, kind, dtype, st);
   }
   const dim3 grid((unsigned)rows);
-#define B200_LN2(YT, HT)                                                                                                     \
-  B200_CUDA(launch_pdl(stack_layernorm2_kernel<YT, HT>, grid, dim3(256), 0, st, stack_pdl(), x, (const YT*)y, w_post, (HT*)h, \
+#define B200_LN2_R(YT, HT, RMS, REGS)                                                                                         \
+  B200_CUDA(launch_pdl(stack_norm2_kernel<YT, HT, RMS, REGS>, grid, dim3(256), 0, st, stack_pdl(), x, (const YT*)y, w_post, (HT*)h, \
                        w_next, dim, eps, offset, mult))
+#define B200_LN2(YT, HT)                                                   \
+  do {                                                                     \
+    if (kind == B200_NORM_LAYER) B200_LN2_R(YT, HT, false, kLn2Regs);      \
+    else if (dim <= 256 * 8) B200_LN2_R(YT, HT, true, 8);                  \
+    else if (dim <= 256 * 16) B200_LN2_R(YT, HT, true, 16);                \
+    else B200_LN2_R(YT, HT, true, kLn2Regs);                               \
+  } while (0)
   if (y_bf16 && dtype == B200_F32) B200_LN2(__nv_bfloat16, float);
   else if (y_bf16) B200_LN2(__nv_bfloat16, __nv_bfloat16);
   else if (dtype == B200_F32) B200_LN2(float, float);
   else B200_LN2(float, __nv_bfloat16);
+#undef B200_LN2_R
 #undef B200_LN2
   return B200_OK;
 }

@@ -270,7 +270,14 @@ __global__ void __launch_bounds__(128) stack_kv_store_kernel(const StackAttn p) 
   T* kd = static_cast<T*>(p.kcache) + (int64_t)p.slot[t] * p.k_slot_stride + (int64_t)p.pos[t] * nk;
   T* vd = static_cast<T*>(p.vcache) + (int64_t)p.slot[t] * p.v_slot_stride + (int64_t)p.pos[t] * nv;
   for (int i = threadIdx.x; i < nk; i += blockDim.x) kd[i] = row[p.off_k + i];
+  if (p.a.values_are_keys) return;
   for (int i = threadIdx.x; i < nv; i += blockDim.x) vd[i] = row[p.off_v + i];
+}
+
+// What happens to (q·k)·scale of the key at distance `dist`: the cap, then the distance bias.
+__device__ __forceinline__ float finish_score(const b200_attn_desc& a, float s, float slope, int dist) {
+  if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+  return a.slopes != nullptr ? s - slope * (float)dist : s;
 }
 
 // One warp merges the key splits' partial softmaxes {max, sum, weighted values} of a (token, head) pair, applies the
@@ -347,8 +354,10 @@ __global__ void __launch_bounds__(128) stack_attn_kernel(const StackAttn p) {
     T* kd = static_cast<T*>(p.kcache) + (int64_t)slot * p.k_slot_stride + (int64_t)i * krs + kvh * dim;
     T* vd = static_cast<T*>(p.vcache) + (int64_t)slot * p.v_slot_stride + (int64_t)i * vrs + kvh * vdim;
     for (int d = lane; d < dim; d += 32) kd[d] = own_k[d];
-    for (int d = lane; d < vdim; d += 32) vd[d] = own_v[d];
+    if (!p.a.values_are_keys)
+      for (int d = lane; d < vdim; d += 32) vd[d] = own_v[d];
   }
+  const float slope = p.a.slopes != nullptr ? p.a.slopes[h] : 0.f;
   const int begin = split ? (int)blockIdx.y * p.keys_per_split : 0;
   const int end = split ? min(total, begin + p.keys_per_split) : total;
   constexpr int NA = VEC ? 8 : VR;
@@ -400,7 +409,7 @@ __global__ void __launch_bounds__(128) stack_attn_kernel(const StackAttn p) {
       } else {
         for (int d = 0; d < dim; ++d) dot = fmaf(qs[d], ldf<T>(kr + d), dot);
       }
-      s = dot * p.a.scale;
+      s = finish_score(p.a, dot * p.a.scale, slope, i - j);
     }
     const float mn = fmaxf(m, warp_max(s));
     const float corr = m == -INFINITY ? 0.f : expf(m - mn);
@@ -510,6 +519,7 @@ __global__ void __launch_bounds__(128) stack_attn_kernel(const StackAttn p) {
 
 // Decode-shaped steps (every row its sequence's only new row) of bf16 engines with key size <= 128 and value size 64 or
 // 128: one CTA per (row, head, split of 128 visible keys), warp w takes keys 32w … of the split, ONE key per lane.
+// (Rows whose own key and value are cached already — own_cached — read them behind the wait, as they read q.)
 // The cached rows a lane needs — its key's 16-byte pieces and its row group's value pieces — are requested BEFORE the
 // programmatic-dependency wait: they were written by earlier steps, and the row's slot and position by the step's
 // first kernel, so all of it is stable while the projection that produces q still runs.  After the wait: q, the row's
@@ -560,8 +570,8 @@ __global__ void __launch_bounds__(128) stack_attn_decode_kernel(const StackAttn 
   float* qs = smem_f;                          // [dim], shared by the four warps
   const T* prow = static_cast<const T*>(p.proj) + (int64_t)t * p.ld_proj;
   for (int d = threadIdx.x; d < dim; d += 128) qs[d] = __bfloat162float(prow[p.off_q + h * dim + d]);
-  const T* own_k = prow + p.off_k + kvh * dim;
-  const T* own_v = prow + p.off_v + kvh * vdim;
+  const T* own_k = p.own_from_proj ? prow + p.off_k + kvh * dim : kb + (int64_t)i * krs;
+  const T* own_v = p.own_from_proj ? prow + p.off_v + kvh * vdim : vb + (int64_t)i * vrs;
   if (valid && j == i) {
 #pragma unroll
     for (int u = 0; u < 16; ++u)
@@ -570,11 +580,12 @@ __global__ void __launch_bounds__(128) stack_attn_decode_kernel(const StackAttn 
 #pragma unroll
   for (int u = 0; u < 16; ++u)
     if (u < G && u * KP + grp < cn && vj[u] == i) vq[u] = *reinterpret_cast<const uint4*>(own_v + gl * 8);
-  if (warp == 0 && blockIdx.y == 0 && h % (p.a.heads / p.a.kv_heads) == 0) {
+  if (p.own_from_proj && warp == 0 && blockIdx.y == 0 && h % (p.a.heads / p.a.kv_heads) == 0) {
     T* kd = static_cast<T*>(p.kcache) + (int64_t)slot * p.k_slot_stride + (int64_t)i * krs + kvh * dim;
     T* vd = static_cast<T*>(p.vcache) + (int64_t)slot * p.v_slot_stride + (int64_t)i * vrs + kvh * vdim;
     for (int d = lane; d < dim; d += 32) kd[d] = own_k[d];
-    for (int d = lane; d < vdim; d += 32) vd[d] = own_v[d];
+    if (!p.a.values_are_keys)
+      for (int d = lane; d < vdim; d += 32) vd[d] = own_v[d];
   }
   __syncthreads();
   // ---- scores and the warp's softmax
@@ -588,7 +599,7 @@ __global__ void __launch_bounds__(128) stack_attn_decode_kernel(const StackAttn 
       for (int e = 0; e < 8; ++e) dot = fmaf(qs[u * 8 + e], kf[e], dot);
     }
   }
-  const float sc_ = valid ? dot * p.a.scale : -INFINITY;
+  const float sc_ = valid ? finish_score(p.a, dot * p.a.scale, p.a.slopes != nullptr ? p.a.slopes[h] : 0.f, i - j) : -INFINITY;
   const float m = warp_max(sc_);
   const float pj = valid ? expf(sc_ - m) : 0.f;
   const float l = warp_sum(pj);
@@ -816,6 +827,9 @@ static int check_attn(const StackAttn& p) {
   B200_CHECK_ARG(a.window >= 0 && a.keep_first >= 0, "stack attention: negative window");
   B200_CHECK_ARG(a.vdim <= 256 && a.dim <= 1024, "stack attention: head sizes above 1024 / 256 are not built");
   B200_CHECK_ARG(p.proj && p.kcache && p.vcache && p.slot && p.pos && p.n_tok > 0, "stack attention: null argument");
+  B200_CHECK_ARG(a.softcap >= 0.f, "stack attention: negative softcap");
+  B200_CHECK_ARG(!a.values_are_keys || (a.vdim == a.dim && p.vcache == p.kcache && p.v_slot_stride == p.k_slot_stride && p.off_v == p.off_k),
+                 "stack attention: values that are the keys have the keys' size, rows and cache");
   return B200_OK;
 }
 
@@ -857,7 +871,7 @@ int launch_stack_attention(const StackAttn& p, int dtype, cudaStream_t st) {
                    (!p.own_from_proj || (p.off_k % 8 == 0 && p.off_v % 8 == 0 && p.ld_proj % 8 == 0 &&
                                          (reinterpret_cast<uintptr_t>(p.proj) & 15) == 0)) &&
                    ((reinterpret_cast<uintptr_t>(p.kcache) | reinterpret_cast<uintptr_t>(p.vcache)) & 15) == 0;
-  if (vec && p.split_ws != nullptr && p.own_from_proj && p.a.dim <= 128 && (vd == 64 || vd == 128) &&
+  if (vec && p.split_ws != nullptr && (p.own_from_proj || p.own_cached) && p.a.dim <= 128 && (vd == 64 || vd == 128) &&
       p.keys_per_split <= 128 && (int64_t)p.n_tok * p.a.heads * p.nsplit <= 2 * 148) {
     // the decode shape, and few enough CTAs to be resident together (the prefetch costs 242 registers per thread: two
     // CTAs per SM): cached rows requested ahead of the dependency wait

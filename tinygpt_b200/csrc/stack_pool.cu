@@ -17,61 +17,85 @@ template <typename T> __device__ __forceinline__ T cvt(float v);
 template <> __device__ __forceinline__ float cvt<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 cvt<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
-// One warp: the norm of one head's convolved channels x (query head g·per + hh, or hh == per: key head g), the turn of its first
-// rot_dims entries, and the row it leaves: q, or the cache row.  A key's entries stay in x as the cache holds them.
+// What one CTA of the preparation works on: key/value head g, query heads [h0, h0 + nh) of those that read it, and — in the first
+// CTA of the group — key head and value head g.  Its channels, in order: [nh·dk: q | dk: k | dv: v].
+struct PrepUnit {
+  int g, h0, nh, nq, mine;
+  bool kv;
+};
+__device__ __forceinline__ PrepUnit prep_unit(const PoolAttn& p, int y) {
+  const int per = p.a.heads / p.a.kv_heads, hc = p.heads_per_cta, nc = (per + hc - 1) / hc;
+  PrepUnit u;
+  u.g = y / nc;
+  const int first = (y % nc) * hc;
+  u.h0 = u.g * per + first;
+  u.nh = min(hc, per - first);
+  u.nq = u.nh * p.a.dim;
+  u.kv = first == 0 && !p.q_only;
+  u.mine = u.nq + (u.kv ? p.a.dim + p.a.vdim : 0);
+  return u;
+}
+// the projection column of the CTA's e-th channel
+__device__ __forceinline__ int prep_col(const PoolAttn& p, const PrepUnit& u, int e) {
+  const int dk = p.a.dim, dv = p.a.vdim;
+  return e < u.nq ? p.off_q + u.h0 * dk + e : e < u.nq + dk ? p.off_k + u.g * dk + (e - u.nq) : p.off_v + u.g * dv + (e - u.nq - dk);
+}
+
+// One warp: the norm of one head's convolved channels x, the turn of its first rot_dims entries, and the row it leaves: a query's
+// in q, or a key's cache row.  A key's entries stay in x as the cache holds them.
 template <typename T>
-__device__ __forceinline__ void finish_head(const PoolAttn& p, int t, int ps, int g, int hh, float* x, T* kc, int lane) {
-  const int H = p.a.heads, G = p.a.kv_heads, dk = p.a.dim, per = H / G, half = p.d.rot_dims / 2;
+__device__ __forceinline__ void finish_head(const PoolAttn& p, int ps, bool key, float* x, T* dst, int lane) {
+  const int dk = p.a.dim, half = p.d.rot_dims / 2;
   const float* tab = half > 0 ? p.d.rot_table + (int64_t)ps * half * 2 : nullptr;
-  const float* w = hh < per ? p.d.q_norm : p.d.k_norm;
+  const float* w = key ? p.d.k_norm : p.d.q_norm;
   float inv = 1.f;
-  if (p.d.q_norm != nullptr) {
+  if (w != nullptr) {
     float ss = 0.f;
     for (int i = lane; i < dk; i += 32) ss += x[i] * x[i];
     inv = 1.f / sqrtf(warp_sum(ss) / (float)dk + p.eps);
   }
-  T* dst = hh < per ? static_cast<T*>(p.q) + ((int64_t)t * H + g * per + hh) * dk : kc + ((int64_t)ps * G + g) * dk;
   for (int i = lane; i < dk - half; i += 32) {   // half pairs, then the entries that do not turn
     if (i < half) {
-      float u = x[i] * inv, v = x[i + half] * inv;
-      if (p.d.q_norm != nullptr) {
-        u *= w[i];
-        v *= w[i + half];
+      const int i0 = p.d.rot_interleaved ? 2 * i : i, i1 = p.d.rot_interleaved ? 2 * i + 1 : i + half;
+      float u = x[i0] * inv, v = x[i1] * inv;
+      if (w != nullptr) {
+        u *= w[i0];
+        v *= w[i1];
       }
       const float c = tab[2 * i], s = tab[2 * i + 1];
       const T a = cvt<T>(u * c - v * s), b = cvt<T>(v * c + u * s);
-      dst[i] = a;
-      dst[i + half] = b;
-      if (hh == per) {
-        x[i] = ldf<T>(&a);
-        x[i + half] = ldf<T>(&b);
+      dst[i0] = a;
+      dst[i1] = b;
+      if (key) {
+        x[i0] = ldf<T>(&a);
+        x[i1] = ldf<T>(&b);
       }
     } else {
       float u = x[i + half] * inv;
-      if (p.d.q_norm != nullptr) u *= w[i + half];
+      if (w != nullptr) u *= w[i + half];
       const T a = cvt<T>(u);
       dst[i + half] = a;
-      if (hh == per) x[i + half] = ldf<T>(&a);
+      if (key) x[i + half] = ldf<T>(&a);
     }
   }
 }
 
-// One CTA per (token, key/value head g): the channels of the query heads that read g, of key head g and of value head g.  The
-// convolution of every channel goes to shared memory; then one warp per query / key head takes the head's norm and turns
-// its first rot_dims entries.  Queries leave for q, keys and values for the slot's cache rows.
+// One CTA per (token, PrepUnit).  The convolution of every channel goes to shared memory; then one warp per query / key head takes
+// the head's norm and turns its first rot_dims entries.  Queries leave for q, keys and values for the slot's cache rows.
 template <typename T>
 __global__ void __launch_bounds__(256) pool_prep_kernel(const PoolAttn p) {
   pdl_trigger();
   pdl_wait();
-  extern __shared__ float sm[];   // [per·dk: q | dk: k | dv: v]
-  const int t = blockIdx.x, g = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int H = p.a.heads, G = p.a.kv_heads, dk = p.a.dim, dv = p.a.vdim, per = H / G, taps = p.d.conv_w != nullptr ? p.d.taps : 1;
-  const int nq = per * dk, mine = nq + dk + dv, ps = p.pos[t];
+  extern __shared__ float sm[];   // [nh·dk: q | dk: k | dv: v]
+  const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const PrepUnit un = prep_unit(p, blockIdx.y);
+  const int H = p.a.heads, G = p.a.kv_heads, dk = p.a.dim, dv = p.a.vdim, g = un.g, taps = p.d.conv_w != nullptr ? p.d.taps : 1;
+  const int nq = un.nq, mine = un.mine, ps = p.pos[t];
   const T* row = static_cast<const T*>(p.proj) + (int64_t)t * p.ld_proj;
   float* cs = p.conv_state + (int64_t)p.slot[t] * p.conv_slot_stride;
   const int front = p.single ? 0 : rows_in_front(p.slot, p.pos, t, taps - 1);
   for (int e = tid; e < mine; e += 256) {
-    const int col = e < nq ? p.off_q + g * nq + e : e < nq + dk ? p.off_k + g * dk + (e - nq) : p.off_v + g * dv + (e - nq - dk);
+    const int col = prep_col(p, un, e);
     auto back = [&](int j) {
       if (j <= front) return ldf<T>(row - (int64_t)j * p.ld_proj + col);
       return ps - j >= 0 ? cs[(int64_t)(taps - 1 - (j - front)) * p.ld_proj + col] : 0.f;
@@ -91,7 +115,11 @@ __global__ void __launch_bounds__(256) pool_prep_kernel(const PoolAttn p) {
   __syncthreads();
   T* kc = static_cast<T*>(p.kcache) + (int64_t)p.slot[t] * p.k_slot_stride;
   T* vc = static_cast<T*>(p.vcache) + (int64_t)p.slot[t] * p.v_slot_stride;
-  for (int hh = warp; hh <= per; hh += 8) finish_head<T>(p, t, ps, g, hh, sm + hh * dk, kc, lane);
+  for (int hh = warp; hh < un.nh + (un.kv ? 1 : 0); hh += 8) {
+    const bool key = hh == un.nh;
+    finish_head<T>(p, ps, key, sm + hh * dk, key ? kc + ((int64_t)ps * G + g) * dk : static_cast<T*>(p.q) + ((int64_t)t * H + un.h0 + hh) * dk, lane);
+  }
+  if (!un.kv) return;
   float* v = sm + nq + dk;
   for (int i = tid; i < dv; i += 256) {
     const T a = cvt<T>(v[i]);
@@ -118,14 +146,15 @@ constexpr int kPrepStrip = 8;
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(256) pool_prep_strip_kernel(const PoolAttn p) {
   pdl_trigger();
-  extern __shared__ float sm[];   // [kPrepStrip][per·dk: q | dk: k | dv: v]
-  const int t0 = blockIdx.x * kPrepStrip, g = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int H = p.a.heads, G = p.a.kv_heads, dk = p.a.dim, dv = p.a.vdim, per = H / G;
-  const int nq = per * dk, mine = nq + dk + dv, n = min(kPrepStrip, p.n_tok - t0);
+  extern __shared__ float sm[];   // [kPrepStrip][nh·dk: q | dk: k | dv: v]
+  const int t0 = blockIdx.x * kPrepStrip, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const PrepUnit un = prep_unit(p, blockIdx.y);
+  const int H = p.a.heads, G = p.a.kv_heads, dk = p.a.dim, dv = p.a.vdim, g = un.g;
+  const int nq = un.nq, mine = un.mine, n = min(kPrepStrip, p.n_tok - t0);
   pdl_wait();
   const bool one = rows_one_seq(p.slot, p.pos, t0, t0 + n);
   for (int e = tid; e < mine; e += 256) {
-    const int col = e < nq ? p.off_q + g * nq + e : e < nq + dk ? p.off_k + g * dk + (e - nq) : p.off_v + g * dv + (e - nq - dk);
+    const int col = prep_col(p, un, e);
     const T* x = static_cast<const T*>(p.proj) + (int64_t)t0 * p.ld_proj + col;
     float w[TAPS], win[TAPS];   // win[j]: the row j positions back
 #pragma unroll
@@ -150,10 +179,15 @@ __global__ void __launch_bounds__(256) pool_prep_strip_kernel(const PoolAttn p) 
     }
   }
   __syncthreads();
-  for (int u = warp; u < n * (per + 1); u += 8) {
-    const int r = u / (per + 1), hh = u % (per + 1), t = t0 + r;
-    finish_head<T>(p, t, p.pos[t], g, hh, sm + r * mine + hh * dk, static_cast<T*>(p.kcache) + (int64_t)p.slot[t] * p.k_slot_stride, lane);
+  const int rows = un.nh + (un.kv ? 1 : 0);
+  for (int u = warp; u < n * rows; u += 8) {
+    const int r = u / rows, hh = u % rows, t = t0 + r, ps = p.pos[t];
+    const bool key = hh == un.nh;
+    T* kc = static_cast<T*>(p.kcache) + (int64_t)p.slot[t] * p.k_slot_stride;
+    finish_head<T>(p, ps, key, sm + r * mine + hh * dk, key ? kc + ((int64_t)ps * G + g) * dk : static_cast<T*>(p.q) + ((int64_t)t * H + un.h0 + hh) * dk,
+                   lane);
   }
+  if (!un.kv) return;
   for (int r = warp; r < n; r += 8) {
     const int t = t0 + r;
     T* vd = static_cast<T*>(p.vcache) + (int64_t)p.slot[t] * p.v_slot_stride + ((int64_t)p.pos[t] * G + g) * dv;
@@ -397,7 +431,7 @@ int check_pool(const PoolAttn& p) {
                  "pool attention: bad sizes (heads %d, kv_heads %d, dim %d, vdim %d)", a.heads, a.kv_heads, a.dim, a.vdim);
   B200_CHECK_ARG(p.d.rot_dims >= 0 && p.d.rot_dims % 2 == 0 && p.d.rot_dims <= a.dim && (p.d.rot_dims == 0 || p.d.rot_table),
                  "pool attention: rot_dims %d must be even, at most the head size %d, with a table", p.d.rot_dims, a.dim);
-  B200_CHECK_ARG((p.d.q_norm == nullptr) == (p.d.k_norm == nullptr), "pool attention: one of the two head norms is missing");
+  B200_CHECK_ARG(p.q_only || (p.d.q_norm == nullptr) == (p.d.k_norm == nullptr), "pool attention: one of the two head norms is missing");
   B200_CHECK_ARG(p.d.softcap >= 0.f, "pool attention: negative softcap");
   B200_CHECK_ARG(p.q && p.kcache && p.vcache && p.slot && p.pos && p.n_tok > 0 && p.max_ctx > 0, "pool attention: null argument");
   return B200_OK;
@@ -408,17 +442,24 @@ int check_pool(const PoolAttn& p) {
 #define POOL_DTYPE_CHECK(dtype) \
   B200_CHECK_ARG((dtype) == B200_BF16 || (dtype) == B200_F32, "stack op: unknown dtype %d", (int)(dtype))
 
-int launch_pool_prep(const PoolAttn& p, int dtype, cudaStream_t st) {
+int launch_pool_prep(const PoolAttn& run, int dtype, cudaStream_t st) {
   POOL_DTYPE_CHECK(dtype);
+  PoolAttn p = run;
   int rc = check_pool(p);
   if (rc != B200_OK) return rc;
   B200_CHECK_ARG(p.proj != nullptr, "pool attention: null projection");
   B200_CHECK_ARG(p.d.conv_w == nullptr || (p.d.taps >= 1 && p.d.taps <= kConvMaxTaps && (p.d.taps == 1 || p.conv_state)),
                  "pool attention: 1 … %d convolution taps with a state", kConvMaxTaps);
-  const size_t smem = (size_t)((p.a.heads / p.a.kv_heads + 1) * p.a.dim + p.a.vdim) * 4;
-  B200_CHECK_ARG(smem <= 48 * 1024, "pool attention: the heads that share one key/value head exceed 12288 channels");
-  if (!p.single && p.n_tok > kPrepStrip && p.d.conv_w != nullptr && p.d.taps <= 4 && kPrepStrip * smem <= 48 * 1024) {
-    const dim3 sg((p.n_tok + kPrepStrip - 1) / kPrepStrip, p.a.kv_heads);
+  // query heads per CTA: the strip's channels within 48 KB, and few rows spread over many CTAs
+  const int per = p.a.heads / p.a.kv_heads, dk = p.a.dim, kv = p.q_only ? 0 : dk + p.a.vdim, limit = 12 * 1024;   // floats
+  B200_CHECK_ARG(dk + kv <= limit, "pool attention: one query head and one key/value head exceed %d channels", limit);
+  const bool strips = !p.single && p.n_tok > kPrepStrip && p.d.conv_w != nullptr && p.d.taps <= 4 && kPrepStrip * (dk + kv) <= limit;
+  const int fit = ((strips ? limit / kPrepStrip : limit) - kv) / dk;
+  p.heads_per_cta = std::max(1, std::min({per, fit, p.n_tok <= 16 ? 4 : 8}));
+  const size_t smem = (size_t)(p.heads_per_cta * dk + kv) * 4;
+  const unsigned units = (unsigned)(p.a.kv_heads * ((per + p.heads_per_cta - 1) / p.heads_per_cta));
+  if (strips) {
+    const dim3 sg((p.n_tok + kPrepStrip - 1) / kPrepStrip, units);
 #define B200_PP(T, TAPS) B200_CUDA(launch_pdl(pool_prep_strip_kernel<T, TAPS>, sg, dim3(256), kPrepStrip * smem, st, stack_pdl(), p))
 #define B200_PP_T(T)                    \
   do {                                  \
@@ -433,7 +474,7 @@ int launch_pool_prep(const PoolAttn& p, int dtype, cudaStream_t st) {
 #undef B200_PP
     return B200_OK;
   }
-  const dim3 grid(p.n_tok, p.a.kv_heads);
+  const dim3 grid(p.n_tok, units);
   if (dtype == B200_F32) B200_CUDA(launch_pdl(pool_prep_kernel<float>, grid, dim3(256), smem, st, stack_pdl(), p));
   else B200_CUDA(launch_pdl(pool_prep_kernel<__nv_bfloat16>, grid, dim3(256), smem, st, stack_pdl(), p));
   return B200_OK;

@@ -1,12 +1,12 @@
 // stack_pool.cuh — attention with pooled blocks behind its window and mixed heads (stack_pool.cu): the per-token preparation of
-// q | k | v (short causal convolution, per-head norms, rotate-half rotary positions) straight into the caches, the block
+// q | k | v (short causal convolution, per-head norms, rotary positions of either pair layout) straight into the caches, the block
 // means, and the attention itself.  Storage type T = bf16 or fp32; convolutions, norms, angles, scores, the softmax and the mixing of
 // its weights are fp32.
 //
 // The key list of a query at position i is [blocks 0 … nb − 1 | tokens lo … i]: lo = max(0, i − window + 1), and nb = the
 // blocks of `pool` positions that end before the window, floor((i − window + 1) / pool).  The caches of a run hold max_ctx token
 // rows and behind them max_ctx / pool block rows; block b is written when its last token is, so it is complete before any
-// position that sees it.
+// position that sees it.  (The preparation, launch_pool_prep, also serves the plain attention of sandwich blocks.)
 #pragma once
 #include "stack.cuh"
 
@@ -29,6 +29,8 @@ struct PoolAttn {
   int max_ctx = 0;
   float* conv_state = nullptr;   // slot 0's [taps − 1][ld_proj] fp32
   int64_t conv_slot_stride = 0;
+  int q_only = 0;                // 1: the rows hold queries only (a layer that reads another layer's cached keys and values)
+  int heads_per_cta = 0;         // launch_pool_prep: query heads one CTA prepares (set by the launcher)
   int single = 0;                // 1: every row is its sequence's only new one — the preparation moves the convolution's state
                                  // on and pools a finished block itself
   const int32_t* slot = nullptr;

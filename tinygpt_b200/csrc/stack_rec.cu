@@ -113,9 +113,9 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnPrep p) {
 // multiply-adds per operand and column, and the output's dot with the NEW columns.  Columns never read each other, so
 // the result of a sequence does not depend on what else is in the step; the order of the sums inside a column is fixed by
 // dk alone (lane l sums rows l, l + 32, …, then the butterfly), whatever NC is.
-// OLD: the output reads the columns BEFORE the token joins them, plus the token's bonus times its value; d holds the decay
-// minus one, so that a decay close to one keeps all its digits.
-template <int DR, bool REMOVE, int NC, bool OLD = false>
+// OLD: the output reads the columns BEFORE the token joins them, plus the token's bonus times its value.  DM1: d holds the
+// decay minus one, so that a decay close to one keeps all its digits.
+template <int DR, bool REMOVE, int NC, bool OLD = false, bool DM1 = OLD>
 __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
   pdl_trigger();
   pdl_wait();
@@ -228,7 +228,7 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
 #pragma unroll
           for (int c = 0; c < NC; ++c) {
             if constexpr (OLD) dot[u][c] = fmaf(S[c][i], rr, dot[u][c]);
-            float sn = OLD ? fmaf(dd, S[c][i], S[c][i]) : dd * S[c][i];
+            float sn = DM1 ? fmaf(dd, S[c][i], S[c][i]) : dd * S[c][i];
             if constexpr (REMOVE) sn = fmaf(-pp, rem[c], sn);
             sn = fmaf(bb, vj[c], sn);
             S[c][i] = sn;
@@ -580,6 +580,153 @@ __global__ void __launch_bounds__(128) wkv_out_kernel(const WkvRun p) {
     for (int c = (int)n + lane; c < p.n_pad; c += 32) static_cast<T*>(p.mid)[(int64_t)t * p.ld_mid + c] = cvt<T>(0.f);
 }
 
+// ------------------------------------------------------------------------------------------------- gated linear attention
+// log sigmoid(z)
+__device__ __forceinline__ float log_sigmoidf(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+
+// Prompts: kGlaStrip tokens × 256 columns per CTA.  A column is one of the heads·dim key channels (its decay minus one, from the
+// strip's bottleneck rows in shared memory and its row of a2, and its key and query entries) or one of the heads·vdim value
+// channels.  The scan's fp32 rows are [decay − 1 | k | q | v].
+constexpr int kGlaStrip = 8;
+template <typename T>
+__global__ void __launch_bounds__(256) gla_prep_kernel(const GlaRun p) {
+  pdl_trigger();
+  pdl_wait();
+  extern __shared__ float sm[];   // [kGlaStrip][rank]
+  const int t0 = blockIdx.x * kGlaStrip, n = min(kGlaStrip, p.scan.n_tok - t0), tid = threadIdx.x;
+  const int H = p.a.heads, nk = H * p.a.dim, nv = H * p.a.vdim, rk = p.d.rank, ldw = (rk + 7) / 8 * 8;
+  const int c = blockIdx.y * 256 + tid;
+  const T* row = static_cast<const T*>(p.proj) + (int64_t)t0 * p.ld_proj;
+  float* f = p.f + (int64_t)t0 * p.scan.ld;
+  if (blockIdx.y * 256 < nk) {   // the same for the whole CTA
+    for (int e = tid; e < kGlaStrip * rk; e += 256) sm[e] = e / rk < n ? ldf<T>(row + (int64_t)(e / rk) * p.ld_proj + p.off_a + e % rk) : 0.f;
+    __syncthreads();
+  }
+  if (c < nk) {
+    const float scale = 1.f / sqrtf((float)p.a.dim), inv_tau = 1.f / p.d.tau, b = p.d.a2_b[c];
+    const T* w = static_cast<const T*>(p.d.a2) + (int64_t)c * ldw;
+    float z[kGlaStrip];
+#pragma unroll
+    for (int u = 0; u < kGlaStrip; ++u) z[u] = b;
+#pragma unroll 4
+    for (int r = 0; r < rk; ++r) {
+      const float wr = ldf<T>(w + r);
+#pragma unroll
+      for (int u = 0; u < kGlaStrip; ++u) z[u] = fmaf(wr, sm[u * rk + r], z[u]);
+    }
+#pragma unroll
+    for (int u = 0; u < kGlaStrip; ++u) {
+      if (u >= n) break;
+      const T* x = row + (int64_t)u * p.ld_proj;
+      float* o = f + (int64_t)u * p.scan.ld;
+      o[c] = expm1f(log_sigmoidf(z[u]) * inv_tau);
+      o[nk + c] = ldf<T>(x + p.off_k + c);
+      o[2 * nk + c] = ldf<T>(x + p.off_q + c) * scale;
+    }
+  } else if (c >= (nk + 255) / 256 * 256) {
+    const int cv = c - (nk + 255) / 256 * 256;
+    if (cv < nv)
+      for (int u = 0; u < n; ++u) f[(int64_t)u * p.scan.ld + 3 * nk + cv] = ldf<T>(row + (int64_t)u * p.ld_proj + p.off_v + cv);
+  }
+}
+
+// One warp per (token, head): o / rms(o) · head_norm (shared by the heads) · silu(out gate).
+template <typename T>
+__global__ void __launch_bounds__(256) gla_out_kernel(const GlaRun p) {
+  pdl_trigger();
+  pdl_wait();
+  const int64_t pair = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31, H = p.a.heads, dv = p.a.vdim;
+  if (pair >= (int64_t)p.scan.n_tok * H) return;
+  const int t = (int)(pair / H), hd = (int)(pair % H);
+  const float* o = p.scan.o + (int64_t)t * p.scan.ld_o + hd * dv;
+  float ss = 0.f;
+  for (int c = lane; c < dv; c += 32) ss += o[c] * o[c];
+  const float inv = 1.f / sqrtf(warp_sum(ss) / (float)dv + p.eps);
+  const T* g = static_cast<const T*>(p.proj) + (int64_t)t * p.ld_proj + p.off_g + hd * dv;
+  T* y = static_cast<T*>(p.mid) + (int64_t)t * p.ld_mid + hd * dv;
+  for (int c = lane; c < dv; c += 32) y[c] = cvt<T>(o[c] * inv * p.d.head_norm[c] * siluf(ldf<T>(g + c)));
+}
+
+// Steps in which every row is its sequence's only new one: the whole mixer between its two products in one launch.  One CTA per
+// (row, head).  The state's entries a thread owns — one column, every `slices`-th … of kGlaRows rows — are requested ahead of
+// the dependency wait (an earlier step left them there, and the row's slot and position come from the step's first kernel);
+// behind it decays, keys, queries and values go to shared memory, the state moves on in registers and back to memory, the
+// slices' sums of a column meet in shared memory, and the head's norm and gate follow.
+constexpr int kGlaThreads = 512;
+constexpr int kGlaRows = 32;
+template <typename T>
+__global__ void __launch_bounds__(kGlaThreads) gla_step_kernel(const GlaRun p) {
+  pdl_trigger();
+  extern __shared__ float sm[];
+  __shared__ float red[kGlaThreads / 32];
+  const int t = blockIdx.x, hd = blockIdx.y, tid = threadIdx.x;
+  const int H = p.a.heads, dk = p.a.dim, dv = p.a.vdim, rk = p.d.rank, ldw = (rk + 7) / 8 * 8;
+  const int cw = min(kGlaThreads, (dv + 31) / 32 * 32), slices = kGlaThreads / cw;   // columns side by side; row slices
+  const int per = (dk + slices - 1) / slices;
+  float* s_d = sm;               // [dk] decay − 1
+  float* s_k = s_d + dk;         // [dk]
+  float* s_q = s_k + dk;         // [dk]
+  float* s_u = s_q + dk;         // [rk]
+  float* s_o = s_u + rk;         // [dv]
+  float* s_p = s_o + dv;         // [slices][cw]
+  const int slice = tid / cw, col = tid % cw;
+  float* st = p.scan.state + (int64_t)p.scan.slot[t] * p.scan.slot_stride + (int64_t)hd * dk * dv;
+  const bool fresh = p.scan.pos[t] == 0;
+  const int d0 = slice * per, d1 = slice < slices ? min(dk, d0 + per) : d0;
+  float S[kGlaRows];
+  auto fetch = [&](int j, int d) {
+#pragma unroll
+    for (int i = 0; i < kGlaRows; ++i) S[i] = d + i < d1 && j < dv && !fresh ? st[(int64_t)(d + i) * dv + j] : 0.f;
+  };
+  fetch(col, d0);
+  pdl_wait();
+  const T* row = static_cast<const T*>(p.proj) + (int64_t)t * p.ld_proj;
+  for (int i = tid; i < rk; i += kGlaThreads) s_u[i] = ldf<T>(row + p.off_a + i);
+  for (int i = tid; i < dk; i += kGlaThreads) {
+    s_k[i] = ldf<T>(row + p.off_k + hd * dk + i);
+    s_q[i] = ldf<T>(row + p.off_q + hd * dk + i) * (1.f / sqrtf((float)dk));
+  }
+  __syncthreads();
+  for (int i = tid; i < dk; i += kGlaThreads) {
+    const T* w = static_cast<const T*>(p.d.a2) + (int64_t)(hd * dk + i) * ldw;
+    float z = p.d.a2_b[hd * dk + i];
+#pragma unroll 8
+    for (int r = 0; r < rk; ++r) z = fmaf(ldf<T>(w + r), s_u[r], z);
+    s_d[i] = expm1f(log_sigmoidf(z) * (1.f / p.d.tau));
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int j0 = 0; j0 < dv; j0 += cw) {
+    const int j = j0 + col;
+    const float v = j < dv ? ldf<T>(row + p.off_v + hd * dv + j) : 0.f;
+    float acc = 0.f;
+    for (int d = d0; d < d1; d += kGlaRows) {
+      if (j0 > 0 || d > d0) fetch(j, d);
+#pragma unroll
+      for (int i = 0; i < kGlaRows; ++i) {
+        if (d + i < d1 && j < dv) {
+          const float sn = fmaf(s_k[d + i], v, fmaf(s_d[d + i], S[i], S[i]));
+          st[(int64_t)(d + i) * dv + j] = sn;
+          acc = fmaf(sn, s_q[d + i], acc);
+        }
+      }
+    }
+    if (slice < slices) s_p[tid] = acc;
+    __syncthreads();
+    if (tid < cw && j < dv) {
+      float o = 0.f;
+      for (int s = 0; s < slices; ++s) o += s_p[s * cw + tid];
+      s_o[j] = o;
+      ss += o * o;
+    }
+    __syncthreads();
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)dv + p.eps);
+  T* y = static_cast<T*>(p.mid) + (int64_t)t * p.ld_mid + hd * dv;
+  for (int c = tid; c < dv; c += kGlaThreads) y[c] = cvt<T>(s_o[c] * inv * p.d.head_norm[c] * siluf(ldf<T>(row + p.off_g + hd * dv + c)));
+}
+
 // ------------------------------------------------------------------------------------------------------ selective scan
 // One thread per (row, channel): convolution over the row's own input and the taps − 1 before it, bias, SiLU.
 template <typename T>
@@ -903,6 +1050,7 @@ int launch_lin_scan(const LinScan& p, cudaStream_t st) {
   B200_CHECK_ARG((p.p == nullptr) == (p.q == nullptr), "linear scan: the removal needs both of its vectors");
   B200_CHECK_ARG(p.heads > 0 && p.dk > 0 && p.dv > 0 && p.share > 0 && p.heads % p.share == 0, "linear scan: bad sizes");
   B200_CHECK_ARG(!p.read_old || (p.p == nullptr && p.bonus && p.vscale == nullptr), "linear scan: reading the old state takes a bonus and no removal");
+  B200_CHECK_ARG(!p.d_minus_one || p.p == nullptr, "linear scan: a decay minus one takes no removal");
   B200_CHECK_ARG(p.dk <= kScanMaxDim, "linear scan: more than %d key channels not built", kScanMaxDim);
   // two columns per warp where the value size fills them and the registers hold them: half the CTAs stage the same rows
   const int nc = (p.dv >= 32 && p.dk <= 256) ? 2 : 1;
@@ -911,6 +1059,7 @@ int launch_lin_scan(const LinScan& p, cudaStream_t st) {
   do {                                                                                                             \
     if (p.p != nullptr) B200_CUDA(launch_pdl(lin_scan_kernel<DR, true, NC>, grid, dim3(256), 0, st, stack_pdl(), p));  \
     else if (p.read_old) B200_CUDA(launch_pdl(lin_scan_kernel<DR, false, NC, true>, grid, dim3(256), 0, st, stack_pdl(), p)); \
+    else if (p.d_minus_one) B200_CUDA(launch_pdl(lin_scan_kernel<DR, false, NC, false, true>, grid, dim3(256), 0, st, stack_pdl(), p)); \
     else B200_CUDA(launch_pdl(lin_scan_kernel<DR, false, NC>, grid, dim3(256), 0, st, stack_pdl(), p));           \
   } while (0)
 #define B200_SCAN(DR)              \
@@ -1021,6 +1170,37 @@ int run_wkv(const WkvRun& p, int dtype, cudaStream_t st) {
   if (rc != B200_OK) return rc;
   if (dtype == B200_F32) B200_CUDA(launch_pdl(wkv_out_kernel<float>, grid, dim3(128), 0, st, stack_pdl(), p));
   else B200_CUDA(launch_pdl(wkv_out_kernel<__nv_bfloat16>, grid, dim3(128), 0, st, stack_pdl(), p));
+  return B200_OK;
+}
+
+int run_gla(const GlaRun& p, int dtype, cudaStream_t st) {
+  REC_DTYPE_CHECK(dtype);
+  const int H = p.a.heads, dk = p.a.dim, dv = p.a.vdim, rk = p.d.rank;
+  B200_CHECK_ARG(p.proj && p.f && p.mid && p.scan.n_tok > 0 && p.scan.state && H > 0 && dk > 0 && dv > 0, "gated linear attention: null argument");
+  B200_CHECK_ARG(p.d.a2 && p.d.a2_b && p.d.head_norm && p.d.tau > 0.f && rk > 0 && rk <= kGlaMaxRank && dk <= kScanMaxDim,
+                 "gated linear attention: null weight, or a bottleneck above %d / a key above %d", kGlaMaxRank, kScanMaxDim);
+  const int cw = std::min(kGlaThreads, (dv + 31) / 32 * 32);
+  const size_t step_smem = (size_t)(3 * dk + rk + dv + kGlaThreads / cw * cw) * 4;
+  if (p.single && step_smem <= 40 * 1024) {
+    const dim3 sg(p.scan.n_tok, H);
+    if (dtype == B200_F32) B200_CUDA(launch_pdl(gla_step_kernel<float>, sg, dim3(kGlaThreads), step_smem, st, stack_pdl(), p));
+    else B200_CUDA(launch_pdl(gla_step_kernel<__nv_bfloat16>, sg, dim3(kGlaThreads), step_smem, st, stack_pdl(), p));
+    return B200_OK;
+  }
+  const int nk = H * dk, nv = H * dv;
+  const dim3 pg((p.scan.n_tok + kGlaStrip - 1) / kGlaStrip, (nk + 255) / 256 + (nv + 255) / 256);
+  const size_t smem = (size_t)kGlaStrip * rk * 4;
+  if (dtype == B200_F32) B200_CUDA(launch_pdl(gla_prep_kernel<float>, pg, dim3(256), smem, st, stack_pdl(), p));
+  else B200_CUDA(launch_pdl(gla_prep_kernel<__nv_bfloat16>, pg, dim3(256), smem, st, stack_pdl(), p));
+  LinScan s = p.scan;
+  s.heads = H; s.dk = dk; s.dv = dv; s.share = 1; s.d_scalar = 0; s.d_minus_one = 1;
+  s.d = p.f; s.b = p.f + nk; s.r = p.f + 2 * (int64_t)nk; s.v = p.f + 3 * (int64_t)nk;
+  s.p = s.q = s.vscale = nullptr;
+  int rc = launch_lin_scan(s, st);
+  if (rc != B200_OK) return rc;
+  const dim3 og((unsigned)(((int64_t)p.scan.n_tok * H + 7) / 8));
+  if (dtype == B200_F32) B200_CUDA(launch_pdl(gla_out_kernel<float>, og, dim3(256), 0, st, stack_pdl(), p));
+  else B200_CUDA(launch_pdl(gla_out_kernel<__nv_bfloat16>, og, dim3(256), 0, st, stack_pdl(), p));
   return B200_OK;
 }
 

@@ -39,6 +39,7 @@ constexpr int kScanMaxDim = 512;
 struct LinScan {
   int heads = 0, dk = 0, dv = 0, share = 1, d_scalar = 0;
   int read_old = 0;
+  int d_minus_one = 0;   // 1 (no removal): d holds the decay minus one
   const float* bonus = nullptr;
   int q_shared = 0;   // 1: q is [heads / share][dk] like b and r (the removal reads along a shared key)
   const float *d = nullptr, *p = nullptr, *q = nullptr, *b = nullptr, *r = nullptr, *v = nullptr, *vscale = nullptr;
@@ -137,6 +138,24 @@ struct WkvRun {
 };
 inline int64_t wkv_row_floats(int heads, int dim) { return (int64_t)heads * (4 * dim + 1); }
 int run_wkv(const WkvRun& p, int dtype, cudaStream_t st);
+
+// ---- gated linear attention around the scan: everything between the in-projection and the out-projection
+constexpr int kGlaMaxRank = 1024;
+struct GlaRun {
+  b200_attn_desc a{};            // heads, dim, vdim
+  b200_gla_desc d{};
+  float eps = 1e-5f;
+  const void* proj = nullptr;    // [n_tok, ld_proj] T: q | k | v | out-gate logits | decay bottleneck at off_q / off_k / off_v / off_g / off_a
+  int64_t ld_proj = 0;
+  int off_q = 0, off_k = 0, off_v = 0, off_g = 0, off_a = 0;
+  int single = 0;                // 1: every row is its sequence's only new one
+  float* f = nullptr;            // [n_tok, gla_row_floats] fp32 workspace: decay − 1 | k | q | v
+  LinScan scan{};                // state, slots, positions, sequences, o
+  void* mid = nullptr;           // [n_tok, ld_mid] T
+  int64_t ld_mid = 0;
+};
+inline int64_t gla_row_floats(int heads, int dim, int vdim) { return (int64_t)heads * (3 * dim + vdim); }
+int run_gla(const GlaRun& p, int dtype, cudaStream_t st);
 
 // ---- Mamba's selective scan: the convolution in front of w_x, then everything between the step-size logits and the
 // out-projection

@@ -18,7 +18,7 @@ import torch
 
 from . import models
 from ._lib import (AttnDesc, AttnPrepDesc, B200Error, DeltaDesc, GatedDeltaDesc, HyperDesc, LatentDesc, LayerWeights, Mamba1Desc,
-                   MambaDesc, MlstmDesc, ModelDesc, MoeDesc, PoolAttnDesc, WkvDesc, StackDesc, StackLayer, WeightTable, check, lib, require_device)
+                   GlaDesc, MambaDesc, MlstmDesc, ModelDesc, MoeDesc, PoolAttnDesc, WkvDesc, StackDesc, StackLayer, WeightTable, check, lib, require_device)
 
 
 def align_prompts(token_lists, context_size: int, pad_token: int):
@@ -186,11 +186,11 @@ class DecodeEngine:
         self.slots = SequenceSlots(spec.max_slots)
 
     def _sandwich_layer(self, spec, i, L, ptr, mdt, acts) -> StackLayer:
-        """Descriptor of layer i of a sandwich-block model (latent attention, mLSTM, prepared attention or gated delta rule
-        mixer; dense or routed feed-forward); the rotation tables are built here, for the engine's context length."""
+        """Descriptor of layer i of a sandwich-block model (latent attention, mLSTM, prepared attention, gated delta rule or
+        gated linear attention mixer; dense, gated or routed feed-forward); the rotation tables are built here, for the engine's context length."""
         lay, p = spec.mix_layout(i), f"l{i}."
         f32 = torch.float32
-        lat, rec, moe, prep, gdelta = LatentDesc(), MlstmDesc(), MoeDesc(), AttnPrepDesc(), GatedDeltaDesc()
+        lat, rec, moe, prep, gdelta, gla = LatentDesc(), MlstmDesc(), MoeDesc(), AttnPrepDesc(), GatedDeltaDesc(), GlaDesc()
         kv_share = 0
 
         def table(rot):
@@ -211,13 +211,16 @@ class DecodeEngine:
             mixer = 1
         elif L.mixer == "attention":
             a, q = L.attn, L.prep or models.AttnPrepSpec()
-            attn = AttnDesc(a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.window, a.keep_first, int(a.out_gate), int(a.sink))
+            attn = AttnDesc(a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.window, a.keep_first, int(a.out_gate), int(a.sink), a.softcap,
+                            ptr(p + "slopes", f32) if a.distance_bias else None, int(a.values_are_keys))
             tab = table(q.rot)
             if q.v_mix:
                 raise B200Error(f"DecodeEngine: layer {i}: the value mix-in is built for post-norm blocks")
+            norms = q.qk_norm or q.head_norm
             prep = AttnPrepDesc(int(q.qk_norm), q.rot.dims if q.rot is not None else 0, int(q.v_norm), 0,
-                                ptr(p + "q_norm", f32) if q.qk_norm else None, ptr(p + "k_norm", f32) if q.qk_norm else None,
-                                tab.data_ptr() if tab is not None else None, None, int(q.rot_interleaved))
+                                ptr(p + "q_norm", f32) if norms else None, ptr(p + "k_norm", f32) if norms else None,
+                                tab.data_ptr() if tab is not None else None, None, int(q.rot_interleaved), int(q.head_norm), q.conv,
+                                ptr(p + "conv_w", f32) if q.conv > 0 else None)
             kv_share = 0 if L.kv_from is None else L.kv_from + 1
             mixer = 0
         elif L.mixer == "gated_delta":
@@ -226,6 +229,11 @@ class DecodeEngine:
             gdelta = GatedDeltaDesc(a.conv, a.unit_eps, ptr(p + "conv_w", f32), ptr(p + "A_log", f32), ptr(p + "dt_bias", f32),
                                     ptr(p + "head_norm", f32))
             mixer = 5
+        elif L.mixer == "gla":
+            a = L.gla
+            attn = AttnDesc(a.heads, a.heads, a.dim, a.vdim, 1.0, 0, 0, 0)
+            gla = GlaDesc(a.rank, a.tau, ptr(p + "a2", mdt), ptr(p + "a2_b", f32), ptr(p + "head_norm", f32))
+            mixer = 10
         else:
             a = L.mlstm
             attn = AttnDesc(a.heads, a.heads, a.dim, a.vdim, 1.0, 0, 0, 0)
@@ -238,10 +246,10 @@ class DecodeEngine:
                           ptr(p + "w_exp_in", mdt), ptr(p + "w_exp_out", mdt))
         return StackLayer(attn, L.ff, acts[L.ff_act], lay.off_q, lay.off_k, lay.off_v, lay.off_g, lay.off_gate, lay.off_up, lay.n_in,
                           0, lay.k_out, ptr(p + "norm", f32), ptr(p + "w_in", mdt), ptr(p + "b_in", f32), ptr(p + "w_out", mdt),
-                          0, None, None, None, mixer, 2 if L.ff_kind == "moe" else 1, ptr(p + "post_norm", f32),
+                          0, None, None, None, mixer, {"gated": 0, "dense": 1, "moe": 2}[L.ff_kind], ptr(p + "post_norm", f32),
                           ptr(p + "ff_norm", f32) if has_ff else None, ptr(p + "ff_post_norm", f32) if has_ff else None,
                           ptr(p + "w_ff_in", mdt), ptr(p + "w_ff_out", mdt), lat, rec, moe, prep, DeltaDesc(), MambaDesc(), gdelta,
-                          ptr(p + "b_out", f32), kv_share)
+                          ptr(p + "b_out", f32), kv_share, gla=gla)
 
     def _postnorm_layer(self, spec, i, L, ptr, mdt, acts) -> StackLayer:
         """Descriptor of layer i of a post-norm-block model (prepared attention, generalized delta rule or Mamba-2 mixer;

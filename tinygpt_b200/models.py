@@ -197,6 +197,12 @@ class AttnSpec:
     bias: bool = True        # q/k/v projections carry a bias
     sink: bool = False       # the softmax's denominator gains 1 (a sink of score 0 that has no value)
     out_bias: bool = False   # the out-projection carries a bias (sandwich blocks)
+    softcap: float = 0.0     # > 0: score <- softcap·tanh(score / softcap)
+    distance_bias: bool = False    # then slope_h·(i − j) is taken off the score, slope_h = 2^(−8 (h + 1) / heads)
+    values_are_keys: bool = False  # the value heads are the key heads (sandwich blocks)
+
+    def slopes(self) -> np.ndarray:
+        return np.exp2(-8.0 * np.arange(1, self.heads + 1, dtype=np.float64) / self.heads)
 
     def visible(self, i: int, j: int) -> bool:
         return j <= i and (self.window <= 0 or i - j < self.window or j < self.keep_first)
@@ -323,6 +329,8 @@ class AttnPrepSpec:
     v_norm: bool = False
     v_mix: bool = False
     rot_interleaved: bool = False  # pairs (2i, 2i+1)
+    head_norm: bool = False        # sandwich blocks: every query / key head by its own root mean square, one weight for all heads
+    conv: int = 0                  # sandwich blocks: taps of the causal convolution every channel of q, k and v passes first
 
 
 @dataclass(frozen=True)
@@ -374,6 +382,17 @@ class GatedDeltaSpec:
 
 
 @dataclass(frozen=True)
+class GlaSpec:
+    """Gated linear attention: per head a dim × vdim state with a decay sigmoid(·)^(1/tau) per key channel, its logits through a
+    bottleneck of `rank`."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    rank: int
+
+
+@dataclass(frozen=True)
 class PoolAttnSpec:
     """Attention behind short convolutions: grouped heads with biases, a causal convolution of `conv` taps on q, k and v, per-head
     query / key norms, rotate-half rotary positions, tanh-capped scores (softcap 0: none), a sliding window of `window` tokens
@@ -421,7 +440,7 @@ class StackLayerSpec:
     attn: Optional[AttnSpec] = None  # mixer "attention"
     ff: int = 0                      # feed-forward width (gated / dense), 0 = none
     ff_act: str = "gelu_tanh"        # gelu_tanh | silu | gelu_erf
-    mixer: str = "attention"         # attention | latent_attention | mlstm | general_delta | mamba2 | gated_delta; of
+    mixer: str = "attention"         # attention | latent_attention | mlstm | general_delta | mamba2 | gated_delta | gla; of
                                      # hyper-connected blocks: mamba1 | wkv | pool_attention | parallel
     latent: Optional[LatentSpec] = None
     mlstm: Optional[MlstmSpec] = None
@@ -431,6 +450,7 @@ class StackLayerSpec:
     delta: Optional[DeltaSpec] = None
     mamba: Optional[Mamba2Spec] = None
     gdelta: Optional[GatedDeltaSpec] = None
+    gla: Optional[GlaSpec] = None
     pool: Optional[PoolAttnSpec] = None   # mixers pool_attention and (left half) parallel
     wkv: Optional[WkvSpec] = None         # mixers wkv and (right half) parallel
     mamba1: Optional[Mamba1Spec] = None
@@ -447,7 +467,7 @@ class MixLayout:
     latent attention: [q | down];  mLSTM: [q | k | v | out-gate logits | input-gate, forget-gate logits];  attention:
     [q | k | v];  generalized delta rule: [r | k | v | out-gate logits | removal logits | decay bottleneck] (the last at
     off_up);  Mamba-2: [z | x | B | C | dt] with z at off_g, x at off_v, B at off_k, C at off_q (x | B | C contiguous), dt at
-    off_gate."""
+    off_gate;  gated linear attention: [q | k | v | out-gate logits | decay bottleneck] (the last at off_up)."""
     off_q: int = 0
     off_k: int = 0
     off_v: int = 0
@@ -501,6 +521,7 @@ class StackSpec:
     loop_mix: bool = True            # every pass of the loop starts with x <- mix_in·[x; x0]
     logit_softcap: float = 0.0       # > 0: logits <- cap·tanh(logits / cap)
     streams: int = 1                 # hyper blocks: copies of the residual stream
+    logit_scale: float = 1.0         # logits = logit_scale·(head·norm(x)) (the packer folds it into the final norm's weight)
     layer_scale: bool = False        # every sublayer's normed output is multiplied by a per-channel vector (the packer folds
                                      # it into the post-norm's weight: both are element-wise factors of the same product)
 
@@ -557,7 +578,17 @@ class StackSpec:
             a = L.attn
             off_k = _up8(a.heads * a.dim)
             off_v = off_k + _up8(a.kv_heads * a.dim)
+            if a.values_are_keys:
+                return MixLayout(off_q=0, off_k=off_k, off_v=off_k, n_in=off_v, k_out=a.heads * a.vdim)
             return MixLayout(off_q=0, off_k=off_k, off_v=off_v, n_in=off_v + _up8(a.kv_heads * a.vdim), k_out=a.heads * a.vdim)
+        if L.mixer == "gla":
+            a = L.gla
+            off_k = _up8(a.heads * a.dim)
+            off_v = off_k + _up8(a.heads * a.dim)
+            off_g = off_v + _up8(a.heads * a.vdim)
+            off_up = off_g + _up8(a.heads * a.vdim)
+            return MixLayout(off_q=0, off_k=off_k, off_v=off_v, off_g=off_g, off_up=off_up, n_in=off_up + _up8(a.rank),
+                             k_out=a.heads * a.vdim)
         if L.mixer == "general_delta":
             a = L.delta
             seg = _up8(a.heads * a.dim)
@@ -616,6 +647,9 @@ class StackSpec:
             elif L.mixer == "gated_delta":
                 q = L.gdelta
                 n += self.width * (2 * q.kv_heads * q.dim + 3 * q.heads * q.vdim + 2 * q.heads)
+            elif L.mixer == "gla":
+                q = L.gla
+                n += self.width * (2 * q.heads * q.dim + 3 * q.heads * q.vdim + q.rank) + q.heads * q.dim * q.rank
             elif L.mixer == "mlstm":
                 q = L.mlstm
                 n += self.width * (2 * q.heads * q.dim + 3 * q.heads * q.vdim + 2 * q.heads)
@@ -626,10 +660,13 @@ class StackSpec:
                 q = L.mamba
                 n += self.width * (2 * q.inner + 2 * q.groups * q.state + q.heads + q.inner)
             elif self.block != "parallel":
-                n += self.width * (a.heads * a.dim + (a.kv_heads * (a.dim + a.vdim) if L.kv_from is None else 0) + a.heads * a.vdim)
+                kv = 0 if L.kv_from is not None else a.kv_heads * (a.dim + (0 if a.values_are_keys else a.vdim))
+                n += self.width * (a.heads * a.dim + kv + a.heads * a.vdim)
             if self.block != "parallel":
                 if L.ff_kind == "dense":
                     n += 2 * L.ff * self.width
+                elif L.ff_kind == "gated":
+                    n += 3 * L.ff * self.width
                 elif L.ff_kind == "moe" and L.moe.act == "glu_clamp":   # the router, the chosen experts, the shared expert and its gate
                     n += self.width * (L.moe.experts + 3 * L.moe.top * L.moe.expert_ff + 3 * L.moe.shared_ff + 1)
                 elif L.ff_kind == "moe":
@@ -1590,6 +1627,199 @@ def pack_bibezen_weights(spec: StackSpec, named: Dict[str, torch.Tensor], device
     return out
 
 
+# ---------------------------------------------------------------------------------------------------------- Favudra
+def favudra_from_config(doc: dict, name: str = "Favudra", shapes: Optional[Dict[str, Tuple[int, ...]]] = None) -> StackSpec:
+    """config.json of the Favudra design → StackSpec.  Favudra: sandwich blocks with zero-centred RMS norms and SwiGLU
+    feed-forwards; mixers are a causal attention behind short convolutions and per-head norms (interleaved rotary pairs, capped
+    scores, a sink; a layer may read the keys and values an earlier layer cached), a windowed attention with a distance bias
+    per head whose values are its keys, or gated linear attention; scaled embedding and logits.  `shapes` (tensor name →
+    shape) gives the rank of the decay bottlenecks, which config.json leaves to the tensors."""
+    layers: List[StackLayerSpec] = []
+    for i, lc in enumerate(doc["layers"]):
+        kind, m = lc.get("type"), lc["mixer"]
+        window = int((m.get("mask") or {}).get("size", 0))
+        if kind in ("attention", "attention_2"):
+            heads, kv, dim = int(m["heads"]), int(m["kv_heads"]), int(m["dim"])
+            if kv < 1 or heads % kv:
+                raise ValueError(f"Favudra: layer {i}: {heads} heads over {kv} kv_heads")
+        if kind == "attention":
+            rot = _rotary_from_config(m["rot"]) if m.get("rot") and int(m["rot"]["dims"]) > 0 else None
+            if rot is not None and (rot.dims % 2 or rot.dims > dim):
+                raise ValueError(f"Favudra: layer {i}: rot.dims {rot.dims} must be even and at most dim")
+            src = m.get("kv_from")
+            attn = AttnSpec(heads=heads, kv_heads=kv, dim=dim, vdim=int(m["vdim"]), scale=float(m["scale"]), window=window, out_gate=False,
+                            bias=False, sink=True, softcap=float(m.get("softcap") or 0.0))
+            if src is not None:
+                src = int(src)
+                S = layers[src] if 0 <= src < i else None
+                if S is None or S.mixer != "attention" or S.kv_from is not None or S.attn.values_are_keys:
+                    raise ValueError(f"Favudra: layer {i}: kv_from {src} is not an earlier attention layer with keys and values of its own")
+                if (S.attn.kv_heads, S.attn.dim, S.attn.vdim) != (kv, dim, attn.vdim):
+                    raise ValueError(f"Favudra: layer {i}: the keys and values of layer {src} have other sizes")
+            conv = int(m.get("conv") or 0)
+            if conv < 0:
+                raise ValueError(f"Favudra: layer {i}: {conv} taps")
+            kw = dict(mixer="attention", attn=attn, kv_from=src,
+                      prep=AttnPrepSpec(rot=rot, rot_interleaved=True, head_norm=True, conv=conv))
+        elif kind == "attention_2":
+            if int(m.get("vdim", dim)) != dim:
+                raise ValueError(f"Favudra: layer {i}: the values are the keys, but vdim {m['vdim']} is not dim {dim}")
+            kw = dict(mixer="attention", attn=AttnSpec(heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=float(m["scale"]), window=window,
+                                                       out_gate=False, bias=False, distance_bias=True, values_are_keys=True))
+        elif kind == "gla":
+            rank = (shapes or {}).get(f"l{i}.mix.a1", (0,))[0]
+            rank = int(m.get("rank", rank) if rank == 0 else rank)
+            if rank < 1:
+                raise ValueError(f"Favudra: layer {i}: the rank of the decay bottleneck comes from the tensors, and there are none")
+            kw = dict(mixer="gla", gla=GlaSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), tau=float(m["tau"]), rank=rank))
+            if kw["gla"].tau <= 0:
+                raise ValueError(f"Favudra: layer {i}: tau {kw['gla'].tau}")
+        else:
+            raise ValueError(f"Favudra: layer {i}: mixer type {kind!r} is not part of the design")
+        mlp = lc.get("mlp")
+        if mlp is not None and mlp.get("kind") != "dense":
+            raise ValueError(f"Favudra: layer {i}: feed-forward kind {mlp.get('kind')!r} is not part of the design")
+        layers.append(StackLayerSpec(ff_kind="gated", ff=int(mlp["ff"]) if mlp is not None else 0, ff_act="silu", **kw))
+    return StackSpec(name=name, architecture="Favudra", width=int(doc["width"]), vocab=int(doc["vocab"]), layers=tuple(layers),
+                     embed_scale=float(doc["embedding"]["scale"]), norm_eps=float(doc["norm"]["eps"]), norm_offset=0.0, block="sandwich",
+                     norm_kind="rms", loop_mix=False, logit_scale=float(doc["logit_scale"]))
+
+
+def favudra_config(spec: StackSpec) -> dict:
+    """The config.json a Favudra StackSpec is read from (inverse of favudra_from_config; the bottlenecks' ranks stay with the
+    tensors)."""
+    doc = {"architecture": "Favudra", "embedding": {"scale": spec.embed_scale}, "layers": [], "logit_scale": spec.logit_scale,
+           "norm": {"eps": spec.norm_eps}, "vocab": spec.vocab, "width": spec.width}
+    for L in spec.layers:
+        if L.mixer == "gla":
+            a = L.gla
+            kind, mixer = "gla", {"dim": a.dim, "heads": a.heads, "tau": a.tau, "vdim": a.vdim}
+        else:
+            a = L.attn
+            mixer = {"dim": a.dim, "heads": a.heads, "kv_heads": a.kv_heads, "scale": a.scale, "vdim": a.vdim}
+            if a.window > 0:
+                mixer["mask"] = {"size": a.window}
+            kind = "attention_2" if a.values_are_keys else "attention"
+            if not a.values_are_keys:
+                mixer["conv"], mixer["softcap"] = L.prep.conv, a.softcap
+                if L.prep.rot is not None:
+                    mixer["rot"] = _rotary_config(L.prep.rot)
+                if L.kv_from is not None:
+                    mixer["kv_from"] = L.kv_from
+        doc["layers"].append({"mixer": mixer, "mlp": {"ff": L.ff, "kind": "dense"} if L.ff > 0 else None, "type": kind})
+    return doc
+
+
+def favudra_tensor_shapes(spec: StackSpec) -> Dict[str, Tuple[int, ...]]:
+    """Checkpoint tensor names and shapes of a Favudra model (Linear weights are [out, in])."""
+    W, out = spec.width, {}
+    out["embed"] = (spec.vocab, W)
+    for i, L in enumerate(spec.layers):
+        p, q = f"l{i}.", f"l{i}.mix."
+        out[p + "norm1"], out[p + "norm1b"] = (W,), (W,)
+        if L.mixer == "gla":
+            a = L.gla
+            nk, nv = a.heads * a.dim, a.heads * a.vdim
+            out[q + "q"], out[q + "k"], out[q + "v"], out[q + "g"], out[q + "o"] = (nk, W), (nk, W), (nv, W), (nv, W), (W, nv)
+            out[q + "norm"] = (a.vdim,)
+            out[q + "a1"], out[q + "a2"], out[q + "a2.b"] = (a.rank, W), (nk, a.rank), (nk,)
+        else:
+            a = L.attn
+            segs = [("q", a.heads * a.dim)]
+            if L.kv_from is None:
+                segs += [("k", a.kv_heads * a.dim)] + ([] if a.values_are_keys else [("v", a.kv_heads * a.vdim)])
+            for nm, rows in segs:
+                out[q + nm] = (rows, W)
+                if L.prep is not None and L.prep.conv > 0:
+                    out[q + nm + ".conv"] = (rows, L.prep.conv)
+                if L.prep is not None and nm != "v":
+                    out[q + nm + ".norm"] = (a.dim,)
+            out[q + "o"] = (W, a.heads * a.vdim)
+        if L.ff > 0:
+            out[p + "norm2"], out[p + "norm2b"] = (W,), (W,)
+            out[p + "mlp.gate"], out[p + "mlp.up"], out[p + "mlp.down"] = (L.ff, W), (L.ff, W), (W, L.ff)
+    out["final.norm"] = (W,)
+    out["head"] = (spec.vocab, W)
+    return out
+
+
+def synth_favudra_weights(spec: StackSpec, seed: int = 0, std: float = 0.05) -> Dict[str, torch.Tensor]:
+    """Seeded synthetic Favudra checkpoint (bf16, checkpoint names): matrices N(0, std·√(64/in)), zero-centred norm weights
+    N(0, 0.1), head norms 1 + N(0, 0.1), convolution taps N(0, 0.5), decay biases where states both keep and forget."""
+    g = torch.Generator().manual_seed(seed)
+    w = {}
+    for name, shape in favudra_tensor_shapes(spec).items():
+        t, last = torch.randn(shape, generator=g), name.split(".", 1)[-1]
+        if last.startswith("norm") or name == "final.norm":
+            t = 0.1 * t
+        elif last.startswith("mix.") and last.endswith("norm"):
+            t = 1.0 + 0.1 * t
+        elif last.endswith(".conv"):
+            t = 0.5 * t
+        elif last == "mix.a2.b":
+            t = 2.0 + t
+        elif last == "mix.a2":
+            t = t * 0.5
+        else:
+            t = t * (std * (64.0 / shape[1]) ** 0.5)
+        w[name] = t.to(torch.bfloat16)
+    return w
+
+
+def pack_favudra_weights(spec: StackSpec, named: Dict[str, torch.Tensor], device="cuda",
+                         dtype: torch.dtype = torch.bfloat16) -> Dict[str, torch.Tensor]:
+    """Checkpoint tensors (Favudra names) → the engine's layout on `device`.  Per layer: w_in = the mixer's in-projections merged by
+    rows (StackSpec.mix_layout), w_out = mix.o, gate | up rows of the feed-forward merged; convolution taps with the tap as the
+    slow index over w_in's rows; a2 padded to 8 columns; the slopes of the distance bias; zero-centred norm weights as 1 + w, the
+    final one times logit_scale.  Vectors in fp32, matrices in `dtype`."""
+    W = spec.width
+    out: Dict[str, torch.Tensor] = {}
+
+    def mat(t):
+        return t.to(dtype).contiguous().to(device)
+
+    def vec(t):
+        return t.to(torch.float32).reshape(-1).contiguous().to(device)
+
+    def one_plus(name):
+        return 1.0 + named[name].to(torch.float32)
+
+    out["embed"], out["head"] = mat(named["embed"]), mat(named["head"])
+    out["final_norm"] = vec(one_plus("final.norm") * spec.logit_scale)
+    for i, L in enumerate(spec.layers):
+        lay, p, q = spec.mix_layout(i), f"l{i}.", f"l{i}.mix."
+        segs = [("q", lay.off_q), ("k", lay.off_k), ("v", lay.off_v)]
+        if L.mixer == "gla":
+            a = L.gla
+            segs += [("g", lay.off_g), ("a1", lay.off_up)]
+            a2 = torch.zeros(a.heads * a.dim, _up8(a.rank), dtype=dtype)
+            a2[:, :a.rank] = named[q + "a2"].to(dtype)
+            out[p + "a2"], out[p + "a2_b"], out[p + "head_norm"] = a2.to(device), vec(named[q + "a2.b"]), vec(named[q + "norm"])
+        else:
+            segs = segs[:1] if L.kv_from is not None else segs[:2] if L.attn.values_are_keys else segs
+            if L.attn.distance_bias:
+                out[p + "slopes"] = vec(torch.from_numpy(L.attn.slopes()))
+        w_in = torch.zeros(lay.n_in, W, dtype=dtype)
+        for nm, off in segs:
+            w_in[off:off + named[q + nm].shape[0]] = named[q + nm].to(dtype)
+        if L.prep is not None:
+            if L.prep.conv > 0:
+                conv = torch.zeros(L.prep.conv, lay.n_in)
+                for nm, off in segs:
+                    t = named[q + nm + ".conv"]
+                    conv[:, off:off + t.shape[0]] = t.t().float()
+                out[p + "conv_w"] = vec(conv)
+            for nm in ("q", "k") if L.kv_from is None else ("q",):
+                out[p + nm + "_norm"] = vec(named[q + nm + ".norm"])
+        out[p + "w_in"], out[p + "w_out"] = w_in.to(device), mat(named[q + "o"])
+        out[p + "norm"], out[p + "post_norm"] = vec(one_plus(p + "norm1")), vec(one_plus(p + "norm1b"))
+        if L.ff > 0:
+            out[p + "ff_norm"], out[p + "ff_post_norm"] = vec(one_plus(p + "norm2")), vec(one_plus(p + "norm2b"))
+            out[p + "w_ff_in"] = mat(torch.cat([named[p + "mlp.gate"], named[p + "mlp.up"]], 0))
+            out[p + "w_ff_out"] = mat(named[p + "mlp.down"])
+    return out
+
+
 @dataclass(frozen=True)
 class Architecture:
     """One design of the layer-stack registry: its config reader and writer, checkpoint tensor list, synthetic checkpoint
@@ -1751,6 +1981,8 @@ ARCHITECTURES["Tarudra"] = Architecture(tarudra_from_config, tarudra_config, tar
                                         pack_tarudra_weights)
 ARCHITECTURES["Bibezen"] = Architecture(bibezen_from_config, bibezen_config, bibezen_tensor_shapes, synth_bibezen_weights,
                                         pack_bibezen_weights, with_shapes=True)
+ARCHITECTURES["Favudra"] = Architecture(favudra_from_config, favudra_config, favudra_tensor_shapes, synth_favudra_weights,
+                                        pack_favudra_weights, with_shapes=True)
 
 
 # ------------------------------------------------------------------------------------------- checkpoint writer

@@ -501,6 +501,119 @@ def main_bibezen(sizes: str, steps: int, warmup: int) -> None:
     print(json.dumps(compare_bibezen(names, steps=steps, warmup=warmup)), flush=True)
 
 
+# Favudra sizes: eight layers [attention, windowed attention whose values are its keys, attention reading layer 0's keys and values,
+# gated linear attention] twice, every one with a SwiGLU feed-forward.  The model beside it is the Tarudra design — the
+# framework's other sandwich-block design with a sink attention, interleaved rotary pairs, shared keys and values, windows and a
+# recurrent mixer behind a head norm and a silu gate — with the same head counts, sizes and windows in every attention place, the
+# gated delta rule with a state of the same size in the recurrent places, and a two-matrix feed-forward half again as wide (equal
+# parameters).
+FAVUDRA_SIZES = {
+    "f2048": dict(width=2048, vocab=65536, heads=16, kv_heads=8, dim=128, rot_dims=64, conv=3, window=1024, g_heads=16, g_kv=8, g_dim=128,
+                  g_vdim=128, rank=16, ff=5464),
+    "f3072": dict(width=3072, vocab=65536, heads=24, kv_heads=8, dim=128, rot_dims=64, conv=3, window=1024, g_heads=24, g_kv=8, g_dim=128,
+                  g_vdim=128, rank=16, ff=8192),
+}
+
+
+def favudra_spec(name: str, max_ctx: int, max_slots: int = 8) -> models.StackSpec:
+    z = FAVUDRA_SIZES[name]
+    attn = models.AttnSpec(z["heads"], z["kv_heads"], z["dim"], z["dim"], z["dim"] ** -0.5, 0, 0, out_gate=False, bias=False, sink=True,
+                           softcap=50.0)
+    tied = models.AttnSpec(z["heads"], z["kv_heads"], z["dim"], z["dim"], z["dim"] ** -0.5, z["window"], 0, out_gate=False, bias=False,
+                           distance_bias=True, values_are_keys=True)
+    prep = models.AttnPrepSpec(rot=models.RotarySpec(dims=z["rot_dims"], base=5e5), rot_interleaved=True, head_norm=True, conv=z["conv"])
+    L = models.StackLayerSpec
+    kw = dict(ff_kind="gated", ff=z["ff"], ff_act="silu")
+    t = L(attn=tied, **kw)
+    g = L(mixer="gla", gla=models.GlaSpec(z["g_heads"], z["g_dim"], z["g_vdim"], 16.0, z["rank"]), **kw)
+
+    def span(i):
+        return (L(attn=attn, prep=prep, **kw), t, L(attn=attn, prep=prep, kv_from=i, **kw), g)
+
+    return models.StackSpec(name="favudra-" + name, architecture="Favudra", width=z["width"], vocab=z["vocab"], layers=span(0) + span(4),
+                            embed_scale=8.0, norm_eps=1e-6, block="sandwich", norm_kind="rms", loop_mix=False, logit_scale=0.5,
+                            max_ctx=max_ctx, max_slots=max_slots)
+
+
+def tarudra_beside(name: str, max_ctx: int, max_slots: int = 8) -> models.StackSpec:
+    z = FAVUDRA_SIZES[name]
+
+    def attn(window):
+        return models.AttnSpec(z["heads"], z["kv_heads"], z["dim"], z["dim"], z["dim"] ** -0.5, window, 0, out_gate=False, bias=True,
+                               sink=True, out_bias=True)
+
+    prep = models.AttnPrepSpec(rot=models.RotarySpec(dims=z["rot_dims"], base=5e5), rot_interleaved=True)
+    L = models.StackLayerSpec
+    kw = dict(ff_kind="dense", ff=z["ff"] * 3 // 2, ff_act="relu2")
+    d = L(mixer="gated_delta", gdelta=models.GatedDeltaSpec(z["g_heads"], z["g_kv"], z["g_dim"], z["g_vdim"], 4), **kw)
+
+    def span(i):
+        return (L(attn=attn(0), prep=prep, **kw), L(attn=attn(z["window"]), prep=prep, **kw), L(attn=attn(0), prep=prep, kv_from=i, **kw), d)
+
+    return models.StackSpec(name="tarudra-beside-" + name, architecture="Tarudra", width=z["width"], vocab=z["vocab"],
+                            layers=span(0) + span(4), norm_eps=1e-6, block="sandwich", norm_kind="layer", loop_mix=False,
+                            logit_softcap=15.0, layer_scale=True, max_ctx=max_ctx, max_slots=max_slots)
+
+
+def device_favudra_weights(spec: models.StackSpec, device, seed: int = 0) -> Dict[str, torch.Tensor]:
+    """Random Favudra weights straight in the engine's layout on the device."""
+    g = torch.Generator(device=device).manual_seed(seed)
+    W = spec.width
+
+    def mat(*shape):
+        return (torch.randn(*shape, generator=g, device=device, dtype=torch.float32) * (shape[-1] ** -0.5)).to(torch.bfloat16)
+
+    def vec(n, centre=1.0, spread=0.05):
+        return centre + torch.randn(n, generator=g, device=device, dtype=torch.float32) * spread
+
+    w = {"embed": mat(spec.vocab, W), "head": mat(spec.vocab, W), "final_norm": vec(W)}
+    for i, L in enumerate(spec.layers):
+        lay, p = spec.mix_layout(i), f"l{i}."
+        w[p + "norm"], w[p + "post_norm"], w[p + "ff_norm"], w[p + "ff_post_norm"] = vec(W), vec(W, 0.6), vec(W), vec(W, 0.6)
+        w[p + "w_in"], w[p + "w_out"] = mat(lay.n_in, W), mat(W, lay.k_out)
+        if L.mixer == "gla":
+            a = L.gla
+            w[p + "a2"], w[p + "a2_b"], w[p + "head_norm"] = mat(a.heads * a.dim, (a.rank + 7) // 8 * 8), vec(a.heads * a.dim, 2.0, 1.0), vec(a.vdim)
+        elif L.prep is not None:
+            w[p + "conv_w"], w[p + "q_norm"], w[p + "k_norm"] = vec(L.prep.conv * lay.n_in, 0.3, 0.3), vec(L.attn.dim), vec(L.attn.dim)
+        else:
+            w[p + "slopes"] = torch.from_numpy(L.attn.slopes()).float().to(device)
+        w[p + "w_ff_in"], w[p + "w_ff_out"] = mat(2 * L.ff, W), mat(W, L.ff)
+    return w
+
+
+def compare_favudra(sizes: List[str], steps: int = 5, warmup: int = 3, prompt_len: int = 2048, n_decode: int = 32) -> dict:
+    dev = torch.device("cuda:0")
+    torch.cuda.set_device(dev)
+    timer = _Timer(dev)
+    max_ctx = prompt_len + n_decode + 8
+    rows = {}
+    for name in sizes:
+        def one(spec, weights):
+            eng = engine.DecodeEngine(spec, weights)
+            k = _measure(eng, True, prompt_len, n_decode, timer, steps, warmup, spec.vocab)
+            k["bytes_per_decode_token"] = eng.bytes_per_token(prompt_len)
+            k["launches_per_decode_token"] = eng.launches_per_token
+            k["matrix_params_per_token"] = spec.weight_params()
+            eng.close()
+            del eng
+            torch.cuda.empty_cache()
+            return k
+        fspec = favudra_spec(name, max_ctx)
+        k = one(fspec, device_favudra_weights(fspec, dev))
+        tspec = tarudra_beside(name, max_ctx)
+        l = one(tspec, device_tarudra_weights(tspec, dev))
+        rows[name] = {"favudra": k, "tarudra": l, "ratio": {m: round(k[m] / l[m], 3) for m in k if m.endswith("tok_s")}}
+    return {"metric": "favudra_compare", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic", "prompt_len": prompt_len,
+            "decode_steps": n_decode, "steps": steps, "warmup": warmup, "l2": "flushed between timed iterations",
+            "sizes": rows}
+
+
+def main_favudra(sizes: str, steps: int, warmup: int) -> None:
+    names = [s for s in sizes.split(",") if s] if sizes and sizes != "all" else list(FAVUDRA_SIZES)
+    print(json.dumps(compare_favudra(names, steps=steps, warmup=warmup)), flush=True)
+
+
 class _Timer:
     def __init__(self, device):
         self.device = device

@@ -695,7 +695,17 @@ def main():
                          "blocks, selective scan, time mixing, pooled-block attention with mixed heads, SwiGLU experts) beside the "
                          "Tekosun design of equal width, vocabulary, layers and expert parameters (sizes of "
                          "tinygpt_b200/stack_bench.py, or all)")
+    ap.add_argument("--favudra-compare", nargs="?", const="all", default=None, metavar="SIZES",
+                    help="instead of the headline run: prefill / decode throughput of the Favudra layer-stack design (capped attention "
+                         "behind short convolutions with shared keys / values, attention whose values are its keys, gated linear "
+                         "attention, SwiGLU feed-forwards) beside the Tarudra design of equal width, vocabulary, layers and "
+                         "feed-forward parameters (sizes of tinygpt_b200/stack_bench.py, or all)")
     args = ap.parse_args()
+    if args.favudra_compare is not None:
+        from tinygpt_b200 import build, stack_bench
+        build.build()
+        stack_bench.main_favudra(args.favudra_compare, steps=max(1, min(args.steps, 10)), warmup=max(3, args.warmup))
+        return
     if args.bibezen_compare is not None:
         from tinygpt_b200 import build, stack_bench
         build.build()

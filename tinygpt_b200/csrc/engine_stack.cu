@@ -152,6 +152,7 @@ struct StackEngine {
   struct SPlans {
     GemvPlan in{}, out{}, ff_in{}, ff_out{}, lora{}, uq{};
     bool ok_in = false, ok_out = false, ok_ff_in = false, ok_ff_out = false, ok_lora = false, ok_uq = false;
+    bool ok_glu = false;   // ff_in is the merged gate | up product with its gate
   };
   std::vector<SPlans> splans;
   // ---- hyper-connected blocks
@@ -938,6 +939,11 @@ static int stack_run_sandwich(StackEngine* s, int r, float* x, int n_tok, cudaSt
                               next_run_w, st);
   }
   if (L.ff_kind == B200_FF_GATED) {
+    if (s->fast && n_tok <= kMaxBatch && pl.ok_glu) {   // both halves and the gate in one launch
+      if ((rc = stack_lin(s, hin, L.w_ff_in, nullptr, n_tok, 2 * L.ff, W, &pl.ff_in, s->mid, nullptr, st)) != B200_OK) return rc;
+      return stack_lin_norm_add(s, s->mid, L.w_ff_out, n_tok, L.ff, pl.ok_ff_out ? &pl.ff_out : nullptr, L.ff_post_norm, x,
+                                next_run_w, st);
+    }
     if ((rc = stack_lin(s, hin, L.w_ff_in, nullptr, n_tok, 2 * L.ff, W, pl.ok_ff_in ? &pl.ff_in : nullptr, s->proj, nullptr, st)) != B200_OK)
       return rc;
     if ((rc = launch_stack_glu(s->mid, L.ff, s->proj, 2 * L.ff, n_tok, L.ff, L.ff_act, dt, st)) != B200_OK) return rc;
@@ -1984,9 +1990,9 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
   if (s->fast) {
     if ((rc = gemv_setup_attributes()) != B200_OK || (rc = gemv_batch_setup_attributes()) != B200_OK) return rc;
     // a plan that cannot be made (k not a multiple of 8, an unaligned matrix) leaves that product on the general kernel
-    auto plan = [&](GemvPlan* pl, const void* w, int64_t n, int64_t k, int epi, int pro = PRO_PLAIN) {
+    auto plan = [&](GemvPlan* pl, const void* w, int64_t n, int64_t k, int epi, int pro = PRO_PLAIN, int nseg = 1) {
       if (k % 8 != 0 || (reinterpret_cast<uintptr_t>(w) & 15) != 0) return false;
-      return gemv_make_plan(pl, w, n, n, k, 1, pro, epi, s->num_sms) == B200_OK;
+      return gemv_make_plan(pl, w, nseg * n, n, k, nseg, pro, epi, s->num_sms) == B200_OK;
     };
     for (int l = 0; hyper && l < d.n_layers; ++l) {
       const b200_stack_layer& L = s->layers[l];
@@ -2023,7 +2029,8 @@ static int stack_build(const b200_stack_desc* desc, b200_engine** out) {
         sp.ok_ff_in = plan(&sp.ff_in, L.w_ff_in, L.ff, d.width, EPI_BIAS_F32);
         sp.ok_ff_out = plan(&sp.ff_out, L.w_ff_out, d.width, L.ff, EPI_BIAS_F32);
       } else if (L.ff_kind == B200_FF_GATED && L.ff > 0) {
-        sp.ok_ff_in = plan(&sp.ff_in, L.w_ff_in, 2 * (int64_t)L.ff, d.width, EPI_BIAS_F32);
+        sp.ok_glu = L.ff_act == B200_ACT_SILU && plan(&sp.ff_in, L.w_ff_in, L.ff, d.width, EPI_SWIGLU, PRO_PLAIN, 2);
+        if (!sp.ok_glu) sp.ok_ff_in = plan(&sp.ff_in, L.w_ff_in, 2 * (int64_t)L.ff, d.width, EPI_BIAS_F32);
         sp.ok_ff_out = plan(&sp.ff_out, L.w_ff_out, d.width, L.ff, EPI_BIAS_F32);
       } else if (L.ff_kind == B200_FF_MOE && L.moe.shared_ff > 0) {
         sp.ok_ff_in = plan(&sp.ff_in, L.w_ff_in, L.moe.expert_act != 0 ? up8i(L.moe.shared_ff) : up8i(2 * L.moe.shared_ff + 1),

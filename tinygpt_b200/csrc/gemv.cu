@@ -390,6 +390,8 @@ gemv_stream_kernel(const GemvParams p, const __grid_constant__ CUtensorMap tmap)
         const float g = round_bf16(a0);
         const __nv_bfloat16 sg = f_to_bf16(g / (1.f + expf(-g)));
         p.y[row] = __hmul(sg, f_to_bf16(a1));
+      } else if constexpr (EPI == EPI_SWIGLU) {
+        p.y[row] = f_to_bf16(a0 / (1.f + expf(-a0)) * a1);
       } else if constexpr (EPI == EPI_BIAS_F32) {
         const float v = a0 + (p.fbias != nullptr ? p.fbias[row] : 0.f);
         if (p.yf != nullptr) p.yf[row] = v;   // the unrounded value too (fp32 logits beside the sampler's bf16 copy)
@@ -419,6 +421,7 @@ using KernelFn = void (*)(const GemvParams, const CUtensorMap);
 template <int RPW>
 KernelFn pick_kernel(int nseg, int pro, int epi) {
   if (nseg == 2) {
+    if (pro == PRO_PLAIN && epi == EPI_SWIGLU) return gemv_stream_kernel<RPW, 2, PRO_PLAIN, EPI_SWIGLU>;
     if (epi != EPI_SILU_MUL) return nullptr;
     switch (pro) {
       case PRO_PLAIN: return gemv_stream_kernel<RPW, 2, PRO_PLAIN, EPI_SILU_MUL>;

@@ -20,9 +20,10 @@ constexpr int kGemvProCount = 4;
 //   EPI_BIAS_F32  y = bf16(acc + fbias)                                 (stack models: fp32 bias, one rounding)
 //   EPI_RESID_F32 yf += mult · acc                                      (stack models: fp32 residual stream)
 //   EPI_ACT_TABLE y = bf16(gelu_tanh(acc) · table[tok·table_ld + table_col + row])   (stack models: gated token table)
+//   EPI_SWIGLU    y = bf16(silu(acc_gate) · acc_up)                     (stack models: merged gate|up projection, one rounding)
 enum GemvEpi : int { EPI_PLAIN = 0, EPI_RESIDUAL = 1, EPI_SILU_MUL = 2, EPI_TP_PUSH = 3, EPI_BIAS_F32 = 4,
-                     EPI_RESID_F32 = 5, EPI_ACT_TABLE = 6 };
-constexpr int kGemvEpiCount = 7;
+                     EPI_RESID_F32 = 5, EPI_ACT_TABLE = 6, EPI_SWIGLU = 7 };
+constexpr int kGemvEpiCount = 8;
 
 constexpr int kMaxTpWorld = 8;
 constexpr int kMaxBatch = 8;   // sequences one batched decode step serves (gemv_batch.cu: W streamed once for all of them)

@@ -58,7 +58,7 @@ gemv_batch_kernel(const GemvParams p, const __grid_constant__ CUtensorMap tmap) 
   constexpr bool kHalfTile = kRowsStage == 8;       // rows 8-15 of the only tile do not exist: a1 = a3 = 0
   constexpr int kSliceK = KB * 32;                  // k-elements of a stage one warp owns
   static_assert(PRO == PRO_PLAIN || PRO == PRO_RMSNORM || PRO == PRO_F32, "single-GPU prologues only");
-  static_assert(EPI == EPI_PLAIN || EPI == EPI_RESIDUAL || EPI == EPI_SILU_MUL || EPI == EPI_BIAS_F32 ||
+  static_assert(EPI == EPI_PLAIN || EPI == EPI_RESIDUAL || EPI == EPI_SILU_MUL || EPI == EPI_SWIGLU || EPI == EPI_BIAS_F32 ||
                     EPI == EPI_RESID_F32 || EPI == EPI_ACT_TABLE,
                 "single-GPU epilogues only");
 
@@ -368,6 +368,8 @@ gemv_batch_kernel(const GemvParams p, const __grid_constant__ CUtensorMap tmap) 
         const float z = a[0];
         const float gl = 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
         y[row] = f_to_bf16(gl * bf16_to_f(p.table[(long long)p.tok[it_b] * p.table_ld + p.table_col + row]));
+      } else if constexpr (EPI == EPI_SWIGLU) {
+        y[row] = f_to_bf16(a[0] / (1.f + expf(-a[0])) * a[NSEG - 1]);
       } else {  // EPI_SILU_MUL
         const float gt = round_bf16(a[0]);
         const __nv_bfloat16 sg = f_to_bf16(gt / (1.f + expf(-gt)));
@@ -384,6 +386,7 @@ using KernelFn = void (*)(const GemvParams, const CUtensorMap);
 
 template <int RPW>
 KernelFn pick_r(int nseg, int pro, int epi) {
+  if (nseg == 2 && pro == PRO_PLAIN && epi == EPI_SWIGLU) return gemv_batch_kernel<RPW, 2, PRO_PLAIN, EPI_SWIGLU>;
   if (nseg == 2) return (pro == PRO_RMSNORM && epi == EPI_SILU_MUL) ? gemv_batch_kernel<RPW, 2, PRO_RMSNORM, EPI_SILU_MUL> : nullptr;
   if (pro == PRO_RMSNORM && epi == EPI_PLAIN) return gemv_batch_kernel<RPW, 1, PRO_RMSNORM, EPI_PLAIN>;
   if (pro == PRO_PLAIN && epi == EPI_RESIDUAL) return gemv_batch_kernel<RPW, 1, PRO_PLAIN, EPI_RESIDUAL>;

@@ -509,7 +509,7 @@ def main_bibezen(sizes: str, steps: int, warmup: int) -> None:
 # parameters).
 FAVUDRA_SIZES = {
     "f2048": dict(width=2048, vocab=65536, heads=16, kv_heads=8, dim=128, rot_dims=64, conv=3, window=1024, g_heads=16, g_kv=8, g_dim=128,
-                  g_vdim=128, rank=16, ff=5464),
+                  g_vdim=128, rank=16, ff=5472),
     "f3072": dict(width=3072, vocab=65536, heads=24, kv_heads=8, dim=128, rot_dims=64, conv=3, window=1024, g_heads=24, g_kv=8, g_dim=128,
                   g_vdim=128, rank=16, ff=8192),
 }

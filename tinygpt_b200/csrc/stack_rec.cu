@@ -6,6 +6,7 @@
 #include "stack_rec.cuh"
 
 #include <algorithm>
+#include <type_traits>
 
 #include "stack_hyper.cuh"
 
@@ -105,7 +106,7 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnPrep p) {
 }
 
 // ------------------------------------------------------------------------------------------------------------ the scan
-// One warp per (sequence, head, NC value columns): lane l holds rows l, l + 32, … of its columns of S (DR rows per lane and
+// With a removal: one warp per (sequence, head, NC value columns): lane l holds rows l, l + 32, … of its columns of S (DR rows per lane and
 // column); 8·NC columns per CTA.  The CTA walks its sequence CH tokens at a time: the chunk's decay, key, query (and removal,
 // unit key) rows (fp32, zero past dk) and the CTA's columns of v sit in shared memory, staged once for all eight warps,
 // while the next chunk's values are already on their way into registers — the walk waits for memory once per sequence.  A
@@ -113,24 +114,20 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnPrep p) {
 // multiply-adds per operand and column, and the output's dot with the NEW columns.  Columns never read each other, so
 // the result of a sequence does not depend on what else is in the step; the order of the sums inside a column is fixed by
 // dk alone (lane l sums rows l, l + 32, …, then the butterfly), whatever NC is.
-// OLD: the output reads the columns BEFORE the token joins them, plus the token's bonus times its value.  DM1: d holds the
-// decay minus one, so that a decay close to one keeps all its digits.
-template <int DR, bool REMOVE, int NC, bool OLD = false, bool DM1 = OLD>
+template <int DR, int NC>
 __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
   pdl_trigger();
   pdl_wait();
   constexpr int DK = 32 * DR;
-  // tokens per chunk: what 8 KB (with the removal's two extra rows: 4 KB) of one operand hold, 4 … 32 — the next chunk waits
-  // in registers, and two CTAs share an SM
-  constexpr int CH0 = (REMOVE ? 1024 : 2048) / DK;
+  // tokens per chunk: what 4 KB of one operand hold, 4 … 32 — the next chunk waits in registers, and two CTAs share an SM
+  constexpr int CH0 = 1024 / DK;
   constexpr int CH = CH0 > 32 ? 32 : CH0 < 4 ? 4 : CH0;
-  constexpr int NV = REMOVE ? 5 : 3;                      // staged vectors per token: d, b, r (, p, q)
+  constexpr int NV = 5;                                   // staged vectors per token: d, b, r, p, q
   constexpr int NQ = CH * NV * DK / 256;                  // staged vector elements per thread and chunk
   constexpr int COLS = 8 * NC;
   constexpr int NVR = (CH * COLS + 255) / 256;            // staged values per thread and chunk
   __shared__ float s_x[CH][NV][DK];
   __shared__ float s_v[CH][COLS];
-  __shared__ float s_bonus[CH];
   const int seg = blockIdx.x, hd = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
   const int dk = p.dk, dv = p.dv;
   const int j0 = blockIdx.z * COLS, jw = j0 + warp * NC;
@@ -151,9 +148,9 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
   const float* src_d = p.d_scalar ? p.d + hd : p.d + (int64_t)hd * dk;
   const float* src_b = p.b + (int64_t)hs * dk;
   const float* src_r = p.r + (int64_t)hs * dk;
-  const float* src_p = REMOVE ? p.p + (int64_t)hd * dk : nullptr;
-  const float* src_q = REMOVE ? p.q + (int64_t)(p.q_shared ? hs : hd) * dk : nullptr;
-  float r_x[NQ], r_v[NVR], r_b = 0.f;
+  const float* src_p = p.p + (int64_t)hd * dk;
+  const float* src_q = p.q + (int64_t)(p.q_shared ? hs : hd) * dk;
+  float r_x[NQ], r_v[NVR];
   auto fetch = [&](int c0) {
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
@@ -177,7 +174,6 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
       }
       r_v[i] = val;
     }
-    if constexpr (OLD) r_b = tid < CH && c0 + tid < cnt ? p.bonus[(int64_t)(r0 + c0 + tid) * p.ld + hd] : 0.f;
   };
   fetch(0);
   for (int c0 = 0; c0 < cnt; c0 += CH) {
@@ -188,7 +184,6 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
 #pragma unroll
     for (int i = 0; i < NVR; ++i)
       if (tid + 256 * i < CH * COLS) (&s_v[0][0])[tid + 256 * i] = r_v[i];
-    if (OLD && tid < CH) s_bonus[tid] = r_b;
     __syncthreads();
     if (c0 + CH < cnt) fetch(c0 + CH);
     if (jw >= dv) continue;   // warps past the last column only help with the staging
@@ -206,33 +201,26 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
           rem[c] = 0.f;
           vj[c] = s_v[t][warp * NC + c];
         }
-        if constexpr (REMOVE) {
 #pragma unroll
-          for (int i = 0; i < DR; ++i) {
-            const float qq = s_x[t][4][lane + 32 * i];
+        for (int i = 0; i < DR; ++i) {
+          const float qq = s_x[t][4][lane + 32 * i];
 #pragma unroll
-            for (int c = 0; c < NC; ++c) rem[c] = fmaf(qq, S[c][i], rem[c]);
-          }
+          for (int c = 0; c < NC; ++c) rem[c] = fmaf(qq, S[c][i], rem[c]);
+        }
 #pragma unroll
-          for (int o = 16; o > 0; o >>= 1) {
+        for (int o = 16; o > 0; o >>= 1) {
 #pragma unroll
-            for (int c = 0; c < NC; ++c) rem[c] += __shfl_xor_sync(0xffffffffu, rem[c], o);
-          }
+          for (int c = 0; c < NC; ++c) rem[c] += __shfl_xor_sync(0xffffffffu, rem[c], o);
         }
 #pragma unroll
         for (int i = 0; i < DR; ++i) {
           const int d = lane + 32 * i;
-          const float dd = s_x[t][0][d], bb = s_x[t][1][d], rr = s_x[t][2][d];
-          float pp = 0.f;
-          if constexpr (REMOVE) pp = s_x[t][3][d];
+          const float dd = s_x[t][0][d], bb = s_x[t][1][d], rr = s_x[t][2][d], pp = s_x[t][3][d];
 #pragma unroll
           for (int c = 0; c < NC; ++c) {
-            if constexpr (OLD) dot[u][c] = fmaf(S[c][i], rr, dot[u][c]);
-            float sn = DM1 ? fmaf(dd, S[c][i], S[c][i]) : dd * S[c][i];
-            if constexpr (REMOVE) sn = fmaf(-pp, rem[c], sn);
-            sn = fmaf(bb, vj[c], sn);
+            const float sn = fmaf(bb, vj[c], fmaf(-pp, rem[c], dd * S[c][i]));
             S[c][i] = sn;
-            if constexpr (!OLD) dot[u][c] = fmaf(sn, rr, dot[u][c]);
+            dot[u][c] = fmaf(sn, rr, dot[u][c]);
           }
         }
       }
@@ -252,7 +240,6 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
 #pragma unroll
           for (int cc = 0; cc < NC; ++cc) mine = (uu == u && cc == c) ? dot[uu][cc] : mine;
         }
-        if constexpr (OLD) mine = fmaf(s_bonus[t4 + u], s_v[t4 + u][warp * NC + c], mine);   // t4 + u < CH
         if (t4 + u < n && jw + c < dv) p.o[(int64_t)(r0 + c0 + t4 + u) * p.ld_o + (int64_t)hd * dv + jw + c] = mine;
       }
     }
@@ -266,6 +253,235 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
       if (d < dk) st[(int64_t)d * dv + jw + c] = S[c][i];
     }
   }
+}
+
+// Without a removal no row of S waits for another: a CTA of four warps takes kScanCols value columns of one (sequence, head), a
+// thread a tile of RS neighbouring rows and four neighbouring columns (an operand a thread reads from shared memory serves four
+// multiply-adds: the walk is bound by that traffic).  A token's output parts meet inside a warp by four shuffles per thread and,
+// once per chunk, over the warps through shared memory; nothing the state waits for.  The chunk's decay, key and query rows come
+// in by cp.async while the chunk before is walked (two buffers).  The order of the sums inside a column is fixed by dk alone.
+// MODE 0: d is the decay, 1: the decay minus one (a decay close to one keeps all its digits), 2: the decay minus one, and the
+// output reads the columns BEFORE the token joins them, plus the token's bonus times its value.  SCALAR: one decay per head.
+constexpr int kScanCols = 16, kScanThreads = 128, kScanSlices = kScanThreads / 4;
+template <int RS, bool SCALAR>
+struct ScanCols {
+  static constexpr int DK = kScanSlices * RS, NV = SCALAR ? 2 : 3;   // staged vectors per token: b, r (, d)
+  static constexpr int CH0 = 2048 / DK, CH = CH0 > 32 ? 32 : CH0 < 4 ? 4 : CH0;
+  static constexpr int smem = (2 * CH * NV * DK + CH * 4 * kScanCols + 2 * CH * (kScanCols + 2)) * 4;
+};
+__device__ __forceinline__ void scan_cp(float* dst, const float* src, int bytes, bool wide) {
+  const uint32_t d = smem_u32(dst);
+  if (wide) asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(bytes) : "memory");
+  else asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(d), "l"(src), "r"(bytes) : "memory");
+}
+// two fp32 multiply-adds (products) in one instruction; a pair of neighbouring rows travels as one 64-bit register pair
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ uint64_t pair2(float lo, float hi) {
+  uint64_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ float2 split2(uint64_t a) {
+  float2 d;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(a));
+  return d;
+}
+template <int RS, int MODE, bool SCALAR>
+__global__ void __launch_bounds__(kScanThreads, RS <= 8 ? 4 : 2) lin_scan_cols_kernel(const LinScan p, const bool wide) {
+  using C = ScanCols<RS, SCALAR>;
+  constexpr int DK = C::DK, NV = C::NV, CH = C::CH, NVR = (CH * kScanCols + kScanThreads - 1) / kScanThreads;
+  pdl_trigger();
+  pdl_wait();
+  extern __shared__ __align__(16) float sm[];
+  float* const s_x = sm;                               // [2][CH][NV][DK]
+  float* const s_v = s_x + 2 * CH * NV * DK;           // [2][CH][kScanCols]
+  float* const s_part = s_v + 2 * CH * kScanCols;      // [CH][4][kScanCols]
+  float* const s_s = s_part + CH * 4 * kScanCols;      // [2][CH][2]: the token's scalar decay and bonus
+  const int seg = blockIdx.x, hd = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int dk = p.dk, dv = p.dv, c4 = (tid & 3) * 4, j0 = blockIdx.z * kScanCols + c4, d0 = (tid >> 2) * RS;
+  const int r0 = p.seg_row0 != nullptr ? p.seg_row0[seg] : seg;
+  const int cnt = p.seg_count != nullptr ? p.seg_count[seg] : 1;
+  float* st = p.state + (int64_t)p.slot[r0] * p.slot_stride + (int64_t)hd * dk * dv;
+  const bool fresh = p.pos[r0] == 0;
+  uint64_t S[RS / 2][4];
+  auto held = [&](int i, int c) { return j0 + c < dv && d0 + i < dk; };
+#pragma unroll
+  for (int i = 0; i < RS / 2; ++i)
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+      S[i][c] = pair2(!fresh && held(2 * i, c) ? st[(int64_t)(d0 + 2 * i) * dv + j0 + c] : 0.f,
+                      !fresh && held(2 * i + 1, c) ? st[(int64_t)(d0 + 2 * i + 1) * dv + j0 + c] : 0.f);
+  const int hs = hd / p.share;   // the head whose b / r vectors this head reads
+  const float* src_b = p.b + (int64_t)hs * dk;
+  const float* src_r = p.r + (int64_t)hs * dk;
+  const float* src_d = SCALAR ? p.d + hd : p.d + (int64_t)hd * dk;
+  auto stage = [&](int c0, int buf) {
+    const int n = min(CH, cnt - c0);
+    float* x = s_x + buf * (CH * NV * DK);
+    if (wide) {   // a thread keeps its place in the row and takes every RP-th token
+      constexpr int UN = DK / 4, RP = kScanThreads / UN;
+      const int td = (tid % UN) * 4, tr = tid / UN, bytes = td < dk ? 16 : 0;   // zeros past the key size
+      const int64_t o = (int64_t)(r0 + c0 + tr) * p.ld + (td < dk ? td : 0), ld = p.ld * RP;
+      const float *qb = src_b + o, *qr = src_r + o, *qd = SCALAR ? nullptr : src_d + o;
+      float* dst = x + tr * (NV * DK) + td;
+#pragma unroll
+      for (int u = 0; u < (CH + RP - 1) / RP; ++u) {
+        if (tr + u * RP >= n) break;
+        scan_cp(dst + u * RP * NV * DK, qb + u * ld, bytes, true);
+        scan_cp(dst + u * RP * NV * DK + DK, qr + u * ld, bytes, true);
+        if constexpr (!SCALAR) scan_cp(dst + u * RP * NV * DK + 2 * DK, qd + u * ld, bytes, true);
+      }
+    } else {
+      for (int e = tid; e < n * NV * DK; e += kScanThreads) {
+        const int t = e / (NV * DK), w = (e / DK) % NV, d = e % DK;
+        const float* src = (w == 0 ? src_b : w == 1 ? src_r : src_d) + (int64_t)(r0 + c0 + t) * p.ld;
+        scan_cp(x + e, d < dk ? src + d : src, d < dk ? 4 : 0, false);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  float r_v[NVR], r_s[2];
+  auto fetch = [&](int c0) {
+#pragma unroll
+    for (int i = 0; i < NVR; ++i) {
+      const int e = tid + kScanThreads * i, t = e / kScanCols, c = blockIdx.z * kScanCols + e % kScanCols;
+      float val = 0.f;
+      if (t < CH && c0 + t < cnt && c < dv) {
+        const int64_t base = (int64_t)(r0 + c0 + t) * p.ld;
+        val = p.v[base + (int64_t)hd * dv + c];
+        if (p.vscale != nullptr) val *= p.vscale[base + hd];
+      }
+      r_v[i] = val;
+    }
+    const bool live = tid < CH && c0 + tid < cnt;
+    if constexpr (SCALAR) r_s[0] = live ? src_d[(int64_t)(r0 + c0 + tid) * p.ld] : 0.f;
+    if constexpr (MODE == 2) r_s[1] = live ? p.bonus[(int64_t)(r0 + c0 + tid) * p.ld + hd] : 0.f;
+  };
+  stage(0, 0);
+  fetch(0);
+  for (int c0 = 0, buf = 0; c0 < cnt; c0 += CH, buf ^= 1) {
+    const int n = min(CH, cnt - c0);
+    float* v = s_v + buf * (CH * kScanCols);
+    float* sc = s_s + buf * (CH * 2);
+#pragma unroll
+    for (int i = 0; i < NVR; ++i)
+      if (tid + kScanThreads * i < CH * kScanCols) v[tid + kScanThreads * i] = r_v[i];
+    if (tid < CH) {
+      if constexpr (SCALAR) sc[2 * tid] = r_s[0];
+      if constexpr (MODE == 2) sc[2 * tid + 1] = r_s[1];
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();   // this chunk is there; the chunk before has been walked and handed out
+    if (c0 + CH < cnt) {
+      stage(c0 + CH, buf ^ 1);
+      fetch(c0 + CH);
+    }
+    const float* x = s_x + buf * (CH * NV * DK) + d0;
+    auto walk = [&](int t, auto group) {   // `group` tokens from t on: their operands load, and their parts leave, side by side
+      constexpr int U = decltype(group)::value, W = RS < 4 ? 1 : 2;   // pairs of rows per load
+      float dot[U][4];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const float4 vf = *reinterpret_cast<const float4*>(v + (t + u) * kScanCols + c4);
+        const uint64_t vj[4] = {pair2(vf.x, vf.x), pair2(vf.y, vf.y), pair2(vf.z, vf.z), pair2(vf.w, vf.w)};
+        const uint64_t ds = SCALAR ? pair2(sc[2 * (t + u)], sc[2 * (t + u)]) : 0;
+        const float* xt = x + (t + u) * (NV * DK);
+        uint64_t acc[4];
+#pragma unroll
+        for (int i0 = 0; i0 < RS / 2; i0 += W) {
+          uint64_t b[W], r[W], d[W];
+          auto load = [&](uint64_t(&o)[W], const float* q) {
+            if constexpr (W == 2) {
+              const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(q);
+              o[0] = w.x;
+              o[1] = w.y;
+            } else {
+              o[0] = *reinterpret_cast<const unsigned long long*>(q);
+            }
+          };
+          load(b, xt + 2 * i0);
+          load(r, xt + DK + 2 * i0);
+          if constexpr (!SCALAR) load(d, xt + 2 * DK + 2 * i0);
+#pragma unroll
+          for (int i = 0; i < W; ++i) {
+            const uint64_t dd = SCALAR ? ds : d[i];
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+              const uint64_t old = S[i0 + i][c];
+              const uint64_t sn = fma2(b[i], vj[c], MODE == 0 ? mul2(dd, old) : fma2(dd, old, old));
+              S[i0 + i][c] = sn;
+              const uint64_t w = MODE == 2 ? old : sn;
+              acc[c] = i0 + i == 0 ? mul2(w, r[i]) : fma2(w, r[i], acc[c]);
+            }
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const float2 a = split2(acc[c]);
+          dot[u][c] = a.x + a.y;
+        }
+      }
+      // four columns over the warp's eight row slices (lane bits 2 … 4): halves of the columns change hands twice, then a sum
+      const bool h4 = lane & 16, h3 = lane & 8;
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        float k0 = h4 ? dot[u][2] : dot[u][0], k1 = h4 ? dot[u][3] : dot[u][1];
+        k0 += __shfl_xor_sync(0xffffffffu, h4 ? dot[u][0] : dot[u][2], 16);
+        k1 += __shfl_xor_sync(0xffffffffu, h4 ? dot[u][1] : dot[u][3], 16);
+        float k = h3 ? k1 : k0;
+        k += __shfl_xor_sync(0xffffffffu, h3 ? k0 : k1, 8);
+        k += __shfl_xor_sync(0xffffffffu, k, 4);
+        if (!(lane & 4)) s_part[((t + u) * 4 + warp) * kScanCols + c4 + (h4 ? 2 : 0) + (h3 ? 1 : 0)] = k;
+      }
+    };
+    constexpr int G = RS <= 4 ? 4 : RS <= 8 ? 2 : 1;
+    int t = 0;
+    for (; t + G <= n; t += G) walk(t, std::integral_constant<int, G>{});
+    for (; t < n; ++t) walk(t, std::integral_constant<int, 1>{});
+    __syncthreads();
+    for (int e = tid; e < n * kScanCols; e += kScanThreads) {
+      const int t = e / kScanCols, c = e % kScanCols, cj = blockIdx.z * kScanCols + c;
+      const float* q = s_part + t * 4 * kScanCols + c;
+      float o = (q[0] + q[kScanCols]) + (q[2 * kScanCols] + q[3 * kScanCols]);
+      if constexpr (MODE == 2) o = fmaf(sc[2 * t + 1], v[e], o);
+      if (cj < dv) p.o[(int64_t)(r0 + c0 + t) * p.ld_o + (int64_t)hd * dv + cj] = o;
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < RS / 2; ++i)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      const float2 a = split2(S[i][c]);
+      if (held(2 * i, c)) st[(int64_t)(d0 + 2 * i) * dv + j0 + c] = a.x;
+      if (held(2 * i + 1, c)) st[(int64_t)(d0 + 2 * i + 1) * dv + j0 + c] = a.y;
+    }
+}
+
+template <int RS, int MODE, bool SCALAR>
+int launch_scan_cols(const LinScan& p, cudaStream_t st) {
+  constexpr int smem = ScanCols<RS, SCALAR>::smem;
+  static cudaError_t attr = cudaFuncSetAttribute(lin_scan_cols_kernel<RS, MODE, SCALAR>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  B200_CUDA(attr);
+  auto al = [](const float* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  const bool wide = p.dk % 4 == 0 && p.ld % 4 == 0 && al(p.b) && al(p.r) && (SCALAR || al(p.d));
+  const dim3 grid(p.n_seg, p.heads, (p.dv + kScanCols - 1) / kScanCols);
+  B200_CUDA(launch_pdl(lin_scan_cols_kernel<RS, MODE, SCALAR>, grid, dim3(kScanThreads), smem, st, stack_pdl(), p, wide));
+  return B200_OK;
+}
+template <int RS>
+int launch_scan_cols(const LinScan& p, cudaStream_t st) {
+  if (p.read_old) return launch_scan_cols<RS, 2, false>(p, st);
+  if (p.d_minus_one) return launch_scan_cols<RS, 1, false>(p, st);
+  return p.d_scalar ? launch_scan_cols<RS, 0, true>(p, st) : launch_scan_cols<RS, 0, false>(p, st);
 }
 
 // ------------------------------------------------------------------------------------------- generalized delta rule
@@ -1049,23 +1265,23 @@ int launch_lin_scan(const LinScan& p, cudaStream_t st) {
                  "linear scan: null argument");
   B200_CHECK_ARG((p.p == nullptr) == (p.q == nullptr), "linear scan: the removal needs both of its vectors");
   B200_CHECK_ARG(p.heads > 0 && p.dk > 0 && p.dv > 0 && p.share > 0 && p.heads % p.share == 0, "linear scan: bad sizes");
+  B200_CHECK_ARG(!p.d_scalar || (!p.read_old && !p.d_minus_one), "linear scan: a scalar decay is given as it is");
   B200_CHECK_ARG(!p.read_old || (p.p == nullptr && p.bonus && p.vscale == nullptr), "linear scan: reading the old state takes a bonus and no removal");
   B200_CHECK_ARG(!p.d_minus_one || p.p == nullptr, "linear scan: a decay minus one takes no removal");
   B200_CHECK_ARG(p.dk <= kScanMaxDim, "linear scan: more than %d key channels not built", kScanMaxDim);
+  if (p.p == nullptr) {
+    if (p.dk <= 64) return launch_scan_cols<2>(p, st);
+    if (p.dk <= 128) return launch_scan_cols<4>(p, st);
+    if (p.dk <= 256) return launch_scan_cols<8>(p, st);
+    return launch_scan_cols<16>(p, st);
+  }
   // two columns per warp where the value size fills them and the registers hold them: half the CTAs stage the same rows
   const int nc = (p.dv >= 32 && p.dk <= 256) ? 2 : 1;
   const dim3 grid(p.n_seg, p.heads, (p.dv + 8 * nc - 1) / (8 * nc));
-#define B200_SCAN_NC(DR, NC)                                                                                       \
-  do {                                                                                                             \
-    if (p.p != nullptr) B200_CUDA(launch_pdl(lin_scan_kernel<DR, true, NC>, grid, dim3(256), 0, st, stack_pdl(), p));  \
-    else if (p.read_old) B200_CUDA(launch_pdl(lin_scan_kernel<DR, false, NC, true>, grid, dim3(256), 0, st, stack_pdl(), p)); \
-    else if (p.d_minus_one) B200_CUDA(launch_pdl(lin_scan_kernel<DR, false, NC, false, true>, grid, dim3(256), 0, st, stack_pdl(), p)); \
-    else B200_CUDA(launch_pdl(lin_scan_kernel<DR, false, NC>, grid, dim3(256), 0, st, stack_pdl(), p));           \
-  } while (0)
-#define B200_SCAN(DR)              \
-  do {                             \
-    if (nc == 2) B200_SCAN_NC(DR, 2); \
-    else B200_SCAN_NC(DR, 1);      \
+#define B200_SCAN(DR)                                                                                           \
+  do {                                                                                                          \
+    if (nc == 2) B200_CUDA(launch_pdl(lin_scan_kernel<DR, 2>, grid, dim3(256), 0, st, stack_pdl(), p));          \
+    else B200_CUDA(launch_pdl(lin_scan_kernel<DR, 1>, grid, dim3(256), 0, st, stack_pdl(), p));                  \
   } while (0)
   if (p.dk <= 32) B200_SCAN(1);
   else if (p.dk <= 64) B200_SCAN(2);
@@ -1073,7 +1289,6 @@ int launch_lin_scan(const LinScan& p, cudaStream_t st) {
   else if (p.dk <= 256) B200_SCAN(8);
   else B200_SCAN(16);
 #undef B200_SCAN
-#undef B200_SCAN_NC
   return B200_OK;
 }
 

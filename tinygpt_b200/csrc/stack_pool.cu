@@ -195,6 +195,123 @@ __global__ void __launch_bounds__(256) pool_prep_strip_kernel(const PoolAttn p) 
   }
 }
 
+// The same preparation without shared memory, for bf16 rows whose head sizes are multiples of four up to 128 and whose pairs are
+// neighbours: one warp per (strip of tokens, head), a lane holds four neighbouring channels.  The strip's rows are requested
+// together; a token then costs the convolution in registers, one warp sum for the norm, the turn inside the lane and one
+// eight-byte store.  single: a strip is one row, whose convolution state — requested ahead of the dependency wait, an earlier step
+// left it there — moves on here.
+constexpr int kHeadStrip = 8;
+template <int TAPS, bool SINGLE>
+__global__ void __launch_bounds__(256) head_prep_kernel(const PoolAttn p) {
+  using T = __nv_bfloat16;
+  constexpr int STRIP = SINGLE ? 1 : kHeadStrip;
+  pdl_trigger();
+  const int H = p.a.heads, G = p.a.kv_heads, unit = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (unit >= H + (p.q_only ? 0 : 2 * G)) return;
+  const bool is_q = unit < H, is_v = unit >= H + G;
+  const int head = is_q ? unit : is_v ? unit - H - G : unit - H, ch = is_v ? p.a.vdim : p.a.dim, c = lane * 4;
+  const bool act = c < ch;
+  const int col = (is_q ? p.off_q : is_v ? p.off_v : p.off_k) + head * ch + (act ? c : 0);
+  const int t0 = blockIdx.x * STRIP, n = min(STRIP, p.n_tok - t0);
+  float w[TAPS][4], nw[4] = {1.f, 1.f, 1.f, 1.f}, win[TAPS][4];   // win[j]: the row j positions back
+  auto load4 = [](float(&o)[4], const float* q) {
+    const float4 v = *reinterpret_cast<const float4*>(q);
+    o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w;
+  };
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) load4(w[j], p.d.conv_w + (int64_t)j * p.ld_proj + col);
+  const float* norm_w = is_v ? nullptr : is_q ? p.d.q_norm : p.d.k_norm;
+  if (norm_w != nullptr && act) load4(nw, norm_w + c);
+  float* cs = p.conv_state + col;   // the slot's part is added below
+  if constexpr (SINGLE) {
+    cs += (int64_t)p.slot[t0] * p.conv_slot_stride;
+    const int ps = p.pos[t0];
+#pragma unroll
+    for (int j = 1; j < TAPS; ++j) {
+      if (ps - j >= 0) load4(win[j], cs + (int64_t)(TAPS - 1 - j) * p.ld_proj);
+      else win[j][0] = win[j][1] = win[j][2] = win[j][3] = 0.f;
+    }
+  }
+  pdl_wait();
+  const T* x = static_cast<const T*>(p.proj) + (int64_t)t0 * p.ld_proj + col;
+  uint2 raw[STRIP];
+#pragma unroll
+  for (int r = 0; r < STRIP; ++r) raw[r] = r < n ? *reinterpret_cast<const uint2*>(x + (int64_t)r * p.ld_proj) : make_uint2(0, 0);
+  auto unpack4 = [](float(&o)[4], uint2 v) {
+    o[0] = bf16_lo(v.x); o[1] = bf16_hi(v.x); o[2] = bf16_lo(v.y); o[3] = bf16_hi(v.y);
+  };
+  const bool one = SINGLE || rows_one_seq(p.slot, p.pos, t0, t0 + n);
+  const float inv_n = 1.f / (float)ch;
+#pragma unroll
+  for (int r = 0; r < STRIP; ++r) {
+    if (r >= n) break;
+    const int t = t0 + r, ps = p.pos[t];
+    if constexpr (!SINGLE) {
+      if (r == 0 || (!one && !row_same_seq(p.slot, p.pos, t, 1))) {
+        const int front = rows_in_front(p.slot, p.pos, t, TAPS - 1);
+        const float* st = cs + (int64_t)p.slot[t] * p.conv_slot_stride;
+#pragma unroll
+        for (int j = 1; j < TAPS; ++j) {
+          if (j <= front) unpack4(win[j], *reinterpret_cast<const uint2*>(x + (int64_t)(r - j) * p.ld_proj));
+          else if (ps - j >= 0) load4(win[j], st + (int64_t)(TAPS - 1 - (j - front)) * p.ld_proj);
+          else win[j][0] = win[j][1] = win[j][2] = win[j][3] = 0.f;
+        }
+      } else {
+#pragma unroll
+        for (int j = TAPS - 1; j > 0; --j)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) win[j][i] = win[j - 1][i];
+      }
+    }
+    unpack4(win[0], raw[r]);
+    float y[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      y[i] = 0.f;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) y[i] = fmaf(w[TAPS - 1 - j][i], win[j][i], y[i]);
+    }
+    if (norm_w != nullptr) {
+      const float ss = warp_sum(act ? fmaf(y[0], y[0], fmaf(y[1], y[1], fmaf(y[2], y[2], y[3] * y[3]))) : 0.f);
+      const float inv = 1.f / sqrtf(ss * inv_n + p.eps);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) y[i] *= inv * nw[i];
+    }
+    if (!is_v && c < p.d.rot_dims) {   // two pairs; their {cos, sin} lie side by side
+      float cs4[4];
+      load4(cs4, p.d.rot_table + (int64_t)ps * p.d.rot_dims + c);
+#pragma unroll
+      for (int i = 0; i < 4; i += 2) {
+        const float a = y[i], b = y[i + 1];
+        y[i] = a * cs4[i] - b * cs4[i + 1];
+        y[i + 1] = b * cs4[i] + a * cs4[i + 1];
+      }
+    }
+    if (act) {
+      T* dst = is_q ? static_cast<T*>(p.q) + ((int64_t)t * H + head) * ch
+                    : (is_v ? static_cast<T*>(p.vcache) + (int64_t)p.slot[t] * p.v_slot_stride
+                            : static_cast<T*>(p.kcache) + (int64_t)p.slot[t] * p.k_slot_stride) + ((int64_t)ps * G + head) * ch;
+      *reinterpret_cast<uint2*>(dst + c) = make_uint2(pack2(y[0], y[1]), pack2(y[2], y[3]));
+      if constexpr (SINGLE) {
+#pragma unroll
+        for (int i = 0; i < TAPS - 1; ++i)   // entry i: the row TAPS − 2 − i positions back
+          *reinterpret_cast<float4*>(cs + (int64_t)i * p.ld_proj) =
+              make_float4(win[TAPS - 2 - i][0], win[TAPS - 2 - i][1], win[TAPS - 2 - i][2], win[TAPS - 2 - i][3]);
+      }
+    }
+  }
+}
+// what head_prep_kernel takes
+bool head_prep_ok(const PoolAttn& p, int dtype) {
+  const b200_attn_desc& a = p.a;
+  auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };   // null pointers are aligned
+  return dtype == B200_BF16 && p.d.conv_w != nullptr && p.d.taps <= 4 && !(p.single && p.d.pool > 0) && a.dim % 4 == 0 && a.dim <= 128 &&
+         a.vdim % 4 == 0 && a.vdim <= 128 && p.d.rot_dims % 4 == 0 && (p.d.rot_dims == 0 || p.d.rot_interleaved) && p.off_q % 4 == 0 &&
+         p.off_k % 4 == 0 && p.off_v % 4 == 0 && p.ld_proj % 4 == 0 && p.k_slot_stride % 4 == 0 && p.v_slot_stride % 4 == 0 &&
+         p.conv_slot_stride % 4 == 0 && al(p.proj) && al(p.q) && al(p.kcache) && al(p.vcache) && al(p.conv_state) && al(p.d.conv_w) &&
+         al(p.d.q_norm) && al(p.d.k_norm) && al(p.d.rot_table);
+}
+
 // The blocks whose last position is among a sequence's rows of this step: the means of their cached keys and values (rows of
 // this step or of earlier ones).
 template <typename T>
@@ -450,6 +567,20 @@ int launch_pool_prep(const PoolAttn& run, int dtype, cudaStream_t st) {
   B200_CHECK_ARG(p.proj != nullptr, "pool attention: null projection");
   B200_CHECK_ARG(p.d.conv_w == nullptr || (p.d.taps >= 1 && p.d.taps <= kConvMaxTaps && (p.d.taps == 1 || p.conv_state)),
                  "pool attention: 1 … %d convolution taps with a state", kConvMaxTaps);
+  if (head_prep_ok(p, dtype)) {
+    const dim3 hg((p.n_tok + (p.single ? 1 : kHeadStrip) - 1) / (p.single ? 1 : kHeadStrip), (p.a.heads + (p.q_only ? 0 : 2 * p.a.kv_heads) + 7) / 8);
+#define B200_HP(TAPS)                                                                                                   \
+  do {                                                                                                                  \
+    if (p.single) B200_CUDA(launch_pdl(head_prep_kernel<TAPS, true>, hg, dim3(256), 0, st, stack_pdl(), p));            \
+    else B200_CUDA(launch_pdl(head_prep_kernel<TAPS, false>, hg, dim3(256), 0, st, stack_pdl(), p));                    \
+  } while (0)
+    if (p.d.taps == 1) B200_HP(1);
+    else if (p.d.taps == 2) B200_HP(2);
+    else if (p.d.taps == 3) B200_HP(3);
+    else B200_HP(4);
+#undef B200_HP
+    return B200_OK;
+  }
   // query heads per CTA: the strip's channels within 48 KB, and few rows spread over many CTAs
   const int per = p.a.heads / p.a.kv_heads, dk = p.a.dim, kv = p.q_only ? 0 : dk + p.a.vdim, limit = 12 * 1024;   // floats
   B200_CHECK_ARG(dk + kv <= limit, "pool attention: one query head and one key/value head exceed %d channels", limit);

@@ -255,19 +255,19 @@ __global__ void __launch_bounds__(256, 2) lin_scan_kernel(const LinScan p) {
   }
 }
 
-// Without a removal no row of S waits for another: a CTA of four warps takes kScanCols value columns of one (sequence, head), a
+// Without a removal no row of S waits for another: a CTA of NT threads takes kScanCols value columns of one (sequence, head), a
 // thread a tile of RS neighbouring rows and four neighbouring columns (an operand a thread reads from shared memory serves four
 // multiply-adds: the walk is bound by that traffic).  A token's output parts meet inside a warp by four shuffles per thread and,
 // once per chunk, over the warps through shared memory; nothing the state waits for.  The chunk's decay, key and query rows come
 // in by cp.async while the chunk before is walked (two buffers).  The order of the sums inside a column is fixed by dk alone.
 // MODE 0: d is the decay, 1: the decay minus one (a decay close to one keeps all its digits), 2: the decay minus one, and the
 // output reads the columns BEFORE the token joins them, plus the token's bonus times its value.  SCALAR: one decay per head.
-constexpr int kScanCols = 16, kScanThreads = 128, kScanSlices = kScanThreads / 4;
-template <int RS, bool SCALAR>
+constexpr int kScanCols = 16;
+template <int RS, int NT, bool SCALAR>
 struct ScanCols {
-  static constexpr int DK = kScanSlices * RS, NV = SCALAR ? 2 : 3;   // staged vectors per token: b, r (, d)
+  static constexpr int DK = NT / 4 * RS, NV = SCALAR ? 2 : 3;   // staged vectors per token: b, r (, d)
   static constexpr int CH0 = 2048 / DK, CH = CH0 > 32 ? 32 : CH0 < 4 ? 4 : CH0;
-  static constexpr int smem = (2 * CH * NV * DK + CH * 4 * kScanCols + 2 * CH * (kScanCols + 2)) * 4;
+  static constexpr int smem = (2 * CH * NV * DK + CH * (NT / 32) * kScanCols + 2 * CH * (kScanCols + 2)) * 4;
 };
 __device__ __forceinline__ void scan_cp(float* dst, const float* src, int bytes, bool wide) {
   const uint32_t d = smem_u32(dst);
@@ -295,17 +295,17 @@ __device__ __forceinline__ float2 split2(uint64_t a) {
   asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(a));
   return d;
 }
-template <int RS, int MODE, bool SCALAR>
-__global__ void __launch_bounds__(kScanThreads, RS <= 8 ? 4 : 2) lin_scan_cols_kernel(const LinScan p, const bool wide) {
-  using C = ScanCols<RS, SCALAR>;
-  constexpr int DK = C::DK, NV = C::NV, CH = C::CH, NVR = (CH * kScanCols + kScanThreads - 1) / kScanThreads;
+template <int RS, int NT, int MODE, bool SCALAR>
+__global__ void __launch_bounds__(NT, RS <= 8 ? 512 / NT : 2) lin_scan_cols_kernel(const LinScan p, const bool wide) {
+  using C = ScanCols<RS, NT, SCALAR>;
+  constexpr int DK = C::DK, NV = C::NV, CH = C::CH, NW = NT / 32, NVR = (CH * kScanCols + NT - 1) / NT;
   pdl_trigger();
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
   float* const s_x = sm;                               // [2][CH][NV][DK]
   float* const s_v = s_x + 2 * CH * NV * DK;           // [2][CH][kScanCols]
-  float* const s_part = s_v + 2 * CH * kScanCols;      // [CH][4][kScanCols]
-  float* const s_s = s_part + CH * 4 * kScanCols;      // [2][CH][2]: the token's scalar decay and bonus
+  float* const s_part = s_v + 2 * CH * kScanCols;      // [CH][NW][kScanCols]
+  float* const s_s = s_part + CH * NW * kScanCols;      // [2][CH][2]: the token's scalar decay and bonus
   const int seg = blockIdx.x, hd = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int dk = p.dk, dv = p.dv, c4 = (tid & 3) * 4, j0 = blockIdx.z * kScanCols + c4, d0 = (tid >> 2) * RS;
   const int r0 = p.seg_row0 != nullptr ? p.seg_row0[seg] : seg;
@@ -328,7 +328,7 @@ __global__ void __launch_bounds__(kScanThreads, RS <= 8 ? 4 : 2) lin_scan_cols_k
     const int n = min(CH, cnt - c0);
     float* x = s_x + buf * (CH * NV * DK);
     if (wide) {   // a thread keeps its place in the row and takes every RP-th token
-      constexpr int UN = DK / 4, RP = kScanThreads / UN;
+      constexpr int UN = DK / 4, RP = NT / UN;
       const int td = (tid % UN) * 4, tr = tid / UN, bytes = td < dk ? 16 : 0;   // zeros past the key size
       const int64_t o = (int64_t)(r0 + c0 + tr) * p.ld + (td < dk ? td : 0), ld = p.ld * RP;
       const float *qb = src_b + o, *qr = src_r + o, *qd = SCALAR ? nullptr : src_d + o;
@@ -341,7 +341,7 @@ __global__ void __launch_bounds__(kScanThreads, RS <= 8 ? 4 : 2) lin_scan_cols_k
         if constexpr (!SCALAR) scan_cp(dst + u * RP * NV * DK + 2 * DK, qd + u * ld, bytes, true);
       }
     } else {
-      for (int e = tid; e < n * NV * DK; e += kScanThreads) {
+      for (int e = tid; e < n * NV * DK; e += NT) {
         const int t = e / (NV * DK), w = (e / DK) % NV, d = e % DK;
         const float* src = (w == 0 ? src_b : w == 1 ? src_r : src_d) + (int64_t)(r0 + c0 + t) * p.ld;
         scan_cp(x + e, d < dk ? src + d : src, d < dk ? 4 : 0, false);
@@ -353,7 +353,7 @@ __global__ void __launch_bounds__(kScanThreads, RS <= 8 ? 4 : 2) lin_scan_cols_k
   auto fetch = [&](int c0) {
 #pragma unroll
     for (int i = 0; i < NVR; ++i) {
-      const int e = tid + kScanThreads * i, t = e / kScanCols, c = blockIdx.z * kScanCols + e % kScanCols;
+      const int e = tid + NT * i, t = e / kScanCols, c = blockIdx.z * kScanCols + e % kScanCols;
       float val = 0.f;
       if (t < CH && c0 + t < cnt && c < dv) {
         const int64_t base = (int64_t)(r0 + c0 + t) * p.ld;
@@ -374,7 +374,7 @@ __global__ void __launch_bounds__(kScanThreads, RS <= 8 ? 4 : 2) lin_scan_cols_k
     float* sc = s_s + buf * (CH * 2);
 #pragma unroll
     for (int i = 0; i < NVR; ++i)
-      if (tid + kScanThreads * i < CH * kScanCols) v[tid + kScanThreads * i] = r_v[i];
+      if (tid + NT * i < CH * kScanCols) v[tid + NT * i] = r_v[i];
     if (tid < CH) {
       if constexpr (SCALAR) sc[2 * tid] = r_s[0];
       if constexpr (MODE == 2) sc[2 * tid + 1] = r_s[1];
@@ -440,7 +440,7 @@ __global__ void __launch_bounds__(kScanThreads, RS <= 8 ? 4 : 2) lin_scan_cols_k
         float k = h3 ? k1 : k0;
         k += __shfl_xor_sync(0xffffffffu, h3 ? k0 : k1, 8);
         k += __shfl_xor_sync(0xffffffffu, k, 4);
-        if (!(lane & 4)) s_part[((t + u) * 4 + warp) * kScanCols + c4 + (h4 ? 2 : 0) + (h3 ? 1 : 0)] = k;
+        if (!(lane & 4)) s_part[((t + u) * NW + warp) * kScanCols + c4 + (h4 ? 2 : 0) + (h3 ? 1 : 0)] = k;
       }
     };
     constexpr int G = RS <= 4 ? 4 : RS <= 8 ? 2 : 1;
@@ -448,10 +448,12 @@ __global__ void __launch_bounds__(kScanThreads, RS <= 8 ? 4 : 2) lin_scan_cols_k
     for (; t + G <= n; t += G) walk(t, std::integral_constant<int, G>{});
     for (; t < n; ++t) walk(t, std::integral_constant<int, 1>{});
     __syncthreads();
-    for (int e = tid; e < n * kScanCols; e += kScanThreads) {
+    for (int e = tid; e < n * kScanCols; e += NT) {
       const int t = e / kScanCols, c = e % kScanCols, cj = blockIdx.z * kScanCols + c;
-      const float* q = s_part + t * 4 * kScanCols + c;
-      float o = (q[0] + q[kScanCols]) + (q[2 * kScanCols] + q[3 * kScanCols]);
+      const float* q = s_part + t * NW * kScanCols + c;
+      float o = 0.f;
+#pragma unroll
+      for (int w = 0; w < NW; ++w) o += q[w * kScanCols];
       if constexpr (MODE == 2) o = fmaf(sc[2 * t + 1], v[e], o);
       if (cj < dv) p.o[(int64_t)(r0 + c0 + t) * p.ld_o + (int64_t)hd * dv + cj] = o;
     }
@@ -466,22 +468,22 @@ __global__ void __launch_bounds__(kScanThreads, RS <= 8 ? 4 : 2) lin_scan_cols_k
     }
 }
 
-template <int RS, int MODE, bool SCALAR>
+template <int RS, int NT, int MODE, bool SCALAR>
 int launch_scan_cols(const LinScan& p, cudaStream_t st) {
-  constexpr int smem = ScanCols<RS, SCALAR>::smem;
-  static cudaError_t attr = cudaFuncSetAttribute(lin_scan_cols_kernel<RS, MODE, SCALAR>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  constexpr int smem = ScanCols<RS, NT, SCALAR>::smem;
+  static cudaError_t attr = cudaFuncSetAttribute(lin_scan_cols_kernel<RS, NT, MODE, SCALAR>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   B200_CUDA(attr);
   auto al = [](const float* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
   const bool wide = p.dk % 4 == 0 && p.ld % 4 == 0 && al(p.b) && al(p.r) && (SCALAR || al(p.d));
   const dim3 grid(p.n_seg, p.heads, (p.dv + kScanCols - 1) / kScanCols);
-  B200_CUDA(launch_pdl(lin_scan_cols_kernel<RS, MODE, SCALAR>, grid, dim3(kScanThreads), smem, st, stack_pdl(), p, wide));
+  B200_CUDA(launch_pdl(lin_scan_cols_kernel<RS, NT, MODE, SCALAR>, grid, dim3(NT), smem, st, stack_pdl(), p, wide));
   return B200_OK;
 }
-template <int RS>
+template <int RS, int NT>
 int launch_scan_cols(const LinScan& p, cudaStream_t st) {
-  if (p.read_old) return launch_scan_cols<RS, 2, false>(p, st);
-  if (p.d_minus_one) return launch_scan_cols<RS, 1, false>(p, st);
-  return p.d_scalar ? launch_scan_cols<RS, 0, true>(p, st) : launch_scan_cols<RS, 0, false>(p, st);
+  if (p.read_old) return launch_scan_cols<RS, NT, 2, false>(p, st);
+  if (p.d_minus_one) return launch_scan_cols<RS, NT, 1, false>(p, st);
+  return p.d_scalar ? launch_scan_cols<RS, NT, 0, true>(p, st) : launch_scan_cols<RS, NT, 0, false>(p, st);
 }
 
 // ------------------------------------------------------------------------------------------- generalized delta rule
@@ -1270,10 +1272,10 @@ int launch_lin_scan(const LinScan& p, cudaStream_t st) {
   B200_CHECK_ARG(!p.d_minus_one || p.p == nullptr, "linear scan: a decay minus one takes no removal");
   B200_CHECK_ARG(p.dk <= kScanMaxDim, "linear scan: more than %d key channels not built", kScanMaxDim);
   if (p.p == nullptr) {
-    if (p.dk <= 64) return launch_scan_cols<2>(p, st);
-    if (p.dk <= 128) return launch_scan_cols<4>(p, st);
-    if (p.dk <= 256) return launch_scan_cols<8>(p, st);
-    return launch_scan_cols<16>(p, st);
+    if (p.dk <= 64) return launch_scan_cols<2, 128>(p, st);
+    if (p.dk <= 128) return launch_scan_cols<4, 128>(p, st);
+    if (p.dk <= 256) return launch_scan_cols<4, 256>(p, st);
+    return launch_scan_cols<8, 256>(p, st);
   }
   // two columns per warp where the value size fills them and the registers hold them: half the CTAs stage the same rows
   const int nc = (p.dv >= 32 && p.dk <= 256) ? 2 : 1;

@@ -200,9 +200,9 @@ __global__ void __launch_bounds__(256) pool_prep_strip_kernel(const PoolAttn p) 
 // together; a token then costs the convolution in registers, one warp sum for the norm, the turn inside the lane and one
 // eight-byte store.  single: a strip is one row, whose convolution state — requested ahead of the dependency wait, an earlier step
 // left it there — moves on here.
-constexpr int kHeadStrip = 8;
+constexpr int kHeadStrip = 4;
 template <int TAPS, bool SINGLE>
-__global__ void __launch_bounds__(256) head_prep_kernel(const PoolAttn p) {
+__global__ void __launch_bounds__(256, 4) head_prep_kernel(const PoolAttn p) {
   using T = __nv_bfloat16;
   constexpr int STRIP = SINGLE ? 1 : kHeadStrip;
   pdl_trigger();

@@ -1,11 +1,12 @@
 // stack_rec.cuh — mixers of post-norm blocks (stack_rec.cu): the per-token preparation of an attention mixer (query / key
 // norms over the whole projection, rotate-half rotary positions, unit-rms values, value mix-in), and the linear
-// recurrences — ONE scan kernel for every recurrence of the form  S ← diag(d) S − p (qᵀS) + b vᵀ,  o = Sᵀr  (generalized
+// recurrences — ONE scan for every recurrence of the form  S ← diag(d) S − p (qᵀS) + b vᵀ,  o = Sᵀr  (generalized
 // delta rule: all terms; Mamba-2: a scalar d per head, no removal, b and r shared by a group of heads), with the
 // design-specific passes before it (gates, decays, unit keys, the short convolution) and behind it (head norms, gates).
 // Storage type T = bf16 or fp32; everything that enters a recurrence, its state and every norm are fp32.
 // Also the recurrences of hyper-connected blocks: RWKV-style time mixing (the same scan, its output read from the state
 // before the token joins it) and Mamba's selective scan (a decay per channel and state entry, a kernel of its own).
+// Recurrences without a removal — Mamba-2, time mixing, gated linear attention — take the scan's column-tile kernel.
 #pragma once
 #include "stack.cuh"
 

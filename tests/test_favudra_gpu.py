@@ -185,7 +185,7 @@ def test_crafted_scores_at_the_window_edge_and_far_away(dtype, decode, case, dim
     and without a window a key 296 positions back must be found — in a prompt and when the last token is decoded alone; also at
     head sizes that send the bf16 engine's prompts to the tensor-core attention kernel and its decode steps to the split-key
     kernels."""
-    n, window = 300, 136 if dim == 64 else 61
+    n, window = 300, 150 if dim == 64 else 61
     cfg = config([(tied(heads, kv_heads, dim, 0 if case == "far" else window, scale=4.0), None)])
     target = {"last_inside": n - window, "first_outside": n - 1 - window, "far": 3}[case]
     w, toks = aimed(cfg, 2, n, target)

@@ -518,20 +518,20 @@ FAVUDRA_SIZES = {
 def favudra_spec(name: str, max_ctx: int, max_slots: int = 8) -> models.StackSpec:
     z = FAVUDRA_SIZES[name]
     attn = models.AttnSpec(z["heads"], z["kv_heads"], z["dim"], z["dim"], z["dim"] ** -0.5, 0, 0, out_gate=False, bias=False, sink=True,
-                           softcap=50.0)
+                           softcap=30.0)
     tied = models.AttnSpec(z["heads"], z["kv_heads"], z["dim"], z["dim"], z["dim"] ** -0.5, z["window"], 0, out_gate=False, bias=False,
                            distance_bias=True, values_are_keys=True)
-    prep = models.AttnPrepSpec(rot=models.RotarySpec(dims=z["rot_dims"], base=5e5), rot_interleaved=True, head_norm=True, conv=z["conv"])
+    prep = models.AttnPrepSpec(rot=models.RotarySpec(dims=z["rot_dims"], base=1e4), rot_interleaved=True, head_norm=True, conv=z["conv"])
     L = models.StackLayerSpec
     kw = dict(ff_kind="gated", ff=z["ff"], ff_act="silu")
     t = L(attn=tied, **kw)
-    g = L(mixer="gla", gla=models.GlaSpec(z["g_heads"], z["g_dim"], z["g_vdim"], 16.0, z["rank"]), **kw)
+    g = L(mixer="gla", gla=models.GlaSpec(z["g_heads"], z["g_dim"], z["g_vdim"], 8.0, z["rank"]), **kw)
 
     def span(i):
         return (L(attn=attn, prep=prep, **kw), t, L(attn=attn, prep=prep, kv_from=i, **kw), g)
 
     return models.StackSpec(name="favudra-" + name, architecture="Favudra", width=z["width"], vocab=z["vocab"], layers=span(0) + span(4),
-                            embed_scale=8.0, norm_eps=1e-6, block="sandwich", norm_kind="rms", loop_mix=False, logit_scale=0.5,
+                            embed_scale=8.0, norm_eps=1e-5, block="sandwich", norm_kind="rms", loop_mix=False, logit_scale=0.25,
                             max_ctx=max_ctx, max_slots=max_slots)
 
 
